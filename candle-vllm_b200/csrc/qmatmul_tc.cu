@@ -605,7 +605,7 @@ qmatmul_tc_kernel(const __grid_constant__ CUtensorMap wmap0, const __grid_consta
                 const int gs = p.group_size;
                 if (gs <= 0 || (gs >= 64 && (gs & (gs - 1)) == 0)) {
                     // the usual groups (64 / 128 / one per column): a quarter (64 weights, 64-aligned) lies in ONE group -- one fetch, a shift
-                    // instead of the integer division (ncu: MUFU.RCP + ~20 IMAD per division, IMAD the most executed opcode of the kernel)
+                    // instead of an integer division per fetch (the kernel is bound by instruction issue)
                     const uint32_t g = gs > 0 ? (uint32_t)kq >> (31 - __clz(gs)) : 0u;
                     const uint32_t bits = static_cast<const unsigned short*>(c.scales)[g * (uint32_t)nn + (uint32_t)marlin_scale_pos(c.n_idx, gs > 0)];
                     m4_next[0] = m4_next[1] = __uint_as_float(bits);
