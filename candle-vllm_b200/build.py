@@ -48,7 +48,10 @@ GROUPS = {"ragged": ["lib", "linear_generic", "dense_gemm", "norm_act", "gated_d
           # kernels (the tcgen05 one also grouped), norms, the per-head preparation and pooled-cache kernels, the SIMT attention over the paged cache and the
           # tensor-core kernels it hands 128-wide heads to, the latent mixers incl. the split-KV latent decode kernel, the expert kernels
           "window": ["lib", "linear_generic", "dense_gemm", "norm_act", "attention_window", "attention_varlen", "attention_prefill", "attention_decode",
-                     "attention_generic", "attention_api", "latent_attention", "mla", "moe_ragged", "elementwise"]}
+                     "attention_generic", "attention_api", "latent_attention", "mla", "moe_ragged", "elementwise"],
+          # linear attention with a decay per key row beside attention whose heads mix their scores: both linear kernels, norms, the recurrences, the query / key /
+          # value preparation (with the paged attention it shares a file with) and the score-mixing attention, argmax
+          "talking": ["lib", "linear_generic", "dense_gemm", "norm_act", "linear_recurrence", "attention_varlen", "attention_prefill", "attention_talking", "elementwise"]}
 
 
 def so_path(group=None) -> str:

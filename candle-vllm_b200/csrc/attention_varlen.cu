@@ -10,7 +10,8 @@
 //                           already carries any frequency scaling and magnitude factor (optional), q written out in f32, k and v
 //                           written into the paged cache at slot_mapping[t] (K [nb, bs, G, dk], V [nb, bs, G, dv]).  The _ex form
 //                           adds a query temperature (q times 1 + coef ln(floor((p + 1) / every) + 1) at position p) and values
-//                           stored at unit root mean square per head.
+//                           stored at unit root mean square per head; the qkv_ form also turns the values by their own table [max_pos, dv/2] over
+//                           all dv entries, and with num_kv_heads = 0 prepares queries alone (a layer that attends over another layer's cache).
 //   paged_attention_varlen  one warp per (token, head); keys in tiles of 32 (a lane scores one key, the tile's values are then
 //                           accumulated with lanes across the value columns), online softmax in f32.  The _sink form puts exp(sink[h]) into
 //                           the denominator of head h (a key without a value; its score is not scaled).
@@ -28,7 +29,7 @@ qk_norm_rope_cache_kernel(const float* __restrict__ qkv, int64_t ld, const float
                           const float* __restrict__ cos_t, const float* __restrict__ sin_t, const int32_t* __restrict__ positions,
                           const int64_t* __restrict__ slot_mapping, TQ* __restrict__ q_out, TC* __restrict__ k_cache,
                           TC* __restrict__ v_cache, int H, int G, int dk, int dv, int rot_dims, float eps, float q_temp_coef, int q_temp_every,
-                          int v_unit_rms) {
+                          int v_unit_rms, const float* __restrict__ v_cos, const float* __restrict__ v_sin) {
     pdl_wait();
     pdl_trigger();
     __shared__ float red[2][8];
@@ -81,6 +82,17 @@ qk_norm_rope_cache_kernel(const float* __restrict__ qkv, int64_t ld, const float
             for (int i = lane; i < dv; i += 32) { const float v = vr[i]; ss = fmaf(v, v, ss); }
             const float sc = 1.0f / sqrtf(warp_sum(ss) / (float)dv + eps);
             for (int i = lane; i < dv; i += 32) v_cache[slot * nv + g * dv + i] = from_f32<TC>(vr[i] * sc);
+        }
+        return;
+    }
+    if (v_cos) {
+        // values turn with their position too, over all of their entries (i with i + dv/2)
+        const int vh = dv >> 1;
+        for (int i = threadIdx.x; i < nv; i += 256) {
+            const int d = i % dv, f = d < vh ? d : d - vh;
+            const float val = row[nq + nk + i], other = row[nq + nk + (d < vh ? i + vh : i - vh)];
+            const float c = v_cos[(int64_t)pos * vh + f], s = v_sin[(int64_t)pos * vh + f];
+            v_cache[slot * nv + i] = from_f32<TC>(d < vh ? val * c - other * s : val * c + other * s);
         }
         return;
     }
@@ -192,16 +204,27 @@ void qk_norm_rope_cache_ex(const float* qkv, int64_t ld, const float* q_norm_w, 
                            int32_t max_pos, const int32_t* positions, const int64_t* slot_mapping, void* q_out, void* key_cache, void* value_cache,
                            int32_t num_tokens, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t rot_dims, float eps,
                            float q_temp_coef, int32_t q_temp_every, int32_t v_unit_rms, int32_t cache_dtype, int32_t q_dtype, int64_t stream) {
+    B200_REQUIRE(num_tokens == 0 || (key_cache && value_cache && num_kv_heads > 0), kErrBadArg, "qk_norm_rope_cache: no cache");
+    qkv_norm_rope_cache(qkv, ld, q_norm_w, k_norm_w, cos_t, sin_t, nullptr, nullptr, max_pos, positions, slot_mapping, q_out, key_cache, value_cache, num_tokens,
+                        num_heads, num_kv_heads, dk, dv, rot_dims, eps, q_temp_coef, q_temp_every, v_unit_rms, cache_dtype, q_dtype, stream);
+}
+
+void qkv_norm_rope_cache(const float* qkv, int64_t ld, const float* q_norm_w, const float* k_norm_w, const float* cos_t, const float* sin_t, const float* v_cos,
+                         const float* v_sin, int32_t max_pos, const int32_t* positions, const int64_t* slot_mapping, void* q_out, void* key_cache, void* value_cache,
+                         int32_t num_tokens, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t rot_dims, float eps,
+                         float q_temp_coef, int32_t q_temp_every, int32_t v_unit_rms, int32_t cache_dtype, int32_t q_dtype, int64_t stream) {
     if (num_tokens == 0) return;
-    B200_REQUIRE(qkv && positions && slot_mapping && q_out && key_cache && value_cache, kErrBadArg, "qk_norm_rope_cache: null pointer");
+    B200_REQUIRE(qkv && positions && slot_mapping && q_out && ((key_cache && value_cache) || num_kv_heads == 0), kErrBadArg, "qk_norm_rope_cache: null pointer");
+    B200_REQUIRE((v_cos == nullptr) == (v_sin == nullptr) && (!v_cos || (dv % 2 == 0 && !v_unit_rms)), kErrBadArg,
+                 "qk_norm_rope_cache: value rotation needs both tables, an even value size and no value norm");
     B200_REQUIRE((q_norm_w == nullptr) == (k_norm_w == nullptr) && (cos_t == nullptr) == (sin_t == nullptr), kErrBadArg,
                  "qk_norm_rope_cache: norm weights / tables come in pairs");
-    B200_REQUIRE(num_heads > 0 && num_kv_heads > 0 && dk > 0 && dv > 0 && rot_dims >= 0 && rot_dims <= dk && rot_dims % 2 == 0 &&
-                 ld >= (int64_t)num_heads * dk + (int64_t)num_kv_heads * (dk + dv) && (!cos_t || max_pos > 0),
+    B200_REQUIRE(num_heads > 0 && num_kv_heads >= 0 && dk > 0 && dv > 0 && rot_dims >= 0 && rot_dims <= dk && rot_dims % 2 == 0 &&
+                 ld >= (int64_t)num_heads * dk + (int64_t)num_kv_heads * (dk + dv) && (!(cos_t || v_cos) || max_pos > 0),
                  kErrBadArg, "qk_norm_rope_cache: bad sizes");
     cudaStream_t st = as_stream(stream);
 #define QNRC(TC, TQ) launch_pdl(qk_norm_rope_cache_kernel<TC, TQ>, dim3(num_tokens), dim3(256), 0, st, qkv, ld, q_norm_w, k_norm_w, cos_t, sin_t, positions, \
-        slot_mapping, (TQ*)q_out, (TC*)key_cache, (TC*)value_cache, num_heads, num_kv_heads, dk, dv, rot_dims, eps, q_temp_coef, q_temp_every, v_unit_rms)
+        slot_mapping, (TQ*)q_out, (TC*)key_cache, (TC*)value_cache, num_heads, num_kv_heads, dk, dv, rot_dims, eps, q_temp_coef, q_temp_every, v_unit_rms, v_cos, v_sin)
     if (cache_dtype == B200_F32 && q_dtype == B200_F32) QNRC(float, float);
     else if (cache_dtype == B200_BF16 && q_dtype == B200_F32) QNRC(__nv_bfloat16, float);
     else if (cache_dtype == B200_BF16 && q_dtype == B200_BF16) QNRC(__nv_bfloat16, __nv_bfloat16);

@@ -11,12 +11,14 @@
 //                         the block-diagonal products;  out_t = S_t * gelu_tanh(y_t + y_bias).  One kernel for steps of few rows per entry;
 //                         for portions of prompts a row-parallel pass first turns gates and y into a_t, the input term and the GELU (in place);
 //                         from 512 rows per entry the bare scan that follows runs over chunks of 128 rows, all chunks at once.
-//   linear_attention      per head, S [dk, dv]:  S_t = a_t S_(t-1) + b_t k_t v_t^T,  o_t = S_t^T q_t, in two gatings:
+//   linear_attention      per head, S [dk, dv]:  S_t = a_t S_(t-1) + b_t k_t v_t^T,  o_t = S_t^T q_t, in two gatings (a third below):
 //                           fixed decay      a = decay[h], b = 1;
 //                           exponential      a_t = e^(f_t + m_(t-1) - m_t), b_t = e^(i_t - m_t) with the running maximum m_t = max(f_t + m_(t-1), i_t),
 //                                            m_0 = 0, i = cap tanh(. / cap), f = logsigmoid(cap tanh(. / cap)); a normaliser n_t = a_t n_(t-1) + b_t k_t
 //                                            rides along and o_t = S_t^T q_t / (max(|n_t . q_t|, e^(-m_t)) + 1e-6).  n and m are stored once per
 //                                            block of 16 value columns, so that no block reads what another one writes.
+//   linear_attention_channel  the same with a decay per token AND key row, S_t = diag(a_t) S_(t-1) + k_t v_t^T (a handed in as f32 [T, H dk]).
+//   low_rank_decay        those decays: a = sigmoid(w y + bias)^(1/tau), y a low-rank inner value per token.
 //                         A block of four warps owns 16 value columns of one head of one entry; inside a warp the key rows are split eight
 //                         ways (lane = 4 * part + column) with the lane's rows of S (and of n) in registers; tokens come in tiles of 16
 //                         staged through shared memory with the activation already applied, the per-token coefficients worked out once
@@ -414,18 +416,22 @@ struct LinAttnArgs {
     float* out;                                  // [T, H dv]
     const int32_t* cu_seqlens; const int32_t* seq_slots; const int32_t* seq_start;
     int H, dk, dv;
+    const float* alpha; int64_t lda;             // [T, H dk] row pitch lda: one decay per token and key row (channel decay)
 };
 
-template <int kR, bool kExp>
+// kG: 0 = a fixed decay per head, 1 = exponential gating, 2 = a decay per key row and token
+template <int kR, int kG>
 __global__ void __launch_bounds__(128)
 linear_attention_kernel(const LinAttnArgs A) {
     pdl_wait();
     pdl_trigger();
+    constexpr bool kExp = kG == 1, kChan = kG == 2;
     constexpr int kP = 8 * kR;                   // padded key rows
     extern __shared__ __align__(16) float smem[];
     float* sq = smem;                            // [kTile][kP]
     float* sk = sq + kTile * kP;                 // [kTile][kP]
-    float* sv = sk + kTile * kP;                 // [kTile][16]
+    float* sal = sk + kTile * kP;                // [kTile][kP] decays of the key rows (channel decay only)
+    float* sv = sal + (kChan ? kTile * kP : 0);  // [kTile][16]
     float* sa = sv + kTile * 16;                 // [kTile] decay of the state
     float* sb = sa + kTile;                      // [kTile] weight of the new outer product
     float* se = sb + kTile;                      // [kTile] e^(-m_t)
@@ -469,10 +475,10 @@ linear_attention_kernel(const LinAttnArgs A) {
         }
     }
     if (kExp && threadIdx.x == 0) sm[0] = fresh ? 0.f : A.mx[own];
-    const float fixed_a = kExp ? 0.f : A.decay[h];
+    const float fixed_a = kG == 0 ? A.decay[h] : 0.f;
     // the next tile's operands travel in registers while the current tile is walked: element e = thread + 128 i of the tile's [16][kP] q and k
     // rows, two of its [16][16] values, and (lanes 0..15 of the last warp) the two gate pre-activations of a token
-    float pq[kR], pk[kR], pv[2], pgi = 0.f, pgf = 0.f;
+    float pq[kR], pk[kR], pal[kChan ? kR : 1], pv[2], pgi = 0.f, pgf = 0.f;
     auto fetch = [&](int tb) {
         const int nt = min(kTile, t1 - tb);
 #pragma unroll
@@ -482,6 +488,7 @@ linear_attention_kernel(const LinAttnArgs A) {
             const float* row = A.proj + (int64_t)(tb + (ok ? tt : 0)) * A.ld;
             pq[i] = ok ? row[A.off_q + h * dk + r] : 0.f;
             pk[i] = ok ? row[A.off_k + h * dk + r] : 0.f;
+            if (kChan) pal[i] = ok ? A.alpha[(int64_t)(tb + tt) * A.lda + h * dk + r] : 0.f;
         }
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -504,6 +511,7 @@ linear_attention_kernel(const LinAttnArgs A) {
             float qv = pq[i], kv = pk[i];
             if (A.act == 1) { qv = silu_f(qv); kv = silu_f(kv); }
             sq[e] = qv * A.q_scale; sk[e] = kv;
+            if (kChan) sal[e] = pal[i];
         }
 #pragma unroll
         for (int i = 0; i < 2; ++i) sv[threadIdx.x + 128 * i] = A.act == 1 ? silu_f(pv[i]) : pv[i];
@@ -541,14 +549,15 @@ linear_attention_kernel(const LinAttnArgs A) {
             float acc[2] = {0.f, 0.f}, nq[2] = {0.f, 0.f};
             const float4* q4 = reinterpret_cast<const float4*>(sq + tt * kP + part * kR);
             const float4* k4 = reinterpret_cast<const float4*>(sk + tt * kP + part * kR);
+            const float4* a4 = reinterpret_cast<const float4*>(sal + tt * kP + part * kR);
 #pragma unroll
             for (int r4 = 0; r4 < kR / 4; ++r4) {
-                const float4 qq = q4[r4], kk = k4[r4];
-                const float qa[4] = {qq.x, qq.y, qq.z, qq.w}, ka[4] = {kk.x, kk.y, kk.z, kk.w};
+                const float4 qq = q4[r4], kk = k4[r4], aa = kChan ? a4[r4] : make_float4(a, a, a, a);
+                const float qa[4] = {qq.x, qq.y, qq.z, qq.w}, ka[4] = {kk.x, kk.y, kk.z, kk.w}, da[4] = {aa.x, aa.y, aa.z, aa.w};
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     const int r = r4 * 4 + j;
-                    S[r] = fmaf(a, S[r], ka[j] * bv);
+                    S[r] = fmaf(da[j], S[r], ka[j] * bv);
                     acc[j & 1] = fmaf(S[r], qa[j], acc[j & 1]);
                     if (kExp) { nv[r] = fmaf(a, nv[r], ka[j] * bn); nq[j & 1] = fmaf(nv[r], qa[j], nq[j & 1]); }
                 }
@@ -602,11 +611,12 @@ linear_attention_kernel(const LinAttnArgs A) {
 // Steps in which every entry brings one token (row b belongs to entry b): nothing is staged and no thread waits for another -- a lane reads its
 // own rows of q and k, its column's value and (exponential gating) the two gate values straight from the projection, takes one pass over its
 // rows of the state and writes them back.  Same lane layout and state layout as the kernel above.
-template <int kR, bool kExp>
+template <int kR, int kG>
 __global__ void __launch_bounds__(128)
 linear_attention_step_kernel(const LinAttnArgs A) {
     pdl_wait();
     pdl_trigger();
+    constexpr bool kExp = kG == 1, kChan = kG == 2;
     const int h = blockIdx.y, b = blockIdx.z;
     const int H = A.H, dk = A.dk, dv = A.dv;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -620,7 +630,7 @@ linear_attention_step_kernel(const LinAttnArgs A) {
     const int64_t own = (slot * H + h) * (int64_t)gridDim.x + blockIdx.x;
     float* np = kExp ? A.nrm + own * dk + part * kR : nullptr;
     const float* row = A.proj + (int64_t)b * A.ld;
-    float S[kR], nv[kR], q[kR], k[kR];
+    float S[kR], nv[kR], q[kR], k[kR], al[kChan ? kR : 1];
 #pragma unroll
     for (int r = 0; r < kR; ++r) {
         const int g = part * kR + r;
@@ -628,6 +638,7 @@ linear_attention_step_kernel(const LinAttnArgs A) {
         S[r] = 0.f; nv[r] = 0.f;
         q[r] = ok ? row[A.off_q + h * dk + g] : 0.f;
         k[r] = ok ? row[A.off_k + h * dk + g] : 0.f;
+        if (kChan) al[r] = ok ? A.alpha[(int64_t)b * A.lda + h * dk + g] : 0.f;
     }
     float v = col_ok ? row[A.off_v + h * dv + col] : 0.f;
     float zi = 0.f, zf = 0.f, m_prev = 0.f;
@@ -653,7 +664,7 @@ linear_attention_step_kernel(const LinAttnArgs A) {
             }
         }
     }
-    float a = kExp ? 0.f : A.decay[h], bw = 1.0f, em = 0.f, m_new = 0.f;
+    float a = kG == 0 ? A.decay[h] : 0.f, bw = 1.0f, em = 0.f, m_new = 0.f;
     if (kExp) {
         const float gi = A.cap * tanhf(zi / A.cap), gf = log_sigmoid_f(A.cap * tanhf(zf / A.cap));
         m_new = fmaxf(gf + m_prev, gi);
@@ -667,7 +678,7 @@ linear_attention_step_kernel(const LinAttnArgs A) {
         float qv = q[r], kv = k[r];
         if (A.act == 1) { qv = silu_f(qv); kv = silu_f(kv); }
         qv *= A.q_scale;
-        S[r] = fmaf(a, S[r], kv * bv);
+        S[r] = fmaf(kChan ? al[r] : a, S[r], kv * bv);
         acc[r & 1] = fmaf(S[r], qv, acc[r & 1]);
         if (kExp) { nv[r] = fmaf(a, nv[r], kv * bw); nq[r & 1] = fmaf(nv[r], qv, nq[r & 1]); }
     }
@@ -716,11 +727,11 @@ struct ChunkArgs {
     LinAttnArgs A;
     float* gc;            // [T, H, 3]: F_t, li_t, m_t (exponential gating)
     float* U;             // [chunk slots, H, dv, dk]
-    float* un;            // [chunk slots, H, dk] a chunk's own term of the normaliser
+    float* un;            // [chunk slots, H, dk] a chunk's own term of the normaliser; with channel decay the product of the chunk's decays per key row
     float* un_in;         // [chunk slots, H, dk] the normaliser that enters the chunk
     float* m0;            // [entries, H] the maximum every entry starts this step with (the slot's copy changes while the kernels run)
     int max_chunks;       // the most chunks any entry has
-    int gating;
+    int gating;           // 0 fixed decay, 1 exponential, 2 channel decay
 };
 
 __device__ __forceinline__ int chunk_base(const int32_t* cu, int b) {      // chunk slots of the entries before b
@@ -782,12 +793,12 @@ __global__ void la_gate_chain_kernel(const ChunkArgs C) {
 
 // F, li, m of row t (tt = its index inside the chunk)
 __device__ __forceinline__ void token_gate(const ChunkArgs& C, int h, int t, int tt, float lnd, float& F, float& li, float& m) {
-    if (C.gating == 0) { F = (float)(tt + 1) * lnd; li = 0.f; m = 0.f; return; }
+    if (C.gating != 1) { F = (float)(tt + 1) * lnd; li = 0.f; m = 0.f; return; }
     const float* g = C.gc + ((int64_t)t * C.A.H + h) * 3;
     F = g[0]; li = g[1]; m = g[2];
 }
 __device__ __forceinline__ float chunk_m_in(const ChunkArgs& C, int b, int h, int t_first, int c) {
-    if (C.gating == 0) return 0.f;
+    if (C.gating != 1) return 0.f;
     if (c > 0) return C.gc[((int64_t)(t_first - 1) * C.A.H + h) * 3 + 2];
     return C.m0[(int64_t)b * C.A.H + h];
 }
@@ -895,7 +906,7 @@ la_chunk_scan_kernel(const ChunkArgs C) {
     for (int a = 0; a < kAhead; ++a) {
         const int c = min(a, nc - 1);
         nu[a] = u0[c * ustride];
-        nn[a] = carries_n ? C.un[n0 + c * nstride] : 0.f;
+        nn[a] = (carries_n || C.gating == 2) ? C.un[n0 + c * nstride] : 0.f;      // channel decay: the product of the chunk's decays of this key row
     }
     for (int cb = 0; cb < nc; cb += kAhead) {
         float cu[kAhead], cn[kAhead];
@@ -905,7 +916,7 @@ la_chunk_scan_kernel(const ChunkArgs C) {
         for (int a = 0; a < kAhead; ++a) {
             const int c = min(cb + kAhead + a, nc - 1);
             nu[a] = u0[c * ustride];
-            nn[a] = carries_n ? C.un[n0 + c * nstride] : 0.f;
+            nn[a] = (carries_n || C.gating == 2) ? C.un[n0 + c * nstride] : 0.f;
         }
 #pragma unroll
         for (int a = 0; a < kAhead; ++a) {
@@ -914,7 +925,7 @@ la_chunk_scan_kernel(const ChunkArgs C) {
             const int nt = min(kChunk, rows - c * kChunk);
             float FL, liL, mL;
             token_gate(C, h, t0 + c * kChunk + nt - 1, nt - 1, lnd, FL, liL, mL);
-            const float g = expf(FL + m_in - mL);
+            const float g = C.gating == 2 ? cn[a] : expf(FL + m_in - mL);
             u0[c * ustride] = S;
             S = fmaf(g, S, cu[a]);
             if (carries_n) {
@@ -1090,24 +1101,295 @@ la_chunk_output_kernel(const ChunkArgs C) {
     }
 }
 
-template <int kR, bool kExp>
-void launch_linear_attention(const LinAttnArgs& A, int num_seqs, bool single_rows, cudaStream_t st) {
-    if (single_rows) {
-        launch_pdl(linear_attention_step_kernel<kR, kExp>, dim3(ceil_div(A.dv, 16), A.H, num_seqs), dim3(128), 0, st, A);
-        return;
+// ---- a decay per token and key row (gated linear attention) over chunks --------------------------------------------------------------------------
+// S_t = diag(a_t) S_(t-1) + k_t v_t^T.  Everything is built from PRODUCTS of decays, all of them in [0, 1], so nothing overflows whatever the decays are
+// and a product that underflows is a contribution that has died.  With tokens grouped in runs of four, run c's product E_c, the product P_t of a
+// token's own run up to and including t and the product R_j of a token's own run after j:
+//     chunk state term     sum_j (prod_{i > j} a_i * k_j) v_j^T                                       (la_chan_state_kernel; E of the whole chunk beside it)
+//     score of t over j    sum_r q_t P_t (prod_{runs between} E) R_j k_j, j in an earlier run; inside one run the products of at most three decays
+//     entering state       q_t P_t prod_{runs before} E against S_in                                      (la_chan_output_kernel)
+// The walk over the chunks is la_chunk_scan_kernel with the chunk's product per key row in place of the scalar decay.
+__global__ void __launch_bounds__(256)
+low_rank_decay_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ alpha, int T, int N,
+                      int R, float inv_tau) {
+    pdl_wait();
+    pdl_trigger();
+    // 256 channels x 8 tokens per block: a thread keeps 16 weights of its channel at a time and meets eight tokens' inner values with them
+    __shared__ float ys[8][16];
+    const int n = blockIdx.x * 256 + threadIdx.x, t0 = blockIdx.y * 8;
+    float z[8];
+    const float b = (n < N && bias) ? bias[n] : 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) z[i] = 0.f;
+    for (int r0 = 0; r0 < R; r0 += 16) {
+        float wr[16];
+#pragma unroll
+        for (int r = 0; r < 16; ++r) wr[r] = (n < N && r0 + r < R) ? w[(int64_t)n * R + r0 + r] : 0.f;
+        __syncthreads();
+        if (threadIdx.x < 128) {
+            const int i = threadIdx.x >> 4, r = threadIdx.x & 15;
+            ys[i][r] = (t0 + i < T && r0 + r < R) ? y[(int64_t)(t0 + i) * ldy + r0 + r] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+#pragma unroll
+            for (int r = 0; r < 16; ++r) z[i] = fmaf(wr[r], ys[i][r], z[i]);
     }
-    const int smem = (2 * kTile * 8 * kR + kTile * 16 + 6 * kTile + 1) * (int)sizeof(float);
-    ensure_dynamic_smem(reinterpret_cast<const void*>(linear_attention_kernel<kR, kExp>), smem);
-    launch_pdl(linear_attention_kernel<kR, kExp>, dim3(ceil_div(A.dv, 16), A.H, num_seqs), dim3(128), (size_t)smem, st, A);
+    if (n >= N) return;
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+        if (t0 + i < T) alpha[(int64_t)(t0 + i) * N + n] = expf(log_sigmoid_f(z[i] + b) * inv_tau);
 }
 
-template <bool kExp>
+__global__ void __launch_bounds__(256)
+la_chan_state_kernel(const ChunkArgs C) {
+    pdl_wait();
+    pdl_trigger();
+    const LinAttnArgs& A = C.A;
+    __shared__ __align__(16) float vs[kChunk][64 + 4], ks[kChunk][64 + 4];
+    __shared__ float es[4][64];
+    const int h = blockIdx.y, b = blockIdx.z / C.max_chunks, c = blockIdx.z % C.max_chunks;
+    const int t0 = A.cu_seqlens[b], rows = A.cu_seqlens[b + 1] - t0;
+    if (c * kChunk >= rows) return;
+    const int tf = t0 + c * kChunk, nt = min(kChunk, rows - c * kChunk);
+    const int dk = A.dk, dv = A.dv, H = A.H;
+    const int tiles_r = (dk + 63) / 64;
+    const int cv0 = (blockIdx.x / tiles_r) * 64, r0 = (blockIdx.x % tiles_r) * 64;
+    const int slot = chunk_base(A.cu_seqlens, b) + c;
+    // a thread takes sixteen neighbouring tokens of one key row: the products of the decays after each of them, then after their quarter of the chunk
+    const int x = threadIdx.x & 63, quarter = threadIdx.x >> 6;
+    float k[16], a[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const int j = quarter * 16 + i;
+        const bool ok = j < nt && r0 + x < dk;
+        const int64_t t = tf + (ok ? j : 0);
+        k[i] = ok ? A.proj[t * A.ld + A.off_k + h * dk + r0 + x] : 0.f;
+        a[i] = ok ? A.alpha[t * A.lda + h * dk + r0 + x] : 1.f;
+    }
+    for (int e = threadIdx.x; e < kChunk * 64; e += 256) {
+        const int j = e >> 6, cx = e & 63;
+        vs[j][cx] = (j < nt && cv0 + cx < dv) ? A.proj[(int64_t)(tf + j) * A.ld + A.off_v + h * dv + cv0 + cx] : 0.f;
+    }
+    float run = 1.f;
+#pragma unroll
+    for (int i = 15; i >= 0; --i) { k[i] *= run; run *= a[i]; }
+    es[quarter][x] = run;
+    __syncthreads();
+    float tail = 1.f;
+    for (int s = quarter + 1; s < 4; ++s) tail *= es[s][x];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) ks[quarter * 16 + i][x] = k[i] * tail;
+    if (quarter == 0 && cv0 == 0 && r0 + x < dk) C.un[((int64_t)slot * H + h) * dk + r0 + x] = run * tail;
+    __syncthreads();
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    float acc[4][4] = {};
+    for (int j = 0; j < nt; ++j) {
+        const float4 a4 = *reinterpret_cast<const float4*>(&vs[j][ty * 4]), k4 = *reinterpret_cast<const float4*>(&ks[j][tx * 4]);
+        const float va[4] = {a4.x, a4.y, a4.z, a4.w}, ka[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int l = 0; l < 4; ++l) acc[i][l] = fmaf(va[i], ka[l], acc[i][l]);
+    }
+    float* U = C.U + ((int64_t)slot * H + h) * dv * dk;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int cv = cv0 + ty * 4 + i;
+        if (cv >= dv) continue;
+#pragma unroll
+        for (int l = 0; l < 4; ++l) {
+            const int r = r0 + tx * 4 + l;
+            if (r < dk) U[(int64_t)cv * dk + r] = acc[i][l];
+        }
+    }
+}
+
+constexpr int kRunPitch = 257;                   // floats per key row of the table of run products: 16 x 16, padded against bank conflicts
+constexpr int kChanOutFloats = 3 * 32 * 68 + 2 * 64 * 68 + 32 * 17;
+
+__global__ void __launch_bounds__(256, 2)
+la_chan_output_kernel(const ChunkArgs C) {
+    pdl_wait();
+    pdl_trigger();
+    const LinAttnArgs& A = C.A;
+    extern __shared__ __align__(16) float sm[];
+    float (*qs)[68] = reinterpret_cast<float (*)[68]>(sm);                          // [32][68] q_t P_t of a slab of 32 key rows: [key row][token]
+    float (*ks)[68] = reinterpret_cast<float (*)[68]>(sm + 32 * 68);                // [32][68] k_j R_j
+    float (*us)[68] = reinterpret_cast<float (*)[68]>(sm + 2 * 32 * 68);            // [32][68] the entering state: [key row][value column]
+    float* mm = sm + 3 * 32 * 68;                                                   // [32][257] products of the runs between run b and run a at a * 16 + b (a > b); before run a at a * 17
+    float (*pw)[68] = reinterpret_cast<float (*)[68]>(sm + 3 * 32 * 68);            // [64][68] scores: [key token][query token], over the table once the slabs are done
+    float (*vs)[68] = reinterpret_cast<float (*)[68]>(sm + 3 * 32 * 68 + 64 * 68);  // [64][68] values: [token][column]
+    float* es = sm + 3 * 32 * 68 + 2 * 64 * 68;                                     // [32][17] E of the sixteen runs
+    static_assert(32 * kRunPitch <= 2 * 64 * 68, "the table of run products fits under the score and value tiles");
+    const int h = blockIdx.y, b = blockIdx.z / C.max_chunks, c = blockIdx.z % C.max_chunks;
+    const int t0 = A.cu_seqlens[b], rows = A.cu_seqlens[b + 1] - t0;
+    if (c * kChunk >= rows) return;
+    const int tf = t0 + c * kChunk, nt = min(kChunk, rows - c * kChunk);
+    const int dk = A.dk, dv = A.dv, H = A.H;
+    const int cv0 = blockIdx.x * 64;
+    const int slot = chunk_base(A.cu_seqlens, b) + c;
+    const float* Uin = C.U + ((int64_t)slot * H + h) * dv * dk;
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    // a thread prepares two runs (warp and warp + 8) of one key row (lane) per slab; the next slab's operands are fetched ahead
+    float rq[2][4], rk[2][4], ra[2][4], ru[8];
+    auto fetch = [&](int r0) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const int j = (warp + 8 * i) * 4 + t;
+                const bool ok = j < nt && r0 + lane < dk;
+                const int64_t row = tf + (ok ? j : 0);
+                rq[i][t] = ok ? A.proj[row * A.ld + A.off_q + h * dk + r0 + lane] * A.q_scale : 0.f;
+                rk[i][t] = ok ? A.proj[row * A.ld + A.off_k + h * dk + r0 + lane] : 0.f;
+                ra[i][t] = ok ? A.alpha[row * A.lda + h * dk + r0 + lane] : 1.f;
+            }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int e = threadIdx.x + 256 * i, j = e >> 5, x = e & 31;
+            ru[i] = (cv0 + j < dv && r0 + x < dk) ? Uin[(int64_t)(cv0 + j) * dk + r0 + x] : 0.f;
+        }
+    };
+    float acc[4][4] = {}, o[4][4] = {};
+    float dg[2][10] = {};                        // scores inside the thread's two runs: (j, t) for j <= t < 4, this lane's key rows
+    fetch(0);
+    for (int r0 = 0; r0 < dk; r0 += 32) {
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int a = warp + 8 * i;
+            float p = 1.f, q4[4], k4[4];
+#pragma unroll
+            for (int t = 0; t < 4; ++t) { p *= ra[i][t]; q4[t] = rq[i][t] * p; }
+            es[lane * 17 + a] = p;
+            float s = 1.f;
+#pragma unroll
+            for (int t = 3; t >= 0; --t) { k4[t] = rk[i][t] * s; s *= ra[i][t]; }
+            *reinterpret_cast<float4*>(&qs[lane][a * 4]) = make_float4(q4[0], q4[1], q4[2], q4[3]);
+            *reinterpret_cast<float4*>(&ks[lane][a * 4]) = make_float4(k4[0], k4[1], k4[2], k4[3]);
+            int n = 0;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                float kj = rk[i][j];
+#pragma unroll
+                for (int t = j; t < 4; ++t) {
+                    if (t > j) kj *= ra[i][t];
+                    dg[i][n] = fmaf(rq[i][t], kj, dg[i][n]);
+                    ++n;
+                }
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int e = threadIdx.x + 256 * i;
+            us[e & 31][e >> 5] = ru[i];
+        }
+        __syncthreads();
+        // the table of run products of every key row of the slab: chains of equal total length per warp
+        {
+            const float* er = es + lane * 17;
+            float* mr = mm + lane * kRunPitch;
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int rb = i == 0 ? warp : 15 - warp;
+                float m = 1.f;
+                for (int a = rb + 1; a < 16; ++a) { mr[a * 16 + rb] = m; m *= er[a]; }
+            }
+            if (warp == 7) {
+                float m = 1.f;
+                for (int a = 0; a < 16; ++a) { mr[a * 17] = m; m *= er[a]; }
+            }
+        }
+        __syncthreads();
+        if (r0 + 32 < dk) fetch(r0 + 32);
+#pragma unroll 4
+        for (int x = 0; x < 32; ++x) {
+            const float4 q4 = *reinterpret_cast<const float4*>(&qs[x][ty * 4]), k4 = *reinterpret_cast<const float4*>(&ks[x][tx * 4]),
+                         u4 = *reinterpret_cast<const float4*>(&us[x][tx * 4]);
+            const float m = mm[x * kRunPitch + ty * 16 + tx], before = mm[x * kRunPitch + ty * 17];
+            const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x * m, k4.y * m, k4.z * m, k4.w * m}, u[4] = {u4.x * before, u4.y * before, u4.z * before, u4.w * before};
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int l = 0; l < 4; ++l) { acc[i][l] = fmaf(q[i], k[l], acc[i][l]); o[i][l] = fmaf(q[i], u[l], o[i][l]); }
+        }
+    }
+    float rv[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const int e = threadIdx.x + 256 * i, j = e >> 6, x = e & 63;
+        rv[i] = (j < nt && cv0 + x < dv) ? A.proj[(int64_t)(tf + j) * A.ld + A.off_v + h * dv + cv0 + x] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int n = 0; n < 10; ++n) dg[i][n] = warp_sum(dg[i][n]);
+    __syncthreads();                             // the table has been read: its place takes the scores and the values
+    if (tx != ty) {                              // an earlier run's keys as summed, a later run's not at all (what was summed there is not a score)
+        const bool seen = tx < ty;
+#pragma unroll
+        for (int l = 0; l < 4; ++l)
+            *reinterpret_cast<float4*>(&pw[tx * 4 + l][ty * 4]) = seen ? make_float4(acc[0][l], acc[1][l], acc[2][l], acc[3][l]) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (lane == 0) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int a = (warp + 8 * i) * 4;
+            *reinterpret_cast<float4*>(&pw[a][a]) = make_float4(dg[i][0], dg[i][1], dg[i][2], dg[i][3]);
+            *reinterpret_cast<float4*>(&pw[a + 1][a]) = make_float4(0.f, dg[i][4], dg[i][5], dg[i][6]);
+            *reinterpret_cast<float4*>(&pw[a + 2][a]) = make_float4(0.f, 0.f, dg[i][7], dg[i][8]);
+            *reinterpret_cast<float4*>(&pw[a + 3][a]) = make_float4(0.f, 0.f, 0.f, dg[i][9]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const int e = threadIdx.x + 256 * i;
+        vs[e >> 6][e & 63] = rv[i];
+    }
+    __syncthreads();
+    const int last = min(nt, ty * 4 + 4);        // no key after the thread's last query
+#pragma unroll 4
+    for (int j = 0; j < last; ++j) {
+        const float4 p4 = *reinterpret_cast<const float4*>(&pw[j][ty * 4]), v4 = *reinterpret_cast<const float4*>(&vs[j][tx * 4]);
+        const float p[4] = {p4.x, p4.y, p4.z, p4.w}, v[4] = {v4.x, v4.y, v4.z, v4.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int l = 0; l < 4; ++l) o[i][l] = fmaf(p[i], v[l], o[i][l]);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int t = ty * 4 + i;
+        if (t >= nt) continue;
+#pragma unroll
+        for (int l = 0; l < 4; ++l) {
+            const int cv = cv0 + tx * 4 + l;
+            if (cv < dv) A.out[(int64_t)(tf + t) * H * dv + h * dv + cv] = o[i][l];
+        }
+    }
+}
+
+template <int kR, int kG>
+void launch_linear_attention(const LinAttnArgs& A, int num_seqs, bool single_rows, cudaStream_t st) {
+    if (single_rows) {
+        launch_pdl(linear_attention_step_kernel<kR, kG>, dim3(ceil_div(A.dv, 16), A.H, num_seqs), dim3(128), 0, st, A);
+        return;
+    }
+    const int smem = ((kG == 2 ? 3 : 2) * kTile * 8 * kR + kTile * 16 + 6 * kTile + 1) * (int)sizeof(float);
+    ensure_dynamic_smem(reinterpret_cast<const void*>(linear_attention_kernel<kR, kG>), smem);
+    launch_pdl(linear_attention_kernel<kR, kG>, dim3(ceil_div(A.dv, 16), A.H, num_seqs), dim3(128), (size_t)smem, st, A);
+}
+
+template <int kG>
 bool dispatch_linear_attention(const LinAttnArgs& A, int num_seqs, bool single_rows, cudaStream_t st) {
-    if (A.dk <= 32) launch_linear_attention<4, kExp>(A, num_seqs, single_rows, st);
-    else if (A.dk <= 64) launch_linear_attention<8, kExp>(A, num_seqs, single_rows, st);
-    else if (A.dk <= 128) launch_linear_attention<16, kExp>(A, num_seqs, single_rows, st);
-    else if (A.dk <= 256) launch_linear_attention<32, kExp>(A, num_seqs, single_rows, st);
-    else if (A.dk <= 512) launch_linear_attention<64, kExp>(A, num_seqs, single_rows, st);      // spills its staging registers: a path for correctness, not speed
+    if (A.dk <= 32) launch_linear_attention<4, kG>(A, num_seqs, single_rows, st);
+    else if (A.dk <= 64) launch_linear_attention<8, kG>(A, num_seqs, single_rows, st);
+    else if (A.dk <= 128) launch_linear_attention<16, kG>(A, num_seqs, single_rows, st);
+    else if (A.dk <= 256) launch_linear_attention<32, kG>(A, num_seqs, single_rows, st);
+    else if (A.dk <= 512) launch_linear_attention<64, kG>(A, num_seqs, single_rows, st);      // spills its staging registers: a path for correctness, not speed
     else return false;
     return true;
 }
@@ -1235,10 +1517,10 @@ void linear_attention(const float* proj, int64_t ld, int32_t off_q, int32_t off_
                  "linear_attention: fixed decay needs decay[H]; exponential gating needs the normaliser, the maximum and a positive cap");
     B200_REQUIRE(dk <= 512, kErrUnsupported, "linear_attention: key size %d > 512", dk);
     LinAttnArgs A{proj, ld, off_q, off_k, off_v, off_i, off_f, decay, i_bias, f_bias, gate_cap, q_scale, act, state, normaliser, maximum, out,
-                  cu_seqlens, seq_slots, seq_start, num_heads, dk, dv};
+                  cu_seqlens, seq_slots, seq_start, num_heads, dk, dv, nullptr, 0};
     cudaStream_t st = as_stream(stream);
-    if (gating == 0) dispatch_linear_attention<false>(A, num_seqs, single_rows != 0, st);
-    else dispatch_linear_attention<true>(A, num_seqs, single_rows != 0, st);
+    if (gating == 0) dispatch_linear_attention<0>(A, num_seqs, single_rows != 0, st);
+    else dispatch_linear_attention<1>(A, num_seqs, single_rows != 0, st);
     count_launch();
     check_launch("linear_attention");
 }
@@ -1264,7 +1546,7 @@ void linear_attention_chunked(const float* proj, int64_t ld, int32_t off_q, int3
     const int64_t slots = (int64_t)(num_tokens + kChunk - 1) / kChunk + num_seqs;
     ChunkArgs C;
     C.A = LinAttnArgs{proj, ld, off_q, off_k, off_v, off_i, off_f, decay, i_bias, f_bias, gate_cap, q_scale, act, state, normaliser, maximum, out,
-                      cu_seqlens, seq_slots, seq_start, num_heads, dk, dv};
+                      cu_seqlens, seq_slots, seq_start, num_heads, dk, dv, nullptr, 0};
     C.U = scratch;
     C.un = C.U + slots * num_heads * dv * dk;
     C.un_in = C.un + slots * num_heads * dk;
@@ -1287,6 +1569,53 @@ void linear_attention_chunked(const float* proj, int64_t ld, int32_t off_q, int3
     launch_pdl(la_chunk_output_kernel, dim3(ceil_div(dv, 64), num_heads, z), dim3(256), (size_t)smem, st, C);
     count_launch(launches);
     check_launch("linear_attention_chunked");
+}
+
+void low_rank_decay(const float* y, int64_t ldy, const float* weight, const float* bias, float* alpha, int32_t num_tokens, int32_t channels, int32_t rank, float tau,
+                    int64_t stream) {
+    if (num_tokens == 0) return;
+    B200_REQUIRE(y && weight && alpha && channels > 0 && rank > 0 && ldy >= rank && tau > 0.f && num_tokens <= 8 * 65535, kErrBadArg, "low_rank_decay: bad arguments");
+    launch_pdl(low_rank_decay_kernel, dim3(ceil_div(channels, 256), ceil_div(num_tokens, 8)), dim3(256), 0, as_stream(stream), y, ldy, weight, bias, alpha,
+               (int)num_tokens, (int)channels, (int)rank, 1.0f / tau);
+    count_launch();
+    check_launch("low_rank_decay");
+}
+
+void linear_attention_channel(const float* proj, int64_t ld, int32_t off_q, int32_t off_k, int32_t off_v, const float* alpha, int64_t lda, float q_scale, float* state,
+                              float* out, float* scratch, const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens,
+                              int32_t num_seqs, int32_t max_rows, int32_t mode, int32_t num_heads, int32_t dk, int32_t dv, int64_t stream) {
+    if (num_seqs == 0 || num_tokens == 0) return;
+    B200_REQUIRE(proj && alpha && state && out && cu_seqlens && seq_slots && seq_start && num_heads > 0 && num_heads <= 65535 && num_seqs <= 65535 && dk > 0 && dv > 0 &&
+                 lda >= (int64_t)num_heads * dk && mode >= 0 && mode <= 2, kErrBadArg, "linear_attention_channel: bad arguments");
+    LinAttnArgs A{proj, ld, off_q, off_k, off_v, 0, 0, nullptr, nullptr, nullptr, 0.f, q_scale, 0, state, nullptr, nullptr, out,
+                  cu_seqlens, seq_slots, seq_start, num_heads, dk, dv, alpha, lda};
+    cudaStream_t st = as_stream(stream);
+    if (mode != 2) {
+        B200_REQUIRE(mode == 0 || num_tokens == num_seqs, kErrBadArg, "linear_attention_channel: the single-row kernel takes one row per entry");
+        B200_REQUIRE(dk <= 512, kErrUnsupported, "linear_attention_channel: key size %d > 512", dk);
+        dispatch_linear_attention<2>(A, num_seqs, mode == 1, st);
+        count_launch();
+        check_launch("linear_attention_channel");
+        return;
+    }
+    B200_REQUIRE(scratch && max_rows > 0, kErrBadArg, "linear_attention_channel: the chunked form needs scratch and max_rows");
+    const int max_chunks = (max_rows + kChunk - 1) / kChunk;
+    B200_REQUIRE((int64_t)max_chunks * num_seqs <= 65535, kErrUnsupported, "linear_attention_channel: %d chunks x %d entries exceed the grid", max_chunks, num_seqs);
+    const int64_t slots = (int64_t)(num_tokens + kChunk - 1) / kChunk + num_seqs;
+    ChunkArgs C{};
+    C.A = A;
+    C.U = scratch;
+    C.un = C.U + slots * num_heads * dv * dk;
+    C.max_chunks = max_chunks;
+    C.gating = 2;
+    const unsigned z = (unsigned)(max_chunks * num_seqs);
+    launch_pdl(la_chan_state_kernel, dim3(ceil_div(dv, 64) * ceil_div(dk, 64), num_heads, z), dim3(256), 0, st, C);
+    launch_pdl(la_chunk_scan_kernel, dim3(ceil_div((int64_t)num_heads * dv * dk, 256), num_seqs), dim3(256), 0, st, C);
+    const int smem = kChanOutFloats * (int)sizeof(float);
+    ensure_dynamic_smem(reinterpret_cast<const void*>(la_chan_output_kernel), smem);
+    launch_pdl(la_chan_output_kernel, dim3(ceil_div(dv, 64), num_heads, z), dim3(256), (size_t)smem, st, C);
+    count_launch(3);
+    check_launch("linear_attention_channel");
 }
 
 }  // extern "C"

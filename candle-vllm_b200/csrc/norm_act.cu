@@ -23,7 +23,11 @@
 //                    with `row_index` only the selected rows are summed and normed and x is left as it is; w null = the sum alone;
 //   group_rms_norm_gate  out = o / rms(o over a group of neighbours) * w * act(gate): the closing norm of the linear-attention mixers,
 //                    one group per head or one for the whole row;
-//   head_gate        out[t, h, :] = src[t, h, :] * sigmoid(gate[t, h]): one gate per attention head.
+//   head_gate        out[t, h, :] = src[t, h, :] * sigmoid(gate[t, h]): one gate per attention head;
+//   post_norm_add_rms_norm  x <- x + rms(y + y_bias) * w_post, then out = rms(x) * w: the norm AFTER a sublayer, its sum and the norm before the next
+//                    sublayer in one pass (with `row_index` only the selected rows, x left as it is; w null = the sum alone);
+//   xielu_rows       out = xIELU(x + bias): pos z^2 + z / 2 for z > 0, neg (e^z - 1 - z) + z / 2 otherwise;
+//   softcap_inplace  x <- cap tanh(x / cap).
 // Any row length (no vector-width rule): the rows these models use are a few hundred to a few thousand floats and every kernel
 // here is one pass over them from L2.
 #include "common.cuh"
@@ -381,6 +385,114 @@ relu2_rows_kernel(const float* __restrict__ x, TOut* __restrict__ out, int ff, i
     }
 }
 
+// the closing norm and sum of one sublayer and the opening norm of the next: x <- x + rms(y + y_bias) * w_post, out = rms(x) * w.  A block per row;
+// rows of up to 1024 kV floats whose four-float groups are aligned stay in registers between the passes (kV groups per thread; 0 = any row, read again).
+template <typename TOut, int kV>
+__global__ void __launch_bounds__(256)
+post_norm_add_rms_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int64_t ldy, const float* __restrict__ y_bias, const float* __restrict__ w_post,
+                              const float* __restrict__ w, TOut* __restrict__ out, const int32_t* __restrict__ row_index, int n, float eps) {
+    pdl_wait();
+    pdl_trigger();
+    __shared__ float red[8];
+    const int row = blockIdx.x;
+    const int64_t src = row_index ? row_index[row] : row;
+    float* xr = x + src * n;
+    const float* yr = y + src * ldy;
+    float ss = 0.f;
+    if constexpr (kV > 0) {
+        float4 yv[kV], xv[kV];
+#pragma unroll
+        for (int v = 0; v < kV; ++v) {
+            const int i = (threadIdx.x + 256 * v) * 4;
+            yv[v] = xv[v] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < n) {
+                yv[v] = *reinterpret_cast<const float4*>(yr + i);
+                xv[v] = *reinterpret_cast<const float4*>(xr + i);
+                if (y_bias) {
+                    const float4 bv = *reinterpret_cast<const float4*>(y_bias + i);
+                    yv[v].x += bv.x; yv[v].y += bv.y; yv[v].z += bv.z; yv[v].w += bv.w;
+                }
+            }
+            ss = fmaf(yv[v].x, yv[v].x, fmaf(yv[v].y, yv[v].y, fmaf(yv[v].z, yv[v].z, fmaf(yv[v].w, yv[v].w, ss))));
+        }
+        const float sy = 1.0f / sqrtf(block_sum_256(ss, red) / (float)n + eps);
+        ss = 0.f;
+#pragma unroll
+        for (int v = 0; v < kV; ++v) {
+            const int i = (threadIdx.x + 256 * v) * 4;
+            if (i < n) {
+                const float4 wp = *reinterpret_cast<const float4*>(w_post + i);
+                xv[v].x += yv[v].x * sy * wp.x; xv[v].y += yv[v].y * sy * wp.y; xv[v].z += yv[v].z * sy * wp.z; xv[v].w += yv[v].w * sy * wp.w;
+                if (!row_index) *reinterpret_cast<float4*>(xr + i) = xv[v];
+            }
+            ss = fmaf(xv[v].x, xv[v].x, fmaf(xv[v].y, xv[v].y, fmaf(xv[v].z, xv[v].z, fmaf(xv[v].w, xv[v].w, ss))));
+        }
+        if (!out) return;
+        const float sx = 1.0f / sqrtf(block_sum_256(ss, red) / (float)n + eps);
+#pragma unroll
+        for (int v = 0; v < kV; ++v) {
+            const int i = (threadIdx.x + 256 * v) * 4;
+            if (i >= n) continue;
+            const float4 wv = *reinterpret_cast<const float4*>(w + i);
+            const float r[4] = {xv[v].x * sx * wv.x, xv[v].y * sx * wv.y, xv[v].z * sx * wv.z, xv[v].w * sx * wv.w};
+            TOut o[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) o[j] = from_f32<TOut>(r[j]);
+            if (sizeof(TOut) == 4) *reinterpret_cast<float4*>(out + (int64_t)row * n + i) = *reinterpret_cast<const float4*>(o);
+            else *reinterpret_cast<uint2*>(out + (int64_t)row * n + i) = *reinterpret_cast<const uint2*>(o);
+        }
+    } else {
+        for (int i = threadIdx.x; i < n; i += 256) { const float v = yr[i] + (y_bias ? y_bias[i] : 0.f); ss = fmaf(v, v, ss); }
+        const float sy = 1.0f / sqrtf(block_sum_256(ss, red) / (float)n + eps);
+        ss = 0.f;
+        for (int i = threadIdx.x; i < n; i += 256) {
+            const float v = xr[i] + (yr[i] + (y_bias ? y_bias[i] : 0.f)) * sy * w_post[i];
+            if (!row_index) xr[i] = v;
+            ss = fmaf(v, v, ss);
+        }
+        if (!out) return;
+        const float sx = 1.0f / sqrtf(block_sum_256(ss, red) / (float)n + eps);
+        for (int i = threadIdx.x; i < n; i += 256) {
+            float v = xr[i];
+            if (row_index) v += (yr[i] + (y_bias ? y_bias[i] : 0.f)) * sy * w_post[i];     // x was not updated: form the sum again
+            out[(int64_t)row * n + i] = from_f32<TOut>(v * sx * w[i]);
+        }
+    }
+}
+
+// xIELU with its two numbers already through softplus: pos z^2 + z / 2 for z > 0, neg (e^z - 1 - z) + z / 2 otherwise
+__device__ __forceinline__ float xielu_f(float z, float pos, float neg) {
+    return z > 0.f ? fmaf(pos * z, z, 0.5f * z) : fmaf(neg, expm1f(z) - z, 0.5f * z);
+}
+
+template <typename TOut>
+__global__ void __launch_bounds__(256)
+xielu_rows_kernel(const float* __restrict__ x, int64_t ld, const float* __restrict__ bias, TOut* __restrict__ out, int ff, float pos, float neg, int vec) {
+    pdl_wait();
+    pdl_trigger();
+    const int64_t r = blockIdx.x;
+    const int c = (blockIdx.y * 256 + threadIdx.x) * 4;
+    if (c >= ff) return;
+    const float* src = x + r * ld + c;
+    TOut* dst = out + r * ff + c;
+    if (vec) {
+        float4 v = *reinterpret_cast<const float4*>(src);
+        if (bias) { const float4 b = *reinterpret_cast<const float4*>(bias + c); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+        TOut o[4] = {from_f32<TOut>(xielu_f(v.x, pos, neg)), from_f32<TOut>(xielu_f(v.y, pos, neg)), from_f32<TOut>(xielu_f(v.z, pos, neg)), from_f32<TOut>(xielu_f(v.w, pos, neg))};
+        if (sizeof(TOut) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(o);
+        else *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(o);
+    } else {
+        for (int i = 0; i < 4 && c + i < ff; ++i) dst[i] = from_f32<TOut>(xielu_f(src[i] + (bias ? bias[c + i] : 0.f), pos, neg));
+    }
+}
+
+__global__ void softcap_kernel(float* __restrict__ x, int64_t total, float cap) {
+    pdl_wait();
+    pdl_trigger();
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < total) x[i] = cap * tanhf(x[i] / cap);
+}
+
 }  // namespace
 }  // namespace b200
 
@@ -594,6 +706,47 @@ void add_rms_norm(float* x, const float* y1, int64_t ld1, const float* y2, int64
     else { set_error(kErrUnsupported, "add_rms_norm: out dtype %d (f32 / bf16)", out_dtype); return; }
     count_launch();
     check_launch("add_rms_norm");
+}
+
+void post_norm_add_rms_norm(float* x, const float* y, int64_t ldy, const float* y_bias, const float* post_weight, const float* weight, void* out, const int32_t* row_index,
+                            int32_t rows, int32_t n, float eps, int32_t out_dtype, int64_t stream) {
+    if (rows == 0) return;
+    B200_REQUIRE(x && y && post_weight && rows > 0 && n > 0 && ldy >= n && ((weight == nullptr) == (out == nullptr)) && (out || !row_index), kErrBadArg,
+                 "post_norm_add_rms_norm: bad arguments");
+    B200_REQUIRE(!out || out_dtype == B200_F32 || out_dtype == B200_BF16, kErrUnsupported, "post_norm_add_rms_norm: out dtype %d (f32 / bf16)", out_dtype);
+    const bool vec = n % 4 == 0 && ldy % 4 == 0 &&
+                     (((uintptr_t)x | (uintptr_t)y | (uintptr_t)y_bias | (uintptr_t)post_weight | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+    const int kv = !vec ? 0 : n <= 1024 ? 1 : n <= 2048 ? 2 : n <= 4096 ? 4 : n <= 8192 ? 8 : 0;
+    cudaStream_t st = as_stream(stream);
+#define PNA(TO, KV) launch_pdl(post_norm_add_rms_norm_kernel<TO, KV>, dim3(rows), dim3(256), 0, st, x, y, ldy, y_bias, post_weight, weight, (TO*)out, row_index, (int)n, eps)
+#define PNA_ALL(TO) do { if (kv == 1) PNA(TO, 1); else if (kv == 2) PNA(TO, 2); else if (kv == 4) PNA(TO, 4); else if (kv == 8) PNA(TO, 8); else PNA(TO, 0); } while (0)
+    if (!out || out_dtype == B200_F32) PNA_ALL(float);
+    else PNA_ALL(__nv_bfloat16);
+#undef PNA_ALL
+#undef PNA
+    count_launch();
+    check_launch("post_norm_add_rms_norm");
+}
+
+void xielu_rows(const float* x, int64_t ld, const float* bias, void* out, int32_t rows, int32_t ff, float pos, float neg, int32_t out_dtype, int64_t stream) {
+    if (rows == 0 || ff == 0) return;
+    B200_REQUIRE(x && out && rows > 0 && ff > 0 && ld >= ff, kErrBadArg, "xielu_rows: bad arguments");
+    const int vec = ff % 4 == 0 && ld % 4 == 0 && (((uintptr_t)x | (uintptr_t)bias | (uintptr_t)out) & 15) == 0;
+    const dim3 grid((unsigned)rows, (unsigned)((ff + 1023) / 1024));
+    cudaStream_t st = as_stream(stream);
+    if (out_dtype == B200_F32) launch_pdl(xielu_rows_kernel<float>, grid, dim3(256), 0, st, x, ld, bias, (float*)out, (int)ff, pos, neg, vec);
+    else if (out_dtype == B200_BF16) launch_pdl(xielu_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, x, ld, bias, (__nv_bfloat16*)out, (int)ff, pos, neg, vec);
+    else { set_error(kErrUnsupported, "xielu_rows: out dtype %d (f32 / bf16)", out_dtype); return; }
+    count_launch();
+    check_launch("xielu_rows");
+}
+
+void softcap_inplace(float* x, int64_t total, float cap, int64_t stream) {
+    if (total == 0) return;
+    B200_REQUIRE(x && total > 0 && cap > 0.f, kErrBadArg, "softcap_inplace: bad arguments");
+    launch_pdl(softcap_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, as_stream(stream), x, total, cap);
+    count_launch();
+    check_launch("softcap_inplace");
 }
 
 }  // extern "C"

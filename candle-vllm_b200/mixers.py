@@ -16,6 +16,9 @@ kernels of ``seq_ops``.  Sizes and constants are constructor arguments so that a
                        input gates are block-diagonal maps of the convolved branch (csrc/linear_recurrence.cu)
   DecayLinearAttention linear attention over an f32 matrix state with one fixed decay per head, SiLU on q / k / v, all heads normed together, sigmoid gate
   MatrixMemoryMixer    linear attention with exponential input / forget gates held stable by a running maximum, a normaliser vector, per-head norm
+  ChannelDecayLinearAttention  linear attention with a decay per token and key row from a low-rank map, per-head norm times a SiLU gate
+  TalkingAttentionMixer  softmax attention whose heads mix their scores, values cached turned by their position, optionally over another layer's cache
+                       (csrc/attention_talking.cu)
   ParallelMixer        two mixers side by side on one input (one fused projection), half the sum of their normed outputs
 
 Activations that feed a matrix product are of the model's compute dtype (bf16 or f32); products come back in f32 and everything
@@ -245,12 +248,22 @@ class GatedMlp:
 
 
 class UngatedMlp:
-    """down(act(up x)) with act = relu(.)^2; up [ff, D], down [D, ff]."""
+    """down(act(up x)) with act = relu(.)^2, or "xielu" with the two numbers (p, q) of w["act"]: softplus(p) z^2 + z / 2 for z > 0, (1/2 + softplus(q))
+    (e^z - 1 - z) + z / 2 otherwise; up [ff, D], down [D, ff].  A bias up.b [ff] joins the activation's kernel (xielu only); a bias down.b [D] is left to the
+    caller (``down_bias``), who adds it where the output is read next."""
 
     def __init__(self, w: Dict[str, torch.Tensor], dtype: torch.dtype, act: str = "relu2"):
-        if act != "relu2":
-            raise BackendError(f"UngatedMlp: unknown activation {act!r}")
+        if act not in ("relu2", "xielu") or (act == "relu2" and ("up.b" in w or "down.b" in w)):
+            raise BackendError(f"UngatedMlp: activation {act!r} (relu2 without biases / xielu)")
         self.dtype, self.act = dtype, act
+        self.up_bias = w["up.b"].float().contiguous() if "up.b" in w else None
+        self.down_bias = w["down.b"].float().contiguous() if "down.b" in w else None
+        if act == "xielu":
+            if w["act"].numel() != 2:
+                raise BackendError(f"UngatedMlp: xielu takes two numbers, the tensor has {w['act'].numel()}")
+            p, q = (float(v) for v in w["act"].double().cpu().flatten())
+            softplus = lambda a: math.log1p(math.exp(-abs(a))) + max(a, 0.0)
+            self.act_pos, self.act_neg = softplus(p), 0.5 + softplus(q)
         self.w_in = w["up"].to(dtype).contiguous()
         self.w_down = w["down"].to(dtype).contiguous()
         self.ff = self.w_in.shape[0]
@@ -259,6 +272,8 @@ class UngatedMlp:
         """``proj``: the product of ``w_in`` with the input when the caller has it already (columns of a wider fused projection)"""
         if proj is None:
             proj = ops.linear(h, self.w_in)
+        if self.act == "xielu":
+            return ops.linear(ops.xielu(proj, self.up_bias, self.act_pos, self.act_neg, self.dtype), self.w_down)
         return ops.linear(ops.glu_packed(proj, self.act, self.dtype), self.w_down)
 
 
@@ -554,6 +569,101 @@ class MatrixMemoryMixer:
                                  kernel=self.kernel)
         z = ops.group_rms_norm_gate(o, self.norm, proj[:, self.off_g:], self.H, self.eps, self.dtype)
         return ops.linear(z, self.w_o)
+
+
+class ChannelDecayLinearAttention:
+    """Gated linear attention: q = W_q h dk^-1/2, k, v plain; a decay per token and key row alpha = sigmoid(a2 (a1 h) + a2.b)^(1/tau); per head
+    S <- diag(alpha) S + k v^T, o = S^T q; each head's o over its root mean square, times norm [dv] (shared by the heads), times silu(g h), then o [D, H dv].
+    weights: q, k [H dk, D], v, g [H dv, D], a1 [rank, D], a2 [H dk, rank], optional a2.b [H dk].  The second map of the decay runs in 32 bits whatever the
+    compute dtype."""
+    kind = "state"
+
+    def __init__(self, w: Dict[str, torch.Tensor], heads: int, dk: int, dv: int, tau: float, eps: float, dtype: torch.dtype):
+        self.H, self.dk, self.dv, self.tau, self.eps, self.dtype = heads, dk, dv, float(tau), eps, dtype
+        self.rank = w["a1"].shape[0]
+        want = {"q": heads * dk, "k": heads * dk, "v": heads * dv, "g": heads * dv, "a2": heads * dk}
+        for name, n in want.items():
+            if w[name].shape[0] != n:
+                raise BackendError(f"ChannelDecayLinearAttention: {name} is {tuple(w[name].shape)}, expected {n} rows")
+        if w["a2"].shape[1] != self.rank or w["norm"].numel() != dv or tuple(w["o"].shape)[1] != heads * dv:
+            raise BackendError(f"ChannelDecayLinearAttention: a2 {tuple(w['a2'].shape)} / norm {tuple(w['norm'].shape)} / o {tuple(w['o'].shape)} for rank {self.rank}, {heads} x {dv}")
+        self.w_in = torch.cat([w["q"], w["k"], w["v"], w["g"], w["a1"]], 0).to(dtype).contiguous()
+        self.off_g = 2 * heads * dk + heads * dv
+        self.off_a = self.off_g + heads * dv
+        self.a2, self.a2_bias = w["a2"].float().contiguous(), (w["a2.b"].float().contiguous() if "a2.b" in w else None)
+        self.norm = w["norm"].float().flatten().repeat(heads).contiguous()
+        self.w_o = w["o"].to(dtype).contiguous()
+        self.kernel = None                       # None: chosen by the step's shape (tests force one)
+
+    def state_shapes(self):
+        return ((self.H, self.dv, self.dk),)
+
+    def forward(self, h: torch.Tensor, batch: StepBatch, cache, proj: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if proj is None:
+            proj = ops.linear(h, self.w_in)
+        alpha = ops.low_rank_decay(proj[:, self.off_a:self.off_a + self.rank], self.a2, self.a2_bias, self.tau)
+        o = ops.linear_attention_channel(proj, 0, self.H * self.dk, 2 * self.H * self.dk, alpha, cache[0], batch, self.H, self.dk, self.dv, q_scale=self.dk ** -0.5,
+                                         kernel=self.kernel)
+        z = ops.group_rms_norm_gate(o, self.norm, proj[:, self.off_g:self.off_g + self.H * self.dv], self.H, self.eps, self.dtype, gate_act="silu")
+        return ops.linear(z, self.w_o)
+
+
+class TalkingAttentionMixer:
+    """Grouped-query softmax attention over the paged cache whose heads mix their scores before the softmax: s'[h] = sum_g talk[h, g] s[g].  q and k are rotated on
+    their first rot.dims entries; with ``rotate_values`` the values are cached turned by their own position over all of their entries (same base) and every head's
+    output is turned back by the query's.  ``one_sink``: one is added to the softmax denominator.  chunk / window = 0 for none.
+
+    weights: q [H dk, D], o [D, H dv], optional talk [H, H]; k [G dk, D] and v [G dv, D] unless ``shared`` (the layer attends over the cache another layer writes)."""
+    kind = "kv"
+
+    def __init__(self, w: Dict[str, torch.Tensor], heads: int, kv_heads: int, dk: int, dv: int, scale: float, dtype: torch.dtype, rot: Optional[dict] = None,
+                 rotate_values: bool = False, one_sink: bool = False, shared: bool = False, chunk: int = 0, window: int = 0, block_size: int = 64, max_pos: int = 4096):
+        if heads % kv_heads:
+            raise BackendError("TalkingAttentionMixer: heads must be a multiple of kv_heads")
+        self.H, self.G, self.dk, self.dv, self.scale, self.dtype = heads, kv_heads, dk, dv, float(scale), dtype
+        self.rot, self.rotate_values, self.one_sink, self.shared = rot, bool(rotate_values and rot), bool(one_sink), bool(shared)
+        self.chunk, self.window, self.block_size = int(chunk), int(window), block_size
+        self.rot_dims = int(rot["dims"]) if rot else 0
+        if self.rot_dims % 2 or self.rot_dims > dk or dv % 2:
+            raise BackendError(f"TalkingAttentionMixer: {self.rot_dims} rotary dims on a head of {dk}, value size {dv} (both even)")
+        want = {"q": heads * dk, **({} if shared else {"k": kv_heads * dk, "v": kv_heads * dv})}
+        for name, n in want.items():
+            if w[name].shape[0] != n:
+                raise BackendError(f"TalkingAttentionMixer: {name} is {tuple(w[name].shape)}, expected {n} rows")
+        if tuple(w["o"].shape)[1] != heads * dv or ("talk" in w and tuple(w["talk"].shape) != (heads, heads)):
+            raise BackendError(f"TalkingAttentionMixer: o {tuple(w['o'].shape)} / talk for {heads} heads of {dv}")
+        self.w_in = torch.cat([w[n] for n in want], 0).to(dtype).contiguous()
+        self.talk = w["talk"].float().contiguous() if "talk" in w else None
+        self.w_o = w["o"].to(dtype).contiguous()
+        self.splits = None                       # None: chosen by the step's shape (tests force a number)
+        self.cos = self.sin = self.v_cos = self.v_sin = None
+        self._device = self.w_in.device
+        if rot:
+            self.ensure_positions(max_pos)
+
+    def ensure_positions(self, max_pos: int) -> None:
+        if self.rot and (self.cos is None or self.cos.shape[0] < max_pos):
+            base = float(self.rot["base"])
+            self.cos, self.sin = yarn_rotary_tables(self.rot_dims, base, max_pos, self.rot.get("scaling"), self._device)
+            if self.rotate_values:
+                self.v_cos, self.v_sin = yarn_rotary_tables(self.dv, base, max_pos, None, self._device)
+
+    def cache_shape(self):
+        return (self.G, self.dk, self.dv)
+
+    def forward(self, h: torch.Tensor, batch: StepBatch, cache, proj: Optional[torch.Tensor] = None) -> torch.Tensor:
+        k_cache, v_cache = cache
+        if self.rot and batch.max_position >= self.cos.shape[0]:
+            self.ensure_positions(max(2 * self.cos.shape[0], batch.max_position + 1))
+        if proj is None:
+            proj = ops.linear(h, self.w_in)
+        tables = (self.cos, self.sin) if self.rot_dims else None
+        v_tables = (self.v_cos, self.v_sin) if self.rotate_values else None
+        q = ops.qkv_rope_cache(proj, tables, v_tables, batch, None if self.shared else k_cache, None if self.shared else v_cache, self.H, self.G, self.dk, self.dv,
+                               self.rot_dims, self.dtype)
+        a = ops.talking_attention(q, k_cache, v_cache, batch, self.talk, v_tables, self.H, self.scale, self.chunk, self.window, self.one_sink, self.dtype,
+                                  splits=self.splits)
+        return ops.linear(a, self.w_o)
 
 
 class ParallelMixer:

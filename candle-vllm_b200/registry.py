@@ -26,7 +26,7 @@ def architecture_of(config: dict) -> str:
 
 
 # the source group (build.GROUPS) whose library alone serves an architecture, for a first start from a source-only checkout
-_BUILD_GROUP = {"Gobesun": "ragged", "Guvusun": "latent", "Panarax": "hybrid", "Dofevik": "window"}
+_BUILD_GROUP = {"Gobesun": "ragged", "Guvusun": "latent", "Panarax": "hybrid", "Dofevik": "window", "Sigalorn": "talking"}
 
 
 def build_group_of(path: str) -> str:
@@ -66,6 +66,11 @@ def _dofevik(path, **kw):
     return DofevikModel.from_pretrained(path, **kw)
 
 
+def _sigalorn(path, **kw):
+    from .sigalorn import SigalornModel
+    return SigalornModel.from_pretrained(path, **kw)
+
+
 def _llama(path, **kw):
     from .llama import load_dense_checkpoint
     return load_dense_checkpoint(path, **kw)
@@ -75,4 +80,5 @@ register_model("Gobesun", _gobesun)
 register_model("Guvusun", _guvusun)
 register_model("Panarax", _panarax)
 register_model("Dofevik", _dofevik)
+register_model("Sigalorn", _sigalorn)
 register_model("LlamaForCausalLM", _llama)

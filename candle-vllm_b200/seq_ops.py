@@ -786,3 +786,136 @@ def paged_attention_sigmoid_pooled(q: torch.Tensor, k_cache: torch.Tensor, v_cac
                                          _stream(q.device))
     check("paged_attention_sigmoid_pooled")
     return out
+
+
+# ---- norm after and before a sublayer in one pass, xIELU, logit cap, decays per key row, heads that mix their scores --------------------------
+
+def post_norm_add_rms_norm(x: torch.Tensor, y: torch.Tensor, post_weight: torch.Tensor, weight: Optional[torch.Tensor], eps: float, out_dtype: Optional[torch.dtype] = None,
+                           y_bias: Optional[torch.Tensor] = None, row_index: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """The step between two sublayers that are normed before and after, on the f32 stream x [T, n] (contiguous): x += rms_norm(y + y_bias) * post_weight in place,
+    then rms_norm(x) * weight -> [T, n] of ``out_dtype``.  ``weight`` None: the sum alone (returns None).  ``row_index`` (i32 [R]): only those rows are summed and
+    normed ([R, n] comes back) and x is left as it is."""
+    T, n = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous() or y.dtype != torch.float32 or y.shape != x.shape or y.stride(1) != 1:
+        raise BackendError("post_norm_add_rms_norm: an f32 contiguous stream and an f32 sublayer output of its shape")
+    if weight is None and row_index is not None:
+        return None
+    rows = T if row_index is None else row_index.shape[0]
+    out = None if weight is None else torch.empty((rows, n), dtype=out_dtype, device=x.device)
+    lib().post_norm_add_rms_norm(_ptr(x), _ptr(y), C.c_int64(y.stride(0) if T > 1 else max(n, y.stride(0))), _ptr(y_bias), _ptr(post_weight), _ptr(weight), _ptr(out),
+                                 _ptr(row_index), C.c_int32(rows), C.c_int32(n), C.c_float(eps), C.c_int32(_tag(out_dtype) if out is not None else DType.F32), _stream(x.device))
+    check("post_norm_add_rms_norm")
+    return out
+
+
+def xielu(x: torch.Tensor, bias: Optional[torch.Tensor], pos: float, neg: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """z = x + bias (x f32 [rows, ff], row stride allowed): pos z^2 + z / 2 where z > 0, neg (e^z - 1 - z) + z / 2 elsewhere"""
+    rows, ff = x.shape
+    if x.dtype != torch.float32 or x.stride(1) != 1 or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != ff)):
+        raise BackendError(f"xielu: x {tuple(x.shape)} {x.dtype}")
+    out = torch.empty((rows, ff), dtype=out_dtype, device=x.device)
+    lib().xielu_rows(_ptr(x), C.c_int64(x.stride(0) if rows > 1 else max(ff, x.stride(0))), _ptr(bias), _ptr(out), C.c_int32(rows), C.c_int32(ff), C.c_float(pos), C.c_float(neg),
+                     C.c_int32(_tag(out_dtype)), _stream(x.device))
+    check("xielu_rows")
+    return out
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """cap tanh(x / cap) in place on a contiguous f32 tensor"""
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise BackendError("softcap: a contiguous f32 tensor")
+    lib().softcap_inplace(_ptr(x), C.c_int64(x.numel()), C.c_float(cap), _stream(x.device))
+    check("softcap_inplace")
+    return x
+
+
+def low_rank_decay(y: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], tau: float) -> torch.Tensor:
+    """sigmoid(weight y + bias)^(1 / tau): y f32 [T, rank] (row stride allowed), weight f32 [channels, rank] -> f32 [T, channels]; 32-bit throughout"""
+    T, R = y.shape
+    N = weight.shape[0]
+    if y.dtype != torch.float32 or weight.dtype != torch.float32 or y.stride(1) != 1 or weight.shape[1] != R or not weight.is_contiguous():
+        raise BackendError(f"low_rank_decay: y {tuple(y.shape)} {y.dtype}, weight {tuple(weight.shape)} {weight.dtype}")
+    alpha = torch.empty((T, N), dtype=torch.float32, device=y.device)
+    lib().low_rank_decay(_ptr(y), C.c_int64(y.stride(0) if T > 1 else max(R, y.stride(0))), _ptr(weight), _ptr(bias), _ptr(alpha), C.c_int32(T), C.c_int32(N), C.c_int32(R),
+                         C.c_float(tau), _stream(y.device))
+    check("low_rank_decay")
+    return alpha
+
+
+def linear_attention_channel(proj: torch.Tensor, off_q: int, off_k: int, off_v: int, alpha: torch.Tensor, state: torch.Tensor, batch: StepBatch, heads: int, dk: int, dv: int,
+                             q_scale: float = 1.0, kernel: Optional[str] = None) -> torch.Tensor:
+    """``linear_attention`` with a decay per token and key row: S <- diag(alpha_t) S + k v^T, o = S^T q per head; alpha f32 [T, H dk], state f32 [slots, H, dv, dk]
+    advanced in place -> f32 [T, H dv].  The same three kernels ("step", "token", "chunked"), chosen by the step's shape the same way."""
+    T = proj.shape[0]
+    if alpha.dtype != torch.float32 or alpha.shape != (T, heads * dk) or not alpha.is_contiguous():
+        raise BackendError(f"linear_attention_channel: decays {tuple(alpha.shape)} {alpha.dtype} for {T} rows of {heads} x {dk}")
+    out = torch.empty((T, heads * dv), dtype=torch.float32, device=proj.device)
+    need = int(lib().linear_attention_chunked_scratch(C.c_int32(T), C.c_int32(batch.num_seqs), C.c_int32(heads), C.c_int32(dk), C.c_int32(dv)))
+    if kernel is None:
+        kernel = "step" if batch.pure_decode else "token"
+        if (batch.max_rows >= CHUNKED_LINEAR_ATTENTION_MIN_ROWS and -(-batch.max_rows // 64) * batch.num_seqs <= 65535 and need * 4 <= CHUNKED_LINEAR_ATTENTION_SCRATCH):
+            kernel = "chunked"
+    try:
+        mode = {"token": 0, "step": 1, "chunked": 2}[kernel]
+    except KeyError:
+        raise BackendError(f"linear_attention_channel: unknown kernel {kernel!r}")
+    scratch = torch.empty((need,), dtype=torch.float32, device=proj.device) if mode == 2 else None
+    lib().linear_attention_channel(_ptr(proj), C.c_int64(proj.stride(0) if T > 1 else proj.shape[1]), C.c_int32(off_q), C.c_int32(off_k), C.c_int32(off_v), _ptr(alpha),
+                                   C.c_int64(heads * dk), C.c_float(q_scale), _ptr(state), _ptr(out), _ptr(scratch), _ptr(batch.cu_seqlens), _ptr(batch.seq_slots),
+                                   _ptr(batch.seq_start), C.c_int32(T), C.c_int32(batch.num_seqs), C.c_int32(batch.max_rows), C.c_int32(mode), C.c_int32(heads),
+                                   C.c_int32(dk), C.c_int32(dv), _stream(proj.device))
+    check("linear_attention_channel")
+    return out
+
+
+def qkv_rope_cache(qkv: torch.Tensor, tables: Optional[tuple], value_tables: Optional[tuple], batch: StepBatch, k_cache: Optional[torch.Tensor],
+                   v_cache: Optional[torch.Tensor], heads: int, kv_heads: int, dk: int, dv: int, rot_dims: int, cache_dtype: torch.dtype,
+                   q_dtype: torch.dtype = torch.float32) -> torch.Tensor:
+    """qkv f32 [T, H dk | G dk | G dv]: q and k turned on their first ``rot_dims`` entries by ``tables`` = (cos, sin) [max_pos, rot_dims / 2], the values over all dv
+    entries by ``value_tables`` [max_pos, dv / 2] (None = not turned); k and v go to the paged cache, q [T, H dk] comes back.  ``k_cache`` None: qkv holds query
+    columns alone (a layer that attends over another layer's cache)."""
+    T = qkv.shape[0]
+    cos, sin = tables if tables else (None, None)
+    v_cos, v_sin = value_tables if value_tables else (None, None)
+    rows = min([t.shape[0] for t in (cos, v_cos) if t is not None], default=0)
+    if rows and batch.max_position >= rows:
+        raise BackendError(f"position {batch.max_position} is outside the rotary table ({rows} rows)")
+    if k_cache is not None and k_cache.dtype != cache_dtype:
+        raise BackendError(f"qkv_rope_cache: cache of {k_cache.dtype}, expected {cache_dtype}")
+    q = torch.empty((T, heads * dk), dtype=q_dtype, device=qkv.device)
+    lib().qkv_norm_rope_cache(_ptr(qkv), C.c_int64(qkv.stride(0) if T > 1 else qkv.shape[1]), _ptr(None), _ptr(None), _ptr(cos), _ptr(sin), _ptr(v_cos), _ptr(v_sin),
+                              C.c_int32(rows), _ptr(batch.positions), _ptr(batch.slot_mapping), _ptr(q), _ptr(k_cache), _ptr(v_cache), C.c_int32(T), C.c_int32(heads),
+                              C.c_int32(kv_heads if k_cache is not None else 0), C.c_int32(dk), C.c_int32(dv), C.c_int32(rot_dims), C.c_float(0.0), C.c_float(0.0),
+                              C.c_int32(0), C.c_int32(0), C.c_int32(_tag(cache_dtype)), C.c_int32(_tag(q_dtype)), _stream(qkv.device))
+    check("qkv_norm_rope_cache")
+    return q
+
+
+TALKING_BLOCKS = 444           # three blocks per SM: steps with fewer rows cut the keys of every row into runs
+
+
+def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: StepBatch, talk: Optional[torch.Tensor], value_tables: Optional[tuple], heads: int,
+                      scale: float, chunk: int, window: int, one_sink: bool, out_dtype: torch.dtype, splits: Optional[int] = None) -> torch.Tensor:
+    """Softmax attention whose heads mix their scores by ``talk`` (f32 [H, H]) before the softmax; ``one_sink``: one is added to every denominator; ``value_tables``: the
+    cached values were turned by their position and every output is turned back by its own.  q f32 [T, H dk] -> [T, H dv] of ``out_dtype`` (the cache's).
+    ``splits``: runs every row's keys are cut into (None: enough blocks to fill the device, from the table width, so that a captured step keeps its choice)."""
+    T = q.shape[0]
+    nb, bs, G, dk = k_cache.shape
+    dv = v_cache.shape[3]
+    v_cos, v_sin = value_tables if value_tables else (None, None)
+    if q.dtype != torch.float32 or k_cache.dtype != out_dtype or (talk is not None and (talk.dtype != torch.float32 or tuple(talk.shape) != (heads, heads))):
+        raise BackendError(f"talking_attention: q {q.dtype}, cache {k_cache.dtype}, out {out_dtype}")
+    if splits is None:
+        longest = batch.block_tables.shape[1] * bs
+        for limit in (chunk, window):
+            if limit > 0:
+                longest = min(longest, limit)
+        splits = max(1, min(-(-TALKING_BLOCKS // T), longest // 64, 64)) if T < TALKING_BLOCKS else 1
+    part = torch.empty((T * splits * heads * (dv + 2),), dtype=torch.float32, device=q.device) if splits > 1 else None
+    out = torch.empty((T, heads * dv), dtype=out_dtype, device=q.device)
+    lib().talking_attention_rows(_ptr(out), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), C.c_int32(batch.block_tables.shape[1]), _ptr(batch.token_seq),
+                                 _ptr(batch.positions), _ptr(talk), _ptr(v_cos), _ptr(v_sin), C.c_int32(T), C.c_int32(heads), C.c_int32(G), C.c_int32(dk), C.c_int32(dv),
+                                 C.c_int32(bs), C.c_float(scale), C.c_int32(chunk), C.c_int32(window), C.c_int32(1 if one_sink else 0), C.c_int32(splits), _ptr(part),
+                                 C.c_int32(_tag(k_cache.dtype)), C.c_int32(_tag(out_dtype)), _stream(q.device))
+    check("talking_attention_rows")
+    return out

@@ -688,6 +688,39 @@ void mla_paged_attention_window(void* out, const void* q_absorbed, const void* q
                                 int32_t num_heads, int32_t kv_lora_rank, int32_t qk_rope_head_dim, int32_t block_size, int32_t max_blocks_per_seq, int64_t num_blocks,
                                 float sm_scale, int32_t dtype, void* workspace, size_t workspace_bytes, int64_t stream);
 
+/* ---- norm after and before a sublayer in one pass, xIELU, logit cap, decays per key row, heads that mix their scores ------------------------------
+ * post_norm_add_rms_norm: x f32 [rows, n] contiguous, in place: x += rms_norm(y + y_bias) * post_weight (y f32, row pitch ldy; y_bias f32 [n] or null), then
+ *   out = rms_norm(x) * weight of out_dtype (weight and out both null: the sum alone).  With row_index (i32 [rows]) only those rows are read, x stays as it is.
+ * xielu_rows: out[r, :ff] = pos z^2 + z / 2 for z > 0, neg (e^z - 1 - z) + z / 2 otherwise, z = x[r] + bias (bias f32 [ff] or null); out F32 / BF16.
+ * softcap_inplace: x = cap tanh(x / cap).
+ * low_rank_decay: alpha f32 [T, channels] = sigmoid(weight y + bias)^(1 / tau); y f32 [T, rank] (row pitch ldy), weight f32 [channels, rank].
+ * linear_attention_channel: linear_attention with a decay per token and key row: S <- diag(alpha_t) S + k v^T, o = S^T (q q_scale), alpha f32 [T, H dk] (row pitch
+ *   lda).  mode 0: token by token, any step; 1: every entry brings exactly one row; 2: over chunks of 64 tokens, all chunks at once (scratch =
+ *   linear_attention_chunked_scratch(...) floats, max_rows = the most rows any entry brings).  dk <= 512 in modes 0 and 1.
+ * qkv_norm_rope_cache: qk_norm_rope_cache_ex with v_cos / v_sin f32 [max_pos, dv / 2] (or null): values are turned over all dv entries (i with i + dv/2) before
+ *   they are cached.  num_kv_heads 0: qkv holds query columns alone and nothing is cached.
+ * talking_attention_rows: s[h, j] = scale q[t, h] . k_j, s' = talk s (talk f32 [H, H] or null = as they are), p = exp(s') / (one_sink + sum exp(s')), out[t, h] = sum p v_j
+ *   turned back by the position's angles of v_cos / v_sin (null = not turned), over the keys with j <= i, j / chunk == i / chunk (chunk > 0), i - j < window (window
+ *   > 0).  q f32 [T, H dk]; cache and out F32 or both BF16.  splits > 1: every row's keys are cut into that many runs, part = T * splits * H * (dv + 2) floats.
+ *   H <= 64, dv even and <= 256, dk <= 1024. */
+void post_norm_add_rms_norm(float* x, const float* y, int64_t ldy, const float* y_bias, const float* post_weight, const float* weight, void* out, const int32_t* row_index,
+                            int32_t rows, int32_t n, float eps, int32_t out_dtype, int64_t stream);
+void xielu_rows(const float* x, int64_t ld, const float* bias, void* out, int32_t rows, int32_t ff, float pos, float neg, int32_t out_dtype, int64_t stream);
+void softcap_inplace(float* x, int64_t total, float cap, int64_t stream);
+void low_rank_decay(const float* y, int64_t ldy, const float* weight, const float* bias, float* alpha, int32_t num_tokens, int32_t channels, int32_t rank, float tau,
+                    int64_t stream);
+void linear_attention_channel(const float* proj, int64_t ld, int32_t off_q, int32_t off_k, int32_t off_v, const float* alpha, int64_t lda, float q_scale, float* state,
+                              float* out, float* scratch, const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens,
+                              int32_t num_seqs, int32_t max_rows, int32_t mode, int32_t num_heads, int32_t dk, int32_t dv, int64_t stream);
+void qkv_norm_rope_cache(const float* qkv, int64_t ld, const float* q_norm_w, const float* k_norm_w, const float* cos_t, const float* sin_t, const float* v_cos,
+                         const float* v_sin, int32_t max_pos, const int32_t* positions, const int64_t* slot_mapping, void* q_out, void* key_cache, void* value_cache,
+                         int32_t num_tokens, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t rot_dims, float eps,
+                         float q_temp_coef, int32_t q_temp_every, int32_t v_unit_rms, int32_t cache_dtype, int32_t q_dtype, int64_t stream);
+void talking_attention_rows(void* out, const float* q, const void* key_cache, const void* value_cache, const int32_t* block_tables, int32_t table_width,
+                            const int32_t* token_seq, const int32_t* positions, const float* talk, const float* v_cos, const float* v_sin, int32_t num_tokens,
+                            int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t block_size, float scale, int32_t chunk, int32_t window,
+                            int32_t one_sink, int32_t splits, float* part, int32_t cache_dtype, int32_t out_dtype, int64_t stream);
+
 #ifdef __cplusplus
 }
 #endif
