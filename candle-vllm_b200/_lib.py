@@ -42,6 +42,7 @@ SYMBOLS = [
     "qk_head_norm_rope_cache", "paged_attention_varlen_sink", "pooled_cache_update", "paged_attention_sigmoid_pooled", "latent_out_gate_ex", "moe_route_bias", "add_rms_norm",
     "mla_paged_attention_window",
     "post_norm_add_rms_norm", "xielu_rows", "softcap_inplace", "low_rank_decay", "linear_attention_channel", "qkv_norm_rope_cache", "talking_attention_rows",
+    "talking_attention_prefill_supported", "talking_attention_prefill",
 ]
 
 
@@ -63,7 +64,8 @@ GROUP_SYMBOLS = {
                          "latent_q_absorb", "latent_attention_varlen", "latent_out_gate_ex", "repack_heads", "token_tables", "mla_decode_kernel_supported",
                          "mla_paged_attention_sink", "mla_paged_attention_window", "mla_paged_decode_workspace_bytes", "moe_route_bias", "moe_gate_up_ex", "moe_down", "linear_grouped", "moe_align_rows",
                          "moe_align", "moe_gather_rows", "moe_combine_rows"],
-    "talking": _COMMON + ["low_rank_decay", "linear_attention_channel", "linear_attention_chunked_scratch", "qkv_norm_rope_cache", "talking_attention_rows"],
+    "talking": _COMMON + ["low_rank_decay", "linear_attention_channel", "linear_attention_chunked_scratch", "qkv_norm_rope_cache", "talking_attention_rows",
+                         "talking_attention_prefill_supported", "talking_attention_prefill"],
 }
 _RESTYPES = {"b200_last_error_message": C.c_char_p, "paged_attention_decode_workspace_bytes": C.c_size_t, "qmatmul_workspace_bytes": C.c_size_t,
              "moe_gemm_workspace_bytes": C.c_size_t, "moe_gemm_fp8_workspace_bytes": C.c_size_t, "mla_paged_decode_workspace_bytes": C.c_size_t,

@@ -9,6 +9,12 @@
 //   talking_rows_kernel     a block per (row, run of keys), f32 arithmetic, any sizes, f32 or bf16 cache: scores (a warp per kv head and 32 keys, four lanes
 //                           share a key's row in 16-byte pieces), mixing and online softmax (a warp per head, a lane per key), values (a warp per run of
 //                           heads, lanes across the columns).  Few rows: the keys of a row are cut into runs and talking_merge_kernel joins them.
+//   talking_prefill_kernel  portions of prompts in 16 bits: a block per 8 query rows with ALL heads, mma.sync m16n8k16 with keys (or value columns) on the
+//                           16-row side and queries on the 8-column side, so that 32 heads' accumulators of 128 value columns fit the register file.  A warp
+//                           owns H / 8 heads in both products; raw scores meet in shared memory, a thread mixes one (query, key) pair over all heads in
+//                           f32, and every warp reads its heads' mixed scores back in the operand layout of the second product.  The first product of the
+//                           next tile is issued before the mixing of this one (scores double-buffered), so a tile costs one barrier; keys and values
+//                           arrive by cp.async while earlier tiles are worked on.
 #include <cuda.h>
 
 #include "common.cuh"
@@ -315,6 +321,318 @@ talking_merge_kernel(const float* __restrict__ part, const int32_t* __restrict__
     }
 }
 
+// ---- portions of prompts on tensor cores --------------------------------------------------------------------------------------------------------
+struct TalkTcArgs {
+    const __nv_bfloat16* q; const __nv_bfloat16* kc; const __nv_bfloat16* vc;
+    const int32_t* block_tables; int table_width;
+    const int32_t* cu_q; const int32_t* cu_k; int num_seqs;
+    const float* talk; const float* cos_t; const float* sin_t;
+    __nv_bfloat16* out;
+    int H, G, dk, dv, bs;
+    float scale_log2;
+    int chunk, window, one_sink;
+    int kst, vst;                                // key / value tiles kept in shared memory (1 or 2)
+    int pk, pv;                                  // row pitches in bytes, multiples of 128
+};
+
+constexpr int kTcRows = 8;                       // query rows of a block
+
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+__device__ __forceinline__ uint4 lds16(uint32_t a) {
+    uint4 v;
+    asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "r"(a));
+    return v;
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ float exp2_fast(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) { const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi); return *reinterpret_cast<const uint32_t*>(&v); }
+
+// kHW: heads per warp (8 warps), kKT: keys per tile
+template <int kHW, int kKT>
+__global__ void __launch_bounds__(256, 1)
+talking_prefill_kernel(const TalkTcArgs A) {
+    pdl_wait();
+    pdl_trigger();
+    constexpr int kMT = kKT / 16, kSP = kKT + 4;                       // 16-key pieces per tile; pitch of a score row
+    extern __shared__ __align__(1024) uint8_t smem_tc[];
+    const int H = A.H, G = A.G, dk = A.dk, dv = A.dv, group = H / G;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    // which (sequence, 8-row tile) is this block?  the last tiles of a sequence see the most keys and start first
+    int seq = -1, tile = 0, base = 0;
+    for (int s = 0; s < A.num_seqs; ++s) {
+        const int nt = (A.cu_q[s + 1] - A.cu_q[s] + kTcRows - 1) / kTcRows;
+        if ((int)blockIdx.x < base + nt) { seq = s; tile = nt - 1 - ((int)blockIdx.x - base); break; }
+        base += nt;
+    }
+    if (seq < 0) return;
+    const int q_begin = A.cu_q[seq], qlen = A.cu_q[seq + 1] - q_begin, klen = A.cu_k[seq + 1] - A.cu_k[seq];
+    const int q0 = tile * kTcRows, rows = min(kTcRows, qlen - q0), pos0 = klen - qlen + q0, last_pos = pos0 + rows - 1;
+    const int key0 = first_visible(pos0, A.chunk, A.window);
+    const int ntiles = (last_pos - key0) / kKT + 1;
+    const int32_t* table = A.block_tables + (int64_t)seq * A.table_width;
+
+    const int kbytes = G * kKT * A.pk, vbytes = G * kKT * A.pv;
+    const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(smem_tc);
+    const uint32_t sQ = sbase, sK = sQ + H * kTcRows * A.pk, sV = sK + A.kst * kbytes;
+    float* S = reinterpret_cast<float*>(smem_tc + (sV - sbase) + A.vst * vbytes);                   // [2][H][8][kSP]
+    const int sstage = H * kTcRows * kSP;
+    float* tk = S + 2 * sstage;                                                                      // [H][Hp]
+    const int Hp = (H + 3) & ~3;
+
+    // a tile of keys (or values) of every kv head: a warp takes whole cache rows; rows past the last visible key repeat it (their weight is 0)
+    auto load_tile = [&](const __nv_bfloat16* cache, int d, uint32_t dst, int pitch, int tl, bool values) {
+        const int d8 = d >> 3, pieces = G * d8, magic = (65536 + d8 - 1) / d8;                       // p / d8 exactly for p < 1024, d8 <= 32
+#pragma unroll
+        for (int kk = 0; kk < kKT / 8; ++kk) {
+            const int key = warp + 8 * kk, j = min(key0 + tl * kKT + key, last_pos);
+            const __nv_bfloat16* src = cache + ((int64_t)table[j / A.bs] * A.bs + j % A.bs) * G * d;
+            for (int p = lane; p < pieces; p += 32) {
+                const int kv = (p * magic) >> 16, c = p - kv * d8;
+                const int cs = values ? c ^ (key & 7) : c ^ ((key & 1) << 2);
+                cp16(dst + (kv * kKT + key) * pitch + cs * 16, src + p * 8);
+            }
+        }
+    };
+    auto load_k = [&](int tl) { if (tl < ntiles) load_tile(A.kc, dk, sK + (A.kst == 2 ? (tl & 1) * kbytes : 0), A.pk, tl, false); };
+    auto load_v = [&](int tl) { if (tl < ntiles) load_tile(A.vc, dv, sV + (A.vst == 2 ? (tl & 1) * vbytes : 0), A.pv, tl, true); };
+
+    {
+        const int d8 = dk >> 3;
+        for (int r = warp; r < H * kTcRows; r += 8) {
+            const int h = r >> 3, qr = r & 7;
+            const __nv_bfloat16* src = A.q + ((int64_t)(q_begin + q0 + min(qr, rows - 1)) * H + h) * dk;
+            for (int c = lane; c < d8; c += 32) cp16(sQ + r * A.pk + (c ^ ((qr & 1) << 2)) * 16, src + c * 8);
+        }
+    }
+    load_k(0);
+    load_v(0);
+    if (A.kst == 2) load_k(1);
+    cp_commit();
+    if (A.talk)
+        for (int i = threadIdx.x; i < H * Hp; i += 256) { const int h = i / Hp, x = i - h * Hp; tk[i] = x < H ? A.talk[h * H + x] : 0.f; }
+
+    const int h0 = warp * kHW;
+    float o[kHW][8][4];
+    float m[kHW], l[kHW];
+#pragma unroll
+    for (int a = 0; a < kHW; ++a) {
+#pragma unroll
+        for (int n = 0; n < 8; ++n) o[a][n][0] = o[a][n][1] = o[a][n][2] = o[a][n][3] = 0.f;
+        m[a] = A.one_sink ? 0.f : -INFINITY;                           // the sink: a key of score 0 without a value, counted by one lane of the query's four
+        l[a] = A.one_sink && t == 0 ? 1.f : 0.f;
+    }
+
+    // raw scores of this warp's heads for tile tl, times scale log2 e, into score stage tl & 1.  The four lanes of a row take 16-byte pieces of it: both operands
+    // permute the contraction index the same way, so no transposing load is needed.
+    auto scores = [&](int tl) {
+        float acc[kHW][kMT][4] = {};
+        const uint32_t kb = sK + (A.kst == 2 ? (tl & 1) * kbytes : 0);
+        const uint32_t sw = (uint32_t)((g & 1) << 2);
+        for (int d0 = 0; d0 < dk; d0 += 32) {
+            const int c = (d0 >> 3) + t;
+            const bool ok = c * 8 < dk;
+            const uint32_t off = (((uint32_t)c) ^ sw) * 16;
+            uint4 ka[kMT][2];
+            int kv_loaded = -1;
+#pragma unroll
+            for (int a = 0; a < kHW; ++a) {
+                const int h = h0 + a;
+                if (h >= H) continue;
+                const int kv = h / group;
+                if (kv != kv_loaded) {
+                    kv_loaded = kv;
+#pragma unroll
+                    for (int mt = 0; mt < kMT; ++mt)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e)
+                            ka[mt][e] = ok ? lds16(kb + (kv * kKT + mt * 16 + e * 8 + g) * A.pk + off) : make_uint4(0u, 0u, 0u, 0u);
+                }
+                const uint4 qb = ok ? lds16(sQ + (h * kTcRows + g) * A.pk + off) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+                for (int mt = 0; mt < kMT; ++mt) {
+                    mma_bf16(acc[a][mt], ka[mt][0].x, ka[mt][1].x, ka[mt][0].y, ka[mt][1].y, qb.x, qb.y);
+                    mma_bf16(acc[a][mt], ka[mt][0].z, ka[mt][1].z, ka[mt][0].w, ka[mt][1].w, qb.z, qb.w);
+                }
+            }
+        }
+        float* Sd = S + (tl & 1) * sstage;
+#pragma unroll
+        for (int a = 0; a < kHW; ++a) {
+            if (h0 + a >= H) continue;
+            float* r0 = Sd + ((h0 + a) * kTcRows + 2 * t) * kSP;
+#pragma unroll
+            for (int mt = 0; mt < kMT; ++mt) {
+                r0[mt * 16 + g] = acc[a][mt][0] * A.scale_log2;
+                r0[kSP + mt * 16 + g] = acc[a][mt][1] * A.scale_log2;
+                r0[mt * 16 + g + 8] = acc[a][mt][2] * A.scale_log2;
+                r0[kSP + mt * 16 + g + 8] = acc[a][mt][3] * A.scale_log2;
+            }
+        }
+    };
+    // every (query, key) pair of score stage st: s'[h] = sum_g talk[h, g] s[g], in place, one thread per pair
+    auto mix = [&](int st) {
+        if (!A.talk || (int)threadIdx.x >= kTcRows * kKT) return;
+        float* col = S + st * sstage + (threadIdx.x / kKT) * kSP + (threadIdx.x % kKT);
+        float s[8 * kHW];
+#pragma unroll
+        for (int x = 0; x < 8 * kHW; ++x) s[x] = x < H ? col[x * kTcRows * kSP] : 0.f;
+#pragma unroll 2
+        for (int h = 0; h < H; ++h) {
+            const float4* w4 = reinterpret_cast<const float4*>(tk + h * Hp);
+            float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+#pragma unroll
+            for (int x = 0; x < 2 * kHW; ++x) {
+                if (x * 4 >= H) break;
+                const float4 w = w4[x];
+                a0 = fmaf(w.x, s[4 * x], a0); a1 = fmaf(w.y, s[4 * x + 1], a1); a2 = fmaf(w.z, s[4 * x + 2], a2); a3 = fmaf(w.w, s[4 * x + 3], a3);
+            }
+            col[h * kTcRows * kSP] = (a0 + a1) + (a2 + a3);
+        }
+    };
+
+    cp_wait_all();
+    __syncthreads();
+    scores(0);
+    __syncthreads();                                                   // all warps are done with key tile 0
+    if (A.kst == 2) load_k(2); else load_k(1);
+    cp_commit();
+    if (A.kst != 2) { cp_wait_all(); __syncthreads(); }
+    const int pos = pos0 + g, lo = first_visible(pos, A.chunk, A.window);       // of this lane's query in the second product
+    for (int i = 0; i < ntiles; ++i) {
+        if (i + 1 < ntiles) scores(i + 1);
+        mix(i & 1);
+        cp_wait_all();
+        __syncthreads();
+        // keys two tiles on (three when two tiles are kept: the other one holds tile i + 2) and the next values travel while this tile is finished
+        load_k(A.kst == 2 ? i + 3 : i + 2);
+        if (A.vst == 2) load_v(i + 1);
+        cp_commit();
+        const float* Sd = S + (i & 1) * sstage;
+        uint32_t pb[kHW][kMT][2];
+#pragma unroll
+        for (int a = 0; a < kHW; ++a) {
+            if (h0 + a >= H) continue;
+            const float* row = Sd + ((h0 + a) * kTcRows + g) * kSP;
+            const int j0 = key0 + i * kKT + 2 * t;
+            float v[kMT][4], mx = -INFINITY;
+#pragma unroll
+            for (int mt = 0; mt < kMT; ++mt) {
+                const float2 x = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t), y = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t + 8);
+                v[mt][0] = x.x; v[mt][1] = x.y; v[mt][2] = y.x; v[mt][3] = y.y;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int j = j0 + mt * 16 + (e >> 1) * 8 + (e & 1);
+                    if (j < lo || j > pos) v[mt][e] = -INFINITY;
+                    mx = fmaxf(mx, v[mt][e]);
+                }
+            }
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+            const float mn = fmaxf(m[a], mx), subtr = mn == -INFINITY ? 0.f : mn;
+            const float corr = exp2_fast(m[a] - subtr);
+            m[a] = mn;
+            float sum = 0.f;
+#pragma unroll
+            for (int mt = 0; mt < kMT; ++mt) {
+                const float p0 = exp2_fast(v[mt][0] - subtr), p1 = exp2_fast(v[mt][1] - subtr), p2 = exp2_fast(v[mt][2] - subtr), p3 = exp2_fast(v[mt][3] - subtr);
+                sum += (p0 + p1) + (p2 + p3);
+                pb[a][mt][0] = pack_bf16(p0, p1); pb[a][mt][1] = pack_bf16(p2, p3);
+            }
+            l[a] = fmaf(l[a], corr, sum);
+            const float c0 = __shfl_sync(0xffffffffu, corr, 8 * t), c1 = __shfl_sync(0xffffffffu, corr, 8 * t + 4);      // of the accumulators' queries 2t, 2t + 1
+#pragma unroll
+            for (int n = 0; n < 8; ++n) { o[a][n][0] *= c0; o[a][n][1] *= c1; o[a][n][2] *= c0; o[a][n][3] *= c1; }
+        }
+        const uint32_t vb = sV + (A.vst == 2 ? (i & 1) * vbytes : 0);
+#pragma unroll
+        for (int mt = 0; mt < kMT; ++mt) {
+            const int key = mt * 16 + (lane & 7) + ((lane >> 4) << 3);
+#pragma unroll
+            for (int n = 0; n < 8; ++n) {
+                if (n * 16 >= dv) break;
+                const uint32_t piece = (uint32_t)((n * 2 + ((lane >> 3) & 1)) ^ (key & 7));
+                uint32_t va[4];
+                int kv_loaded = -1;
+#pragma unroll
+                for (int a = 0; a < kHW; ++a) {
+                    if (h0 + a >= H) continue;
+                    const int kv = (h0 + a) / group;
+                    if (kv != kv_loaded) { kv_loaded = kv; ldsm_x4_trans(va, vb + (kv * kKT + key) * A.pv + piece * 16); }
+                    mma_bf16(o[a][n], va[0], va[1], va[2], va[3], pb[a][mt][0], pb[a][mt][1]);
+                }
+            }
+        }
+        if (A.kst != 2 || A.vst != 2) {                                // a single buffer: everybody is done with it, then it is filled again
+            if (A.kst != 2) cp_wait_all();
+            __syncthreads();
+            if (A.vst != 2) { load_v(i + 1); cp_commit(); }
+        }
+    }
+    cp_wait_all();
+    __syncthreads();
+    // ---- normalise, turn back, store: head by head through a warp's own rows of shared memory --------------------------------------------------
+    const int op = ((dv + 31) & ~31) + 4;                              // floats; 8 query rows per warp
+    float* os = reinterpret_cast<float*>(smem_tc) + warp * kTcRows * op;
+    const int half = dv >> 1;
+#pragma unroll
+    for (int a = 0; a < kHW; ++a) {
+        const int h = h0 + a;
+        if (h >= H) continue;
+        float lt = l[a];
+        lt += __shfl_xor_sync(0xffffffffu, lt, 1);
+        lt += __shfl_xor_sync(0xffffffffu, lt, 2);
+        const float inv = lt > 0.f ? 1.0f / lt : 0.f;
+        const float i0 = __shfl_sync(0xffffffffu, inv, 8 * t), i1 = __shfl_sync(0xffffffffu, inv, 8 * t + 4);
+        __syncwarp();
+#pragma unroll
+        for (int n = 0; n < 8; ++n) {
+            if (n * 16 >= dv) break;
+            os[(2 * t) * op + n * 16 + g] = o[a][n][0] * i0; os[(2 * t + 1) * op + n * 16 + g] = o[a][n][1] * i1;
+            os[(2 * t) * op + n * 16 + g + 8] = o[a][n][2] * i0; os[(2 * t + 1) * op + n * 16 + g + 8] = o[a][n][3] * i1;
+        }
+        __syncwarp();
+        for (int r = 0; r < rows; ++r) {
+            __nv_bfloat16* dst = A.out + ((int64_t)(q_begin + q0 + r) * H + h) * dv;
+            for (int x = lane; x < half; x += 32) {
+                float u = os[r * op + x], w = os[r * op + x + half];
+                if (A.cos_t) {
+                    const float c = A.cos_t[(int64_t)(pos0 + r) * half + x], sn = A.sin_t[(int64_t)(pos0 + r) * half + x];
+                    const float u2 = u * c + w * sn;
+                    w = w * c - u * sn; u = u2;
+                }
+                dst[x] = __float2bfloat16_rn(u); dst[x + half] = __float2bfloat16_rn(w);
+            }
+        }
+    }
+}
+
+// the tile and stage choice of a shape: heads per warp, keys per tile, stages of keys and values, bytes of shared memory (0 = not taken)
+struct TcPlan { int hw, kt, kst, vst, pk, pv; size_t smem; };
+TcPlan tc_plan(int H, int G, int dk, int dv) {
+    TcPlan none{0, 0, 0, 0, 0, 0, 0};
+    if (H > 32 || H % G || dk % 8 || dv % 16 || dv > 128 || dk > 256 || (int64_t)G * (dk > dv ? dk : dv) / 8 > 1024) return none;
+    const int hw = H <= 8 ? 1 : H <= 16 ? 2 : 4;
+    const int pk = (dk * 2 + 127) / 128 * 128, pv = (dv * 2 + 127) / 128 * 128;
+    const int tries[6][3] = {{32, 2, 2}, {32, 2, 1}, {16, 2, 2}, {16, 2, 1}, {32, 1, 1}, {16, 1, 1}};
+    for (const auto& c : tries) {
+        if (hw == 4 && c[0] != 16) continue;
+        size_t b = (size_t)H * kTcRows * pk + (size_t)c[1] * G * c[0] * pk + (size_t)c[2] * G * c[0] * pv + (size_t)2 * H * kTcRows * (c[0] + 4) * 4 +
+                   (size_t)H * ((H + 3) / 4 * 4) * 4;
+        const size_t outb = (size_t)8 * kTcRows * ((dv + 31) / 32 * 32 + 4) * 4;
+        if (b < outb) b = outb;
+        if (b <= 227 * 1024) return TcPlan{hw, c[0], c[1], c[2], pk, pv, b};
+    }
+    return none;
+}
+
 template <typename TC, typename TOut>
 bool launch_rows(const TalkArgs& A, int T, size_t smem, cudaStream_t st) {
     const int hw = (A.H + 7) / 8, pairs = (A.dv + 63) / 64;
@@ -372,6 +690,37 @@ void talking_attention_rows(void* out, const float* q, const void* key_cache, co
         count_launch();
     }
     check_launch("talking_attention_rows");
+}
+
+int32_t talking_attention_prefill_supported(int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv) {
+    return num_heads > 0 && num_kv_heads > 0 && dk > 0 && dv > 0 && tc_plan(num_heads, num_kv_heads, dk, dv).smem > 0 ? 1 : 0;
+}
+
+void talking_attention_prefill(void* out, const void* q, const void* key_cache, const void* value_cache, const int32_t* block_tables, int32_t table_width,
+                               const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, const float* talk, const float* v_cos, const float* v_sin, int32_t num_seqs,
+                               int32_t num_tokens, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t block_size, float scale, int32_t chunk,
+                               int32_t window, int32_t one_sink, int64_t stream) {
+    if (num_tokens == 0 || num_seqs == 0) return;
+    B200_REQUIRE(out && q && key_cache && value_cache && block_tables && cu_seqlens_q && cu_seqlens_k && (v_cos == nullptr) == (v_sin == nullptr), kErrBadArg,
+                 "talking_attention_prefill: null pointer");
+    B200_REQUIRE(num_heads > 0 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && dk > 0 && dv > 0 && block_size > 0 && table_width > 0, kErrBadArg,
+                 "talking_attention_prefill: bad sizes");
+    const TcPlan P = tc_plan(num_heads, num_kv_heads, dk, dv);
+    B200_REQUIRE(P.smem > 0 && (((uintptr_t)q | (uintptr_t)key_cache | (uintptr_t)value_cache) & 15) == 0, kErrUnsupported,
+                 "talking_attention_prefill: %d / %d heads of %d / %d (at most 32 heads, dk a multiple of 8, dv of 16 and <= 128)", num_heads, num_kv_heads, dk, dv);
+    TalkTcArgs A{(const __nv_bfloat16*)q, (const __nv_bfloat16*)key_cache, (const __nv_bfloat16*)value_cache, block_tables, table_width, cu_seqlens_q, cu_seqlens_k,
+                 num_seqs, talk, v_cos, v_sin, (__nv_bfloat16*)out, num_heads, num_kv_heads, dk, dv, block_size, scale * 1.4426950408889634f, chunk, window, one_sink,
+                 P.kst, P.vst, P.pk, P.pv};
+    cudaStream_t st = as_stream(stream);
+    const dim3 grid((unsigned)(num_tokens / kTcRows + num_seqs));
+#define TTC(HW, KT) do { ensure_dynamic_smem((const void*)talking_prefill_kernel<HW, KT>, (int)P.smem); \
+        launch_pdl(talking_prefill_kernel<HW, KT>, grid, dim3(256), P.smem, st, A); } while (0)
+    if (P.hw == 1) { if (P.kt == 32) TTC(1, 32); else TTC(1, 16); }
+    else if (P.hw == 2) { if (P.kt == 32) TTC(2, 32); else TTC(2, 16); }
+    else TTC(4, 16);
+#undef TTC
+    count_launch();
+    check_launch("talking_attention_prefill");
 }
 
 }  // extern "C"

@@ -636,6 +636,8 @@ class TalkingAttentionMixer:
         self.talk = w["talk"].float().contiguous() if "talk" in w else None
         self.w_o = w["o"].to(dtype).contiguous()
         self.splits = None                       # None: chosen by the step's shape (tests force a number)
+        # portions of prompts in 16 bits: the tensor-core kernel, when it takes these sizes
+        self.prefill_kernel = ops.talking_prefill_kernel_supported(heads, kv_heads, dk, dv, dtype)
         self.cos = self.sin = self.v_cos = self.v_sin = None
         self._device = self.w_in.device
         if rot:
@@ -660,7 +662,7 @@ class TalkingAttentionMixer:
         tables = (self.cos, self.sin) if self.rot_dims else None
         v_tables = (self.v_cos, self.v_sin) if self.rotate_values else None
         q = ops.qkv_rope_cache(proj, tables, v_tables, batch, None if self.shared else k_cache, None if self.shared else v_cache, self.H, self.G, self.dk, self.dv,
-                               self.rot_dims, self.dtype)
+                               self.rot_dims, self.dtype, torch.bfloat16 if self.prefill_kernel and batch.max_rows >= ops.TALKING_PREFILL_MIN_ROWS else torch.float32)
         a = ops.talking_attention(q, k_cache, v_cache, batch, self.talk, v_tables, self.H, self.scale, self.chunk, self.window, self.one_sink, self.dtype,
                                   splits=self.splits)
         return ops.linear(a, self.w_o)

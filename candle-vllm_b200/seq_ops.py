@@ -891,18 +891,33 @@ def qkv_rope_cache(qkv: torch.Tensor, tables: Optional[tuple], value_tables: Opt
     return q
 
 
+TALKING_PREFILL_MIN_ROWS = 8   # steps in which some entry brings at least this many rows take the tensor-core kernel (bf16)
+
+
+def talking_prefill_kernel_supported(heads: int, kv_heads: int, dk: int, dv: int, dtype: torch.dtype) -> bool:
+    return dtype == torch.bfloat16 and bool(lib().talking_attention_prefill_supported(C.c_int32(heads), C.c_int32(kv_heads), C.c_int32(dk), C.c_int32(dv)))
+
+
 TALKING_BLOCKS = 444           # three blocks per SM: steps with fewer rows cut the keys of every row into runs
 
 
 def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: StepBatch, talk: Optional[torch.Tensor], value_tables: Optional[tuple], heads: int,
                       scale: float, chunk: int, window: int, one_sink: bool, out_dtype: torch.dtype, splits: Optional[int] = None) -> torch.Tensor:
     """Softmax attention whose heads mix their scores by ``talk`` (f32 [H, H]) before the softmax; ``one_sink``: one is added to every denominator; ``value_tables``: the
-    cached values were turned by their position and every output is turned back by its own.  q f32 [T, H dk] -> [T, H dv] of ``out_dtype`` (the cache's).
-    ``splits``: runs every row's keys are cut into (None: enough blocks to fill the device, from the table width, so that a captured step keeps its choice)."""
+    cached values were turned by their position and every output is turned back by its own.  q f32 [T, H dk] -> [T, H dv] of ``out_dtype`` (the cache's); a bf16 q
+    takes the tensor-core kernel for portions of prompts (``talking_prefill_kernel_supported``).  ``splits``: runs every row's keys are cut into (None: enough blocks to fill the device, from the table width, so that a captured step keeps its choice)."""
     T = q.shape[0]
     nb, bs, G, dk = k_cache.shape
     dv = v_cache.shape[3]
     v_cos, v_sin = value_tables if value_tables else (None, None)
+    if q.dtype == torch.bfloat16 and k_cache.dtype == out_dtype == torch.bfloat16:
+        out = torch.empty((T, heads * dv), dtype=out_dtype, device=q.device)
+        lib().talking_attention_prefill(_ptr(out), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), C.c_int32(batch.block_tables.shape[1]), _ptr(batch.cu_seqlens),
+                                        _ptr(batch.cu_seqlens_k), _ptr(talk), _ptr(v_cos), _ptr(v_sin), C.c_int32(batch.num_seqs), C.c_int32(T), C.c_int32(heads), C.c_int32(G),
+                                        C.c_int32(dk), C.c_int32(dv), C.c_int32(bs), C.c_float(scale), C.c_int32(chunk), C.c_int32(window), C.c_int32(1 if one_sink else 0),
+                                        _stream(q.device))
+        check("talking_attention_prefill")
+        return out
     if q.dtype != torch.float32 or k_cache.dtype != out_dtype or (talk is not None and (talk.dtype != torch.float32 or tuple(talk.shape) != (heads, heads))):
         raise BackendError(f"talking_attention: q {q.dtype}, cache {k_cache.dtype}, out {out_dtype}")
     if splits is None:

@@ -508,3 +508,61 @@ def dofevik_weights(cfg: dict, seed: int = 0, device="cpu") -> dict:
                 sf = L["mlp"]["shared"]["ff"]
                 out[p + "mlp.shared.up"], out[p + "mlp.shared.down"] = lin(sf, D), lin(D, sf)
     return {k: v.to(torch.bfloat16).to(device) for k, v in out.items()}
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Sigalorn: random checkpoints of any shape (tests and bench.py)
+# ---------------------------------------------------------------------------------------------------------------------
+def sigalorn_gla_layer(heads: int, dim: int, vdim: int, tau: float = 16.0, ff: int = 0) -> dict:
+    return dict(type="gla", mixer=dict(heads=heads, dim=dim, vdim=vdim, tau=tau), mlp=dict(ff=ff, kind="dense") if ff else None)
+
+
+def sigalorn_attention_layer(heads: int, kv_heads: int, dim: int, vdim: int, chunk: int = 0, rot_dims: int = 0, base: float = 10000.0, scale: float = None, ff: int = 0,
+                             kv_from: int = None) -> dict:
+    mixer = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=dim ** -0.5 if scale is None else scale, rot=dict(base=base, dims=rot_dims or dim))
+    if chunk:
+        mixer["mask"] = dict(size=chunk)
+    if kv_from is not None:
+        mixer["kv_from"] = kv_from
+    return dict(type="attention", mixer=mixer, mlp=dict(ff=ff, kind="dense") if ff else None)
+
+
+def sigalorn_config(width: int, vocab: int, layers: list, eps: float = 1e-6, embedding_scale: float = 1.0, softcap: float = 20.0) -> dict:
+    cfg = dict(architecture="Sigalorn", embedding=dict(scale=embedding_scale), layers=layers, norm=dict(eps=eps), vocab=vocab, width=width)
+    if softcap:
+        cfg["logit_softcap"] = softcap
+    return cfg
+
+
+def sigalorn_weights(cfg: dict, seed: int = 0, rank: int = 16, device="cpu") -> dict:
+    """name -> bf16 tensor with magnitudes that keep every mechanism visible in the logits: scores of a few units whose heads mix strongly, decays from nearly one
+    to nearly zero within a layer, logits that reach into the cap."""
+    g = torch.Generator().manual_seed(seed)
+    D, V = cfg["width"], cfg["vocab"]
+    out = {}
+    rnd = lambda *shape, std=1.0: (torch.randn(*shape, generator=g) * std)
+    lin = lambda n, k, gain=1.0: rnd(n, k, std=gain * k ** -0.5)
+    norm = lambda n: 1.0 + rnd(n, std=0.25)
+    out["embed"], out["head"], out["final.norm"] = rnd(V, D), lin(V, D, 6.0), norm(D)
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        H, dk, dv = m["heads"], m["dim"], m["vdim"]
+        out[p + "norm1"], out[p + "norm1b"] = norm(D), norm(D)
+        if L["type"] == "gla":
+            out[p + "mix.q"], out[p + "mix.k"], out[p + "mix.v"], out[p + "mix.g"] = lin(H * dk, D), lin(H * dk, D), lin(H * dv, D), lin(H * dv, D)
+            out[p + "mix.a1"], out[p + "mix.a2"] = lin(rank, D), lin(H * dk, rank, 1.5)
+            out[p + "mix.a2.b"] = torch.rand(H * dk, generator=g) * 9.0 - 3.0
+            out[p + "mix.norm"], out[p + "mix.o"] = norm(dv), lin(D, H * dv)
+        else:
+            G = m["kv_heads"]
+            out[p + "mix.q"] = lin(H * dk, D, 1.5)
+            if m.get("kv_from") is None:
+                out[p + "mix.k"], out[p + "mix.v"] = lin(G * dk, D), lin(G * dv, D)
+            out[p + "mix.talk"] = torch.eye(H) * 0.8 + rnd(H, H, std=0.6 * H ** -0.5)
+            out[p + "mix.o"] = lin(D, H * dv)
+        if L.get("mlp"):
+            ff = L["mlp"]["ff"]
+            out[p + "norm2"], out[p + "norm2b"] = norm(D), norm(D)
+            out[p + "mlp.up"], out[p + "mlp.up.b"], out[p + "mlp.down"], out[p + "mlp.down.b"] = lin(ff, D), rnd(ff, std=0.3), lin(D, ff), rnd(D, std=0.3)
+            out[p + "mlp.act"] = rnd(2)
+    return {k: v.to(torch.bfloat16).to(device) for k, v in out.items()}
