@@ -49,7 +49,7 @@ def parse():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--cpu-seconds", type=float, default=20.0)
     ap.add_argument("--parity-steps", type=int, default=3, help="decode steps compared against a TP=1 engine before timing (0 = off)")
-    ap.add_argument("--arch", default="llama", choices=["llama", "gobesun", "guvusun", "panarax", "dofevik"],
+    ap.add_argument("--arch", default="llama", choices=["llama", "gobesun", "guvusun", "panarax", "dofevik", "sigalorn"],
                     help="llama = the metric (default, unchanged).  gobesun = prefill / decode throughput of the Gobesun decoder at layer sizes of real "
                          "models (random weights), beside a dense bf16 Llama of equal width / heads / ff / depth, with a per-kernel roofline table; "
                          "one JSON line, single GPU.  guvusun / panarax / dofevik = the same for those decoders (panarax beside a Gobesun, dofevik beside a Guvusun of "
@@ -1499,10 +1499,211 @@ def run_dofevik(args):
                       "gpu_launches": int(pkg.lib().b200_total_kernel_launches() - l0), "sizes": results}))
 
 
+# ------------------------------------------------------------------------------------------------
+# --arch sigalorn: linear attention with a decay per key row and attention whose heads mix their scores, beside a Gobesun (recurrent + chunk-masked attention
+# layers, the same norms around every sublayer) of equal size
+# ------------------------------------------------------------------------------------------------
+SIGALORN_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv=4, ff=5632, vocab=32000, layers=8, chunk=2048, rank=16),
+    "w4096": dict(width=4096, heads=32, kv=8, ff=11008, vocab=32000, layers=4, chunk=2048, rank=16),
+}
+
+
+def run_sigalorn(args):
+    import torch
+    import candle_vllm_b200 as pkg
+    from candle_vllm_b200 import seq_ops as ops, synthetic as S
+    from candle_vllm_b200.engine import ModelRunner
+    from candle_vllm_b200.gobesun import GobesunConfig, GobesunModel
+    from candle_vllm_b200.inputs import prepare_step
+    from candle_vllm_b200.sigalorn import SigalornConfig, SigalornModel
+
+    torch.cuda.set_device(0)
+    dev = "cuda"
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else \
+        {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "fallback": True}
+    HBM, TC = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    props = torch.cuda.get_device_properties(0)
+    F32 = props.multi_processor_count * 128 * 2 * 1.965e9            # nominal f32 multiply-add rate: the recurrences are 32-bit by definition
+    K, W = max(args.steps, 1), max(args.warmup, 3)
+    P, B, CTX, hd = 4096, 32, 1024, 128
+    bf = torch.bfloat16
+    l0 = pkg.lib().b200_total_kernel_launches()
+
+    def timed(fn, reps, warm=3):
+        for _ in range(warm):
+            fn()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(reps):
+            fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / reps * 1e-3
+
+    def once(fn):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize(); e0.record()
+        r = fn()
+        e1.record(); torch.cuda.synchronize()
+        return r, e0.elapsed_time(e1) * 1e-3
+
+    names = ["linear", "rms_norm_ex", "post_norm_add_rms_norm", "gelu_tanh_mul", "xielu", "embedding_scaled", "causal_conv_silu", "gated_delta_rule", "gated_rms_norm",
+             "group_rms_norm_gate", "low_rank_decay", "linear_attention_channel", "qk_norm_rope_cache", "qkv_rope_cache", "paged_attention_varlen_sink",
+             "paged_attention_decode_chunked", "talking_attention", "softcap"]
+
+    def measure(model, V):
+        """(prefill s, decode s per step incl. host, decode s per step device, {(tag, kernel): [s]})"""
+        blocks_per = -(-(CTX + K + W + 8) // 64)
+        runner = ModelRunner(model, B * blocks_per + P // 64 + 1, B + 1, 64, decode_graphs=True, max_blocks_per_seq=blocks_per)
+        toks = torch.randint(0, V, (P,), generator=torch.Generator().manual_seed(1)).tolist()
+
+        def prefill():
+            runner.admit(10 ** 6)
+            runner.execute([dict(seq_id=10 ** 6, tokens=toks, want=[P - 1])])
+            runner.release(10 ** 6)
+        pre = timed(prefill, 3, 2)
+        for i in range(B):
+            runner.admit(i)
+        for i in range(0, B, 4):
+            runner.execute([dict(seq_id=j, tokens=toks[:CTX], want=[]) for j in range(i, i + 4)])
+        step_entries = lambda: [dict(seq_id=j, tokens=[toks[j]], want=[0]) for j in range(B)]
+        dec = timed(lambda: runner.execute(step_entries()), K, W)
+        dec_dev = timed(runner._graphs[B].graph.replay, K, 3)
+        kern = {}
+        orig = {n: getattr(ops, n) for n in names}
+
+        def instrument(tag):
+            def wrap(n):
+                def f(*a, **k):
+                    r, s = once(lambda: orig[n](*a, **k))
+                    kern.setdefault((tag, n if n != "linear" else f"linear[{a[1].shape[0]}x{a[1].shape[1]}]"), []).append(s)
+                    return r
+                return f
+            for n in names:
+                setattr(ops, n, wrap(n))
+        instrument("prefill")
+        prefill(); kern.clear(); prefill()
+        runner.decode_graphs = False
+        instrument("decode")
+        runner.execute(step_entries())
+        for k in [k for k in kern if k[0] == "decode"]:
+            kern.pop(k)
+        runner.execute(step_entries())
+        for n in names:
+            setattr(ops, n, orig[n])
+        del runner
+        torch.cuda.empty_cache()
+        return pre, dec, dec_dev, kern
+
+    sampler = ClockSampler(0); sampler.start()
+    results = {}
+    for name in [n for n in args.arch_sizes.split(",") if n in SIGALORN_SIZES]:
+        z = SIGALORN_SIZES[name]
+        D, H, G, ff, V, NL, R = z["width"], z["heads"], z["kv"], z["ff"], z["vocab"], z["layers"], z["rank"]
+        # ---- three recurrent layers to one attention layer, every layer with a feed-forward; the last attention layer uses the first one's keys when there are two
+        layers = []
+        for i in range(NL):
+            layers.append(S.sigalorn_attention_layer(H, G, hd, hd, chunk=z["chunk"], base=1e6, ff=ff, kv_from=3 if i > 3 else None) if i % 4 == 3 else
+                          S.sigalorn_gla_layer(H, hd, hd, ff=ff))
+        cfg = S.sigalorn_config(D, V, layers)
+        model = SigalornModel(SigalornConfig.from_dict(cfg), S.sigalorn_weights(cfg, 0, rank=R), dtype=bf, block_size=64, max_pos=P + 64, device=dev)
+        s_pre, s_dec, s_dec_dev, s_kern = measure(model, V)
+        del model
+        torch.cuda.empty_cache()
+        # ---- Gobesun of equal width / heads / ff / depth
+        glayers = [S.gobesun_attention_layer(H, G, hd, hd, z["chunk"], hd, ff=ff, base=1e6) if i % 4 == 3 else S.gobesun_delta_layer(H, H // 2, hd, hd, conv=4, ff=ff)
+                   for i in range(NL)]
+        gcfg = S.gobesun_config(D, V, glayers)
+        gmodel = GobesunModel(GobesunConfig.from_dict(gcfg), S.gobesun_weights(gcfg, 0), dtype=bf, block_size=64, max_pos=P + 64, device=dev)
+        g_pre, g_dec, g_dec_dev, g_kern = measure(gmodel, V)
+        del gmodel
+        torch.cuda.empty_cache()
+        # ---- the like kernel of the linear attention: the one with a fixed decay per head (Panarax), same heads and sizes, timed alone the way the models' calls are
+        like = {}
+        for tag, entries, T in (("prefill", [dict(tokens=[0] * P, start=0, block_table=list(range(P // 64)), state_slot=0, want=[])], P),
+                                ("decode", [dict(tokens=[0], start=CTX, block_table=list(range(CTX // 64 + 1)), state_slot=j, want=[]) for j in range(B)], B)):
+            bt = ops.StepBatch.from_host(prepare_step(entries, 64), dev)
+            pr = torch.randn(T, 4 * H * hd, device=dev) * 0.1
+            st, de = torch.zeros(B, H, hd, hd, device=dev), torch.full((H,), 0.97, device=dev)
+            call = lambda: ops.linear_attention(pr, 0, H * hd, 2 * H * hd, st, bt, H, hd, hd, act="silu", decay=de)
+            for _ in range(3):
+                call()
+            like[(tag, "linear_attention[decay]")] = [once(call)[1] for _ in range(5)]
+            del pr, st
+        torch.cuda.empty_cache()
+        med = lambda v: (sorted(v)[(len(v) - 1) // 2] + sorted(v)[len(v) // 2]) / 2
+        esz, Gd = 2, H // 2
+        Cd = 2 * Gd * hd + H * hd
+
+        def work(tag, key, T):
+            """algorithmic work of one call: ("bytes", n) against the measured copy bandwidth, ("flops", n) against the measured bf16 GEMM rate, ("f32", n) against
+            the nominal f32 multiply-add rate"""
+            pre = tag == "prefill"
+            if key.startswith("linear["):
+                n, k = (int(v) for v in key[7:-1].split("x"))
+                if n == V and pre:
+                    T = 1
+                return ("flops", 2.0 * T * n * k) if (pre and T > 1) else ("bytes", n * k * esz + T * (k * esz + n * 4))
+            state = (1 if pre else T) * 2 * H * hd * hd * 4                # one read and one write of every entry's state
+            seen = sum(i % z["chunk"] + 1 for i in range(T)) if pre else T * (CTX % z["chunk"] + 1)
+            att = ("flops", 4.0 * H * hd * seen) if pre else ("bytes", seen * 2 * G * hd * esz)
+            qkv = T * ((H + 2 * G) * hd * 4 + H * hd * esz + 2 * G * hd * esz)
+            return {
+                "rms_norm_ex": ("bytes", T * D * (4 + esz)), "post_norm_add_rms_norm": ("bytes", T * D * (12 + esz)),
+                "gelu_tanh_mul": ("bytes", T * ff * (8 + esz)), "xielu": ("bytes", T * ff * (4 + esz)), "embedding_scaled": ("bytes", T * D * (esz + 4)),
+                "causal_conv_silu": ("bytes", T * Cd * 8), "gated_rms_norm": ("bytes", T * H * hd * (8 + esz)), "group_rms_norm_gate": ("bytes", T * H * hd * (8 + esz)),
+                "low_rank_decay": ("bytes", T * (H * hd + R) * 4 + H * hd * R * 4),
+                "gated_delta_rule": ("f32", 6.0 * T * H * hd * hd) if pre else ("bytes", T * (Cd + H * hd) * 4 + state),
+                "linear_attention[decay]": ("f32", 4.0 * T * H * hd * hd) if pre else ("bytes", T * 4 * H * hd * 4 + state),
+                "linear_attention_channel": ("f32", 4.0 * T * H * hd * hd) if pre else ("bytes", T * 5 * H * hd * 4 + state),
+                "qk_norm_rope_cache": ("bytes", qkv), "qkv_rope_cache": ("bytes", qkv),
+                "paged_attention_varlen_sink": att, "paged_attention_decode_chunked": att, "talking_attention": att,
+                "softcap": ("bytes", (1 if pre else T) * V * 8),
+            }.get(key)
+
+        def table(kern, tag, T):
+            out = {}
+            for (tg, key), v in kern.items():
+                if tg != tag:
+                    continue
+                t = med(v)
+                e = {"us": round(t * 1e6, 1), "calls_per_step": len(v)}
+                w = work(tag, key, T)
+                if w:
+                    roof = w[1] / {"bytes": HBM, "flops": TC, "f32": F32}[w[0]]
+                    e.update(bound=w[0], roofline_us=round(roof * 1e6, 2), frac_of_roofline=round(roof / t, 3))
+                if key == "talking_attention" and tag == "prefill":
+                    # mixing is 32-bit by definition: H multiply-adds per head, query and key on the FMA pipe, beside the two products on the tensor cores
+                    mix = 2.0 * H * H * sum(i % z["chunk"] + 1 for i in range(T)) / F32
+                    e.update(f32_mixing_roofline_us=round(mix * 1e6, 2), frac_of_mixing_roofline=round(mix / t, 3))
+                out[key] = e
+            return out
+        side = lambda pre, dec, dec_dev, kern: {
+            "prefill_tokens_per_s": round(P / pre), "prefill_ms": round(pre * 1e3, 2), "decode_tokens_per_s": round(B / dec), "decode_ms_per_step": round(dec * 1e3, 3),
+            "decode": "CUDA-graph replay incl. host metadata and H2D", "decode_ms_per_step_device": round(dec_dev * 1e3, 3),
+            "decode_tokens_per_s_device": round(B / dec_dev), "kernels_prefill": table(kern, "prefill", P), "kernels_decode": table(kern, "decode", B)}
+        results[name] = {"sigalorn": side(s_pre, s_dec, s_dec_dev, s_kern), "gobesun": side(g_pre, g_dec, g_dec_dev, g_kern),
+                         "like_kernels": {"prefill": table(like, "prefill", P), "decode": table(like, "decode", B)},
+                         "shape": dict(z, prompt=P, decode_batch=B, decode_ctx=CTX, head_dim=hd)}
+    clocks = sampler.stop()
+    first = results[next(iter(results))]
+    print(json.dumps({"metric": "Sigalorn prefill / decode tokens/s beside a Gobesun of equal size", "value": first["sigalorn"]["decode_tokens_per_s"],
+                      "unit": UNIT, "n_gpus": 1, "steps": K, "warmup": W, "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "arch": "sigalorn",
+                      "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "f32_fma_tflops_nominal": round(F32 / 1e12, 1),
+                                "source": "fallback" if peaks.get("fallback") else "MEASURED_PEAKS.json"},
+                      "l2": "weights and activations of a step exceed L2 (126 MB)", "clocks": clocks,
+                      "gpu_launches": int(pkg.lib().b200_total_kernel_launches() - l0), "sizes": results}))
+
+
 def main():
     args = parse()
     if args.arch == "gobesun":
         run_gobesun(args)
+        return
+    if args.arch == "sigalorn":
+        run_sigalorn(args)
         return
     if args.arch == "dofevik":
         run_dofevik(args)
