@@ -11,7 +11,7 @@
 //                           heads, lanes across the columns).  Few rows: the keys of a row are cut into runs and talking_merge_kernel joins them.
 //   talking_prefill_kernel  portions of prompts in 16 bits: a block per 8 query rows with ALL heads, mma.sync m16n8k16 with keys (or value columns) on the
 //                           16-row side and queries on the 8-column side, so that 32 heads' accumulators of 128 value columns fit the register file.  A warp
-//                           owns H / 8 heads in both products; raw scores meet in shared memory, a thread mixes one (query, key) pair over all heads in
+//                           owns H / 16 heads in both products; raw scores meet in shared memory, a thread mixes one (query, key) pair over all heads in
 //                           f32, and every warp reads its heads' mixed scores back in the operand layout of the second product.  The first product of the
 //                           next tile is issued before the mixing of this one (scores double-buffered), so a tile costs one barrier; keys and values
 //                           arrive by cp.async while earlier tiles are worked on.
@@ -33,9 +33,14 @@ struct TalkArgs {
     float* part;                                 // splits > 1: [T, splits, H, dv + 2]: unnormalised sum, maximum, denominator
     int H, G, dk, dv, bs;
     float scale;
-    int chunk, window, one_sink, splits, tile, qpitch;
+    int chunk, window, one_sink, splits, tile, qpitch, bs_shift;
 };
 
+// cache row of a position (shift >= 0: the block size is 1 << shift, otherwise it is divided by)
+__device__ __forceinline__ int64_t cache_row(const int32_t* table, int j, int bs, int shift) {
+    const int b = shift >= 0 ? j >> shift : j / bs;
+    return (int64_t)table[b] * bs + (j - b * bs);
+}
 __device__ __forceinline__ int first_visible(int pos, int chunk, int window) {
     int lo = chunk > 0 ? (pos / chunk) * chunk : 0;
     if (window > 0 && pos - window + 1 > lo) lo = pos - window + 1;
@@ -101,7 +106,7 @@ talking_rows_kernel(const TalkArgs A) {
     auto place = [&](int j0, int buf) {          // keys past the run's end stand for its first one (their weight is 0, what they read is finite)
         for (int i = threadIdx.x; i < KT; i += 256) {
             const int j = j0 + i < je ? j0 + i : jb;
-            ph[buf * KT + i] = (int64_t)table[j / A.bs] * A.bs + j % A.bs;
+            ph[buf * KT + i] = cache_row(table, j, A.bs, A.bs_shift);
         }
     };
     if (jb < je) place(jb, 0);
@@ -109,6 +114,9 @@ talking_rows_kernel(const TalkArgs A) {
     const int slices = H < 8 ? 8 / H : 1;
     const int h0 = H < 8 ? warp % H : warp * kHW, slice = H < 8 ? warp / H : 0;
     const bool has_values = slice < slices && h0 < H;
+    int kvh[kHW];                                // their kv heads
+#pragma unroll
+    for (int a = 0; a < kHW; ++a) kvh[a] = min(h0 + a, H - 1) / group;
     float2 acc[kHW][kC];
 #pragma unroll
     for (int a = 0; a < kHW; ++a)
@@ -229,7 +237,7 @@ talking_rows_kernel(const TalkArgs A) {
                 float2 vv[4][kC];
 #pragma unroll
                 for (int a = 0; a < kHW; ++a) {
-                    const int g = min(h0 + a, H - 1) / group;
+                    const int g = kvh[a];
                     if (g != g_loaded) {
                         g_loaded = g;
 #pragma unroll
@@ -333,9 +341,10 @@ struct TalkTcArgs {
     int chunk, window, one_sink;
     int kst, vst;                                // key / value tiles kept in shared memory (1 or 2)
     int pk, pv;                                  // row pitches in bytes, multiples of 128
+    int bs_shift;
 };
 
-constexpr int kTcRows = 8;                       // query rows of a block
+constexpr int kTcRows = 8, kTcWarps = 16, kTcThreads = kTcWarps * 32;        // query rows and warps of a block
 
 __device__ __forceinline__ void cp16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
@@ -355,15 +364,15 @@ __device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
 __device__ __forceinline__ float exp2_fast(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) { const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi); return *reinterpret_cast<const uint32_t*>(&v); }
 
-// kHW: heads per warp (8 warps), kKT: keys per tile
-template <int kHW, int kKT>
-__global__ void __launch_bounds__(256, 1)
+// kHW: heads per warp (16 warps), kKT: keys per tile, k128: keys and values of 128 entries (the addresses are then constants)
+template <int kHW, int kKT, bool k128>
+__global__ void __launch_bounds__(kTcThreads, 1)
 talking_prefill_kernel(const TalkTcArgs A) {
     pdl_wait();
     pdl_trigger();
     constexpr int kMT = kKT / 16, kSP = kKT + 4;                       // 16-key pieces per tile; pitch of a score row
     extern __shared__ __align__(1024) uint8_t smem_tc[];
-    const int H = A.H, G = A.G, dk = A.dk, dv = A.dv, group = H / G;
+    const int H = A.H, G = A.G, dk = k128 ? 128 : A.dk, dv = k128 ? 128 : A.dv, pk = k128 ? 256 : A.pk, pv = k128 ? 256 : A.pv, group = H / G;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     // which (sequence, 8-row tile) is this block?  the last tiles of a sequence see the most keys and start first
     int seq = -1, tile = 0, base = 0;
@@ -379,21 +388,33 @@ talking_prefill_kernel(const TalkTcArgs A) {
     const int ntiles = (last_pos - key0) / kKT + 1;
     const int32_t* table = A.block_tables + (int64_t)seq * A.table_width;
 
-    const int kbytes = G * kKT * A.pk, vbytes = G * kKT * A.pv;
+    const int kbytes = G * kKT * pk, vbytes = G * kKT * pv;
     const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(smem_tc);
-    const uint32_t sQ = sbase, sK = sQ + H * kTcRows * A.pk, sV = sK + A.kst * kbytes;
-    float* S = reinterpret_cast<float*>(smem_tc + (sV - sbase) + A.vst * vbytes);                   // [2][H][8][kSP]
-    const int sstage = H * kTcRows * kSP;
-    float* tk = S + 2 * sstage;                                                                      // [H][Hp]
-    const int Hp = (H + 3) & ~3;
+    const uint32_t sQ = sbase, sK = sQ + H * kTcRows * pk, sV = sK + A.kst * kbytes;
+    float* S = reinterpret_cast<float*>(smem_tc + (sV - sbase) + A.vst * vbytes);                   // [2][Hp][8][kSP]
+    const int Hp = (H + 3) & ~3, tp = Hp + 4;                          // heads rounded up to whole groups of four (rows of zeros); row pitch of the mixing matrix
+    const int sstage = Hp * kTcRows * kSP;
+    float* tk = S + 2 * sstage;                                                                      // [8 kNP][tp] talk times scale log2 e, zeros past H
+    const int magic_k = (65536 + (dk >> 3) - 1) / (dk >> 3), magic_v = (65536 + (dv >> 3) - 1) / (dv >> 3);
 
     // a tile of keys (or values) of every kv head: a warp takes whole cache rows; rows past the last visible key repeat it (their weight is 0)
     auto load_tile = [&](const __nv_bfloat16* cache, int d, uint32_t dst, int pitch, int tl, bool values) {
-        const int d8 = d >> 3, pieces = G * d8, magic = (65536 + d8 - 1) / d8;                       // p / d8 exactly for p < 1024, d8 <= 32
+        const int d8 = d >> 3, pieces = G * d8, magic = values ? magic_v : magic_k;                  // (p * magic) >> 16 = p / d8 exactly for p < 1024, d8 <= 32
+        const __nv_bfloat16* rows_of[kKT / kTcWarps];
 #pragma unroll
-        for (int kk = 0; kk < kKT / 8; ++kk) {
-            const int key = warp + 8 * kk, j = min(key0 + tl * kKT + key, last_pos);
-            const __nv_bfloat16* src = cache + ((int64_t)table[j / A.bs] * A.bs + j % A.bs) * G * d;
+        for (int kk = 0; kk < kKT / kTcWarps; ++kk)
+            rows_of[kk] = cache + cache_row(table, min(key0 + tl * kKT + warp + kTcWarps * kk, last_pos), A.bs, A.bs_shift) * G * d;
+#pragma unroll
+        for (int kk = 0; kk < kKT / kTcWarps; ++kk) {
+            const int key = warp + kTcWarps * kk;
+            const __nv_bfloat16* src = rows_of[kk];
+            if constexpr (k128) {                                      // a lane's pieces lie two kv heads apart, at the same place of their rows
+                const int c = lane & 15, cs = values ? c ^ (key & 7) : c ^ ((key & 1) << 2);
+                uint32_t at = dst + ((lane >> 4) * kKT + key) * 256 + cs * 16;
+                src += lane * 8;
+                for (int p = lane; p < pieces; p += 32, at += 2 * kKT * 256, src += 256) cp16(at, src);
+                continue;
+            }
             for (int p = lane; p < pieces; p += 32) {
                 const int kv = (p * magic) >> 16, c = p - kv * d8;
                 const int cs = values ? c ^ (key & 7) : c ^ ((key & 1) << 2);
@@ -401,15 +422,15 @@ talking_prefill_kernel(const TalkTcArgs A) {
             }
         }
     };
-    auto load_k = [&](int tl) { if (tl < ntiles) load_tile(A.kc, dk, sK + (A.kst == 2 ? (tl & 1) * kbytes : 0), A.pk, tl, false); };
-    auto load_v = [&](int tl) { if (tl < ntiles) load_tile(A.vc, dv, sV + (A.vst == 2 ? (tl & 1) * vbytes : 0), A.pv, tl, true); };
+    auto load_k = [&](int tl) { if (tl < ntiles) load_tile(A.kc, dk, sK + (A.kst == 2 ? (tl & 1) * kbytes : 0), pk, tl, false); };
+    auto load_v = [&](int tl) { if (tl < ntiles) load_tile(A.vc, dv, sV + (A.vst == 2 ? (tl & 1) * vbytes : 0), pv, tl, true); };
 
     {
         const int d8 = dk >> 3;
-        for (int r = warp; r < H * kTcRows; r += 8) {
+        for (int r = warp; r < H * kTcRows; r += kTcWarps) {
             const int h = r >> 3, qr = r & 7;
             const __nv_bfloat16* src = A.q + ((int64_t)(q_begin + q0 + min(qr, rows - 1)) * H + h) * dk;
-            for (int c = lane; c < d8; c += 32) cp16(sQ + r * A.pk + (c ^ ((qr & 1) << 2)) * 16, src + c * 8);
+            for (int c = lane; c < d8; c += 32) cp16(sQ + r * pk + (c ^ ((qr & 1) << 2)) * 16, src + c * 8);
         }
     }
     load_k(0);
@@ -417,45 +438,51 @@ talking_prefill_kernel(const TalkTcArgs A) {
     if (A.kst == 2) load_k(1);
     cp_commit();
     if (A.talk)
-        for (int i = threadIdx.x; i < H * Hp; i += 256) { const int h = i / Hp, x = i - h * Hp; tk[i] = x < H ? A.talk[h * H + x] : 0.f; }
+        for (int i = threadIdx.x; i < 8 * (kTcThreads / (kTcRows * kKT)) * tp; i += kTcThreads) {
+            const int h = i / tp, x = i - h * tp;
+            tk[i] = h < H && x < H ? A.talk[h * H + x] * A.scale_log2 : 0.f;
+        }
+    for (int i = threadIdx.x; i < (Hp - H) * kTcRows * kSP; i += kTcThreads) S[H * kTcRows * kSP + i] = S[sstage + H * kTcRows * kSP + i] = 0.f;
 
     const int h0 = warp * kHW;
     float o[kHW][8][4];
     float m[kHW], l[kHW];
+    int kvh[kHW];                                                      // kv heads of this warp's heads
 #pragma unroll
     for (int a = 0; a < kHW; ++a) {
+        kvh[a] = min(h0 + a, H - 1) / group;
 #pragma unroll
         for (int n = 0; n < 8; ++n) o[a][n][0] = o[a][n][1] = o[a][n][2] = o[a][n][3] = 0.f;
         m[a] = A.one_sink ? 0.f : -INFINITY;                           // the sink: a key of score 0 without a value, counted by one lane of the query's four
         l[a] = A.one_sink && t == 0 ? 1.f : 0.f;
     }
 
-    // raw scores of this warp's heads for tile tl, times scale log2 e, into score stage tl & 1.  The four lanes of a row take 16-byte pieces of it: both operands
+    // raw scores of this warp's heads for tile tl into score stage tl & 1.  The four lanes of a row take 16-byte pieces of it: both operands
     // permute the contraction index the same way, so no transposing load is needed.
+    const uint32_t off_a = (uint32_t)((t ^ ((g & 1) << 2)) * 16), off_b = off_a ^ 64u;       // of the even and odd 32-entry parts of a row pair
     auto scores = [&](int tl) {
         float acc[kHW][kMT][4] = {};
         const uint32_t kb = sK + (A.kst == 2 ? (tl & 1) * kbytes : 0);
-        const uint32_t sw = (uint32_t)((g & 1) << 2);
-        for (int d0 = 0; d0 < dk; d0 += 32) {
-            const int c = (d0 >> 3) + t;
-            const bool ok = c * 8 < dk;
-            const uint32_t off = (((uint32_t)c) ^ sw) * 16;
+#pragma unroll (k128 ? 4 : 1)
+        for (int d = 0; d < (dk + 31) / 32; ++d) {
+            const bool ok = k128 || (4 * d + t) * 8 < dk;
+            const uint32_t off = ((d & 1) ? off_b : off_a) + (d >> 1) * 128;
             uint4 ka[kMT][2];
             int kv_loaded = -1;
 #pragma unroll
             for (int a = 0; a < kHW; ++a) {
                 const int h = h0 + a;
                 if (h >= H) continue;
-                const int kv = h / group;
+                const int kv = kvh[a];
                 if (kv != kv_loaded) {
                     kv_loaded = kv;
+                    const uint32_t at = kb + (kv * kKT + g) * pk + off;
 #pragma unroll
                     for (int mt = 0; mt < kMT; ++mt)
 #pragma unroll
-                        for (int e = 0; e < 2; ++e)
-                            ka[mt][e] = ok ? lds16(kb + (kv * kKT + mt * 16 + e * 8 + g) * A.pk + off) : make_uint4(0u, 0u, 0u, 0u);
+                        for (int e = 0; e < 2; ++e) ka[mt][e] = ok ? lds16(at + (mt * 16 + e * 8) * pk) : make_uint4(0u, 0u, 0u, 0u);
                 }
-                const uint4 qb = ok ? lds16(sQ + (h * kTcRows + g) * A.pk + off) : make_uint4(0u, 0u, 0u, 0u);
+                const uint4 qb = ok ? lds16(sQ + (h * kTcRows + g) * pk + off) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
                 for (int mt = 0; mt < kMT; ++mt) {
                     mma_bf16(acc[a][mt], ka[mt][0].x, ka[mt][1].x, ka[mt][0].y, ka[mt][1].y, qb.x, qb.y);
@@ -470,34 +497,39 @@ talking_prefill_kernel(const TalkTcArgs A) {
             float* r0 = Sd + ((h0 + a) * kTcRows + 2 * t) * kSP;
 #pragma unroll
             for (int mt = 0; mt < kMT; ++mt) {
-                r0[mt * 16 + g] = acc[a][mt][0] * A.scale_log2;
-                r0[kSP + mt * 16 + g] = acc[a][mt][1] * A.scale_log2;
-                r0[mt * 16 + g + 8] = acc[a][mt][2] * A.scale_log2;
-                r0[kSP + mt * 16 + g + 8] = acc[a][mt][3] * A.scale_log2;
+                r0[mt * 16 + g] = acc[a][mt][0];
+                r0[kSP + mt * 16 + g] = acc[a][mt][1];
+                r0[mt * 16 + g + 8] = acc[a][mt][2];
+                r0[kSP + mt * 16 + g + 8] = acc[a][mt][3];
             }
         }
     };
-    // every (query, key) pair of score stage st: s'[h] = sum_g talk[h, g] s[g], in place, one thread per pair
+    // every (query, key) pair of score stage st: s'[h] = scale log2 e sum_g talk[h, g] s[g], in place.  kNP lanes of one warp share a pair: all of them read its H
+    // raw scores, then every one writes its share of the heads.
+    constexpr int kNP = kTcThreads / (kTcRows * kKT), kPW = 32 / kNP;
+    static_assert(8 * kNP >= 16 * kHW, "eight heads per lane cover all of them");
     auto mix = [&](int st) {
-        if (!A.talk || (int)threadIdx.x >= kTcRows * kKT) return;
-        float* col = S + st * sstage + (threadIdx.x / kKT) * kSP + (threadIdx.x % kKT);
-        float s[8 * kHW];
-#pragma unroll
-        for (int x = 0; x < 8 * kHW; ++x) s[x] = x < H ? col[x * kTcRows * kSP] : 0.f;
+        if (!A.talk) return;
+        const int pair = warp * kPW + lane % kPW, part = lane / kPW;
+        float* col = S + st * sstage + (pair / kKT) * kSP + pair % kKT;
+        float r[8] = {};                                               // heads part, part + kNP, ... of the mixing matrix's padded rows
+        const float* w0 = tk + part * tp;
 #pragma unroll 2
-        for (int h = 0; h < H; ++h) {
-            const float4* w4 = reinterpret_cast<const float4*>(tk + h * Hp);
-            float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+        for (int x = 0; x < Hp; x += 4) {
+            float s[4];
 #pragma unroll
-            for (int x = 0; x < 2 * kHW; ++x) {
-                if (x * 4 >= H) break;
-                const float4 w = w4[x];
-                a0 = fmaf(w.x, s[4 * x], a0); a1 = fmaf(w.y, s[4 * x + 1], a1); a2 = fmaf(w.z, s[4 * x + 2], a2); a3 = fmaf(w.w, s[4 * x + 3], a3);
+            for (int e = 0; e < 4; ++e) s[e] = col[(x + e) * kTcRows * kSP];
+#pragma unroll
+            for (int n = 0; n < 8; ++n) {
+                const float4 w = *reinterpret_cast<const float4*>(w0 + n * kNP * tp + x);
+                r[n] = fmaf(w.x, s[0], fmaf(w.y, s[1], fmaf(w.z, s[2], fmaf(w.w, s[3], r[n]))));
             }
-            col[h * kTcRows * kSP] = (a0 + a1) + (a2 + a3);
         }
+        __syncwarp();
+#pragma unroll
+        for (int n = 0; n < 8; ++n)
+            if (part + n * kNP < H) col[(part + n * kNP) * kTcRows * kSP] = r[n];
     };
-
     cp_wait_all();
     __syncthreads();
     scores(0);
@@ -505,7 +537,14 @@ talking_prefill_kernel(const TalkTcArgs A) {
     if (A.kst == 2) load_k(2); else load_k(1);
     cp_commit();
     if (A.kst != 2) { cp_wait_all(); __syncthreads(); }
+    uint32_t voff[4];                                                  // a lane's row and swizzled 16-byte piece of a value tile, for four neighbouring pairs of pieces
+    {
+        const int key = (lane & 7) + ((lane >> 4) << 3);
+#pragma unroll
+        for (int n = 0; n < 4; ++n) voff[n] = (uint32_t)(key * pv + (((n * 2 + ((lane >> 3) & 1)) ^ (key & 7)) << 4));
+    }
     const int pos = pos0 + g, lo = first_visible(pos, A.chunk, A.window);       // of this lane's query in the second product
+    const int lo_last = first_visible(last_pos, A.chunk, A.window);
     for (int i = 0; i < ntiles; ++i) {
         if (i + 1 < ntiles) scores(i + 1);
         mix(i & 1);
@@ -517,6 +556,8 @@ talking_prefill_kernel(const TalkTcArgs A) {
         cp_commit();
         const float* Sd = S + (i & 1) * sstage;
         uint32_t pb[kHW][kMT][2];
+        const int jt = key0 + i * kKT;
+        const bool whole = jt + kKT - 1 <= pos0 && jt >= lo_last;      // every key of the tile is seen by every row
 #pragma unroll
         for (int a = 0; a < kHW; ++a) {
             if (h0 + a >= H) continue;
@@ -527,10 +568,11 @@ talking_prefill_kernel(const TalkTcArgs A) {
             for (int mt = 0; mt < kMT; ++mt) {
                 const float2 x = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t), y = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t + 8);
                 v[mt][0] = x.x; v[mt][1] = x.y; v[mt][2] = y.x; v[mt][3] = y.y;
+                if (!A.talk) { v[mt][0] *= A.scale_log2; v[mt][1] *= A.scale_log2; v[mt][2] *= A.scale_log2; v[mt][3] *= A.scale_log2; }      // else in the matrix
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int j = j0 + mt * 16 + (e >> 1) * 8 + (e & 1);
-                    if (j < lo || j > pos) v[mt][e] = -INFINITY;
+                    if (!whole && (j < lo || j > pos)) v[mt][e] = -INFINITY;
                     mx = fmaxf(mx, v[mt][e]);
                 }
             }
@@ -547,25 +589,26 @@ talking_prefill_kernel(const TalkTcArgs A) {
                 pb[a][mt][0] = pack_bf16(p0, p1); pb[a][mt][1] = pack_bf16(p2, p3);
             }
             l[a] = fmaf(l[a], corr, sum);
-            const float c0 = __shfl_sync(0xffffffffu, corr, 8 * t), c1 = __shfl_sync(0xffffffffu, corr, 8 * t + 4);      // of the accumulators' queries 2t, 2t + 1
+            if (__any_sync(0xffffffffu, corr != 1.f)) {                // some row's maximum has moved
+                const float c0 = __shfl_sync(0xffffffffu, corr, 8 * t), c1 = __shfl_sync(0xffffffffu, corr, 8 * t + 4);      // of the accumulators' queries 2t, 2t + 1
 #pragma unroll
-            for (int n = 0; n < 8; ++n) { o[a][n][0] *= c0; o[a][n][1] *= c1; o[a][n][2] *= c0; o[a][n][3] *= c1; }
+                for (int n = 0; n < 8; ++n) { o[a][n][0] *= c0; o[a][n][1] *= c1; o[a][n][2] *= c0; o[a][n][3] *= c1; }
+            }
         }
         const uint32_t vb = sV + (A.vst == 2 ? (i & 1) * vbytes : 0);
 #pragma unroll
         for (int mt = 0; mt < kMT; ++mt) {
-            const int key = mt * 16 + (lane & 7) + ((lane >> 4) << 3);
 #pragma unroll
             for (int n = 0; n < 8; ++n) {
                 if (n * 16 >= dv) break;
-                const uint32_t piece = (uint32_t)((n * 2 + ((lane >> 3) & 1)) ^ (key & 7));
+                const uint32_t off = voff[n & 3] + (n >> 2) * 128 + mt * 16 * pv;
                 uint32_t va[4];
                 int kv_loaded = -1;
 #pragma unroll
                 for (int a = 0; a < kHW; ++a) {
                     if (h0 + a >= H) continue;
-                    const int kv = (h0 + a) / group;
-                    if (kv != kv_loaded) { kv_loaded = kv; ldsm_x4_trans(va, vb + (kv * kKT + key) * A.pv + piece * 16); }
+                    const int kv = kvh[a];
+                    if (kv != kv_loaded) { kv_loaded = kv; ldsm_x4_trans(va, vb + kv * kKT * pv + off); }
                     mma_bf16(o[a][n], va[0], va[1], va[2], va[3], pb[a][mt][0], pb[a][mt][1]);
                 }
             }
@@ -619,18 +662,24 @@ struct TcPlan { int hw, kt, kst, vst, pk, pv; size_t smem; };
 TcPlan tc_plan(int H, int G, int dk, int dv) {
     TcPlan none{0, 0, 0, 0, 0, 0, 0};
     if (H > 32 || H % G || dk % 8 || dv % 16 || dv > 128 || dk > 256 || (int64_t)G * (dk > dv ? dk : dv) / 8 > 1024) return none;
-    const int hw = H <= 8 ? 1 : H <= 16 ? 2 : 4;
+    const int hw = H <= 16 ? 1 : 2, Hp = (H + 3) / 4 * 4;
     const int pk = (dk * 2 + 127) / 128 * 128, pv = (dv * 2 + 127) / 128 * 128;
     const int tries[6][3] = {{32, 2, 2}, {32, 2, 1}, {16, 2, 2}, {16, 2, 1}, {32, 1, 1}, {16, 1, 1}};
     for (const auto& c : tries) {
-        if (hw == 4 && c[0] != 16) continue;
-        size_t b = (size_t)H * kTcRows * pk + (size_t)c[1] * G * c[0] * pk + (size_t)c[2] * G * c[0] * pv + (size_t)2 * H * kTcRows * (c[0] + 4) * 4 +
-                   (size_t)H * ((H + 3) / 4 * 4) * 4;
-        const size_t outb = (size_t)8 * kTcRows * ((dv + 31) / 32 * 32 + 4) * 4;
+        if (hw == 2 && c[0] != 16) continue;                          // the registers of two heads per warp hold one 16-key piece of scores
+        size_t b = (size_t)H * kTcRows * pk + (size_t)c[1] * G * c[0] * pk + (size_t)c[2] * G * c[0] * pv + (size_t)2 * Hp * kTcRows * (c[0] + 4) * 4 +
+                   (size_t)8 * (kTcThreads / (kTcRows * c[0])) * (Hp + 4) * 4;
+        const size_t outb = (size_t)kTcWarps * kTcRows * ((dv + 31) / 32 * 32 + 4) * 4;
         if (b < outb) b = outb;
         if (b <= 227 * 1024) return TcPlan{hw, c[0], c[1], c[2], pk, pv, b};
     }
     return none;
+}
+
+int block_shift(int bs) {
+    for (int i = 0; i < 20; ++i)
+        if (bs == 1 << i) return i;
+    return -1;
 }
 
 template <typename TC, typename TOut>
@@ -667,7 +716,7 @@ void talking_attention_rows(void* out, const float* q, const void* key_cache, co
                  splits >= 1 && splits <= 65535 && (splits == 1 || part), kErrBadArg, "talking_attention_rows: bad sizes (an even value size; scratch for more than one run)");
     B200_REQUIRE(num_heads <= 64 && dv <= 256 && dk <= 1024, kErrUnsupported, "talking_attention_rows: %d heads > 64, value size %d > 256 or key size %d > 1024", num_heads, dv, dk);
     TalkArgs A{q, key_cache, value_cache, block_tables, table_width, token_seq, positions, talk, v_cos, v_sin, out, part, num_heads, num_kv_heads, dk, dv, block_size,
-               scale, chunk, window, one_sink, splits, 32, 0};
+               scale, chunk, window, one_sink, splits, 32, 0, block_shift(block_size)};
     const int subs = num_kv_heads >= 8 ? 1 : num_kv_heads >= 4 ? 2 : 4;                 // 32-key pieces per tile: work for eight warps
     A.tile = 32 * subs;
     const int span = cache_dtype == B200_F32 ? 16 : 32;                                 // entries four lanes take at a time
@@ -710,14 +759,15 @@ void talking_attention_prefill(void* out, const void* q, const void* key_cache, 
                  "talking_attention_prefill: %d / %d heads of %d / %d (at most 32 heads, dk a multiple of 8, dv of 16 and <= 128)", num_heads, num_kv_heads, dk, dv);
     TalkTcArgs A{(const __nv_bfloat16*)q, (const __nv_bfloat16*)key_cache, (const __nv_bfloat16*)value_cache, block_tables, table_width, cu_seqlens_q, cu_seqlens_k,
                  num_seqs, talk, v_cos, v_sin, (__nv_bfloat16*)out, num_heads, num_kv_heads, dk, dv, block_size, scale * 1.4426950408889634f, chunk, window, one_sink,
-                 P.kst, P.vst, P.pk, P.pv};
+                 P.kst, P.vst, P.pk, P.pv, block_shift(block_size)};
     cudaStream_t st = as_stream(stream);
     const dim3 grid((unsigned)(num_tokens / kTcRows + num_seqs));
-#define TTC(HW, KT) do { ensure_dynamic_smem((const void*)talking_prefill_kernel<HW, KT>, (int)P.smem); \
-        launch_pdl(talking_prefill_kernel<HW, KT>, grid, dim3(256), P.smem, st, A); } while (0)
+#define TTC3(HW, KT, W) do { ensure_dynamic_smem((const void*)talking_prefill_kernel<HW, KT, W>, (int)P.smem); \
+        launch_pdl(talking_prefill_kernel<HW, KT, W>, grid, dim3(kTcThreads), P.smem, st, A); } while (0)
+#define TTC(HW, KT) do { if (dk == 128 && dv == 128) TTC3(HW, KT, true); else TTC3(HW, KT, false); } while (0)
     if (P.hw == 1) { if (P.kt == 32) TTC(1, 32); else TTC(1, 16); }
-    else if (P.hw == 2) { if (P.kt == 32) TTC(2, 32); else TTC(2, 16); }
-    else TTC(4, 16);
+    else TTC(2, 16);
+#undef TTC3
 #undef TTC
     count_launch();
     check_launch("talking_attention_prefill");
