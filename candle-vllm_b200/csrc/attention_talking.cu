@@ -9,6 +9,7 @@
 //   talking_rows_kernel     a block per (row, run of keys), f32 arithmetic, any sizes, f32 or bf16 cache: scores (a warp per kv head and 32 keys, four lanes
 //                           share a key's row in 16-byte pieces), mixing and online softmax (a warp per head, a lane per key), values (a warp per run of
 //                           heads, lanes across the columns).  Few rows: the keys of a row are cut into runs and talking_merge_kernel joins them.
+//   talking_decode_kernel   the same for few rows over a 16-bit cache, on mma.sync: every head gets a mixed query as long as a cache row.
 //   talking_prefill_kernel  portions of prompts in 16 bits: a block per 8 query rows with ALL heads, mma.sync m16n8k16 with keys (or value columns) on the
 //                           16-row side and queries on the 8-column side, so that 32 heads' accumulators of 128 value columns fit the register file.  A warp
 //                           owns H / 16 heads in both products; raw scores meet in shared memory, a thread mixes one (query, key) pair over all heads in
@@ -47,29 +48,31 @@ __device__ __forceinline__ int first_visible(int pos, int chunk, int window) {
     return lo;
 }
 
-template <typename TC> struct Piece;             // a 16-byte piece of a cached row as floats
+template <typename TC> struct Piece;             // a 16-byte piece of a cached row as floats, and four neighbouring entries of one
 template <> struct Piece<float> {
     static constexpr int N = 4;
-    static __device__ __forceinline__ void load(const float* p, float (&v)[4]) { const float4 r = *reinterpret_cast<const float4*>(p); v[0] = r.x; v[1] = r.y; v[2] = r.z; v[3] = r.w; }
+    static __device__ __forceinline__ void open(const uint4& r, float (&v)[4]) {
+        v[0] = __uint_as_float(r.x); v[1] = __uint_as_float(r.y); v[2] = __uint_as_float(r.z); v[3] = __uint_as_float(r.w);
+    }
+    typedef float4 Four;
+    static __device__ __forceinline__ float4 four(const float4& w) { return w; }
 };
 template <> struct Piece<__nv_bfloat16> {
     static constexpr int N = 8;
-    static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[8]) {
-        const uint4 r = *reinterpret_cast<const uint4*>(p);
+    static __device__ __forceinline__ void open(const uint4& r, float (&v)[8]) {
         const uint32_t w[4] = {r.x, r.y, r.z, r.w};
 #pragma unroll
         for (int i = 0; i < 4; ++i) { v[2 * i] = __uint_as_float(w[i] << 16); v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
     }
+    typedef uint2 Four;
+    static __device__ __forceinline__ float4 four(const uint2& w) {
+        return make_float4(__uint_as_float(w.x << 16), __uint_as_float(w.x & 0xffff0000u), __uint_as_float(w.y << 16), __uint_as_float(w.y & 0xffff0000u));
+    }
 };
-__device__ __forceinline__ float2 load_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
-__device__ __forceinline__ float2 load_pair(const __nv_bfloat16* p) {
-    const uint32_t w = *reinterpret_cast<const uint32_t*>(p);
-    return make_float2(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u));
-}
 
-// kHW: heads a warp accumulates values for, kC: pairs of value columns per lane (columns 2 lane + 64 c and the next)
+// kHW: heads a warp accumulates values for, kC: groups of four value columns per lane (columns 4 lane + 128 c and the next three)
 template <typename TC, typename TOut, int kHW, int kC>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, kHW * kC <= 2 ? 2 : 1)
 talking_rows_kernel(const TalkArgs A) {
     pdl_wait();
     pdl_trigger();
@@ -117,12 +120,12 @@ talking_rows_kernel(const TalkArgs A) {
     int kvh[kHW];                                // their kv heads
 #pragma unroll
     for (int a = 0; a < kHW; ++a) kvh[a] = min(h0 + a, H - 1) / group;
-    float2 acc[kHW][kC];
+    float4 acc[kHW][kC];
 #pragma unroll
     for (int a = 0; a < kHW; ++a)
 #pragma unroll
-        for (int c = 0; c < kC; ++c) acc[a][c] = make_float2(0.f, 0.f);
-    const bool whole = dk % N == 0;              // rows are whole 16-byte pieces
+        for (int c = 0; c < kC; ++c) acc[a][c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    const bool whole = dk % N == 0, fours = dv % 4 == 0;               // key rows are whole 16-byte pieces, value rows whole groups of four
     __syncthreads();
     for (int j0 = jb, it = 0; j0 < je; j0 += KT, ++it) {
         const int64_t* pht = ph + (it & 1) * KT;
@@ -136,21 +139,24 @@ talking_rows_kernel(const TalkArgs A) {
             for (int i = 0; i < 4; ++i) kp[i] = kc + (pht[sub * 32 + i * 8 + r] * G + g) * dk;
             for (int hb = 0; hb < group; hb += 4) {
                 float a[4][4] = {};
+                uint4 nx[4];                     // the next pieces travel while these are multiplied
+#pragma unroll
+                for (int i = 0; i < 4; ++i) nx[i] = whole && c4 * N < dk ? *reinterpret_cast<const uint4*>(kp[i] + c4 * N) : make_uint4(0u, 0u, 0u, 0u);
                 for (int d0 = 0; d0 < dk; d0 += 4 * N) {
                     const int d = d0 + c4 * N;
                     float kv[4][N];
+                    if (whole) {
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        if (whole) {
-                            if (d < dk) Piece<TC>::load(kp[i] + d, kv[i]);
-                            else {
+                        for (int i = 0; i < 4; ++i) Piece<TC>::open(nx[i], kv[i]);
+                        if (d0 + 4 * N < dk) {
 #pragma unroll
-                                for (int e = 0; e < N; ++e) kv[i][e] = 0.f;
-                            }
-                        } else {
+                            for (int i = 0; i < 4; ++i) nx[i] = d + 4 * N < dk ? *reinterpret_cast<const uint4*>(kp[i] + d + 4 * N) : make_uint4(0u, 0u, 0u, 0u);
+                        }
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i)
 #pragma unroll
                             for (int e = 0; e < N; ++e) kv[i][e] = d + e < dk ? to_f32<TC>(kp[i][d + e]) : 0.f;
-                        }
                     }
 #pragma unroll
                     for (int hh = 0; hh < 4; ++hh) {
@@ -226,35 +232,55 @@ talking_rows_kernel(const TalkArgs A) {
             for (int a = 0; a < kHW; ++a) {
                 const float corr = h0 + a < H ? cs[h0 + a] : 0.f;
 #pragma unroll
-                for (int c = 0; c < kC; ++c) { acc[a][c].x *= corr; acc[a][c].y *= corr; }
+                for (int c = 0; c < kC; ++c) { acc[a][c].x *= corr; acc[a][c].y *= corr; acc[a][c].z *= corr; acc[a][c].w *= corr; }
             }
-            for (int k4 = slice * 4; k4 < nsub * 32; k4 += slices * 4) {
-                if (j0 + k4 >= je) break;
-                float4 p4[kHW];
-#pragma unroll
-                for (int a = 0; a < kHW; ++a) p4[a] = h0 + a < H ? *reinterpret_cast<const float4*>(P + (h0 + a) * KT + k4) : make_float4(0.f, 0.f, 0.f, 0.f);
+            // eight keys at a time: their rows travel together (rows past the run's end repeat its first one, at weight 0)
+            for (int k8 = slice * 8; k8 < nsub * 32; k8 += slices * 8) {
+                if (j0 + k8 >= je) break;
                 int g_loaded = -1;
-                float2 vv[4][kC];
+                float4 vv[8][kC];
 #pragma unroll
                 for (int a = 0; a < kHW; ++a) {
                     const int g = kvh[a];
                     if (g != g_loaded) {
                         g_loaded = g;
+                        if (fours) {                 // all loads first, clamped instead of guarded: columns past dv are not stored
+                            typename Piece<TC>::Four raw[8][kC];
 #pragma unroll
-                        for (int i = 0; i < 4; ++i) {
-                            const TC* vp = vc + (pht[k4 + i] * G + g) * dv;
+                            for (int i = 0; i < 8; ++i)
 #pragma unroll
-                            for (int c = 0; c < kC; ++c) {
-                                const int col = 2 * lane + 64 * c;
-                                vv[i][c] = col < dv ? load_pair(vp + col) : make_float2(0.f, 0.f);
+                                for (int c = 0; c < kC; ++c)
+                                    raw[i][c] = *reinterpret_cast<const typename Piece<TC>::Four*>(vc + (pht[k8 + i] * G + g) * dv + min(4 * lane + 128 * c, dv - 4));
+#pragma unroll
+                            for (int i = 0; i < 8; ++i)
+#pragma unroll
+                                for (int c = 0; c < kC; ++c) vv[i][c] = Piece<TC>::four(raw[i][c]);
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) {
+                                const TC* vp = vc + (pht[k8 + i] * G + g) * dv;
+#pragma unroll
+                                for (int c = 0; c < kC; ++c) {
+                                    const int col = 4 * lane + 128 * c;
+                                    vv[i][c] = make_float4(col < dv ? to_f32<TC>(vp[col]) : 0.f, col + 1 < dv ? to_f32<TC>(vp[col + 1]) : 0.f,
+                                                           col + 2 < dv ? to_f32<TC>(vp[col + 2]) : 0.f, col + 3 < dv ? to_f32<TC>(vp[col + 3]) : 0.f);
+                                }
                             }
                         }
                     }
-                    const float p[4] = {p4[a].x, p4[a].y, p4[a].z, p4[a].w};
 #pragma unroll
-                    for (int i = 0; i < 4; ++i)
+                    for (int i4 = 0; i4 < 2; ++i4) {
+                        const float4 p4 = h0 + a < H ? *reinterpret_cast<const float4*>(P + (h0 + a) * KT + k8 + 4 * i4) : make_float4(0.f, 0.f, 0.f, 0.f);
+                        const float p[4] = {p4.x, p4.y, p4.z, p4.w};
 #pragma unroll
-                        for (int c = 0; c < kC; ++c) { acc[a][c].x = fmaf(p[i], vv[i][c].x, acc[a][c].x); acc[a][c].y = fmaf(p[i], vv[i][c].y, acc[a][c].y); }
+                        for (int i = 0; i < 4; ++i)
+#pragma unroll
+                            for (int c = 0; c < kC; ++c) {
+                                const float4 v = vv[4 * i4 + i][c];
+                                acc[a][c].x = fmaf(p[i], v.x, acc[a][c].x); acc[a][c].y = fmaf(p[i], v.y, acc[a][c].y);
+                                acc[a][c].z = fmaf(p[i], v.z, acc[a][c].z); acc[a][c].w = fmaf(p[i], v.w, acc[a][c].w);
+                            }
+                    }
                 }
             }
         }
@@ -268,8 +294,10 @@ talking_rows_kernel(const TalkArgs A) {
             if (h0 + a >= H) continue;
 #pragma unroll
             for (int c = 0; c < kC; ++c) {
-                const int col = 2 * lane + 64 * c;
-                if (col < dv) *reinterpret_cast<float2*>(O + (slice * H + h0 + a) * dv + col) = acc[a][c];
+                const int col = 4 * lane + 128 * c;
+                float* dst = O + (slice * H + h0 + a) * dv + col;
+                if (col < dv) *reinterpret_cast<float2*>(dst) = make_float2(acc[a][c].x, acc[a][c].y);
+                if (col + 2 < dv) *reinterpret_cast<float2*>(dst + 2) = make_float2(acc[a][c].z, acc[a][c].w);
             }
         }
     }
@@ -349,13 +377,9 @@ constexpr int kTcRows = 8, kTcWarps = 16, kTcThreads = kTcWarps * 32;        // 
 __device__ __forceinline__ void cp16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void cp_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
-__device__ __forceinline__ uint4 lds16(uint32_t a) {
-    uint4 v;
-    asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "r"(a));
-    return v;
-}
 __device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+    // not volatile: a pure function of its operands, which the compiler may move between the loads that feed it
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
@@ -390,6 +414,7 @@ talking_prefill_kernel(const TalkTcArgs A) {
 
     const int kbytes = G * kKT * pk, vbytes = G * kKT * pv;
     const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(smem_tc);
+    auto lds16 = [&](uint32_t a) { return *reinterpret_cast<const uint4*>(smem_tc + (a - sbase)); };
     const uint32_t sQ = sbase, sK = sQ + H * kTcRows * pk, sV = sK + A.kst * kbytes;
     float* S = reinterpret_cast<float*>(smem_tc + (sV - sbase) + A.vst * vbytes);                   // [2][Hp][8][kSP]
     const int Hp = (H + 3) & ~3, tp = Hp + 4;                          // heads rounded up to whole groups of four (rows of zeros); row pitch of the mixing matrix
@@ -676,6 +701,221 @@ TcPlan tc_plan(int H, int G, int dk, int dv) {
     return none;
 }
 
+// ---- few rows in 16 bits on tensor cores --------------------------------------------------------------------------------------------------------
+// A row alone needs no exchange of scores: mixing commutes with the product, s'[h, j] = (sum_g talk[h, g] q[g]) . k_j summed kv head by kv head, so every head gets
+// one mixed query as long as a whole cache row, q'[h] = (talk[h, g] q[g] summed over the heads g of each kv head), and the scores of all heads are one product of
+// q' [H, G dk] with the cache rows.  A block per (row, run of keys), eight warps, 64 keys per tile: a warp scores eight keys (cache rows read straight into the operand
+// layout, four lanes per row in 16-byte pieces), a warp per head takes the online softmax, and a warp multiplies the weights of one kv head's heads with 64 value
+// columns (eight neighbouring columns per lane from four rows, paired in registers; the column order of the product is a permutation undone at the store).
+constexpr int kDecTile = 64, kDecSP = kDecTile + 4, kDecPP = kDecTile + 8;      // keys per tile, pitches of a score row (f32) and of a weight row (bf16)
+constexpr int kDecHead = 2 * kDecTile * 8 + 96 * 4;                             // bytes ahead of the queries: a multiple of 128
+
+template <int kMT, int kU>                       // 16-head tiles, (kv head, 64 columns) units per warp
+__global__ void __launch_bounds__(256, 2)
+talking_decode_kernel(const TalkArgs A) {
+    pdl_wait();
+    pdl_trigger();
+    extern __shared__ __align__(128) uint8_t smem_dec[];
+    const int H = A.H, G = A.G, dk = A.dk, dv = A.dv, group = H / G, row = G * dk, pq = (row * 2 + 127) / 128 * 128;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    int64_t* ph = reinterpret_cast<int64_t*>(smem_dec);                      // [2][64] cache rows of the tile's keys
+    float* cs = reinterpret_cast<float*>(ph + 2 * kDecTile);                 // [32] correction of this tile, [32] maxima (base 2), [32] denominators
+    float* ms = cs + 32; float* ls = ms + 32;
+    uint8_t* qm = smem_dec + kDecHead;                                       // [16 kMT][pq] mixed queries, 16-byte pieces swizzled
+    float* S = reinterpret_cast<float*>(qm + 16 * kMT * pq);                 // [16 kMT][kDecSP]
+    __nv_bfloat16* P = reinterpret_cast<__nv_bfloat16*>(S + 16 * kMT * kDecSP);       // [H + 16][kDecPP]
+    const int tok = blockIdx.x, split = blockIdx.y;
+    const int pos = A.positions[tok];
+    const int lo = first_visible(pos, A.chunk, A.window);
+    const int per = ((pos - lo + A.splits) / A.splits + kDecTile - 1) / kDecTile * kDecTile;
+    const int jb = lo + split * per, je = min(pos + 1, jb + per);
+    const int32_t* table = A.block_tables + (int64_t)A.token_seq[tok] * A.table_width;
+    const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(A.kc);
+    const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(A.vc);
+    auto place = [&](int j0, int buf) {          // keys past the run's end stand for its first one (their weight is 0, what they read is finite)
+        if (threadIdx.x < kDecTile) {
+            const int j = j0 + threadIdx.x < je ? j0 + threadIdx.x : jb;
+            ph[buf * kDecTile + threadIdx.x] = cache_row(table, j, A.bs, A.bs_shift);
+        }
+    };
+    const float scale_log2 = A.scale * 1.4426950408889634f;
+    if (jb < je) {
+        place(jb, 0);
+        // a thread makes 16-byte pieces of the mixed queries: eight neighbouring entries of one head
+        for (int i = threadIdx.x; i < 16 * kMT * (row >> 3); i += 256) {
+            const int h = i / (row >> 3), c = i - h * (row >> 3);
+            const int kv = c * 8 / dk, d = c * 8 - kv * dk;
+            float v[8] = {};
+            if (h < H)
+                for (int e = 0; e < group; ++e) {
+                    const int x = kv * group + e;
+                    const float w = (A.talk ? A.talk[h * H + x] : (x == h ? 1.f : 0.f)) * scale_log2;
+                    const float4* q4 = reinterpret_cast<const float4*>(A.q + ((int64_t)tok * H + x) * dk + d);
+                    const float4 a = q4[0], b = q4[1];
+                    v[0] = fmaf(w, a.x, v[0]); v[1] = fmaf(w, a.y, v[1]); v[2] = fmaf(w, a.z, v[2]); v[3] = fmaf(w, a.w, v[3]);
+                    v[4] = fmaf(w, b.x, v[4]); v[5] = fmaf(w, b.y, v[5]); v[6] = fmaf(w, b.z, v[6]); v[7] = fmaf(w, b.w, v[7]);
+                }
+            *reinterpret_cast<uint4*>(qm + h * pq + ((c ^ ((h & 1) << 2)) << 4)) =
+                make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+        }
+    }
+    if (threadIdx.x < 32) {
+        const bool sink = A.one_sink && split == 0;                          // a key of score 0 without a value, counted by the first run
+        ms[threadIdx.x] = sink ? 0.f : -INFINITY;
+        ls[threadIdx.x] = sink ? 1.f : 0.f;
+    }
+    const int cols = (dv + 63) / 64, units = G * cols;
+    float o[kU][8][4];
+#pragma unroll
+    for (int u = 0; u < kU; ++u)
+#pragma unroll
+        for (int n = 0; n < 8; ++n) o[u][n][0] = o[u][n][1] = o[u][n][2] = o[u][n][3] = 0.f;
+    int ukv[kU], ucol[kU];                       // kv head and first column of this lane's eight
+#pragma unroll
+    for (int u = 0; u < kU; ++u) { const int x = warp + 8 * u; ukv[u] = x < units ? x / cols : -1; ucol[u] = (x % cols) * 64 + g * 8; }
+    __syncthreads();
+    const int nblk = row / 32;
+    const uint8_t* qrow = qm + g * pq + (((uint32_t)t ^ ((g & 1) << 2)) << 4);       // piece t of an even 32-entry part; the odd parts' lie 64 bytes away
+    const int odd = (g & 1) ? -64 : 64;
+    for (int j0 = jb, it = 0; j0 < je; j0 += kDecTile, ++it) {
+        const int64_t* pht = ph + (it & 1) * kDecTile;
+        // ---- scores of eight keys ------------------------------------------------------------------------------------------------------------
+        if (j0 + warp * 8 < je) {
+            const uint4* kr = reinterpret_cast<const uint4*>(kc + pht[warp * 8 + g] * row) + t;
+            float acc[kMT][4] = {};
+            uint4 nx[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) nx[i] = kr[min(i, nblk - 1) * 4];
+            for (int b = 0; b < nblk; b += 4) {
+                uint4 cur[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) { cur[i] = nx[i]; nx[i] = kr[min(b + 4 + i, nblk - 1) * 4]; }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    if (b + i >= nblk) break;
+                    const uint8_t* qa = qrow + ((b + i) >> 1) * 128 + (((b + i) & 1) ? odd : 0);
+#pragma unroll
+                    for (int mt = 0; mt < kMT; ++mt) {
+                        const uint4 x = *reinterpret_cast<const uint4*>(qa + mt * 16 * pq), y = *reinterpret_cast<const uint4*>(qa + (mt * 16 + 8) * pq);
+                        mma_bf16(acc[mt], x.x, y.x, x.y, y.y, cur[i].x, cur[i].y);
+                        mma_bf16(acc[mt], x.z, y.z, x.w, y.w, cur[i].z, cur[i].w);
+                    }
+                }
+            }
+#pragma unroll
+            for (int mt = 0; mt < kMT; ++mt) {
+                *reinterpret_cast<float2*>(S + (mt * 16 + g) * kDecSP + warp * 8 + 2 * t) = make_float2(acc[mt][0], acc[mt][1]);
+                *reinterpret_cast<float2*>(S + (mt * 16 + g + 8) * kDecSP + warp * 8 + 2 * t) = make_float2(acc[mt][2], acc[mt][3]);
+            }
+        }
+        // the first half of the tile's values travels during the softmax: rows 2t, 2t + 1, 2t + 8, 2t + 9 of two sets of sixteen keys
+        uint4 vr[2][4];
+        auto fetch_v = [&](int u, int ks, uint4 (&d)[4]) {
+            const bool ok = ukv[u] >= 0 && ucol[u] < dv;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int key = ks * 16 + 2 * t + (e & 1) + (e >> 1) * 8;
+                d[e] = ok ? *reinterpret_cast<const uint4*>(vc + (pht[key] * G + ukv[u]) * dv + ucol[u]) : make_uint4(0u, 0u, 0u, 0u);
+            }
+        };
+        fetch_v(0, 0, vr[0]);
+        fetch_v(0, 1, vr[1]);
+        __syncthreads();
+        // ---- online softmax, a warp per head ----------------------------------------------------------------------------------------------------
+        for (int h = warp; h < H; h += 8) {
+            float a = j0 + lane < je ? S[h * kDecSP + lane] : -INFINITY, b = j0 + 32 + lane < je ? S[h * kDecSP + 32 + lane] : -INFINITY;
+            const float m_old = ms[h], m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
+            a = exp2f(a - m_new); b = exp2f(b - m_new);
+            P[h * kDecPP + lane] = __float2bfloat16_rn(a);
+            P[h * kDecPP + 32 + lane] = __float2bfloat16_rn(b);
+            const float sum = warp_sum(a + b);
+            __syncwarp();
+            if (lane == 0) {
+                const float corr = exp2f(m_old - m_new);
+                cs[h] = corr; ms[h] = m_new;
+                ls[h] = fmaf(ls[h], corr, sum);
+            }
+        }
+        if (j0 + kDecTile < je) place(j0 + kDecTile, (it + 1) & 1);
+        __syncthreads();
+        // ---- values -----------------------------------------------------------------------------------------------------------------------------
+#pragma unroll
+        for (int u = 0; u < kU; ++u) {
+            if (ukv[u] < 0) continue;
+            const int hb = ukv[u] * group;
+            const float c0 = g < group ? cs[hb + g] : 0.f, c1 = g + 8 < group ? cs[hb + g + 8] : 0.f;
+#pragma unroll
+            for (int n = 0; n < 8; ++n) { o[u][n][0] *= c0; o[u][n][1] *= c0; o[u][n][2] *= c1; o[u][n][3] *= c1; }
+            if (u > 0) { fetch_v(u, 0, vr[0]); fetch_v(u, 1, vr[1]); }
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks) {
+                if (j0 + ks * 16 >= je) break;
+                const __nv_bfloat16* p0 = P + (hb + g) * kDecPP + ks * 16 + 2 * t;       // rows past the group belong to other heads: their products are not stored
+                const __nv_bfloat16* p1 = p0 + 8 * kDecPP;
+                const uint32_t a0 = *reinterpret_cast<const uint32_t*>(p0), a2 = *reinterpret_cast<const uint32_t*>(p0 + 8);
+                const uint32_t a1 = *reinterpret_cast<const uint32_t*>(p1), a3 = *reinterpret_cast<const uint32_t*>(p1 + 8);
+                uint4 r[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) r[e] = vr[ks & 1][e];
+                if (ks < 2) fetch_v(u, ks + 2, vr[ks & 1]);
+                const uint32_t w[4][4] = {{r[0].x, r[0].y, r[0].z, r[0].w}, {r[1].x, r[1].y, r[1].z, r[1].w}, {r[2].x, r[2].y, r[2].z, r[2].w}, {r[3].x, r[3].y, r[3].z, r[3].w}};
+#pragma unroll
+                for (int n2 = 0; n2 < 4; ++n2) {         // columns 2 n2 and 2 n2 + 1 of the lane's eight: pair the rows' low halves, then their high halves
+                    mma_bf16(o[u][2 * n2], a0, a1, a2, a3, __byte_perm(w[0][n2], w[1][n2], 0x5410), __byte_perm(w[2][n2], w[3][n2], 0x5410));
+                    mma_bf16(o[u][2 * n2 + 1], a0, a1, a2, a3, __byte_perm(w[0][n2], w[1][n2], 0x7632), __byte_perm(w[2][n2], w[3][n2], 0x7632));
+                }
+            }
+        }
+    }
+    __syncthreads();
+    // ---- output or the run's partial result: accumulator n of a lane's queries' columns 2t, 2t + 1 is value column 8 (2t) + n, 8 (2t + 1) + n of its 64 -------------
+    float* O = reinterpret_cast<float*>(qm);                                 // [H][dv]
+#pragma unroll
+    for (int u = 0; u < kU; ++u) {
+        if (ukv[u] < 0) continue;
+        const int base = ucol[u] - g * 8;
+#pragma unroll
+        for (int n = 0; n < 8; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int r = g + (e >> 1) * 8, col = base + 8 * (2 * t + (e & 1)) + n;
+                if (r < group && col < dv) O[(ukv[u] * group + r) * dv + col] = o[u][n][e];
+            }
+    }
+    __syncthreads();
+    const int half = dv >> 1;
+    for (int e = threadIdx.x; e < H * half; e += 256) {
+        const int h = e / half, x = e - h * half;
+        float a = O[h * dv + x], b = O[h * dv + x + half];
+        if (A.splits > 1) {
+            float* pp = A.part + (((int64_t)tok * A.splits + split) * H + h) * (dv + 2);
+            pp[x] = a; pp[x + half] = b;
+            if (x == 0) { pp[dv] = ms[h] * 0.6931471805599453f; pp[dv + 1] = ls[h]; }        // the merge takes natural exponents
+            continue;
+        }
+        const float inv = 1.0f / ls[h];
+        a *= inv; b *= inv;
+        if (A.cos_t) {
+            const float c = A.cos_t[(int64_t)pos * half + x], s = A.sin_t[(int64_t)pos * half + x];
+            const float u = a * c + b * s;
+            b = b * c - a * s; a = u;
+        }
+        __nv_bfloat16* op = static_cast<__nv_bfloat16*>(A.out) + ((int64_t)tok * H + h) * dv;
+        op[x] = __float2bfloat16_rn(a); op[x + half] = __float2bfloat16_rn(b);
+    }
+}
+
+// shared memory of the kernel above for these sizes, 0 when it does not take them
+size_t decode_plan(int H, int G, int dk, int dv) {
+    if (H > 32 || H % G || H / G > 16 || (G * dk) % 32 || dk % 8 || dv % 8 || G * ((dv + 63) / 64) > 16) return 0;
+    const int mt = (H + 15) / 16, pq = (G * dk * 2 + 127) / 128 * 128;
+    size_t b = (size_t)16 * mt * pq + (size_t)16 * mt * kDecSP * 4 + (size_t)(H + 16) * kDecPP * 2;
+    const size_t outb = (size_t)H * dv * 4;
+    if (b < outb) b = outb;
+    b += kDecHead;
+    return b <= 110 * 1024 ? b : 0;              // two blocks per SM
+}
+
 int block_shift(int bs) {
     for (int i = 0; i < 20; ++i)
         if (bs == 1 << i) return i;
@@ -684,11 +924,11 @@ int block_shift(int bs) {
 
 template <typename TC, typename TOut>
 bool launch_rows(const TalkArgs& A, int T, size_t smem, cudaStream_t st) {
-    const int hw = (A.H + 7) / 8, pairs = (A.dv + 63) / 64;
+    const int hw = (A.H + 7) / 8;
     const dim3 grid(T, A.splits);
 #define TR(HW, CC) do { ensure_dynamic_smem((const void*)talking_rows_kernel<TC, TOut, HW, CC>, (int)smem); \
         launch_pdl(talking_rows_kernel<TC, TOut, HW, CC>, grid, dim3(256), smem, st, A); return true; } while (0)
-#define TRC(HW) do { if (pairs == 1) TR(HW, 1); if (pairs == 2) TR(HW, 2); if (pairs <= 4) TR(HW, 4); return false; } while (0)
+#define TRC(HW) do { if (A.dv <= 128) TR(HW, 1); if (A.dv <= 256) TR(HW, 2); return false; } while (0)
     if (hw == 1) TRC(1);
     if (hw == 2) TRC(2);
     if (hw <= 4) TRC(4);
@@ -708,13 +948,15 @@ extern "C" {
 void talking_attention_rows(void* out, const float* q, const void* key_cache, const void* value_cache, const int32_t* block_tables, int32_t table_width,
                             const int32_t* token_seq, const int32_t* positions, const float* talk, const float* v_cos, const float* v_sin, int32_t num_tokens,
                             int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t block_size, float scale, int32_t chunk, int32_t window,
-                            int32_t one_sink, int32_t splits, float* part, int32_t cache_dtype, int32_t out_dtype, int64_t stream) {
+                            int32_t one_sink, int32_t splits, float* part, int32_t plain, int32_t cache_dtype, int32_t out_dtype, int64_t stream) {
     if (num_tokens == 0) return;
     B200_REQUIRE(out && q && key_cache && value_cache && block_tables && token_seq && positions && (v_cos == nullptr) == (v_sin == nullptr), kErrBadArg,
                  "talking_attention_rows: null pointer");
     B200_REQUIRE(num_heads > 0 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && dk > 0 && dv > 0 && dv % 2 == 0 && block_size > 0 && table_width > 0 &&
                  splits >= 1 && splits <= 65535 && (splits == 1 || part), kErrBadArg, "talking_attention_rows: bad sizes (an even value size; scratch for more than one run)");
     B200_REQUIRE(num_heads <= 64 && dv <= 256 && dk <= 1024, kErrUnsupported, "talking_attention_rows: %d heads > 64, value size %d > 256 or key size %d > 1024", num_heads, dv, dk);
+    const size_t dec_smem = cache_dtype == B200_BF16 && out_dtype == B200_BF16 && plain == 0 && (((uintptr_t)q | (uintptr_t)key_cache | (uintptr_t)value_cache) & 15) == 0
+                                ? decode_plan(num_heads, num_kv_heads, dk, dv) : 0;
     TalkArgs A{q, key_cache, value_cache, block_tables, table_width, token_seq, positions, talk, v_cos, v_sin, out, part, num_heads, num_kv_heads, dk, dv, block_size,
                scale, chunk, window, one_sink, splits, 32, 0, block_shift(block_size)};
     const int subs = num_kv_heads >= 8 ? 1 : num_kv_heads >= 4 ? 2 : 4;                 // 32-key pieces per tile: work for eight warps
@@ -724,10 +966,19 @@ void talking_attention_rows(void* out, const float* q, const void* key_cache, co
     const int pool = 2 * num_heads * A.tile > (num_heads < 8 ? 8 : num_heads) * dv ? 2 * num_heads * A.tile : (num_heads < 8 ? 8 : num_heads) * dv;
     const size_t floats = (size_t)num_heads * A.qpitch + ((pool + 3) & ~3) + ((3 * num_heads + 3) & ~3) + 4 * (size_t)A.tile + (size_t)num_heads * num_heads;
     const size_t smem = floats * sizeof(float);
-    B200_REQUIRE(smem <= 227 * 1024, kErrUnsupported, "talking_attention_rows: %d heads of key size %d do not fit shared memory", num_heads, dk);
+    B200_REQUIRE(dec_smem > 0 || smem <= 227 * 1024, kErrUnsupported, "talking_attention_rows: %d heads of key size %d do not fit shared memory", num_heads, dk);
     cudaStream_t st = as_stream(stream);
     bool ok = false;
-    if (cache_dtype == B200_F32 && out_dtype == B200_F32) ok = launch_rows<float, float>(A, num_tokens, smem, st);
+    if (dec_smem > 0) {
+        const dim3 grid(num_tokens, splits);
+        const bool two = num_kv_heads * ((dv + 63) / 64) > 8;
+#define TDK(MT, UU) do { ensure_dynamic_smem((const void*)talking_decode_kernel<MT, UU>, (int)dec_smem); \
+        launch_pdl(talking_decode_kernel<MT, UU>, grid, dim3(256), dec_smem, st, A); } while (0)
+        if (num_heads <= 16) { if (two) TDK(1, 2); else TDK(1, 1); }
+        else { if (two) TDK(2, 2); else TDK(2, 1); }
+#undef TDK
+        ok = true;
+    } else if (cache_dtype == B200_F32 && out_dtype == B200_F32) ok = launch_rows<float, float>(A, num_tokens, smem, st);
     else if (cache_dtype == B200_BF16 && out_dtype == B200_BF16) ok = launch_rows<__nv_bfloat16, __nv_bfloat16>(A, num_tokens, smem, st);
     else { set_error(kErrUnsupported, "talking_attention_rows: cache dtype %d / out dtype %d", cache_dtype, out_dtype); return; }
     B200_REQUIRE(ok, kErrUnsupported, "talking_attention_rows: no kernel for %d heads, value size %d", num_heads, dv);

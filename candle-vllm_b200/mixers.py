@@ -635,7 +635,7 @@ class TalkingAttentionMixer:
         self.w_in = torch.cat([w[n] for n in want], 0).to(dtype).contiguous()
         self.talk = w["talk"].float().contiguous() if "talk" in w else None
         self.w_o = w["o"].to(dtype).contiguous()
-        self.splits = None                       # None: chosen by the step's shape (tests force a number)
+        self.splits, self.plain = None, False    # runs of keys chosen by the step's shape, kernels by the sizes (tests force a number / the f32-arithmetic kernel)
         # portions of prompts in 16 bits: the tensor-core kernel, when it takes these sizes
         self.prefill_kernel = ops.talking_prefill_kernel_supported(heads, kv_heads, dk, dv, dtype)
         self.cos = self.sin = self.v_cos = self.v_sin = None
@@ -664,7 +664,7 @@ class TalkingAttentionMixer:
         q = ops.qkv_rope_cache(proj, tables, v_tables, batch, None if self.shared else k_cache, None if self.shared else v_cache, self.H, self.G, self.dk, self.dv,
                                self.rot_dims, self.dtype, torch.bfloat16 if self.prefill_kernel and batch.max_rows >= ops.TALKING_PREFILL_MIN_ROWS else torch.float32)
         a = ops.talking_attention(q, k_cache, v_cache, batch, self.talk, v_tables, self.H, self.scale, self.chunk, self.window, self.one_sink, self.dtype,
-                                  splits=self.splits)
+                                  splits=self.splits, plain=self.plain)
         return ops.linear(a, self.w_o)
 
 

@@ -898,14 +898,15 @@ def talking_prefill_kernel_supported(heads: int, kv_heads: int, dk: int, dv: int
     return dtype == torch.bfloat16 and bool(lib().talking_attention_prefill_supported(C.c_int32(heads), C.c_int32(kv_heads), C.c_int32(dk), C.c_int32(dv)))
 
 
-TALKING_BLOCKS = 444           # three blocks per SM: steps with fewer rows cut the keys of every row into runs
+TALKING_BLOCKS = 296           # two blocks per SM: steps with fewer rows cut the keys of every row into runs
 
 
 def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: StepBatch, talk: Optional[torch.Tensor], value_tables: Optional[tuple], heads: int,
-                      scale: float, chunk: int, window: int, one_sink: bool, out_dtype: torch.dtype, splits: Optional[int] = None) -> torch.Tensor:
+                      scale: float, chunk: int, window: int, one_sink: bool, out_dtype: torch.dtype, splits: Optional[int] = None, plain: bool = False) -> torch.Tensor:
     """Softmax attention whose heads mix their scores by ``talk`` (f32 [H, H]) before the softmax; ``one_sink``: one is added to every denominator; ``value_tables``: the
     cached values were turned by their position and every output is turned back by its own.  q f32 [T, H dk] -> [T, H dv] of ``out_dtype`` (the cache's); a bf16 q
-    takes the tensor-core kernel for portions of prompts (``talking_prefill_kernel_supported``).  ``splits``: runs every row's keys are cut into (None: enough blocks to fill the device, from the table width, so that a captured step keeps its choice)."""
+    takes the tensor-core kernel for portions of prompts (``talking_prefill_kernel_supported``).  ``splits``: runs every row's keys are cut into (None: enough blocks to fill the device, from the table width, so that a captured step keeps its choice);
+    ``plain``: f32 arithmetic over a bf16 cache too."""
     T = q.shape[0]
     nb, bs, G, dk = k_cache.shape
     dv = v_cache.shape[3]
@@ -930,7 +931,7 @@ def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     out = torch.empty((T, heads * dv), dtype=out_dtype, device=q.device)
     lib().talking_attention_rows(_ptr(out), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), C.c_int32(batch.block_tables.shape[1]), _ptr(batch.token_seq),
                                  _ptr(batch.positions), _ptr(talk), _ptr(v_cos), _ptr(v_sin), C.c_int32(T), C.c_int32(heads), C.c_int32(G), C.c_int32(dk), C.c_int32(dv),
-                                 C.c_int32(bs), C.c_float(scale), C.c_int32(chunk), C.c_int32(window), C.c_int32(1 if one_sink else 0), C.c_int32(splits), _ptr(part),
+                                 C.c_int32(bs), C.c_float(scale), C.c_int32(chunk), C.c_int32(window), C.c_int32(1 if one_sink else 0), C.c_int32(splits), _ptr(part), C.c_int32(1 if plain else 0),
                                  C.c_int32(_tag(k_cache.dtype)), C.c_int32(_tag(out_dtype)), _stream(q.device))
     check("talking_attention_rows")
     return out

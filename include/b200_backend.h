@@ -702,7 +702,8 @@ void mla_paged_attention_window(void* out, const void* q_absorbed, const void* q
  * talking_attention_rows: s[h, j] = scale q[t, h] . k_j, s' = talk s (talk f32 [H, H] or null = as they are), p = exp(s') / (one_sink + sum exp(s')), out[t, h] = sum p v_j
  *   turned back by the position's angles of v_cos / v_sin (null = not turned), over the keys with j <= i, j / chunk == i / chunk (chunk > 0), i - j < window (window
  *   > 0).  q f32 [T, H dk]; cache and out F32 or both BF16.  splits > 1: every row's keys are cut into that many runs, part = T * splits * H * (dv + 2) floats.
- *   H <= 64, dv even and <= 256, dk <= 1024.
+ *   H <= 64, dv even and <= 256, dk <= 1024.  A BF16 cache with H <= 32, dk and dv multiples of 8 and at most 16 kv heads x 64-column groups takes a tensor-core
+ *   kernel (plain != 0: not even then).
  * talking_attention_prefill: the same on tensor cores for portions of prompts: q, cache and out BF16, entry b's rows are cu_seqlens_q[b] .. cu_seqlens_q[b + 1] = the
  *   last of its cu_seqlens_k[b + 1] - cu_seqlens_k[b] positions.  talking_attention_prefill_supported: 1 if it takes these sizes (H <= 32, dk a multiple of 8, dv a
  *   multiple of 16 and <= 128, tiles that fit shared memory). */
@@ -722,7 +723,7 @@ void qkv_norm_rope_cache(const float* qkv, int64_t ld, const float* q_norm_w, co
 void talking_attention_rows(void* out, const float* q, const void* key_cache, const void* value_cache, const int32_t* block_tables, int32_t table_width,
                             const int32_t* token_seq, const int32_t* positions, const float* talk, const float* v_cos, const float* v_sin, int32_t num_tokens,
                             int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t block_size, float scale, int32_t chunk, int32_t window,
-                            int32_t one_sink, int32_t splits, float* part, int32_t cache_dtype, int32_t out_dtype, int64_t stream);
+                            int32_t one_sink, int32_t splits, float* part, int32_t plain, int32_t cache_dtype, int32_t out_dtype, int64_t stream);
 int32_t talking_attention_prefill_supported(int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv);
 void talking_attention_prefill(void* out, const void* q, const void* key_cache, const void* value_cache, const int32_t* block_tables, int32_t table_width,
                                const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, const float* talk, const float* v_cos, const float* v_sin, int32_t num_seqs,

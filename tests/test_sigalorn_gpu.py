@@ -316,8 +316,8 @@ WIDE = [  # H, G, dk, dv, chunk, rot_dims: sizes of the tensor-core kernel: one,
 
 @pytest.mark.parametrize("H,G,dk,dv,chunk,rot", WIDE)
 def test_talking_attention_on_the_tensor_core_kernel(H, G, dk, dv, chunk, rot):
-    """bf16: whole prompts, portions that start inside pages, tiles and chunks, and single rows (the f32-arithmetic kernel over the same 16-bit cache), against the
-    oracle and against the f32 run"""
+    """bf16: whole prompts, portions that start inside pages, tiles and chunks, and single rows (the kernel of mixed queries in one and several runs of keys, and the
+    f32-arithmetic kernel over the same 16-bit cache), against the oracle and against the f32 run"""
     T = 230
     L, w, h, want = mixer_case(H, G, dk, dv, chunk, rot, T, seed=H + dk)
     got32, _ = run_attention(make_mixer(L, w, torch.float32), h, [T], TABLE, torch.float32)
@@ -325,10 +325,11 @@ def test_talking_attention_on_the_tensor_core_kernel(H, G, dk, dv, chunk, rot):
     mix = make_mixer(L, w, torch.bfloat16)
     assert mix.prefill_kernel
     scale = float(want.abs().max())
-    for sizes in ([T], [100, 1, 37, 2, 64, 9]):
+    for sizes, splits, plain in (([T], None, False), ([100, 1, 37, 2, 64, 9], None, False), ([97, 1], None, False), ([130, 2, 1], 1, False), ([190, 1], 3, False), ([97, 1, 2], 2, True)):
+        mix.splits, mix.plain = splits, plain
         got = run_attention(mix, h, sizes, TABLE, torch.bfloat16)[0].float().cpu().to(F64)
         err = (got - want).abs().max(-1).values / scale
-        assert float(err.max()) < 5e-2 and float(err.median()) < 1.5e-2, (sizes, float(err.max()), float(err.median()), int(err.argmax()))
+        assert float(err.max()) < 5e-2 and float(err.median()) < 1.5e-2, (sizes, splits, plain, float(err.max()), float(err.median()), int(err.argmax()))
 
 
 def test_entries_of_a_batch_do_not_see_each_other():
