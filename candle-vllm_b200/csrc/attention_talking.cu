@@ -704,26 +704,27 @@ TcPlan tc_plan(int H, int G, int dk, int dv) {
 // ---- few rows in 16 bits on tensor cores --------------------------------------------------------------------------------------------------------
 // A row alone needs no exchange of scores: mixing commutes with the product, s'[h, j] = (sum_g talk[h, g] q[g]) . k_j summed kv head by kv head, so every head gets
 // one mixed query as long as a whole cache row, q'[h] = (talk[h, g] q[g] summed over the heads g of each kv head), and the scores of all heads are one product of
-// q' [H, G dk] with the cache rows.  A block per (row, run of keys), eight warps, 64 keys per tile: a warp scores eight keys (cache rows read straight into the operand
+// q' [H, G dk] with the cache rows.  A block per (row, run of keys), eight or sixteen warps, 64 keys per tile: a warp scores eight keys (cache rows read straight into the operand
 // layout, four lanes per row in 16-byte pieces), a warp per head takes the online softmax, and a warp multiplies the weights of one kv head's heads with 64 value
 // columns (eight neighbouring columns per lane from four rows, paired in registers; the column order of the product is a permutation undone at the store).
 constexpr int kDecTile = 64, kDecSP = kDecTile + 4, kDecPP = kDecTile + 8;      // keys per tile, pitches of a score row (f32) and of a weight row (bf16)
-constexpr int kDecHead = 2 * kDecTile * 8 + 96 * 4;                             // bytes ahead of the queries: a multiple of 128
+constexpr int kDecHead = 4 * kDecTile * 8 + 96 * 4;                             // bytes ahead of the queries: a multiple of 128
 
-template <int kMT, int kU>                       // 16-head tiles, (kv head, 64 columns) units per warp
-__global__ void __launch_bounds__(256, 2)
+// kMT: 16-head tiles; kW: warps, 8 or 16 (two warps then share eight keys' scores, half of the cache row each).  Every warp has one (kv head, 64 columns) unit of the values
+template <int kMT, int kW>
+__global__ void __launch_bounds__(kW * 32, 16 / kW)
 talking_decode_kernel(const TalkArgs A) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(128) uint8_t smem_dec[];
     const int H = A.H, G = A.G, dk = A.dk, dv = A.dv, group = H / G, row = G * dk, pq = (row * 2 + 127) / 128 * 128;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-    int64_t* ph = reinterpret_cast<int64_t*>(smem_dec);                      // [2][64] cache rows of the tile's keys
-    float* cs = reinterpret_cast<float*>(ph + 2 * kDecTile);                 // [32] correction of this tile, [32] maxima (base 2), [32] denominators
+    int64_t* ph = reinterpret_cast<int64_t*>(smem_dec);                      // [4][64] cache rows of the keys of this tile and the ones ahead
+    float* cs = reinterpret_cast<float*>(ph + 4 * kDecTile);                 // [32] correction of this tile, [32] maxima (base 2), [32] denominators
     float* ms = cs + 32; float* ls = ms + 32;
     uint8_t* qm = smem_dec + kDecHead;                                       // [16 kMT][pq] mixed queries, 16-byte pieces swizzled
-    float* S = reinterpret_cast<float*>(qm + 16 * kMT * pq);                 // [16 kMT][kDecSP]
-    __nv_bfloat16* P = reinterpret_cast<__nv_bfloat16*>(S + 16 * kMT * kDecSP);       // [H + 16][kDecPP]
+    float* S = reinterpret_cast<float*>(qm + 16 * kMT * pq);                 // [kW / 8][16 kMT][kDecSP]
+    __nv_bfloat16* P = reinterpret_cast<__nv_bfloat16*>(S + kW / 8 * 16 * kMT * kDecSP);       // [H + 16][kDecPP]
     const int tok = blockIdx.x, split = blockIdx.y;
     const int pos = A.positions[tok];
     const int lo = first_visible(pos, A.chunk, A.window);
@@ -733,30 +734,69 @@ talking_decode_kernel(const TalkArgs A) {
     const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(A.kc);
     const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(A.vc);
     auto place = [&](int j0, int buf) {          // keys past the run's end stand for its first one (their weight is 0, what they read is finite)
-        if (threadIdx.x < kDecTile) {
+        if (j0 < je && threadIdx.x < kDecTile) {
             const int j = j0 + threadIdx.x < je ? j0 + threadIdx.x : jb;
             ph[buf * kDecTile + threadIdx.x] = cache_row(table, j, A.bs, A.bs_shift);
         }
     };
     const float scale_log2 = A.scale * 1.4426950408889634f;
+    const int all_blk = row / 32, kg = warp & 7;                             // this warp's group of eight keys and its 32-entry parts of their rows
+    const int blk0 = kW == 16 ? (warp >> 3) * (all_blk - all_blk / 2) : 0, nblk = kW == 16 ? (warp >> 3 ? all_blk / 2 : all_blk - all_blk / 2) : all_blk;
+    uint4 nx[4];                                 // the next pieces of this warp's eight keys travel while earlier ones are multiplied, across tiles too
+    auto first_pieces = [&](int j0, int buf) {
+        if (j0 + kg * 8 >= je || nblk == 0) return;
+        const uint4* kr = reinterpret_cast<const uint4*>(kc + ph[buf * kDecTile + kg * 8 + g] * row) + t + blk0 * 4;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) nx[i] = kr[min(i, nblk - 1) * 4];
+    };
     if (jb < je) {
         place(jb, 0);
-        // a thread makes 16-byte pieces of the mixed queries: eight neighbouring entries of one head
-        for (int i = threadIdx.x; i < 16 * kMT * (row >> 3); i += 256) {
-            const int h = i / (row >> 3), c = i - h * (row >> 3);
-            const int kv = c * 8 / dk, d = c * 8 - kv * dk;
-            float v[8] = {};
-            if (h < H)
-                for (int e = 0; e < group; ++e) {
-                    const int x = kv * group + e;
-                    const float w = (A.talk ? A.talk[h * H + x] : (x == h ? 1.f : 0.f)) * scale_log2;
-                    const float4* q4 = reinterpret_cast<const float4*>(A.q + ((int64_t)tok * H + x) * dk + d);
-                    const float4 a = q4[0], b = q4[1];
-                    v[0] = fmaf(w, a.x, v[0]); v[1] = fmaf(w, a.y, v[1]); v[2] = fmaf(w, a.z, v[2]); v[3] = fmaf(w, a.w, v[3]);
-                    v[4] = fmaf(w, b.x, v[4]); v[5] = fmaf(w, b.y, v[5]); v[6] = fmaf(w, b.z, v[6]); v[7] = fmaf(w, b.w, v[7]);
-                }
+        place(jb + kDecTile, 1);
+        __syncthreads();
+        first_pieces(jb, 0);
+        // mixed queries in 16-byte pieces, eight neighbouring entries of one head each
+        const int pieces = row >> 3, parts = max(1, kW * 32 / pieces), per_part = (16 * kMT + parts - 1) / parts;
+        auto put = [&](int h, int c, const float (&v)[8]) {
             *reinterpret_cast<uint4*>(qm + h * pq + ((c ^ ((h & 1) << 2)) << 4)) =
                 make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+        };
+        for (int i = threadIdx.x; i < pieces * parts; i += kW * 32) {
+            const int c = i % pieces, part = i / pieces, kv = c * 8 / dk, d = c * 8 - kv * dk;
+            const int ha = part * per_part, hb = min(16 * kMT, ha + per_part);
+            const float* q0 = A.q + ((int64_t)tok * H + kv * group) * dk + d;
+            if (group <= 4) {                    // the kv head's queries stay in registers for all the heads of this thread
+                float qv[4][8];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float4* q4 = reinterpret_cast<const float4*>(q0 + (int64_t)min(e, group - 1) * dk);
+                    const float4 a = q4[0], b = q4[1];
+                    qv[e][0] = a.x; qv[e][1] = a.y; qv[e][2] = a.z; qv[e][3] = a.w; qv[e][4] = b.x; qv[e][5] = b.y; qv[e][6] = b.z; qv[e][7] = b.w;
+                }
+#pragma unroll 4
+                for (int h = ha; h < hb; ++h) {
+                    float w[4], v[8] = {};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        w[e] = e < group && h < H ? (A.talk ? A.talk[h * H + kv * group + e] : (kv * group + e == h ? 1.f : 0.f)) * scale_log2 : 0.f;
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+#pragma unroll
+                        for (int x = 0; x < 8; ++x) v[x] = fmaf(w[e], qv[e][x], v[x]);
+                    put(h, c, v);
+                }
+            } else {
+                for (int h = ha; h < hb; ++h) {
+                    float v[8] = {};
+                    for (int e = 0; e < group && h < H; ++e) {
+                        const float w = (A.talk ? A.talk[h * H + kv * group + e] : (kv * group + e == h ? 1.f : 0.f)) * scale_log2;
+                        const float4* q4 = reinterpret_cast<const float4*>(q0 + (int64_t)e * dk);
+                        const float4 a = q4[0], b = q4[1];
+                        v[0] = fmaf(w, a.x, v[0]); v[1] = fmaf(w, a.y, v[1]); v[2] = fmaf(w, a.z, v[2]); v[3] = fmaf(w, a.w, v[3]);
+                        v[4] = fmaf(w, b.x, v[4]); v[5] = fmaf(w, b.y, v[5]); v[6] = fmaf(w, b.z, v[6]); v[7] = fmaf(w, b.w, v[7]);
+                    }
+                    put(h, c, v);
+                }
+            }
         }
     }
     if (threadIdx.x < 32) {
@@ -765,35 +805,31 @@ talking_decode_kernel(const TalkArgs A) {
         ls[threadIdx.x] = sink ? 1.f : 0.f;
     }
     const int cols = (dv + 63) / 64, units = G * cols;
-    float o[kU][8][4];
+    float o[8][4];
 #pragma unroll
-    for (int u = 0; u < kU; ++u)
-#pragma unroll
-        for (int n = 0; n < 8; ++n) o[u][n][0] = o[u][n][1] = o[u][n][2] = o[u][n][3] = 0.f;
-    int ukv[kU], ucol[kU];                       // kv head and first column of this lane's eight
-#pragma unroll
-    for (int u = 0; u < kU; ++u) { const int x = warp + 8 * u; ukv[u] = x < units ? x / cols : -1; ucol[u] = (x % cols) * 64 + g * 8; }
+    for (int n = 0; n < 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+    const int ukv = warp < units ? warp / cols : -1, ucol = (warp % cols) * 64 + g * 8;      // kv head and first column of this lane's eight
     __syncthreads();
-    const int nblk = row / 32;
     const uint8_t* qrow = qm + g * pq + (((uint32_t)t ^ ((g & 1) << 2)) << 4);       // piece t of an even 32-entry part; the odd parts' lie 64 bytes away
     const int odd = (g & 1) ? -64 : 64;
     for (int j0 = jb, it = 0; j0 < je; j0 += kDecTile, ++it) {
-        const int64_t* pht = ph + (it & 1) * kDecTile;
+        const int64_t* pht = ph + (it & 3) * kDecTile;
         // ---- scores of eight keys ------------------------------------------------------------------------------------------------------------
-        if (j0 + warp * 8 < je) {
-            const uint4* kr = reinterpret_cast<const uint4*>(kc + pht[warp * 8 + g] * row) + t;
+        if (j0 + kg * 8 < je) {
+            const uint4* kr = reinterpret_cast<const uint4*>(kc + pht[kg * 8 + g] * row) + t + blk0 * 4;
             float acc[kMT][4] = {};
-            uint4 nx[4];
-#pragma unroll
-            for (int i = 0; i < 4; ++i) nx[i] = kr[min(i, nblk - 1) * 4];
             for (int b = 0; b < nblk; b += 4) {
                 uint4 cur[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) { cur[i] = nx[i]; nx[i] = kr[min(b + 4 + i, nblk - 1) * 4]; }
+                for (int i = 0; i < 4; ++i) cur[i] = nx[i];
+                if (b + 4 < nblk) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) nx[i] = kr[min(b + 4 + i, nblk - 1) * 4];
+                }
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     if (b + i >= nblk) break;
-                    const uint8_t* qa = qrow + ((b + i) >> 1) * 128 + (((b + i) & 1) ? odd : 0);
+                    const uint8_t* qa = qrow + ((blk0 + b + i) >> 1) * 128 + (((blk0 + b + i) & 1) ? odd : 0);
 #pragma unroll
                     for (int mt = 0; mt < kMT; ++mt) {
                         const uint4 x = *reinterpret_cast<const uint4*>(qa + mt * 16 * pq), y = *reinterpret_cast<const uint4*>(qa + (mt * 16 + 8) * pq);
@@ -804,26 +840,31 @@ talking_decode_kernel(const TalkArgs A) {
             }
 #pragma unroll
             for (int mt = 0; mt < kMT; ++mt) {
-                *reinterpret_cast<float2*>(S + (mt * 16 + g) * kDecSP + warp * 8 + 2 * t) = make_float2(acc[mt][0], acc[mt][1]);
-                *reinterpret_cast<float2*>(S + (mt * 16 + g + 8) * kDecSP + warp * 8 + 2 * t) = make_float2(acc[mt][2], acc[mt][3]);
+                float* sd = S + ((warp >> 3) * 16 * kMT + mt * 16 + g) * kDecSP + kg * 8 + 2 * t;
+                *reinterpret_cast<float2*>(sd) = make_float2(acc[mt][0], acc[mt][1]);
+                *reinterpret_cast<float2*>(sd + 8 * kDecSP) = make_float2(acc[mt][2], acc[mt][3]);
             }
         }
         // the first half of the tile's values travels during the softmax: rows 2t, 2t + 1, 2t + 8, 2t + 9 of two sets of sixteen keys
         uint4 vr[2][4];
-        auto fetch_v = [&](int u, int ks, uint4 (&d)[4]) {
-            const bool ok = ukv[u] >= 0 && ucol[u] < dv;
+        auto fetch_v = [&](int ks, uint4 (&d)[4]) {
+            const bool ok = ukv >= 0 && ucol < dv;
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = ks * 16 + 2 * t + (e & 1) + (e >> 1) * 8;
-                d[e] = ok ? *reinterpret_cast<const uint4*>(vc + (pht[key] * G + ukv[u]) * dv + ucol[u]) : make_uint4(0u, 0u, 0u, 0u);
+                d[e] = ok ? *reinterpret_cast<const uint4*>(vc + (pht[key] * G + ukv) * dv + ucol) : make_uint4(0u, 0u, 0u, 0u);
             }
         };
-        fetch_v(0, 0, vr[0]);
-        fetch_v(0, 1, vr[1]);
+        fetch_v(0, vr[0]);
+        fetch_v(1, vr[1]);
+        first_pieces(j0 + kDecTile, (it + 1) & 3);
         __syncthreads();
         // ---- online softmax, a warp per head ----------------------------------------------------------------------------------------------------
-        for (int h = warp; h < H; h += 8) {
-            float a = j0 + lane < je ? S[h * kDecSP + lane] : -INFINITY, b = j0 + 32 + lane < je ? S[h * kDecSP + 32 + lane] : -INFINITY;
+        for (int h = warp; h < H; h += kW) {
+            float a = S[h * kDecSP + lane], b = S[h * kDecSP + 32 + lane];
+            if (kW == 16) { a += S[(16 * kMT + h) * kDecSP + lane]; b += S[(16 * kMT + h) * kDecSP + 32 + lane]; }
+            if (j0 + lane >= je) a = -INFINITY;                              // (what a skipped group left there is not looked at)
+            if (j0 + 32 + lane >= je) b = -INFINITY;
             const float m_old = ms[h], m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
             a = exp2f(a - m_new); b = exp2f(b - m_new);
             P[h * kDecPP + lane] = __float2bfloat16_rn(a);
@@ -836,17 +877,14 @@ talking_decode_kernel(const TalkArgs A) {
                 ls[h] = fmaf(ls[h], corr, sum);
             }
         }
-        if (j0 + kDecTile < je) place(j0 + kDecTile, (it + 1) & 1);
+        place(j0 + 2 * kDecTile, (it + 2) & 3);
         __syncthreads();
         // ---- values -----------------------------------------------------------------------------------------------------------------------------
-#pragma unroll
-        for (int u = 0; u < kU; ++u) {
-            if (ukv[u] < 0) continue;
-            const int hb = ukv[u] * group;
+        if (ukv >= 0) {
+            const int hb = ukv * group;
             const float c0 = g < group ? cs[hb + g] : 0.f, c1 = g + 8 < group ? cs[hb + g + 8] : 0.f;
 #pragma unroll
-            for (int n = 0; n < 8; ++n) { o[u][n][0] *= c0; o[u][n][1] *= c0; o[u][n][2] *= c1; o[u][n][3] *= c1; }
-            if (u > 0) { fetch_v(u, 0, vr[0]); fetch_v(u, 1, vr[1]); }
+            for (int n = 0; n < 8; ++n) { o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1; }
 #pragma unroll
             for (int ks = 0; ks < 4; ++ks) {
                 if (j0 + ks * 16 >= je) break;
@@ -857,12 +895,12 @@ talking_decode_kernel(const TalkArgs A) {
                 uint4 r[4];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) r[e] = vr[ks & 1][e];
-                if (ks < 2) fetch_v(u, ks + 2, vr[ks & 1]);
+                if (ks < 2) fetch_v(ks + 2, vr[ks & 1]);
                 const uint32_t w[4][4] = {{r[0].x, r[0].y, r[0].z, r[0].w}, {r[1].x, r[1].y, r[1].z, r[1].w}, {r[2].x, r[2].y, r[2].z, r[2].w}, {r[3].x, r[3].y, r[3].z, r[3].w}};
 #pragma unroll
                 for (int n2 = 0; n2 < 4; ++n2) {         // columns 2 n2 and 2 n2 + 1 of the lane's eight: pair the rows' low halves, then their high halves
-                    mma_bf16(o[u][2 * n2], a0, a1, a2, a3, __byte_perm(w[0][n2], w[1][n2], 0x5410), __byte_perm(w[2][n2], w[3][n2], 0x5410));
-                    mma_bf16(o[u][2 * n2 + 1], a0, a1, a2, a3, __byte_perm(w[0][n2], w[1][n2], 0x7632), __byte_perm(w[2][n2], w[3][n2], 0x7632));
+                    mma_bf16(o[2 * n2], a0, a1, a2, a3, __byte_perm(w[0][n2], w[1][n2], 0x5410), __byte_perm(w[2][n2], w[3][n2], 0x5410));
+                    mma_bf16(o[2 * n2 + 1], a0, a1, a2, a3, __byte_perm(w[0][n2], w[1][n2], 0x7632), __byte_perm(w[2][n2], w[3][n2], 0x7632));
                 }
             }
         }
@@ -870,21 +908,19 @@ talking_decode_kernel(const TalkArgs A) {
     __syncthreads();
     // ---- output or the run's partial result: accumulator n of a lane's queries' columns 2t, 2t + 1 is value column 8 (2t) + n, 8 (2t + 1) + n of its 64 -------------
     float* O = reinterpret_cast<float*>(qm);                                 // [H][dv]
-#pragma unroll
-    for (int u = 0; u < kU; ++u) {
-        if (ukv[u] < 0) continue;
-        const int base = ucol[u] - g * 8;
+    if (ukv >= 0) {
+        const int base = ucol - g * 8;
 #pragma unroll
         for (int n = 0; n < 8; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int r = g + (e >> 1) * 8, col = base + 8 * (2 * t + (e & 1)) + n;
-                if (r < group && col < dv) O[(ukv[u] * group + r) * dv + col] = o[u][n][e];
+                if (r < group && col < dv) O[(ukv * group + r) * dv + col] = o[n][e];
             }
     }
     __syncthreads();
     const int half = dv >> 1;
-    for (int e = threadIdx.x; e < H * half; e += 256) {
+    for (int e = threadIdx.x; e < H * half; e += kW * 32) {
         const int h = e / half, x = e - h * half;
         float a = O[h * dv + x], b = O[h * dv + x + half];
         if (A.splits > 1) {
@@ -909,11 +945,12 @@ talking_decode_kernel(const TalkArgs A) {
 size_t decode_plan(int H, int G, int dk, int dv) {
     if (H > 32 || H % G || H / G > 16 || (G * dk) % 32 || dk % 8 || dv % 8 || G * ((dv + 63) / 64) > 16) return 0;
     const int mt = (H + 15) / 16, pq = (G * dk * 2 + 127) / 128 * 128;
-    size_t b = (size_t)16 * mt * pq + (size_t)16 * mt * kDecSP * 4 + (size_t)(H + 16) * kDecPP * 2;
+    const int wide = G * ((dv + 63) / 64) > 8;                               // sixteen warps, one block per SM
+    size_t b = (size_t)16 * mt * pq + (size_t)(1 + wide) * 16 * mt * kDecSP * 4 + (size_t)(H + 16) * kDecPP * 2;
     const size_t outb = (size_t)H * dv * 4;
     if (b < outb) b = outb;
     b += kDecHead;
-    return b <= 110 * 1024 ? b : 0;              // two blocks per SM
+    return b <= (wide ? 220 : 110) * 1024 ? b : 0;
 }
 
 int block_shift(int bs) {
@@ -971,11 +1008,11 @@ void talking_attention_rows(void* out, const float* q, const void* key_cache, co
     bool ok = false;
     if (dec_smem > 0) {
         const dim3 grid(num_tokens, splits);
-        const bool two = num_kv_heads * ((dv + 63) / 64) > 8;
-#define TDK(MT, UU) do { ensure_dynamic_smem((const void*)talking_decode_kernel<MT, UU>, (int)dec_smem); \
-        launch_pdl(talking_decode_kernel<MT, UU>, grid, dim3(256), dec_smem, st, A); } while (0)
-        if (num_heads <= 16) { if (two) TDK(1, 2); else TDK(1, 1); }
-        else { if (two) TDK(2, 2); else TDK(2, 1); }
+        const int units = num_kv_heads * ((dv + 63) / 64);
+#define TDK(MT, WW) do { ensure_dynamic_smem((const void*)talking_decode_kernel<MT, WW>, (int)dec_smem); \
+        launch_pdl(talking_decode_kernel<MT, WW>, grid, dim3(WW * 32), dec_smem, st, A); } while (0)
+        if (num_heads <= 16) { if (units <= 8) TDK(1, 8); else TDK(1, 16); }
+        else { if (units <= 8) TDK(2, 8); else TDK(2, 16); }
 #undef TDK
         ok = true;
     } else if (cache_dtype == B200_F32 && out_dtype == B200_F32) ok = launch_rows<float, float>(A, num_tokens, smem, st);

@@ -1109,37 +1109,51 @@ la_chunk_output_kernel(const ChunkArgs C) {
 //     score of t over j    sum_r q_t P_t (prod_{runs between} E) R_j k_j, j in an earlier run; inside one run the products of at most three decays
 //     entering state       q_t P_t prod_{runs before} E against S_in                                      (la_chan_output_kernel)
 // The walk over the chunks is la_chunk_scan_kernel with the chunk's product per key row in place of the scalar decay.
+template <int kTok>
 __global__ void __launch_bounds__(256)
 low_rank_decay_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ alpha, int T, int N,
                       int R, float inv_tau) {
     pdl_wait();
     pdl_trigger();
-    // 256 channels x 8 tokens per block: a thread keeps 16 weights of its channel at a time and meets eight tokens' inner values with them
-    __shared__ float ys[8][16];
-    const int n = blockIdx.x * 256 + threadIdx.x, t0 = blockIdx.y * 8;
-    float z[8];
+    // 256 channels x kTok tokens per block: a thread keeps 16 weights of its channel at a time and meets the tokens' inner values with them
+    __shared__ __align__(16) float ys[kTok][16];
+    const int n = blockIdx.x * 256 + threadIdx.x, t0 = blockIdx.y * kTok;
+    float z[kTok];
     const float b = (n < N && bias) ? bias[n] : 0.f;
+    const bool fours = R % 4 == 0;               // weight rows are whole 16-byte words
 #pragma unroll
-    for (int i = 0; i < 8; ++i) z[i] = 0.f;
+    for (int i = 0; i < kTok; ++i) z[i] = b;
     for (int r0 = 0; r0 < R; r0 += 16) {
         float wr[16];
+        const float* wp = w + (int64_t)(n < N ? n : 0) * R + r0;
 #pragma unroll
-        for (int r = 0; r < 16; ++r) wr[r] = (n < N && r0 + r < R) ? w[(int64_t)n * R + r0 + r] : 0.f;
+        for (int r = 0; r < 16; r += 4) {
+            if (fours) {
+                const float4 v = r0 + r < R ? *reinterpret_cast<const float4*>(wp + r) : make_float4(0.f, 0.f, 0.f, 0.f);
+                wr[r] = v.x; wr[r + 1] = v.y; wr[r + 2] = v.z; wr[r + 3] = v.w;
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) wr[r + e] = r0 + r + e < R ? wp[r + e] : 0.f;
+            }
+        }
         __syncthreads();
-        if (threadIdx.x < 128) {
-            const int i = threadIdx.x >> 4, r = threadIdx.x & 15;
+        for (int e = threadIdx.x; e < kTok * 16; e += 256) {
+            const int i = e >> 4, r = e & 15;
             ys[i][r] = (t0 + i < T && r0 + r < R) ? y[(int64_t)(t0 + i) * ldy + r0 + r] : 0.f;
         }
         __syncthreads();
 #pragma unroll
-        for (int i = 0; i < 8; ++i)
+        for (int i = 0; i < kTok; ++i)
 #pragma unroll
-            for (int r = 0; r < 16; ++r) z[i] = fmaf(wr[r], ys[i][r], z[i]);
+            for (int r = 0; r < 16; r += 4) {
+                const float4 v = *reinterpret_cast<const float4*>(&ys[i][r]);
+                z[i] = fmaf(wr[r], v.x, fmaf(wr[r + 1], v.y, fmaf(wr[r + 2], v.z, fmaf(wr[r + 3], v.w, z[i]))));
+            }
     }
     if (n >= N) return;
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
-        if (t0 + i < T) alpha[(int64_t)(t0 + i) * N + n] = expf(log_sigmoid_f(z[i] + b) * inv_tau);
+    for (int i = 0; i < kTok; ++i)
+        if (t0 + i < T) alpha[(int64_t)(t0 + i) * N + n] = expf(log_sigmoid_f(z[i]) * inv_tau);
 }
 
 __global__ void __launch_bounds__(256)
@@ -1574,9 +1588,14 @@ void linear_attention_chunked(const float* proj, int64_t ld, int32_t off_q, int3
 void low_rank_decay(const float* y, int64_t ldy, const float* weight, const float* bias, float* alpha, int32_t num_tokens, int32_t channels, int32_t rank, float tau,
                     int64_t stream) {
     if (num_tokens == 0) return;
-    B200_REQUIRE(y && weight && alpha && channels > 0 && rank > 0 && ldy >= rank && tau > 0.f && num_tokens <= 8 * 65535, kErrBadArg, "low_rank_decay: bad arguments");
-    launch_pdl(low_rank_decay_kernel, dim3(ceil_div(channels, 256), ceil_div(num_tokens, 8)), dim3(256), 0, as_stream(stream), y, ldy, weight, bias, alpha,
-               (int)num_tokens, (int)channels, (int)rank, 1.0f / tau);
+    B200_REQUIRE(y && weight && alpha && channels > 0 && rank > 0 && ldy >= rank && tau > 0.f && num_tokens <= 32 * 65535, kErrBadArg, "low_rank_decay: bad arguments");
+    cudaStream_t st = as_stream(stream);
+    if (num_tokens <= 256)                       // few rows: short blocks, many of them
+        launch_pdl(low_rank_decay_kernel<2>, dim3(ceil_div(channels, 256), ceil_div(num_tokens, 2)), dim3(256), 0, st, y, ldy, weight, bias, alpha, (int)num_tokens,
+                   (int)channels, (int)rank, 1.0f / tau);
+    else
+        launch_pdl(low_rank_decay_kernel<32>, dim3(ceil_div(channels, 256), ceil_div(num_tokens, 32)), dim3(256), 0, st, y, ldy, weight, bias, alpha, (int)num_tokens,
+                   (int)channels, (int)rank, 1.0f / tau);
     count_launch();
     check_launch("low_rank_decay");
 }

@@ -276,6 +276,46 @@ group_rms_norm_gate_kernel(const float* __restrict__ o, int64_t ldo, const float
 }
 
 
+// groups of up to 1024 entries in whole aligned groups of four: a warp per (row, group), kV groups of four per lane kept in registers between the passes
+template <typename TOut, int kV>
+__global__ void __launch_bounds__(256)
+group_rms_norm_gate_warp_kernel(const float* __restrict__ o, int64_t ldo, const float* __restrict__ w, const float* __restrict__ gate, int64_t ldg, TOut* __restrict__ out,
+                                int64_t items, int groups, int n, int glen, float eps, int gate_act) {
+    pdl_wait();
+    pdl_trigger();
+    const int64_t item = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (item >= items) return;
+    const int64_t t = item / groups;
+    const int c0 = (int)(item - t * groups) * glen, lane = threadIdx.x & 31;
+    float4 v[kV], z[kV];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < kV; ++k) {
+        const int i = (lane + 32 * k) * 4;
+        v[k] = i < glen ? *reinterpret_cast<const float4*>(o + t * ldo + c0 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        if (gate) z[k] = i < glen ? *reinterpret_cast<const float4*>(gate + t * ldg + c0 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
+    }
+    const float sc = 1.0f / sqrtf(warp_sum(ss) / (float)glen + eps);
+#pragma unroll
+    for (int k = 0; k < kV; ++k) {
+        const int i = (lane + 32 * k) * 4;
+        if (i >= glen) continue;
+        float r[4] = {v[k].x * sc, v[k].y * sc, v[k].z * sc, v[k].w * sc};
+        if (w) { const float4 wv = *reinterpret_cast<const float4*>(w + c0 + i); r[0] *= wv.x; r[1] *= wv.y; r[2] *= wv.z; r[3] *= wv.w; }
+        if (gate) {
+            const float zz[4] = {z[k].x, z[k].y, z[k].z, z[k].w};
+#pragma unroll
+            for (int j = 0; j < 4; ++j) r[j] *= (gate_act == 0 ? 1.0f : zz[j]) / (1.0f + expf(-zz[j]));
+        }
+        TOut q[4] = {from_f32<TOut>(r[0]), from_f32<TOut>(r[1]), from_f32<TOut>(r[2]), from_f32<TOut>(r[3])};
+        TOut* dst = out + t * n + c0 + i;
+        if (sizeof(TOut) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(q);
+        else *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(q);
+    }
+}
+
+
 template <typename TS, typename TOut>
 __global__ void head_gate_kernel(const TS* __restrict__ src, const float* __restrict__ gate, int64_t ldg, TOut* __restrict__ out, int H, int dv) {
     pdl_wait();
@@ -654,6 +694,22 @@ void group_rms_norm_gate(const float* o, int64_t ldo, const float* weight, const
     B200_REQUIRE(o && out && n > 0 && groups > 0 && n % groups == 0 && ldo >= n && (!gate || ld_gate >= n) && groups <= 65535 && (gate_act == 0 || gate_act == 1),
                  kErrBadArg, "group_rms_norm_gate: bad arguments");
     cudaStream_t st = as_stream(stream);
+    const int glen = n / groups;
+    const bool vec = glen % 4 == 0 && glen <= 1024 && ldo % 4 == 0 && (!gate || ld_gate % 4 == 0) &&
+                     (((uintptr_t)o | (uintptr_t)weight | (uintptr_t)gate | (uintptr_t)out) & 15) == 0 && (out_dtype == B200_F32 || out_dtype == B200_BF16);
+    if (vec) {
+        const int64_t items = (int64_t)num_tokens * groups;
+        const dim3 g8((unsigned)((items + 7) / 8));
+#define GRW(TO, KV) launch_pdl(group_rms_norm_gate_warp_kernel<TO, KV>, g8, dim3(256), 0, st, o, ldo, weight, gate, ld_gate, (TO*)out, items, (int)groups, (int)n, glen, eps, (int)gate_act)
+#define GRW_ALL(TO) do { if (glen <= 128) GRW(TO, 1); else if (glen <= 256) GRW(TO, 2); else if (glen <= 512) GRW(TO, 4); else GRW(TO, 8); } while (0)
+        if (out_dtype == B200_F32) GRW_ALL(float);
+        else GRW_ALL(__nv_bfloat16);
+#undef GRW_ALL
+#undef GRW
+        count_launch();
+        check_launch("group_rms_norm_gate");
+        return;
+    }
     const dim3 grid(groups, num_tokens);
     if (out_dtype == B200_F32)
         launch_pdl(group_rms_norm_gate_kernel<float>, grid, dim3(128), 0, st, o, ldo, weight, gate, ld_gate, (float*)out, n, n / groups, eps, gate_act);

@@ -898,7 +898,7 @@ def talking_prefill_kernel_supported(heads: int, kv_heads: int, dk: int, dv: int
     return dtype == torch.bfloat16 and bool(lib().talking_attention_prefill_supported(C.c_int32(heads), C.c_int32(kv_heads), C.c_int32(dk), C.c_int32(dv)))
 
 
-TALKING_BLOCKS = 296           # two blocks per SM: steps with fewer rows cut the keys of every row into runs
+TALKING_BLOCKS = 296           # two blocks per SM: steps with fewer rows cut the keys of every row into runs (blocks of sixteen warps: one per SM)
 
 
 def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: StepBatch, talk: Optional[torch.Tensor], value_tables: Optional[tuple], heads: int,
@@ -926,7 +926,8 @@ def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         for limit in (chunk, window):
             if limit > 0:
                 longest = min(longest, limit)
-        splits = max(1, min(-(-TALKING_BLOCKS // T), longest // 64, 64)) if T < TALKING_BLOCKS else 1
+        wide = out_dtype == torch.bfloat16 and not plain and 8 < G * -(-dv // 64) <= 16
+        splits = max(1, min(-(-(TALKING_BLOCKS // 2) // T) if wide else TALKING_BLOCKS // T, longest // 64, 64))
     part = torch.empty((T * splits * heads * (dv + 2),), dtype=torch.float32, device=q.device) if splits > 1 else None
     out = torch.empty((T, heads * dv), dtype=out_dtype, device=q.device)
     lib().talking_attention_rows(_ptr(out), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), C.c_int32(batch.block_tables.shape[1]), _ptr(batch.token_seq),

@@ -102,6 +102,19 @@ def test_xielu_with_bias_and_two_numbers(ff):
     assert same.dtype == torch.bfloat16 and same.shape == (9, ff)
 
 
+@pytest.mark.parametrize("groups,glen", [(3, 5), (4, 64), (2, 300), (16, 128), (1, 1000), (2, 1030)])
+def test_norm_per_group_times_a_silu_gate(groups, glen):
+    g = torch.Generator().manual_seed(glen)
+    n, T = groups * glen, 11
+    o, z, w = torch.randn(T, n + 4, generator=g) * 2, torch.randn(T, n + 8, generator=g) * 3, 1 + torch.randn(n, generator=g) * 0.3
+    x = o[:, :n].to(F64).view(T, groups, glen)
+    want = (O.rms(x, 1e-3).reshape(T, n) * w.to(F64)) * O.silu(z[:, :n].to(F64))
+    for od, zd in ((dev(o)[:, :n], dev(z)[:, :n]), (dev(o[:, :n]), dev(z[:, :n]))):
+        close(ops.group_rms_norm_gate(od, dev(w), zd, groups, 1e-3, torch.float32, gate_act="silu"), want, 2e-6, "f32")
+        close(ops.group_rms_norm_gate(od, dev(w), zd, groups, 1e-3, torch.bfloat16, gate_act="silu"), want, 6e-3, "bf16")
+    close(ops.group_rms_norm_gate(dev(o[:, :n]), None, None, groups, 1e-3, torch.float32), O.rms(x, 1e-3).reshape(T, n), 2e-6, "norm alone")
+
+
 def test_logit_cap():
     x = torch.randn(5, 77, generator=torch.Generator().manual_seed(0)) * 40
     close(ops.softcap(dev(x), 12.5), 12.5 * torch.tanh(x.to(F64) / 12.5), 1e-6, "cap")
@@ -311,7 +324,7 @@ def test_talking_attention_f32(H, G, dk, dv, chunk, rot, sizes):
 
 WIDE = [  # H, G, dk, dv, chunk, rot_dims: sizes of the tensor-core kernel: one, two and four heads per warp, both tile widths, single and double buffers
     (4, 2, 64, 48, 100, 64), (8, 8, 32, 16, 0, 32), (16, 4, 128, 128, 130, 128), (12, 3, 80, 112, 64, 40), (32, 8, 64, 64, 90, 64), (20, 5, 40, 32, 33, 40),
-    (5, 5, 96, 80, 200, 96), (16, 16, 128, 128, 100, 64), (32, 8, 128, 128, 150, 128), (1, 1, 8, 16, 7, 8), (6, 2, 72, 96, 1, 72), (24, 1, 128, 64, 0, 128)]
+    (5, 5, 96, 80, 200, 96), (16, 16, 128, 128, 100, 64), (32, 8, 128, 128, 150, 128), (1, 1, 8, 16, 7, 8), (6, 2, 72, 96, 1, 72), (24, 1, 128, 64, 0, 128), (16, 2, 64, 80, 70, 32), (18, 9, 24, 128, 90, 24)]
 
 
 @pytest.mark.parametrize("H,G,dk,dv,chunk,rot", WIDE)
