@@ -417,7 +417,8 @@ talking_prefill_kernel(const TalkTcArgs A) {
     auto lds16 = [&](uint32_t a) { return *reinterpret_cast<const uint4*>(smem_tc + (a - sbase)); };
     const uint32_t sQ = sbase, sK = sQ + H * kTcRows * pk, sV = sK + A.kst * kbytes;
     float* S = reinterpret_cast<float*>(smem_tc + (sV - sbase) + A.vst * vbytes);                   // [2][Hp][8][kSP]
-    const int Hp = (H + 3) & ~3, tp = Hp + 4;                          // heads rounded up to whole groups of four (rows of zeros); row pitch of the mixing matrix
+    const int Hp = (H + 3) & ~3;                                       // heads rounded up to whole groups of four (rows of zeros)
+    constexpr int tp = 16 * kHW + 4;                                   // row pitch of the mixing matrix
     const int sstage = Hp * kTcRows * kSP;
     float* tk = S + 2 * sstage;                                                                      // [8 kNP][tp] talk times scale log2 e, zeros past H
     const int magic_k = (65536 + (dk >> 3) - 1) / (dk >> 3), magic_v = (65536 + (dv >> 3) - 1) / (dv >> 3);
@@ -486,6 +487,7 @@ talking_prefill_kernel(const TalkTcArgs A) {
     // permute the contraction index the same way, so no transposing load is needed.
     const uint32_t off_a = (uint32_t)((t ^ ((g & 1) << 2)) * 16), off_b = off_a ^ 64u;       // of the even and odd 32-entry parts of a row pair
     auto scores = [&](int tl) {
+        if (h0 >= H) return;
         float acc[kHW][kMT][4] = {};
         const uint32_t kb = sK + (A.kst == 2 ? (tl & 1) * kbytes : 0);
 #pragma unroll (k128 ? 4 : 1)
@@ -496,10 +498,8 @@ talking_prefill_kernel(const TalkTcArgs A) {
             int kv_loaded = -1;
 #pragma unroll
             for (int a = 0; a < kHW; ++a) {
-                const int h = h0 + a;
-                if (h >= H) continue;
-                const int kv = kvh[a];
-                if (kv != kv_loaded) {
+                const int h = min(h0 + a, H - 1), kv = kvh[a];         // a head past the last repeats it: nothing of it is stored
+                if (a == 0 || kv != kv_loaded) {
                     kv_loaded = kv;
                     const uint32_t at = kb + (kv * kKT + g) * pk + off;
 #pragma unroll
@@ -580,61 +580,66 @@ talking_prefill_kernel(const TalkTcArgs A) {
         if (A.vst == 2) load_v(i + 1);
         cp_commit();
         const float* Sd = S + (i & 1) * sstage;
-        uint32_t pb[kHW][kMT][2];
-        const int jt = key0 + i * kKT;
-        const bool whole = jt + kKT - 1 <= pos0 && jt >= lo_last;      // every key of the tile is seen by every row
+        if (h0 < H) {
+            uint32_t pb[kHW][kMT][2];
+            const int jt = key0 + i * kKT;
+            const bool whole = jt + kKT - 1 <= pos0 && jt >= lo_last;      // every key of the tile is seen by every row
 #pragma unroll
-        for (int a = 0; a < kHW; ++a) {
-            if (h0 + a >= H) continue;
-            const float* row = Sd + ((h0 + a) * kTcRows + g) * kSP;
-            const int j0 = key0 + i * kKT + 2 * t;
-            float v[kMT][4], mx = -INFINITY;
+            for (int a = 0; a < kHW; ++a) {
+                const float* row = Sd + (min(h0 + a, H - 1) * kTcRows + g) * kSP;
+                const int j0 = key0 + i * kKT + 2 * t;
+                float v[kMT][4], mx = -INFINITY;
 #pragma unroll
-            for (int mt = 0; mt < kMT; ++mt) {
-                const float2 x = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t), y = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t + 8);
-                v[mt][0] = x.x; v[mt][1] = x.y; v[mt][2] = y.x; v[mt][3] = y.y;
-                if (!A.talk) { v[mt][0] *= A.scale_log2; v[mt][1] *= A.scale_log2; v[mt][2] *= A.scale_log2; v[mt][3] *= A.scale_log2; }      // else in the matrix
+                for (int mt = 0; mt < kMT; ++mt) {
+                    const float2 x = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t), y = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t + 8);
+                    v[mt][0] = x.x; v[mt][1] = x.y; v[mt][2] = y.x; v[mt][3] = y.y;
+                    if (!A.talk) { v[mt][0] *= A.scale_log2; v[mt][1] *= A.scale_log2; v[mt][2] *= A.scale_log2; v[mt][3] *= A.scale_log2; }      // else in the matrix
+                }
+                if (!whole) {
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int j = j0 + mt * 16 + (e >> 1) * 8 + (e & 1);
-                    if (!whole && (j < lo || j > pos)) v[mt][e] = -INFINITY;
-                    mx = fmaxf(mx, v[mt][e]);
+                    for (int mt = 0; mt < kMT; ++mt)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const int j = j0 + mt * 16 + (e >> 1) * 8 + (e & 1);
+                            if (j < lo || j > pos) v[mt][e] = -INFINITY;
+                        }
+                }
+#pragma unroll
+                for (int mt = 0; mt < kMT; ++mt) mx = fmaxf(mx, fmaxf(fmaxf(v[mt][0], v[mt][1]), fmaxf(v[mt][2], v[mt][3])));
+                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+                const float mn = fmaxf(m[a], mx), subtr = mn == -INFINITY ? 0.f : mn;
+                const float corr = exp2_fast(m[a] - subtr);
+                m[a] = mn;
+                float sum = 0.f;
+#pragma unroll
+                for (int mt = 0; mt < kMT; ++mt) {
+                    const float p0 = exp2_fast(v[mt][0] - subtr), p1 = exp2_fast(v[mt][1] - subtr), p2 = exp2_fast(v[mt][2] - subtr), p3 = exp2_fast(v[mt][3] - subtr);
+                    sum += (p0 + p1) + (p2 + p3);
+                    pb[a][mt][0] = pack_bf16(p0, p1); pb[a][mt][1] = pack_bf16(p2, p3);
+                }
+                l[a] = fmaf(l[a], corr, sum);
+                if (__any_sync(0xffffffffu, corr != 1.f)) {                // some row's maximum has moved
+                    const float c0 = __shfl_sync(0xffffffffu, corr, 8 * t), c1 = __shfl_sync(0xffffffffu, corr, 8 * t + 4);      // of the accumulators' queries 2t, 2t + 1
+#pragma unroll
+                    for (int n = 0; n < 8; ++n) { o[a][n][0] *= c0; o[a][n][1] *= c1; o[a][n][2] *= c0; o[a][n][3] *= c1; }
                 }
             }
-            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-            const float mn = fmaxf(m[a], mx), subtr = mn == -INFINITY ? 0.f : mn;
-            const float corr = exp2_fast(m[a] - subtr);
-            m[a] = mn;
-            float sum = 0.f;
+            const uint32_t vb = sV + (A.vst == 2 ? (i & 1) * vbytes : 0);
 #pragma unroll
             for (int mt = 0; mt < kMT; ++mt) {
-                const float p0 = exp2_fast(v[mt][0] - subtr), p1 = exp2_fast(v[mt][1] - subtr), p2 = exp2_fast(v[mt][2] - subtr), p3 = exp2_fast(v[mt][3] - subtr);
-                sum += (p0 + p1) + (p2 + p3);
-                pb[a][mt][0] = pack_bf16(p0, p1); pb[a][mt][1] = pack_bf16(p2, p3);
-            }
-            l[a] = fmaf(l[a], corr, sum);
-            if (__any_sync(0xffffffffu, corr != 1.f)) {                // some row's maximum has moved
-                const float c0 = __shfl_sync(0xffffffffu, corr, 8 * t), c1 = __shfl_sync(0xffffffffu, corr, 8 * t + 4);      // of the accumulators' queries 2t, 2t + 1
 #pragma unroll
-                for (int n = 0; n < 8; ++n) { o[a][n][0] *= c0; o[a][n][1] *= c1; o[a][n][2] *= c0; o[a][n][3] *= c1; }
-            }
-        }
-        const uint32_t vb = sV + (A.vst == 2 ? (i & 1) * vbytes : 0);
+                for (int n = 0; n < 8; ++n) {
+                    if (n * 16 >= dv) break;
+                    const uint32_t off = voff[n & 3] + (n >> 2) * 128 + mt * 16 * pv;
+                    uint32_t va[4];
+                    int kv_loaded = -1;
 #pragma unroll
-        for (int mt = 0; mt < kMT; ++mt) {
-#pragma unroll
-            for (int n = 0; n < 8; ++n) {
-                if (n * 16 >= dv) break;
-                const uint32_t off = voff[n & 3] + (n >> 2) * 128 + mt * 16 * pv;
-                uint32_t va[4];
-                int kv_loaded = -1;
-#pragma unroll
-                for (int a = 0; a < kHW; ++a) {
-                    if (h0 + a >= H) continue;
-                    const int kv = kvh[a];
-                    if (kv != kv_loaded) { kv_loaded = kv; ldsm_x4_trans(va, vb + kv * kKT * pv + off); }
-                    mma_bf16(o[a][n], va[0], va[1], va[2], va[3], pb[a][mt][0], pb[a][mt][1]);
+                    for (int a = 0; a < kHW; ++a) {
+                        const int kv = kvh[a];
+                        if (a == 0 || kv != kv_loaded) { kv_loaded = kv; ldsm_x4_trans(va, vb + kv * kKT * pv + off); }
+                        mma_bf16(o[a][n], va[0], va[1], va[2], va[3], pb[a][mt][0], pb[a][mt][1]);
+                    }
                 }
             }
         }
@@ -693,7 +698,7 @@ TcPlan tc_plan(int H, int G, int dk, int dv) {
     for (const auto& c : tries) {
         if (hw == 2 && c[0] != 16) continue;                          // the registers of two heads per warp hold one 16-key piece of scores
         size_t b = (size_t)H * kTcRows * pk + (size_t)c[1] * G * c[0] * pk + (size_t)c[2] * G * c[0] * pv + (size_t)2 * Hp * kTcRows * (c[0] + 4) * 4 +
-                   (size_t)8 * (kTcThreads / (kTcRows * c[0])) * (Hp + 4) * 4;
+                   (size_t)8 * (kTcThreads / (kTcRows * c[0])) * (16 * hw + 4) * 4;
         const size_t outb = (size_t)kTcWarps * kTcRows * ((dv + 31) / 32 * 32 + 4) * 4;
         if (b < outb) b = outb;
         if (b <= 227 * 1024) return TcPlan{hw, c[0], c[1], c[2], pk, pv, b};
