@@ -12,8 +12,9 @@
 //   talking_decode_kernel   the same for few rows over a 16-bit cache, on mma.sync: every head gets a mixed query as long as a cache row.
 //   talking_prefill_kernel  portions of prompts in 16 bits: a block per 8 query rows with ALL heads, mma.sync m16n8k16 with keys (or value columns) on the
 //                           16-row side and queries on the 8-column side, so that 32 heads' accumulators of 128 value columns fit the register file.  A warp
-//                           owns H / 16 heads in both products; raw scores meet in shared memory, a thread mixes one (query, key) pair over all heads in
-//                           f32, and every warp reads its heads' mixed scores back in the operand layout of the second product.  The first product of the
+//                           owns H / 16 heads in both products; raw scores meet in shared memory in f32, are mixed there on the tensor
+//                           cores as sums of three 16-bit parts (all 24 bits of a score), and every warp reads its heads' mixed scores back in the operand
+//                           layout of the second product.  The first product of the
 //                           next tile is issued before the mixing of this one (scores double-buffered), so a tile costs one barrier; keys and values
 //                           arrive by cp.async while earlier tiles are worked on.
 #include <cuda.h>
@@ -395,6 +396,7 @@ talking_prefill_kernel(const TalkTcArgs A) {
     pdl_wait();
     pdl_trigger();
     constexpr int kMT = kKT / 16, kSP = kKT + 4;                       // 16-key pieces per tile; pitch of a score row
+    constexpr int kHP = 16 * kHW, kSH = kTcRows * kSP + 4, kTP = kHP + 8;      // heads rounded up (rows of zeros); pitches of a head's scores and of the mixing matrix
     extern __shared__ __align__(1024) uint8_t smem_tc[];
     const int H = A.H, G = A.G, dk = k128 ? 128 : A.dk, dv = k128 ? 128 : A.dv, pk = k128 ? 256 : A.pk, pv = k128 ? 256 : A.pv, group = H / G;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
@@ -416,11 +418,9 @@ talking_prefill_kernel(const TalkTcArgs A) {
     const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(smem_tc);
     auto lds16 = [&](uint32_t a) { return *reinterpret_cast<const uint4*>(smem_tc + (a - sbase)); };
     const uint32_t sQ = sbase, sK = sQ + H * kTcRows * pk, sV = sK + A.kst * kbytes;
-    float* S = reinterpret_cast<float*>(smem_tc + (sV - sbase) + A.vst * vbytes);                   // [2][Hp][8][kSP]
-    const int Hp = (H + 3) & ~3;                                       // heads rounded up to whole groups of four (rows of zeros)
-    constexpr int tp = 16 * kHW + 4;                                   // row pitch of the mixing matrix
-    const int sstage = Hp * kTcRows * kSP;
-    float* tk = S + 2 * sstage;                                                                      // [8 kNP][tp] talk times scale log2 e, zeros past H
+    float* S = reinterpret_cast<float*>(smem_tc + (sV - sbase) + A.vst * vbytes);                   // [2][kHP][kSH]: rows of kSP floats per query
+    constexpr int sstage = kHP * kSH;
+    __nv_bfloat16* tk = reinterpret_cast<__nv_bfloat16*>(S + 2 * sstage);                            // [kHP][kTP] the mixing matrix, zeros past H
     const int magic_k = (65536 + (dk >> 3) - 1) / (dk >> 3), magic_v = (65536 + (dv >> 3) - 1) / (dv >> 3);
 
     // a tile of keys (or values) of every kv head: a warp takes whole cache rows; rows past the last visible key repeat it (their weight is 0)
@@ -464,11 +464,11 @@ talking_prefill_kernel(const TalkTcArgs A) {
     if (A.kst == 2) load_k(1);
     cp_commit();
     if (A.talk)
-        for (int i = threadIdx.x; i < 8 * (kTcThreads / (kTcRows * kKT)) * tp; i += kTcThreads) {
-            const int h = i / tp, x = i - h * tp;
-            tk[i] = h < H && x < H ? A.talk[h * H + x] * A.scale_log2 : 0.f;
+        for (int i = threadIdx.x; i < kHP * kHP; i += kTcThreads) {
+            const int h = i / kHP, x = i % kHP;
+            tk[h * kTP + x] = __float2bfloat16_rn(h < H && x < H ? A.talk[h * H + x] : 0.f);
         }
-    for (int i = threadIdx.x; i < (Hp - H) * kTcRows * kSP; i += kTcThreads) S[H * kTcRows * kSP + i] = S[sstage + H * kTcRows * kSP + i] = 0.f;
+    for (int i = threadIdx.x; i < (kHP - H) * kSH; i += kTcThreads) S[H * kSH + i] = S[sstage + H * kSH + i] = 0.f;
 
     const int h0 = warp * kHW;
     float o[kHW][8][4];
@@ -519,7 +519,7 @@ talking_prefill_kernel(const TalkTcArgs A) {
 #pragma unroll
         for (int a = 0; a < kHW; ++a) {
             if (h0 + a >= H) continue;
-            float* r0 = Sd + ((h0 + a) * kTcRows + 2 * t) * kSP;
+            float* r0 = Sd + (h0 + a) * kSH + 2 * t * kSP;
 #pragma unroll
             for (int mt = 0; mt < kMT; ++mt) {
                 r0[mt * 16 + g] = acc[a][mt][0];
@@ -529,32 +529,47 @@ talking_prefill_kernel(const TalkTcArgs A) {
             }
         }
     };
-    // every (query, key) pair of score stage st: s'[h] = scale log2 e sum_g talk[h, g] s[g], in place.  kNP lanes of one warp share a pair: all of them read its H
-    // raw scores, then every one writes its share of the heads.
-    constexpr int kNP = kTcThreads / (kTcRows * kKT), kPW = 32 / kNP;
-    static_assert(8 * kNP >= 16 * kHW, "eight heads per lane cover all of them");
+    // score stage st: s'[h] = sum_g talk[h, g] s[g] for every (query, key) pair, in place, on the tensor cores without leaving 32 bits: the mixing matrix is exact in
+    // 16 bits, a score is the sum of three 16-bit numbers (8 bits of its 24 each), their products are exact and are summed in f32.  A warp takes eight
+    // neighbouring keys of one query at a time; nobody else touches those columns.
     auto mix = [&](int st) {
         if (!A.talk) return;
-        const int pair = warp * kPW + lane % kPW, part = lane / kPW;
-        float* col = S + st * sstage + (pair / kKT) * kSP + pair % kKT;
-        float r[8] = {};                                               // heads part, part + kNP, ... of the mixing matrix's padded rows
-        const float* w0 = tk + part * tp;
-#pragma unroll 2
-        for (int x = 0; x < Hp; x += 4) {
-            float s[4];
+        constexpr int kTiles = kTcRows * kKT / 8;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) s[e] = col[(x + e) * kTcRows * kSP];
+        for (int nt = warp; nt < kTiles; nt += kTcWarps) {
+            float* col = S + st * sstage + (nt / (kKT / 8)) * kSP + (nt % (kKT / 8)) * 8;
+            float acc[kHW][4] = {};
 #pragma unroll
-            for (int n = 0; n < 8; ++n) {
-                const float4 w = *reinterpret_cast<const float4*>(w0 + n * kNP * tp + x);
-                r[n] = fmaf(w.x, s[0], fmaf(w.y, s[1], fmaf(w.z, s[2], fmaf(w.w, s[3], r[n]))));
+            for (int ks = 0; ks < kHW; ++ks) {
+                uint32_t part[3][2];
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    float x = col[(ks * 16 + 2 * t + 8 * e) * kSH + g], y = col[(ks * 16 + 2 * t + 8 * e + 1) * kSH + g];
+#pragma unroll
+                    for (int p = 0; p < 3; ++p) {
+                        part[p][e] = pack_bf16(x, y);
+                        x -= __uint_as_float(part[p][e] << 16);
+                        y -= __uint_as_float(part[p][e] & 0xffff0000u);
+                    }
+                }
+#pragma unroll
+                for (int mt = 0; mt < kHW; ++mt) {
+                    const uint32_t* w = reinterpret_cast<const uint32_t*>(tk + (mt * 16 + g) * kTP + ks * 16) + t;
+                    const uint32_t a0 = w[0], a1 = w[4 * kTP], a2 = w[4], a3 = w[4 * kTP + 4];
+#pragma unroll
+                    for (int p = 2; p >= 0; --p) mma_bf16(acc[mt], a0, a1, a2, a3, part[p][0], part[p][1]);
+                }
+            }
+            __syncwarp();
+#pragma unroll
+            for (int mt = 0; mt < kHW; ++mt) {
+                float* r0 = col + (mt * 16 + g) * kSH + 2 * t;                 // rows past H stay zero: the matrix has rows of zeros there
+                *reinterpret_cast<float2*>(r0) = make_float2(acc[mt][0], acc[mt][1]);
+                *reinterpret_cast<float2*>(r0 + 8 * kSH) = make_float2(acc[mt][2], acc[mt][3]);
             }
         }
-        __syncwarp();
-#pragma unroll
-        for (int n = 0; n < 8; ++n)
-            if (part + n * kNP < H) col[(part + n * kNP) * kTcRows * kSP] = r[n];
     };
+
     cp_wait_all();
     __syncthreads();
     scores(0);
@@ -586,14 +601,14 @@ talking_prefill_kernel(const TalkTcArgs A) {
             const bool whole = jt + kKT - 1 <= pos0 && jt >= lo_last;      // every key of the tile is seen by every row
 #pragma unroll
             for (int a = 0; a < kHW; ++a) {
-                const float* row = Sd + (min(h0 + a, H - 1) * kTcRows + g) * kSP;
+                const float* row = Sd + min(h0 + a, H - 1) * kSH + g * kSP;
                 const int j0 = key0 + i * kKT + 2 * t;
                 float v[kMT][4], mx = -INFINITY;
 #pragma unroll
                 for (int mt = 0; mt < kMT; ++mt) {
                     const float2 x = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t), y = *reinterpret_cast<const float2*>(row + mt * 16 + 2 * t + 8);
                     v[mt][0] = x.x; v[mt][1] = x.y; v[mt][2] = y.x; v[mt][3] = y.y;
-                    if (!A.talk) { v[mt][0] *= A.scale_log2; v[mt][1] *= A.scale_log2; v[mt][2] *= A.scale_log2; v[mt][3] *= A.scale_log2; }      // else in the matrix
+                    v[mt][0] *= A.scale_log2; v[mt][1] *= A.scale_log2; v[mt][2] *= A.scale_log2; v[mt][3] *= A.scale_log2;
                 }
                 if (!whole) {
 #pragma unroll
@@ -692,13 +707,13 @@ struct TcPlan { int hw, kt, kst, vst, pk, pv; size_t smem; };
 TcPlan tc_plan(int H, int G, int dk, int dv) {
     TcPlan none{0, 0, 0, 0, 0, 0, 0};
     if (H > 32 || H % G || dk % 8 || dv % 16 || dv > 128 || dk > 256 || (int64_t)G * (dk > dv ? dk : dv) / 8 > 1024) return none;
-    const int hw = H <= 16 ? 1 : 2, Hp = (H + 3) / 4 * 4;
+    const int hw = H <= 16 ? 1 : 2;
     const int pk = (dk * 2 + 127) / 128 * 128, pv = (dv * 2 + 127) / 128 * 128;
     const int tries[6][3] = {{32, 2, 2}, {32, 2, 1}, {16, 2, 2}, {16, 2, 1}, {32, 1, 1}, {16, 1, 1}};
     for (const auto& c : tries) {
         if (hw == 2 && c[0] != 16) continue;                          // the registers of two heads per warp hold one 16-key piece of scores
-        size_t b = (size_t)H * kTcRows * pk + (size_t)c[1] * G * c[0] * pk + (size_t)c[2] * G * c[0] * pv + (size_t)2 * Hp * kTcRows * (c[0] + 4) * 4 +
-                   (size_t)8 * (kTcThreads / (kTcRows * c[0])) * (16 * hw + 4) * 4;
+        size_t b = (size_t)H * kTcRows * pk + (size_t)c[1] * G * c[0] * pk + (size_t)c[2] * G * c[0] * pv + (size_t)2 * 16 * hw * (kTcRows * (c[0] + 4) + 4) * 4 +
+                   (size_t)16 * hw * (16 * hw + 8) * 2;
         const size_t outb = (size_t)kTcWarps * kTcRows * ((dv + 31) / 32 * 32 + 4) * 4;
         if (b < outb) b = outb;
         if (b <= 227 * 1024) return TcPlan{hw, c[0], c[1], c[2], pk, pv, b};

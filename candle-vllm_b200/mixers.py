@@ -637,7 +637,8 @@ class TalkingAttentionMixer:
         self.w_o = w["o"].to(dtype).contiguous()
         self.splits, self.plain = None, False    # runs of keys chosen by the step's shape, kernels by the sizes (tests force a number / the f32-arithmetic kernel)
         # portions of prompts in 16 bits: the tensor-core kernel, when it takes these sizes
-        self.prefill_kernel = ops.talking_prefill_kernel_supported(heads, kv_heads, dk, dv, dtype)
+        self.prefill_kernel = ops.talking_prefill_kernel_supported(heads, kv_heads, dk, dv, dtype) and \
+            (self.talk is None or torch.equal(self.talk, self.talk.to(torch.bfloat16).float()))       # its mixing matrix is a 16-bit operand: exact or not used
         self.cos = self.sin = self.v_cos = self.v_sin = None
         self._device = self.w_in.device
         if rot:

@@ -704,7 +704,7 @@ void mla_paged_attention_window(void* out, const void* q_absorbed, const void* q
  *   > 0).  q f32 [T, H dk]; cache and out F32 or both BF16.  splits > 1: every row's keys are cut into that many runs, part = T * splits * H * (dv + 2) floats.
  *   H <= 64, dv even and <= 256, dk <= 1024.  A BF16 cache with H <= 32, dk and dv multiples of 8 and at most 16 kv heads x 64-column groups takes a tensor-core
  *   kernel (plain != 0: not even then).
- * talking_attention_prefill: the same on tensor cores for portions of prompts: q, cache and out BF16, entry b's rows are cu_seqlens_q[b] .. cu_seqlens_q[b + 1] = the
+ * talking_attention_prefill: the same on tensor cores for portions of prompts: q, cache and out BF16, talk representable in BF16 (it is rounded), entry b's rows are cu_seqlens_q[b] .. cu_seqlens_q[b + 1] = the
  *   last of its cu_seqlens_k[b + 1] - cu_seqlens_k[b] positions.  talking_attention_prefill_supported: 1 if it takes these sizes (H <= 32, dk a multiple of 8, dv a
  *   multiple of 16 and <= 128, tiles that fit shared memory). */
 void post_norm_add_rms_norm(float* x, const float* y, int64_t ldy, const float* y_bias, const float* post_weight, const float* weight, void* out, const int32_t* row_index,
