@@ -52,8 +52,8 @@ def parse():
     ap.add_argument("--arch", default="llama", choices=["llama", "gobesun", "guvusun", "panarax", "dofevik", "sigalorn"],
                     help="llama = the metric (default, unchanged).  gobesun = prefill / decode throughput of the Gobesun decoder at layer sizes of real "
                          "models (random weights), beside a dense bf16 Llama of equal width / heads / ff / depth, with a per-kernel roofline table; "
-                         "one JSON line, single GPU.  guvusun / panarax / dofevik = the same for those decoders (panarax beside a Gobesun, dofevik beside a Guvusun of "
-                         "equal size).")
+                         "one JSON line, single GPU.  guvusun / panarax / dofevik / sigalorn = the same for those decoders (panarax and sigalorn beside a Gobesun, dofevik "
+                         "beside a Guvusun of equal size).")
     ap.add_argument("--arch-sizes", default="w2048,w4096")
     return ap.parse_args()
 
@@ -1659,7 +1659,9 @@ def run_sigalorn(args):
                 "linear_attention[decay]": ("f32", 4.0 * T * H * hd * hd) if pre else ("bytes", T * 4 * H * hd * 4 + state),
                 "linear_attention_channel": ("f32", 4.0 * T * H * hd * hd) if pre else ("bytes", T * 5 * H * hd * 4 + state),
                 "qk_norm_rope_cache": ("bytes", qkv), "qkv_rope_cache": ("bytes", qkv),
-                "paged_attention_varlen_sink": att, "paged_attention_decode_chunked": att, "talking_attention": att,
+                "paged_attention_varlen_sink": att, "paged_attention_decode_chunked": att,
+                # mixing: H more multiply-adds per head, query and key
+                "talking_attention": ("flops", (4.0 * H * hd + 2.0 * H * H) * seen) if pre else att,
                 "softcap": ("bytes", (1 if pre else T) * V * 8),
             }.get(key)
 
@@ -1674,10 +1676,6 @@ def run_sigalorn(args):
                 if w:
                     roof = w[1] / {"bytes": HBM, "flops": TC, "f32": F32}[w[0]]
                     e.update(bound=w[0], roofline_us=round(roof * 1e6, 2), frac_of_roofline=round(roof / t, 3))
-                if key == "talking_attention" and tag == "prefill":
-                    # mixing is 32-bit by definition: H multiply-adds per head, query and key on the FMA pipe, beside the two products on the tensor cores
-                    mix = 2.0 * H * H * sum(i % z["chunk"] + 1 for i in range(T)) / F32
-                    e.update(f32_mixing_roofline_us=round(mix * 1e6, 2), frac_of_mixing_roofline=round(mix / t, 3))
                 out[key] = e
             return out
         side = lambda pre, dec, dec_dev, kern: {

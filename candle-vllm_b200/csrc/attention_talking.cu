@@ -39,9 +39,9 @@ struct TalkArgs {
 };
 
 // cache row of a position (shift >= 0: the block size is 1 << shift, otherwise it is divided by)
-__device__ __forceinline__ int64_t cache_row(const int32_t* table, int j, int bs, int shift) {
+__device__ __forceinline__ int cache_row(const int32_t* table, int j, int bs, int shift) {
     const int b = shift >= 0 ? j >> shift : j / bs;
-    return (int64_t)table[b] * bs + (j - b * bs);
+    return table[b] * bs + (j - b * bs);
 }
 __device__ __forceinline__ int first_visible(int pos, int chunk, int window) {
     int lo = chunk > 0 ? (pos / chunk) * chunk : 0;
@@ -429,7 +429,7 @@ talking_prefill_kernel(const TalkTcArgs A) {
         const __nv_bfloat16* rows_of[kKT / kTcWarps];
 #pragma unroll
         for (int kk = 0; kk < kKT / kTcWarps; ++kk)
-            rows_of[kk] = cache + cache_row(table, min(key0 + tl * kKT + warp + kTcWarps * kk, last_pos), A.bs, A.bs_shift) * G * d;
+            rows_of[kk] = cache + (int64_t)cache_row(table, min(key0 + tl * kKT + warp + kTcWarps * kk, last_pos), A.bs, A.bs_shift) * (G * d);
 #pragma unroll
         for (int kk = 0; kk < kKT / kTcWarps; ++kk) {
             const int key = warp + kTcWarps * kk;
@@ -438,6 +438,7 @@ talking_prefill_kernel(const TalkTcArgs A) {
                 const int c = lane & 15, cs = values ? c ^ (key & 7) : c ^ ((key & 1) << 2);
                 uint32_t at = dst + ((lane >> 4) * kKT + key) * 256 + cs * 16;
                 src += lane * 8;
+#pragma unroll 4
                 for (int p = lane; p < pieces; p += 32, at += 2 * kKT * 256, src += 256) cp16(at, src);
                 continue;
             }
