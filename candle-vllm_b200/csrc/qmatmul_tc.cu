@@ -287,8 +287,8 @@ struct F4Quarter {
 };
 
 // Q6_K staging.  A block = ql[128] | qh[64] | scales i8[16] | d f16 = 210 bytes and is only 2-byte aligned
-// in memory, while a TMA box must START 16-byte aligned (probed on B200: an unaligned start raises "illegal
-// instruction", tools/probes/tma_align_test.cu).  So the box starts at the block address rounded down to 16
+// in memory, while a TMA box must START 16-byte aligned (an unaligned start is an illegal instruction on
+// B200).  So the box starts at the block address rounded down to 16
 // and is 240 bytes wide (15 x 16: an odd number of 16-byte units per row keeps LDS.128 conflict-free); the
 // block then sits off = (210 * sb) % 16 bytes into the row slot, off in {0, 2, .., 14}, uniform per stage.
 // Each thread loads its slot with aligned LDS.128 and realigns the words it needs in registers:
