@@ -43,13 +43,16 @@ SYMBOLS = [
     "mla_paged_attention_window",
     "post_norm_add_rms_norm", "xielu_rows", "softcap_inplace", "low_rank_decay", "linear_attention_channel", "qkv_norm_rope_cache", "talking_attention_rows",
     "talking_attention_prefill_supported", "talking_attention_prefill",
+    "paged_attention_varlen_ex", "token_shift_mix", "low_rank_map", "linear_attention_channel_bonus", "gated_delta_rule_channel", "scaled_post_norm_add",
+    "group_rms_norm_gate_into", "cast_rows_bf16",
 ]
 
 
 # what a library built from one source group (build.GROUPS) exports
 _COMMON = ["b200_abi_version", "b200_last_error", "b200_last_error_message", "b200_device_sm_count", "b200_device_cc", "b200_total_kernel_launches", "linear_16bit",
            "linear_f32out", "rms_norm_ex", "gelu_tanh_mul", "embedding_scaled", "argmax_f32", "rms_norm", "cast", "embedding_positional", "layer_norm_ex",
-           "gated_residual_add", "gated_add_layer_norm", "glu_packed", "group_rms_norm_gate", "head_gate", "add_rms_norm", "post_norm_add_rms_norm", "xielu_rows", "softcap_inplace"]
+           "gated_residual_add", "gated_add_layer_norm", "glu_packed", "group_rms_norm_gate", "head_gate", "add_rms_norm", "post_norm_add_rms_norm", "xielu_rows", "softcap_inplace", "scaled_post_norm_add",
+           "group_rms_norm_gate_into", "cast_rows_bf16"]
 GROUP_SYMBOLS = {
     "ragged": _COMMON + ["causal_conv_silu", "gated_delta_rule", "gated_delta_rule_tiled", "gated_delta_rule_step", "gated_rms_norm", "qk_norm_rope_cache",
                          "paged_attention_varlen", "chunk_decode_view", "paged_attention_decode", "paged_attention_decode_workspace_bytes"],
@@ -64,8 +67,10 @@ GROUP_SYMBOLS = {
                          "latent_q_absorb", "latent_attention_varlen", "latent_out_gate_ex", "repack_heads", "token_tables", "mla_decode_kernel_supported",
                          "mla_paged_attention_sink", "mla_paged_attention_window", "mla_paged_decode_workspace_bytes", "moe_route_bias", "moe_gate_up_ex", "moe_down", "linear_grouped", "moe_align_rows",
                          "moe_align", "moe_gather_rows", "moe_combine_rows"],
-    "talking": _COMMON + ["low_rank_decay", "linear_attention_channel", "linear_attention_chunked_scratch", "qkv_norm_rope_cache", "talking_attention_rows",
+    "talking": _COMMON + ["low_rank_decay", "low_rank_map", "linear_attention_channel", "linear_attention_channel_bonus", "linear_attention_chunked_scratch", "qkv_norm_rope_cache", "talking_attention_rows",
                          "talking_attention_prefill_supported", "talking_attention_prefill"],
+    "sliding": _COMMON + ["causal_conv_ex", "gated_delta_rule_channel", "low_rank_map", "token_shift_mix", "linear_attention_channel_bonus", "linear_attention_chunked_scratch",
+                         "qk_head_norm_rope_cache", "paged_attention_varlen_ex", "linear_grouped"],
 }
 _RESTYPES = {"b200_last_error_message": C.c_char_p, "paged_attention_decode_workspace_bytes": C.c_size_t, "qmatmul_workspace_bytes": C.c_size_t,
              "moe_gemm_workspace_bytes": C.c_size_t, "moe_gemm_fp8_workspace_bytes": C.c_size_t, "mla_paged_decode_workspace_bytes": C.c_size_t,

@@ -51,7 +51,11 @@ GROUPS = {"ragged": ["lib", "linear_generic", "dense_gemm", "norm_act", "gated_d
                      "attention_generic", "attention_api", "latent_attention", "mla", "moe_ragged", "elementwise"],
           # linear attention with a decay per key row beside attention whose heads mix their scores: both linear kernels, norms, the recurrences, the query / key /
           # value preparation (with the paged attention it shares a file with) and the score-mixing attention, argmax
-          "talking": ["lib", "linear_generic", "dense_gemm", "norm_act", "linear_recurrence", "attention_varlen", "attention_prefill", "attention_talking", "elementwise"]}
+          "talking": ["lib", "linear_generic", "dense_gemm", "norm_act", "linear_recurrence", "attention_varlen", "attention_prefill", "attention_talking", "elementwise"],
+          # windowed attention with kept first tokens beside token-shift linear attention or a delta rule with a decay per key row: both linear kernels (the tcgen05 one
+          # also grouped), norms, the recurrences, the per-head preparation, the attention over the paged cache, argmax
+          "sliding": ["lib", "linear_generic", "dense_gemm", "norm_act", "linear_recurrence", "gated_delta", "attention_window", "attention_varlen", "attention_prefill",
+                      "elementwise"]}
 
 
 def so_path(group=None) -> str:

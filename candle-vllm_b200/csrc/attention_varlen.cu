@@ -1,7 +1,7 @@
 // attention_varlen.cu -- softmax attention over the paged cache for ragged steps (portions of prompts beside single decoded
 // tokens in one launch), with separate key and value sizes, an f32 or bf16 cache, and a visibility rule per query:
 //     key j is seen by the query at position i  iff  j <= i, floor(j / chunk) == floor(i / chunk) when chunk > 0, and
-//     i - j < window when window > 0.
+//     i - j < window when window > 0 (or j < keep_first).
 // Chunks and windows are counted in sequence positions, so the result does not depend on where a prompt was cut.
 //
 //   qk_norm_rope_cache      from the packed f32 product [T, H dk | G dk | G dv] of a fused q|k|v projection: RMS norm over the WHOLE
@@ -14,7 +14,9 @@
 //                           all dv entries, and with num_kv_heads = 0 prepares queries alone (a layer that attends over another layer's cache).
 //   paged_attention_varlen  one warp per (token, head); keys in tiles of 32 (a lane scores one key, the tile's values are then
 //                           accumulated with lanes across the value columns), online softmax in f32.  The _sink form puts exp(sink[h]) into
-//                           the denominator of head h (a key without a value; its score is not scaled).
+//                           the denominator of head h (a key without a value; its score is not scaled).  The _ex form adds kept first tokens
+//                           (positions below keep_first never leave the window), a cap on the scores, softcap tanh(s / softcap), one sigmoid gate per
+//                           output entry and an output row pitch.
 #include <stdlib.h>
 
 #include "attention.cuh"
@@ -123,7 +125,8 @@ __global__ void __launch_bounds__(128)
 paged_attention_varlen_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_cache, const TC* __restrict__ v_cache,
                               const int32_t* __restrict__ block_tables, int table_width, const int32_t* __restrict__ token_seq,
                               const int32_t* __restrict__ positions, TOut* __restrict__ out, int64_t items, int H, int G, int dk, int dv,
-                              int block_size, float scale, int chunk, int window, const float* __restrict__ sink) {
+                              int block_size, float scale, int chunk, int window, const float* __restrict__ sink, int keep_first, float softcap,
+                              const float* __restrict__ gate, int64_t ld_gate, int64_t ld_out) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ float qsm[];                  // [4 warps][dk]
@@ -141,14 +144,16 @@ paged_attention_varlen_kernel(const TQ* __restrict__ q, const TC* __restrict__ k
     int lo = 0;
     if (chunk > 0) lo = (pos / chunk) * chunk;
     if (window > 0 && pos - window + 1 > lo) lo = pos - window + 1;
+    // visible positions: the kept first ones that lie before the window, then lo .. pos
+    const int kept = min(keep_first, lo), visible = kept + pos - lo + 1;
     // a sink is a key without a value whose score is sink[h] as it stands: the running maximum and sum start from it
     float m = sink ? sink[h] : -INFINITY, l = sink ? 1.f : 0.f;
     float acc[kMaxVPerLane];
 #pragma unroll
     for (int c = 0; c < kMaxVPerLane; ++c) acc[c] = 0.f;
-    for (int j0 = lo; j0 <= pos; j0 += 32) {
-        const int j = j0 + lane;
-        const bool valid = j <= pos;
+    for (int n0 = 0; n0 < visible; n0 += 32) {
+        const int n = n0 + lane, j = n < kept ? n : lo + n - kept;
+        const bool valid = n < visible;
         int64_t phys = 0;
         float s = -INFINITY;
         if (valid) {
@@ -156,7 +161,7 @@ paged_attention_varlen_kernel(const TQ* __restrict__ q, const TC* __restrict__ k
             const TC* kr = k_cache + (phys * G + g) * dk;
             float d = 0.f;
             for (int i = 0; i < dk; ++i) d = fmaf(qs[i], to_f32<TC>(kr[i]), d);
-            s = d;
+            s = softcap > 0.f ? softcap * tanhf(d / softcap) : d;
         }
         const float m_new = fmaxf(m, warp_max(s));
         const float p = valid ? expf(s - m_new) : 0.f;
@@ -165,7 +170,7 @@ paged_attention_varlen_kernel(const TQ* __restrict__ q, const TC* __restrict__ k
         m = m_new;
 #pragma unroll
         for (int c = 0; c < kMaxVPerLane; ++c) acc[c] *= corr;
-        const int cnt = min(32, pos - j0 + 1);
+        const int cnt = min(32, visible - n0);
         for (int kk = 0; kk < cnt; ++kk) {
             const float pk = __shfl_sync(0xffffffffu, p, kk);
             const int64_t ph = __shfl_sync(0xffffffffu, phys, kk);
@@ -181,7 +186,10 @@ paged_attention_varlen_kernel(const TQ* __restrict__ q, const TC* __restrict__ k
 #pragma unroll
     for (int c = 0; c < kMaxVPerLane; ++c) {
         const int i = lane + 32 * c;
-        if (i < dv) out[((int64_t)t * H + h) * dv + i] = from_f32<TOut>(acc[c] * inv);
+        if (i >= dv) continue;
+        float v = acc[c] * inv;
+        if (gate) v *= 1.0f / (1.0f + expf(-gate[t * ld_gate + (int64_t)h * dv + i]));
+        out[t * ld_out + (int64_t)h * dv + i] = from_f32<TOut>(v);
     }
 }
 
@@ -259,9 +267,19 @@ void paged_attention_varlen_sink(void* out, const void* q, const void* key_cache
                                  const int32_t* cu_seqlens_k, int32_t num_seqs, int32_t num_tokens, int32_t num_heads, int32_t num_kv_heads, int32_t dk,
                                  int32_t dv, int32_t block_size, float scale, int32_t chunk, int32_t window, const float* sink, int32_t q_dtype,
                                  int32_t cache_dtype, int32_t out_dtype, int64_t stream) {
+    paged_attention_varlen_ex(out, (int64_t)num_heads * dv, q, key_cache, value_cache, block_tables, table_width, token_seq, positions, cu_seqlens_q, cu_seqlens_k, num_seqs,
+                              num_tokens, num_heads, num_kv_heads, dk, dv, block_size, scale, chunk, window, 0, 0.f, sink, nullptr, 0, q_dtype, cache_dtype, out_dtype, stream);
+}
+
+void paged_attention_varlen_ex(void* out, int64_t ld_out, const void* q, const void* key_cache, const void* value_cache, const int32_t* block_tables, int32_t table_width,
+                               const int32_t* token_seq, const int32_t* positions, const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, int32_t num_seqs,
+                               int32_t num_tokens, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t block_size, float scale, int32_t chunk,
+                               int32_t window, int32_t keep_first, float softcap, const float* sink, const float* gate, int64_t ld_gate, int32_t q_dtype,
+                               int32_t cache_dtype, int32_t out_dtype, int64_t stream) {
     if (num_tokens == 0) return;
     B200_REQUIRE(out && q && key_cache && value_cache && block_tables && token_seq && positions, kErrBadArg, "paged_attention_varlen: null pointer");
-    B200_REQUIRE(num_heads > 0 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && dk > 0 && dv > 0 && block_size > 0 && table_width > 0,
+    B200_REQUIRE(num_heads > 0 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && dk > 0 && dv > 0 && block_size > 0 && table_width > 0 &&
+                 ld_out >= (int64_t)num_heads * dv && keep_first >= 0 && softcap >= 0.f && (!gate || ld_gate >= (int64_t)num_heads * dv),
                  kErrBadArg, "paged_attention_varlen: bad sizes");
     cudaStream_t st = as_stream(stream);
     // 16-bit q / cache / out with 128-wide heads and 64-token blocks: the tensor-core kernel that serves the other models' prefill
@@ -269,7 +287,7 @@ void paged_attention_varlen_sink(void* out, const void* q, const void* key_cache
     static const bool no_tc = [] { const char* e = getenv("B200_VARLEN_SIMT"); return e && atoi(e) != 0; }();
     PrefillExtras extras;
     extras.sink = sink;
-    if (!no_tc && q_dtype == B200_BF16 && out_dtype == B200_BF16 && dk == dv && cu_seqlens_q && cu_seqlens_k && num_seqs > 0 &&
+    if (!no_tc && keep_first == 0 && softcap == 0.f && !gate && ld_out == (int64_t)num_heads * dv && q_dtype == B200_BF16 && out_dtype == B200_BF16 && dk == dv && cu_seqlens_q && cu_seqlens_k && num_seqs > 0 &&
         paged_attention_prefill_tc_supported(dk, block_size, B200_BF16, cache_dtype, B200_KV_FLASH, 0.f, 1, q, key_cache, value_cache)) {
         paged_attention_prefill_tc(out, q, key_cache, value_cache, (const uint32_t*)block_tables, (const uint32_t*)cu_seqlens_q,
                                    (const uint32_t*)cu_seqlens_k, num_seqs, num_tokens, num_heads, num_kv_heads, table_width, (int64_t)1 << 22, scale,
@@ -282,7 +300,8 @@ void paged_attention_varlen_sink(void* out, const void* q, const void* key_cache
     const unsigned grid = (unsigned)((items + 3) / 4);
     const size_t smem = (size_t)4 * dk * sizeof(float);
 #define PAV(TC, TO, TQ) launch_pdl(paged_attention_varlen_kernel<TC, TO, TQ>, dim3(grid), dim3(128), smem, st, (const TQ*)q, (const TC*)key_cache, \
-        (const TC*)value_cache, block_tables, table_width, token_seq, positions, (TO*)out, items, num_heads, num_kv_heads, dk, dv, block_size, scale, chunk, window, sink)
+        (const TC*)value_cache, block_tables, table_width, token_seq, positions, (TO*)out, items, num_heads, num_kv_heads, dk, dv, block_size, scale, chunk, window, sink, \
+        keep_first, softcap, gate, ld_gate, ld_out)
     if (cache_dtype == B200_F32 && out_dtype == B200_F32 && q_dtype == B200_F32) PAV(float, float, float);
     else if (cache_dtype == B200_BF16 && out_dtype == B200_BF16 && q_dtype == B200_F32) PAV(__nv_bfloat16, __nv_bfloat16, float);
     else if (cache_dtype == B200_BF16 && out_dtype == B200_BF16 && q_dtype == B200_BF16) PAV(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16);

@@ -83,10 +83,11 @@ causal_conv_update_kernel(const float* __restrict__ x, int64_t ldx, float* __res
 // Every sum has a fixed order, so portions of any size give the same state bit for bit.
 constexpr int kTile = 16;
 
-template <int kR>
+// kChan: one decay per token and key row, handed in as `chan` f32 [T, H dk] (S <- diag(g) S); off_a, A_log and dt_bias are then not read.
+template <int kR, bool kChan>
 __global__ void __launch_bounds__(128)
 gated_delta_rule_kernel(const float* __restrict__ qkv, const float* __restrict__ proj, int64_t ld_proj, int off_b, int off_a,
-                        const float* __restrict__ A_log, const float* __restrict__ dt_bias, float* __restrict__ state, float* __restrict__ out,
+                        const float* __restrict__ A_log, const float* __restrict__ dt_bias, const float* __restrict__ chan, float* __restrict__ state, float* __restrict__ out,
                         const int32_t* __restrict__ cu_seqlens, const int32_t* __restrict__ seq_slots, const int32_t* __restrict__ seq_start,
                         int H, int G, int dk, int dv) {
     pdl_wait();
@@ -100,6 +101,7 @@ gated_delta_rule_kernel(const float* __restrict__ qkv, const float* __restrict__
     float* bs = vs + kTile * 16;                      // [kTile] b, then beta
     float* ds = bs + kTile;                           // [kTile] a, then decay
     float* kqs = ds + kTile;                          // [kTile] k . q of the unit vectors
+    float* gs = kqs + kTile;                          // [kTile][kDP] decays of the key rows (kChan only)
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, part = lane >> 2;
     const int b = blockIdx.z, h = blockIdx.y;
     const int col = blockIdx.x * 16 + warp * 4 + (lane & 3);
@@ -123,11 +125,11 @@ gated_delta_rule_kernel(const float* __restrict__ qkv, const float* __restrict__
 #pragma unroll
         for (int r = 0; r < kR; ++r) S[r] = (live && !fresh && row0 + r < dk) ? Sg[r] : 0.f;
     }
-    const float neg_rate = -expf(A_log[h]);
-    const float bias = dt_bias[h];
+    const float neg_rate = kChan ? 0.f : -expf(A_log[h]);
+    const float bias = kChan ? 0.f : dt_bias[h];
     const float qscale = 1.0f / sqrtf((float)dk);
 
-    float rq[kNQ], rk[kNQ], rv[kTile * 16 / 128], ra = 0.f, rb = 0.f;
+    float rq[kNQ], rk[kNQ], rg[kChan ? kNQ : 1], rv[kTile * 16 / 128], ra = 0.f, rb = 0.f;
     auto load_tile = [&](int first, int cnt) {        // global -> registers
 #pragma unroll
         for (int j = 0; j < kNQ; ++j) {
@@ -136,6 +138,7 @@ gated_delta_rule_kernel(const float* __restrict__ qkv, const float* __restrict__
             const float* row = qkv + (int64_t)(first + tt) * C + g * dk + i;
             rq[j] = in ? row[0] : 0.f;
             rk[j] = in ? row[G * dk] : 0.f;
+            if (kChan) rg[kChan ? j : 0] = in ? chan[(int64_t)(first + tt) * H * dk + h * dk + i] : 0.f;
         }
 #pragma unroll
         for (int j = 0; j < kTile * 16 / 128; ++j) {
@@ -144,12 +147,15 @@ gated_delta_rule_kernel(const float* __restrict__ qkv, const float* __restrict__
         }
         if (tid < kTile && tid < cnt) {
             rb = proj[(int64_t)(first + tid) * ld_proj + off_b + h];
-            ra = proj[(int64_t)(first + tid) * ld_proj + off_a + h];
+            if (!kChan) ra = proj[(int64_t)(first + tid) * ld_proj + off_a + h];
         }
     };
     auto store_tile = [&]() {                          // registers -> shared memory
 #pragma unroll
-        for (int j = 0; j < kNQ; ++j) { qs[tid + 128 * j] = rq[j]; ks[tid + 128 * j] = rk[j]; }
+        for (int j = 0; j < kNQ; ++j) {
+            qs[tid + 128 * j] = rq[j]; ks[tid + 128 * j] = rk[j];
+            if (kChan) gs[tid + 128 * j] = rg[kChan ? j : 0];
+        }
 #pragma unroll
         for (int j = 0; j < kTile * 16 / 128; ++j) vs[tid + 128 * j] = rv[j];
         if (tid < kTile) { bs[tid] = rb; ds[tid] = ra; }
@@ -167,7 +173,7 @@ gated_delta_rule_kernel(const float* __restrict__ qkv, const float* __restrict__
             if (lane == 0) {
                 kqs[tt] = qk * qn * kn;
                 bs[tt] = 1.0f / (1.0f + expf(-bs[tt]));
-                ds[tt] = expf(neg_rate * softplus_f(ds[tt] + bias));
+                if (!kChan) ds[tt] = expf(neg_rate * softplus_f(ds[tt] + bias));
             }
         }
     };
@@ -192,7 +198,7 @@ gated_delta_rule_kernel(const float* __restrict__ qkv, const float* __restrict__
         for (int tt = 0; tt < cnt; ++tt) {
             const float4* k4 = reinterpret_cast<const float4*>(ks + tt * kDP + row0);
             const float4* q4 = reinterpret_cast<const float4*>(qs + tt * kDP + row0);
-            const float decay = ds[tt], beta = bs[tt], kq = kqs[tt], v = vs[tt * 16 + warp * 4 + (lane & 3)];
+            const float decay = kChan ? 1.f : ds[tt], beta = bs[tt], kq = kqs[tt], v = vs[tt * 16 + warp * 4 + (lane & 3)];
             // both read-outs of the state as the previous token left it, S0: with S = g S0 + k u^T,
             //   S0^T k -> u = beta (v - g S0^T k)   and   S^T q = g S0^T q + u (k . q),
             // so one butterfly round per token joins both sums and the update is one pass
@@ -202,6 +208,10 @@ gated_delta_rule_kernel(const float* __restrict__ qkv, const float* __restrict__
             for (int r = 0; r < kR; r += 4) {
                 const float4 c = k4[r >> 2], a = q4[r >> 2];
                 kd[r] = c.x; kd[r + 1] = c.y; kd[r + 2] = c.z; kd[r + 3] = c.w;
+                if (kChan) {                             // the decay of every key row first; what follows then reads g S
+                    const float4 gg = reinterpret_cast<const float4*>(gs + tt * kDP + row0)[r >> 2];
+                    S[r] *= gg.x; S[r + 1] *= gg.y; S[r + 2] *= gg.z; S[r + 3] *= gg.w;
+                }
                 p[0] = fmaf(S[r], c.x, p[0]); p[1] = fmaf(S[r + 1], c.y, p[1]); p[2] = fmaf(S[r + 2], c.z, p[2]); p[3] = fmaf(S[r + 3], c.w, p[3]);
                 o[0] = fmaf(S[r], a.x, o[0]); o[1] = fmaf(S[r + 1], a.y, o[1]); o[2] = fmaf(S[r + 2], a.z, o[2]); o[3] = fmaf(S[r + 3], a.w, o[3]);
             }
@@ -232,10 +242,10 @@ gated_delta_rule_kernel(const float* __restrict__ qkv, const float* __restrict__
 // norms, k . q, beta and decay for itself (the q / k rows are a few hundred bytes and stay in L1), and a lane reads its own kR entries
 // of q and k straight from the rows.  No shared memory, no block-wide barrier, ~80 registers: six and more blocks per SM keep the state
 // traffic in flight.  The sums are those of gated_delta_rule_kernel in the same order.
-template <int kR>
+template <int kR, bool kChan>
 __global__ void __launch_bounds__(128)
 gated_delta_step_kernel(const float* __restrict__ qkv, const float* __restrict__ proj, int64_t ld_proj, int off_b, int off_a,
-                        const float* __restrict__ A_log, const float* __restrict__ dt_bias, float* __restrict__ state, float* __restrict__ out,
+                        const float* __restrict__ A_log, const float* __restrict__ dt_bias, const float* __restrict__ chan, float* __restrict__ state, float* __restrict__ out,
                         const int32_t* __restrict__ seq_slots, const int32_t* __restrict__ seq_start, int H, int G, int dk, int dv) {
     pdl_wait();
     pdl_trigger();
@@ -279,6 +289,19 @@ gated_delta_step_kernel(const float* __restrict__ qkv, const float* __restrict__
             qd[r] = in ? qrow[row0 + r] : 0.f;
         }
     }
+    if (kChan) {
+        const float* grow = chan + (int64_t)t * H * dk + h * dk + row0;
+        if (vec && ((H * dk) & 3) == 0) {
+#pragma unroll
+            for (int r = 0; r < kR; r += 4) {
+                const float4 gg = *reinterpret_cast<const float4*>(grow + r);
+                S[r] *= gg.x; S[r + 1] *= gg.y; S[r + 2] *= gg.z; S[r + 3] *= gg.w;
+            }
+        } else {
+#pragma unroll
+            for (int r = 0; r < kR; ++r) S[r] *= row0 + r < dk ? grow[r] : 0.f;
+        }
+    }
     const float v = live ? qkv[(int64_t)t * C + 2 * G * dk + h * dv + col] : 0.f;
     float qq = 0.f, kk = 0.f, qk = 0.f;
     for (int i = lane; i < kDP; i += 32) {
@@ -289,7 +312,7 @@ gated_delta_step_kernel(const float* __restrict__ qkv, const float* __restrict__
     const float qn = (1.0f / sqrtf((float)dk)) / sqrtf(qq + 1e-6f), kn = 1.0f / sqrtf(kk + 1e-6f);
     const float kq = qk * qn * kn;
     const float beta = 1.0f / (1.0f + expf(-proj[(int64_t)t * ld_proj + off_b + h]));
-    const float decay = expf(-expf(A_log[h]) * softplus_f(proj[(int64_t)t * ld_proj + off_a + h] + dt_bias[h]));
+    const float decay = kChan ? 1.f : expf(-expf(A_log[h]) * softplus_f(proj[(int64_t)t * ld_proj + off_a + h] + dt_bias[h]));
     float p[4] = {0.f, 0.f, 0.f, 0.f}, o[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
     for (int r = 0; r < kR; r += 4) {
@@ -695,9 +718,9 @@ void gated_delta_rule(const float* qkv, const float* proj, int64_t ld_proj, int3
     const dim3 grid(ceil_div(dv, 16), num_heads, num_seqs);
 #define GDR(R) do { \
         const int smem = (2 * kTile * 8 * R + kTile * 16 + 3 * kTile) * (int)sizeof(float); \
-        ensure_dynamic_smem(reinterpret_cast<const void*>(gated_delta_rule_kernel<R>), smem); \
-        launch_pdl(gated_delta_rule_kernel<R>, grid, dim3(128), smem, st, qkv, proj, ld_proj, off_b, off_a, A_log, dt_bias, state, out, cu_seqlens, seq_slots, \
-                   seq_start, num_heads, num_kv_heads, dk, dv); } while (0)
+        ensure_dynamic_smem(reinterpret_cast<const void*>(gated_delta_rule_kernel<R, false>), smem); \
+        launch_pdl(gated_delta_rule_kernel<R, false>, grid, dim3(128), smem, st, qkv, proj, ld_proj, off_b, off_a, A_log, dt_bias, (const float*)nullptr, state, out, cu_seqlens, \
+                   seq_slots, seq_start, num_heads, num_kv_heads, dk, dv); } while (0)
     if (dk <= 32) GDR(4);
     else if (dk <= 64) GDR(8);
     else if (dk <= 128) GDR(16);
@@ -718,8 +741,8 @@ void gated_delta_rule_step(const float* qkv, const float* proj, int64_t ld_proj,
     B200_REQUIRE(dk <= 512, kErrUnsupported, "gated_delta_rule_step: key size %d > 512", dk);
     cudaStream_t st = as_stream(stream);
     const dim3 grid(ceil_div(dv, 16), num_heads, num_seqs);
-#define GDS(R) launch_pdl(gated_delta_step_kernel<R>, grid, dim3(128), 0, st, qkv, proj, ld_proj, off_b, off_a, A_log, dt_bias, state, out, seq_slots, seq_start, \
-                          num_heads, num_kv_heads, dk, dv)
+#define GDS(R) launch_pdl(gated_delta_step_kernel<R, false>, grid, dim3(128), 0, st, qkv, proj, ld_proj, off_b, off_a, A_log, dt_bias, (const float*)nullptr, state, out, seq_slots, \
+                          seq_start, num_heads, num_kv_heads, dk, dv)
     if (dk <= 32) GDS(4);
     else if (dk <= 64) GDS(8);
     else if (dk <= 128) GDS(16);
@@ -764,6 +787,37 @@ void gated_delta_rule_tiled(const float* qkv, const float* proj, int64_t ld_proj
 #undef GDT
     count_launch();
     check_launch("gated_delta_rule_tiled");
+}
+
+void gated_delta_rule_channel(const float* qkv, const float* proj, int64_t ld_proj, int32_t off_b, const float* decay, float* state, float* out, float* scratch,
+                              const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t max_rows,
+                              int32_t mode, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int64_t stream) {
+    if (num_seqs == 0 || num_tokens == 0) return;
+    B200_REQUIRE(qkv && proj && decay && state && out && cu_seqlens && seq_slots && seq_start, kErrBadArg, "gated_delta_rule_channel: null pointer");
+    B200_REQUIRE(num_heads > 0 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && dk > 0 && dv > 0 && num_seqs <= 65535 && max_rows > 0 && mode >= 0 && mode <= 2 &&
+                 (mode != 1 || num_tokens == num_seqs), kErrBadArg, "gated_delta_rule_channel: bad sizes");
+    B200_REQUIRE(dk <= 512, kErrUnsupported, "gated_delta_rule_channel: key size %d > 512", dk);
+    cudaStream_t st = as_stream(stream);
+    const dim3 grid(ceil_div(dv, 16), num_heads, num_seqs);
+    const float* none = nullptr;
+#define GDC(R) do { \
+        if (mode == 1) { \
+            launch_pdl(gated_delta_step_kernel<R, true>, grid, dim3(128), 0, st, qkv, proj, ld_proj, off_b, 0, none, none, decay, state, out, seq_slots, seq_start, num_heads, \
+                       num_kv_heads, dk, dv); \
+        } else { \
+            const int smem = (3 * kTile * 8 * R + kTile * 16 + 3 * kTile) * (int)sizeof(float); \
+            ensure_dynamic_smem(reinterpret_cast<const void*>(gated_delta_rule_kernel<R, true>), smem); \
+            launch_pdl(gated_delta_rule_kernel<R, true>, grid, dim3(128), smem, st, qkv, proj, ld_proj, off_b, 0, none, none, decay, state, out, cu_seqlens, seq_slots, seq_start, \
+                       num_heads, num_kv_heads, dk, dv); \
+        } } while (0)
+    if (dk <= 32) GDC(4);
+    else if (dk <= 64) GDC(8);
+    else if (dk <= 128) GDC(16);
+    else if (dk <= 256) GDC(32);
+    else GDC(64);                                      // spills its staging registers: a path for correctness, not speed
+#undef GDC
+    count_launch();
+    check_launch("gated_delta_rule_channel");
 }
 
 void gated_rms_norm(const float* o, const float* gate, int64_t ld_gate, const float* weight, void* out, int32_t num_tokens, int32_t num_heads,

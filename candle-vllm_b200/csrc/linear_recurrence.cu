@@ -18,7 +18,10 @@
 //                                            rides along and o_t = S_t^T q_t / (max(|n_t . q_t|, e^(-m_t)) + 1e-6).  n and m are stored once per
 //                                            block of 16 value columns, so that no block reads what another one writes.
 //   linear_attention_channel  the same with a decay per token AND key row, S_t = diag(a_t) S_(t-1) + k_t v_t^T (a handed in as f32 [T, H dk]).
-//   low_rank_decay        those decays: a = sigmoid(w y + bias)^(1/tau), y a low-rank inner value per token.
+//                         The _bonus form reads a token's output before its decay and write: o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t.
+//   low_rank_map          a second low-rank factor in 32 bits, z = w y + bias (y through tanh or not), as one of: sigmoid(z)^(1/tau), exp(-exp(z)),
+//                         exp(-exp(log_rate) softplus(z)), z.  low_rank_decay is the first of them.
+//   token_shift_mix       several copies of a row, each moved its own way towards the previous token's row (which is part of the state).
 //                         A block of four warps owns 16 value columns of one head of one entry; inside a warp the key rows are split eight
 //                         ways (lane = 4 * part + column) with the lane's rows of S (and of n) in registers; tokens come in tiles of 16
 //                         staged through shared memory with the activation already applied, the per-token coefficients worked out once
@@ -408,7 +411,7 @@ constexpr int kScanSplitRows = 16;     // entries with at least this many rows: 
 
 struct LinAttnArgs {
     const float* proj; int64_t ld;
-    int off_q, off_k, off_v, off_i, off_f;      // columns of proj: q, k [H dk], v [H dv], gate pre-activations [H] (exponential gating only)
+    int64_t off_q, off_k, off_v; int off_i, off_f;      // columns of proj: q, k [H dk], v [H dv], gate pre-activations [H] (exponential gating only)
     const float* decay;                          // [H] (fixed decay)
     const float* i_bias; const float* f_bias;    // [H]
     float cap, q_scale; int act;
@@ -417,15 +420,17 @@ struct LinAttnArgs {
     const int32_t* cu_seqlens; const int32_t* seq_slots; const int32_t* seq_start;
     int H, dk, dv;
     const float* alpha; int64_t lda;             // [T, H dk] row pitch lda: one decay per token and key row (channel decay)
+    const float* bonus;                          // [H, dk]: the output is read before the token joins the state, which it enters with this weight (channel decay)
 };
 
-// kG: 0 = a fixed decay per head, 1 = exponential gating, 2 = a decay per key row and token
+// kG: 0 = a fixed decay per head, 1 = exponential gating, 2 = a decay per key row and token, 3 = the same with the output read BEFORE the token's decay and
+// write: o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t
 template <int kR, int kG>
 __global__ void __launch_bounds__(128)
 linear_attention_kernel(const LinAttnArgs A) {
     pdl_wait();
     pdl_trigger();
-    constexpr bool kExp = kG == 1, kChan = kG == 2;
+    constexpr bool kExp = kG == 1, kChan = kG >= 2, kBonus = kG == 3;
     constexpr int kP = 8 * kR;                   // padded key rows
     extern __shared__ __align__(16) float smem[];
     float* sq = smem;                            // [kTile][kP]
@@ -476,6 +481,11 @@ linear_attention_kernel(const LinAttnArgs A) {
     }
     if (kExp && threadIdx.x == 0) sm[0] = fresh ? 0.f : A.mx[own];
     const float fixed_a = kG == 0 ? A.decay[h] : 0.f;
+    float bo[kBonus ? kR : 1];
+    if (kBonus) {
+#pragma unroll
+        for (int r = 0; r < kR; ++r) bo[kBonus ? r : 0] = part * kR + r < dk ? A.bonus[h * dk + part * kR + r] : 0.f;
+    }
     // the next tile's operands travel in registers while the current tile is walked: element e = thread + 128 i of the tile's [16][kP] q and k
     // rows, two of its [16][16] values, and (lanes 0..15 of the last warp) the two gate pre-activations of a token
     float pq[kR], pk[kR], pal[kChan ? kR : 1], pv[2], pgi = 0.f, pgf = 0.f;
@@ -557,8 +567,10 @@ linear_attention_kernel(const LinAttnArgs A) {
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     const int r = r4 * 4 + j;
-                    S[r] = fmaf(da[j], S[r], ka[j] * bv);
-                    acc[j & 1] = fmaf(S[r], qa[j], acc[j & 1]);
+                    const float kv = ka[j] * bv;
+                    if (kBonus) acc[j & 1] = fmaf(fmaf(bo[kBonus ? r : 0], kv, S[r]), qa[j], acc[j & 1]);
+                    S[r] = fmaf(da[j], S[r], kv);
+                    if (!kBonus) acc[j & 1] = fmaf(S[r], qa[j], acc[j & 1]);
                     if (kExp) { nv[r] = fmaf(a, nv[r], ka[j] * bn); nq[j & 1] = fmaf(nv[r], qa[j], nq[j & 1]); }
                 }
             }
@@ -616,7 +628,7 @@ __global__ void __launch_bounds__(128)
 linear_attention_step_kernel(const LinAttnArgs A) {
     pdl_wait();
     pdl_trigger();
-    constexpr bool kExp = kG == 1, kChan = kG == 2;
+    constexpr bool kExp = kG == 1, kChan = kG >= 2, kBonus = kG == 3;
     const int h = blockIdx.y, b = blockIdx.z;
     const int H = A.H, dk = A.dk, dv = A.dv;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -678,8 +690,10 @@ linear_attention_step_kernel(const LinAttnArgs A) {
         float qv = q[r], kv = k[r];
         if (A.act == 1) { qv = silu_f(qv); kv = silu_f(kv); }
         qv *= A.q_scale;
-        S[r] = fmaf(kChan ? al[r] : a, S[r], kv * bv);
-        acc[r & 1] = fmaf(S[r], qv, acc[r & 1]);
+        const float kvv = kv * bv;
+        if (kBonus) acc[r & 1] = fmaf(fmaf(part * kR + r < dk ? A.bonus[h * dk + part * kR + r] : 0.f, kvv, S[r]), qv, acc[r & 1]);
+        S[r] = fmaf(kChan ? al[kChan ? r : 0] : a, S[r], kvv);
+        if (!kBonus) acc[r & 1] = fmaf(S[r], qv, acc[r & 1]);
         if (kExp) { nv[r] = fmaf(a, nv[r], kv * bw); nq[r & 1] = fmaf(nv[r], qv, nq[r & 1]); }
     }
     float o = acc[0] + acc[1], nqs = nq[0] + nq[1];
@@ -1109,10 +1123,18 @@ la_chunk_output_kernel(const ChunkArgs C) {
 //     score of t over j    sum_r q_t P_t (prod_{runs between} E) R_j k_j, j in an earlier run; inside one run the products of at most three decays
 //     entering state       q_t P_t prod_{runs before} E against S_in                                      (la_chan_output_kernel)
 // The walk over the chunks is la_chunk_scan_kernel with the chunk's product per key row in place of the scalar decay.
+// what becomes of z = w y + bias: 0 = sigmoid(z)^(1 / tau); 1 = exp(-exp(z)); 2 = exp(-exp(log_rate) softplus(z)); 3 = z itself
+__device__ __forceinline__ float low_rank_value(float z, int form, float inv_tau, float log_rate) {
+    if (form == 0) return expf(log_sigmoid_f(z) * inv_tau);
+    if (form == 1) return expf(-expf(z));
+    if (form == 2) return expf(-expf(log_rate) * (fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)))));
+    return z;
+}
+
 template <int kTok>
 __global__ void __launch_bounds__(256)
 low_rank_decay_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ alpha, int T, int N,
-                      int R, float inv_tau) {
+                      int R, float inv_tau, int in_tanh, int form, const float* __restrict__ log_rate, int channels_per_rate) {
     pdl_wait();
     pdl_trigger();
     // 256 channels x kTok tokens per block: a thread keeps 16 weights of its channel at a time and meets the tokens' inner values with them
@@ -1139,7 +1161,8 @@ low_rank_decay_kernel(const float* __restrict__ y, int64_t ldy, const float* __r
         __syncthreads();
         for (int e = threadIdx.x; e < kTok * 16; e += 256) {
             const int i = e >> 4, r = e & 15;
-            ys[i][r] = (t0 + i < T && r0 + r < R) ? y[(int64_t)(t0 + i) * ldy + r0 + r] : 0.f;
+            const float v = (t0 + i < T && r0 + r < R) ? y[(int64_t)(t0 + i) * ldy + r0 + r] : 0.f;
+            ys[i][r] = in_tanh ? tanhf(v) : v;
         }
         __syncthreads();
 #pragma unroll
@@ -1151,9 +1174,10 @@ low_rank_decay_kernel(const float* __restrict__ y, int64_t ldy, const float* __r
             }
     }
     if (n >= N) return;
+    const float lr = form == 2 ? log_rate[n / channels_per_rate] : 0.f;
 #pragma unroll
     for (int i = 0; i < kTok; ++i)
-        if (t0 + i < T) alpha[(int64_t)(t0 + i) * N + n] = expf(log_sigmoid_f(z[i]) * inv_tau);
+        if (t0 + i < T) alpha[(int64_t)(t0 + i) * N + n] = low_rank_value(z[i], form, inv_tau, lr);
 }
 
 __global__ void __launch_bounds__(256)
@@ -1223,6 +1247,9 @@ la_chan_state_kernel(const ChunkArgs C) {
 constexpr int kRunPitch = 257;                   // floats per key row of the table of run products: 16 x 16, padded against bank conflicts
 constexpr int kChanOutFloats = 3 * 32 * 68 + 2 * 64 * 68 + 32 * 17;
 
+// kBonus: the output is read before the token's own decay and write, so the products of decays leave out the query's token and a token meets its own key and
+// value with the bonus weight
+template <bool kBonus>
 __global__ void __launch_bounds__(256, 2)
 la_chan_output_kernel(const ChunkArgs C) {
     pdl_wait();
@@ -1248,8 +1275,9 @@ la_chan_output_kernel(const ChunkArgs C) {
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     // a thread prepares two runs (warp and warp + 8) of one key row (lane) per slab; the next slab's operands are fetched ahead
-    float rq[2][4], rk[2][4], ra[2][4], ru[8];
+    float rq[2][4], rk[2][4], ra[2][4], ru[8], rbo = 0.f;
     auto fetch = [&](int r0) {
+        if (kBonus) rbo = r0 + lane < dk ? A.bonus[h * dk + r0 + lane] : 0.f;
 #pragma unroll
         for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -1277,7 +1305,11 @@ la_chan_output_kernel(const ChunkArgs C) {
             const int a = warp + 8 * i;
             float p = 1.f, q4[4], k4[4];
 #pragma unroll
-            for (int t = 0; t < 4; ++t) { p *= ra[i][t]; q4[t] = rq[i][t] * p; }
+            for (int t = 0; t < 4; ++t) {
+                if (kBonus) q4[t] = rq[i][t] * p;
+                p *= ra[i][t];
+                if (!kBonus) q4[t] = rq[i][t] * p;
+            }
             es[lane * 17 + a] = p;
             float s = 1.f;
 #pragma unroll
@@ -1290,8 +1322,9 @@ la_chan_output_kernel(const ChunkArgs C) {
                 float kj = rk[i][j];
 #pragma unroll
                 for (int t = j; t < 4; ++t) {
-                    if (t > j) kj *= ra[i][t];
-                    dg[i][n] = fmaf(rq[i][t], kj, dg[i][n]);
+                    if (!kBonus && t > j) kj *= ra[i][t];
+                    dg[i][n] = fmaf(rq[i][t], kBonus && t == j ? kj * rbo : kj, dg[i][n]);
+                    if (kBonus && t > j) kj *= ra[i][t];
                     ++n;
                 }
             }
@@ -1386,13 +1419,73 @@ la_chan_output_kernel(const ChunkArgs C) {
     }
 }
 
+// ---- every token moved part of the way towards the token before it -------------------------------------------------------------------------------
+// out[m, t] = x[t] + (x[t - 1] - x[t]) * mu[m], m = 0 .. mixes - 1, one slab of slab_rows rows per mix; the row before a portion's first comes from
+// state [slots, dim] (zero for a new sequence), which then takes the portion's last row: the thread that reads a channel of the state for an entry's first
+// row is the one that writes it.  A block walks `rows` rows of kV x 128 channels with the weights and the previous row in registers.
+constexpr int kMaxMixes = 8;
+template <typename TOut, int kV>
+__global__ void __launch_bounds__(128)
+token_shift_mix_kernel(const float* __restrict__ x, int64_t ldx, const float* __restrict__ mu, float* __restrict__ state, TOut* __restrict__ out, int64_t slab_rows,
+                       const int32_t* __restrict__ token_seq, const int32_t* __restrict__ cu_seqlens, const int32_t* __restrict__ seq_slots,
+                       const int32_t* __restrict__ seq_start, int T, int dim, int mixes, int rows) {
+    pdl_wait();
+    pdl_trigger();
+    const int c = (blockIdx.x * 128 + threadIdx.x) * kV;
+    if (c >= dim) return;
+    const int t_begin = blockIdx.y * rows, t_end = min(T, t_begin + rows);
+    auto load = [&](const float* p, float (&v)[kV]) {
+        if constexpr (kV == 4) { const float4 f = *reinterpret_cast<const float4*>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+        else v[0] = *p;
+    };
+    float m[kMaxMixes][kV], prev[kV];
+#pragma unroll
+    for (int i = 0; i < kMaxMixes; ++i)
+        if (i < mixes) load(mu + (int64_t)i * dim + c, m[i]);
+    bool have_prev = false;
+    for (int t = t_begin; t < t_end; ++t) {
+        const int b = token_seq[t], first = cu_seqlens[b];
+        float cur[kV];
+        load(x + (int64_t)t * ldx + c, cur);
+        if (t == first) {
+            float* st = state + (int64_t)seq_slots[b] * dim + c;
+            if (seq_start[b] == 0) {
+#pragma unroll
+                for (int j = 0; j < kV; ++j) prev[j] = 0.f;
+            } else {
+                load(st, prev);
+            }
+            float last[kV];
+            load(x + (int64_t)(cu_seqlens[b + 1] - 1) * ldx + c, last);
+#pragma unroll
+            for (int j = 0; j < kV; ++j) st[j] = last[j];
+        } else if (!have_prev) {
+            load(x + (int64_t)(t - 1) * ldx + c, prev);
+        }
+        have_prev = true;
+#pragma unroll
+        for (int i = 0; i < kMaxMixes; ++i) {
+            if (i >= mixes) break;
+            TOut o[kV];
+#pragma unroll
+            for (int j = 0; j < kV; ++j) o[j] = from_f32<TOut>(fmaf(prev[j] - cur[j], m[i][j], cur[j]));
+            TOut* dst = out + ((int64_t)i * slab_rows + t) * dim + c;
+            if constexpr (kV == 1) *dst = o[0];
+            else if constexpr (sizeof(TOut) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(o);
+            else *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(o);
+        }
+#pragma unroll
+        for (int j = 0; j < kV; ++j) prev[j] = cur[j];
+    }
+}
+
 template <int kR, int kG>
 void launch_linear_attention(const LinAttnArgs& A, int num_seqs, bool single_rows, cudaStream_t st) {
     if (single_rows) {
         launch_pdl(linear_attention_step_kernel<kR, kG>, dim3(ceil_div(A.dv, 16), A.H, num_seqs), dim3(128), 0, st, A);
         return;
     }
-    const int smem = ((kG == 2 ? 3 : 2) * kTile * 8 * kR + kTile * 16 + 6 * kTile + 1) * (int)sizeof(float);
+    const int smem = ((kG >= 2 ? 3 : 2) * kTile * 8 * kR + kTile * 16 + 6 * kTile + 1) * (int)sizeof(float);
     ensure_dynamic_smem(reinterpret_cast<const void*>(linear_attention_kernel<kR, kG>), smem);
     launch_pdl(linear_attention_kernel<kR, kG>, dim3(ceil_div(A.dv, 16), A.H, num_seqs), dim3(128), (size_t)smem, st, A);
 }
@@ -1531,7 +1624,7 @@ void linear_attention(const float* proj, int64_t ld, int32_t off_q, int32_t off_
                  "linear_attention: fixed decay needs decay[H]; exponential gating needs the normaliser, the maximum and a positive cap");
     B200_REQUIRE(dk <= 512, kErrUnsupported, "linear_attention: key size %d > 512", dk);
     LinAttnArgs A{proj, ld, off_q, off_k, off_v, off_i, off_f, decay, i_bias, f_bias, gate_cap, q_scale, act, state, normaliser, maximum, out,
-                  cu_seqlens, seq_slots, seq_start, num_heads, dk, dv, nullptr, 0};
+                  cu_seqlens, seq_slots, seq_start, num_heads, dk, dv, nullptr, 0, nullptr};
     cudaStream_t st = as_stream(stream);
     if (gating == 0) dispatch_linear_attention<0>(A, num_seqs, single_rows != 0, st);
     else dispatch_linear_attention<1>(A, num_seqs, single_rows != 0, st);
@@ -1560,7 +1653,7 @@ void linear_attention_chunked(const float* proj, int64_t ld, int32_t off_q, int3
     const int64_t slots = (int64_t)(num_tokens + kChunk - 1) / kChunk + num_seqs;
     ChunkArgs C;
     C.A = LinAttnArgs{proj, ld, off_q, off_k, off_v, off_i, off_f, decay, i_bias, f_bias, gate_cap, q_scale, act, state, normaliser, maximum, out,
-                      cu_seqlens, seq_slots, seq_start, num_heads, dk, dv, nullptr, 0};
+                      cu_seqlens, seq_slots, seq_start, num_heads, dk, dv, nullptr, 0, nullptr};
     C.U = scratch;
     C.un = C.U + slots * num_heads * dv * dk;
     C.un_in = C.un + slots * num_heads * dk;
@@ -1587,32 +1680,71 @@ void linear_attention_chunked(const float* proj, int64_t ld, int32_t off_q, int3
 
 void low_rank_decay(const float* y, int64_t ldy, const float* weight, const float* bias, float* alpha, int32_t num_tokens, int32_t channels, int32_t rank, float tau,
                     int64_t stream) {
+    low_rank_map(y, ldy, weight, bias, alpha, num_tokens, channels, rank, 0, 0, tau, nullptr, 1, stream);
+}
+
+void low_rank_map(const float* y, int64_t ldy, const float* weight, const float* bias, float* out, int32_t num_tokens, int32_t channels, int32_t rank, int32_t in_tanh,
+                  int32_t form, float tau, const float* log_rate, int32_t channels_per_rate, int64_t stream) {
     if (num_tokens == 0) return;
-    B200_REQUIRE(y && weight && alpha && channels > 0 && rank > 0 && ldy >= rank && tau > 0.f && num_tokens <= 32 * 65535, kErrBadArg, "low_rank_decay: bad arguments");
+    B200_REQUIRE(y && weight && out && channels > 0 && rank > 0 && ldy >= rank && num_tokens <= 32 * 65535 && form >= 0 && form <= 3 && (form != 0 || tau > 0.f) &&
+                 (form != 2 || (log_rate && channels_per_rate > 0 && channels % channels_per_rate == 0)), kErrBadArg, "low_rank_map: bad arguments");
     cudaStream_t st = as_stream(stream);
-    if (num_tokens <= 256)                       // few rows: short blocks, many of them
-        launch_pdl(low_rank_decay_kernel<2>, dim3(ceil_div(channels, 256), ceil_div(num_tokens, 2)), dim3(256), 0, st, y, ldy, weight, bias, alpha, (int)num_tokens,
-                   (int)channels, (int)rank, 1.0f / tau);
+    const float inv_tau = form == 0 ? 1.0f / tau : 0.f;
+    // few rows: short blocks, many of them
+    const int tok = num_tokens <= 256 ? 2 : 32;
+    const dim3 grid(ceil_div(channels, 256), ceil_div(num_tokens, tok));
+    if (tok == 2)
+        launch_pdl(low_rank_decay_kernel<2>, grid, dim3(256), 0, st, y, ldy, weight, bias, out, (int)num_tokens, (int)channels, (int)rank, inv_tau, (int)in_tanh, (int)form,
+                   log_rate, (int)channels_per_rate);
     else
-        launch_pdl(low_rank_decay_kernel<32>, dim3(ceil_div(channels, 256), ceil_div(num_tokens, 32)), dim3(256), 0, st, y, ldy, weight, bias, alpha, (int)num_tokens,
-                   (int)channels, (int)rank, 1.0f / tau);
+        launch_pdl(low_rank_decay_kernel<32>, grid, dim3(256), 0, st, y, ldy, weight, bias, out, (int)num_tokens, (int)channels, (int)rank, inv_tau, (int)in_tanh, (int)form,
+                   log_rate, (int)channels_per_rate);
     count_launch();
-    check_launch("low_rank_decay");
+    check_launch("low_rank_map");
+}
+
+void token_shift_mix(const float* x, int64_t ldx, const float* mu, float* state, void* out, int64_t slab_rows, const int32_t* token_seq, const int32_t* cu_seqlens,
+                     const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens, int32_t dim, int32_t mixes, int32_t out_dtype, int64_t stream) {
+    if (num_tokens == 0) return;
+    B200_REQUIRE(x && mu && state && out && token_seq && cu_seqlens && seq_slots && seq_start && dim > 0 && ldx >= dim && slab_rows >= num_tokens && mixes >= 1 && mixes <= kMaxMixes,
+                 kErrBadArg, "token_shift_mix: bad arguments (1 to %d mixes)", kMaxMixes);
+    B200_REQUIRE(out_dtype == B200_F32 || out_dtype == B200_BF16, kErrUnsupported, "token_shift_mix: out dtype %d (f32 / bf16)", out_dtype);
+    const bool vec = dim % 4 == 0 && ldx % 4 == 0 && (((uintptr_t)x | (uintptr_t)mu | (uintptr_t)state | (uintptr_t)out) & 15) == 0;
+    const int rows = num_tokens <= 256 ? 1 : 8;
+    const dim3 grid(ceil_div(dim, vec ? 512 : 128), ceil_div(num_tokens, rows));
+    cudaStream_t st = as_stream(stream);
+#define TSM(TO, V) launch_pdl(token_shift_mix_kernel<TO, V>, grid, dim3(128), 0, st, x, ldx, mu, state, (TO*)out, slab_rows, token_seq, cu_seqlens, seq_slots, seq_start, \
+                              (int)num_tokens, (int)dim, (int)mixes, rows)
+    if (out_dtype == B200_F32) { if (vec) TSM(float, 4); else TSM(float, 1); }
+    else { if (vec) TSM(__nv_bfloat16, 4); else TSM(__nv_bfloat16, 1); }
+#undef TSM
+    count_launch();
+    check_launch("token_shift_mix");
 }
 
 void linear_attention_channel(const float* proj, int64_t ld, int32_t off_q, int32_t off_k, int32_t off_v, const float* alpha, int64_t lda, float q_scale, float* state,
                               float* out, float* scratch, const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens,
                               int32_t num_seqs, int32_t max_rows, int32_t mode, int32_t num_heads, int32_t dk, int32_t dv, int64_t stream) {
+    linear_attention_channel_bonus(proj, ld, off_q, off_k, off_v, alpha, lda, nullptr, q_scale, state, out, scratch, cu_seqlens, seq_slots, seq_start, num_tokens, num_seqs,
+                                   max_rows, mode, num_heads, dk, dv, stream);
+}
+
+void linear_attention_channel_bonus(const float* proj, int64_t ld, int64_t off_q, int64_t off_k, int64_t off_v, const float* alpha, int64_t lda, const float* bonus,
+                                    float q_scale, float* state, float* out, float* scratch, const int32_t* cu_seqlens, const int32_t* seq_slots,
+                                    const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t max_rows, int32_t mode, int32_t num_heads, int32_t dk,
+                                    int32_t dv, int64_t stream) {
     if (num_seqs == 0 || num_tokens == 0) return;
     B200_REQUIRE(proj && alpha && state && out && cu_seqlens && seq_slots && seq_start && num_heads > 0 && num_heads <= 65535 && num_seqs <= 65535 && dk > 0 && dv > 0 &&
                  lda >= (int64_t)num_heads * dk && mode >= 0 && mode <= 2, kErrBadArg, "linear_attention_channel: bad arguments");
+    // the three operands may be columns of one matrix or matrices of their own with one pitch: an offset is anything from the first to the last element
     LinAttnArgs A{proj, ld, off_q, off_k, off_v, 0, 0, nullptr, nullptr, nullptr, 0.f, q_scale, 0, state, nullptr, nullptr, out,
-                  cu_seqlens, seq_slots, seq_start, num_heads, dk, dv, alpha, lda};
+                  cu_seqlens, seq_slots, seq_start, num_heads, dk, dv, alpha, lda, bonus};
     cudaStream_t st = as_stream(stream);
     if (mode != 2) {
         B200_REQUIRE(mode == 0 || num_tokens == num_seqs, kErrBadArg, "linear_attention_channel: the single-row kernel takes one row per entry");
         B200_REQUIRE(dk <= 512, kErrUnsupported, "linear_attention_channel: key size %d > 512", dk);
-        dispatch_linear_attention<2>(A, num_seqs, mode == 1, st);
+        if (bonus) dispatch_linear_attention<3>(A, num_seqs, mode == 1, st);
+        else dispatch_linear_attention<2>(A, num_seqs, mode == 1, st);
         count_launch();
         check_launch("linear_attention_channel");
         return;
@@ -1631,8 +1763,9 @@ void linear_attention_channel(const float* proj, int64_t ld, int32_t off_q, int3
     launch_pdl(la_chan_state_kernel, dim3(ceil_div(dv, 64) * ceil_div(dk, 64), num_heads, z), dim3(256), 0, st, C);
     launch_pdl(la_chunk_scan_kernel, dim3(ceil_div((int64_t)num_heads * dv * dk, 256), num_seqs), dim3(256), 0, st, C);
     const int smem = kChanOutFloats * (int)sizeof(float);
-    ensure_dynamic_smem(reinterpret_cast<const void*>(la_chan_output_kernel), smem);
-    launch_pdl(la_chan_output_kernel, dim3(ceil_div(dv, 64), num_heads, z), dim3(256), (size_t)smem, st, C);
+    void (*output)(const ChunkArgs) = bonus ? la_chan_output_kernel<true> : la_chan_output_kernel<false>;
+    ensure_dynamic_smem(reinterpret_cast<const void*>(output), smem);
+    launch_pdl(output, dim3(ceil_div(dv, 64), num_heads, z), dim3(256), (size_t)smem, st, C);
     count_launch(3);
     check_launch("linear_attention_channel");
 }

@@ -25,9 +25,11 @@
 //                    one group per head or one for the whole row;
 //   head_gate        out[t, h, :] = src[t, h, :] * sigmoid(gate[t, h]): one gate per attention head;
 //   post_norm_add_rms_norm  x <- x + rms(y + y_bias) * w_post, then out = rms(x) * w: the norm AFTER a sublayer, its sum and the norm before the next
-//                    sublayer in one pass (with `row_index` only the selected rows, x left as it is; w null = the sum alone);
+//                    sublayer in one pass (with `row_index` only the selected rows, x left as it is; w null = the sum alone); the scaled_ form takes
+//                    y times a factor (before the bias) and, with w null and an `out`, also leaves the new x there in the compute dtype;
 //   xielu_rows       out = xIELU(x + bias): pos z^2 + z / 2 for z > 0, neg (e^z - 1 - z) + z / 2 otherwise;
-//   softcap_inplace  x <- cap tanh(x / cap).
+//   softcap_inplace  x <- cap tanh(x / cap);
+//   cast_rows_bf16   out = x for rows with a pitch of their own.
 // Any row length (no vector-width rule): the rows these models use are a few hundred to a few thousand floats and every kernel
 // here is one pass over them from L2.
 #include "common.cuh"
@@ -252,7 +254,7 @@ __global__ void glu_packed_kernel(const float* __restrict__ gu, TOut* __restrict
 template <typename TOut>
 __global__ void __launch_bounds__(128)
 group_rms_norm_gate_kernel(const float* __restrict__ o, int64_t ldo, const float* __restrict__ w, const float* __restrict__ gate, int64_t ldg, TOut* __restrict__ out,
-                           int n, int glen, float eps, int gate_act) {
+                           int64_t ld_out, int glen, float eps, int gate_act) {
     pdl_wait();
     pdl_trigger();
     __shared__ float red[4];
@@ -271,7 +273,7 @@ group_rms_norm_gate_kernel(const float* __restrict__ o, int64_t ldo, const float
             const float z = gate[t * ldg + c0 + i];
             v *= gate_act == 0 ? 1.0f / (1.0f + expf(-z)) : z / (1.0f + expf(-z));
         }
-        out[t * n + c0 + i] = from_f32<TOut>(v);
+        out[t * ld_out + c0 + i] = from_f32<TOut>(v);
     }
 }
 
@@ -280,7 +282,7 @@ group_rms_norm_gate_kernel(const float* __restrict__ o, int64_t ldo, const float
 template <typename TOut, int kV>
 __global__ void __launch_bounds__(256)
 group_rms_norm_gate_warp_kernel(const float* __restrict__ o, int64_t ldo, const float* __restrict__ w, const float* __restrict__ gate, int64_t ldg, TOut* __restrict__ out,
-                                int64_t items, int groups, int n, int glen, float eps, int gate_act) {
+                                int64_t items, int groups, int64_t ld_out, int glen, float eps, int gate_act) {
     pdl_wait();
     pdl_trigger();
     const int64_t item = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -309,7 +311,7 @@ group_rms_norm_gate_warp_kernel(const float* __restrict__ o, int64_t ldo, const 
             for (int j = 0; j < 4; ++j) r[j] *= (gate_act == 0 ? 1.0f : zz[j]) / (1.0f + expf(-zz[j]));
         }
         TOut q[4] = {from_f32<TOut>(r[0]), from_f32<TOut>(r[1]), from_f32<TOut>(r[2]), from_f32<TOut>(r[3])};
-        TOut* dst = out + t * n + c0 + i;
+        TOut* dst = out + t * ld_out + c0 + i;
         if (sizeof(TOut) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(q);
         else *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(q);
     }
@@ -430,7 +432,7 @@ relu2_rows_kernel(const float* __restrict__ x, TOut* __restrict__ out, int ff, i
 template <typename TOut, int kV>
 __global__ void __launch_bounds__(256)
 post_norm_add_rms_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int64_t ldy, const float* __restrict__ y_bias, const float* __restrict__ w_post,
-                              const float* __restrict__ w, TOut* __restrict__ out, const int32_t* __restrict__ row_index, int n, float eps) {
+                              const float* __restrict__ w, TOut* __restrict__ out, const int32_t* __restrict__ row_index, int n, float eps, float y_scale) {
     pdl_wait();
     pdl_trigger();
     __shared__ float red[8];
@@ -447,6 +449,7 @@ post_norm_add_rms_norm_kernel(float* __restrict__ x, const float* __restrict__ y
             yv[v] = xv[v] = make_float4(0.f, 0.f, 0.f, 0.f);
             if (i < n) {
                 yv[v] = *reinterpret_cast<const float4*>(yr + i);
+                yv[v].x *= y_scale; yv[v].y *= y_scale; yv[v].z *= y_scale; yv[v].w *= y_scale;
                 xv[v] = *reinterpret_cast<const float4*>(xr + i);
                 if (y_bias) {
                     const float4 bv = *reinterpret_cast<const float4*>(y_bias + i);
@@ -468,12 +471,12 @@ post_norm_add_rms_norm_kernel(float* __restrict__ x, const float* __restrict__ y
             ss = fmaf(xv[v].x, xv[v].x, fmaf(xv[v].y, xv[v].y, fmaf(xv[v].z, xv[v].z, fmaf(xv[v].w, xv[v].w, ss))));
         }
         if (!out) return;
-        const float sx = 1.0f / sqrtf(block_sum_256(ss, red) / (float)n + eps);
+        const float sx = w ? 1.0f / sqrtf(block_sum_256(ss, red) / (float)n + eps) : 1.0f;
 #pragma unroll
         for (int v = 0; v < kV; ++v) {
             const int i = (threadIdx.x + 256 * v) * 4;
             if (i >= n) continue;
-            const float4 wv = *reinterpret_cast<const float4*>(w + i);
+            const float4 wv = w ? *reinterpret_cast<const float4*>(w + i) : make_float4(1.f, 1.f, 1.f, 1.f);
             const float r[4] = {xv[v].x * sx * wv.x, xv[v].y * sx * wv.y, xv[v].z * sx * wv.z, xv[v].w * sx * wv.w};
             TOut o[4];
 #pragma unroll
@@ -482,19 +485,21 @@ post_norm_add_rms_norm_kernel(float* __restrict__ x, const float* __restrict__ y
             else *reinterpret_cast<uint2*>(out + (int64_t)row * n + i) = *reinterpret_cast<const uint2*>(o);
         }
     } else {
-        for (int i = threadIdx.x; i < n; i += 256) { const float v = yr[i] + (y_bias ? y_bias[i] : 0.f); ss = fmaf(v, v, ss); }
+        auto y_at = [&](int i) { return fmaf(yr[i], y_scale, y_bias ? y_bias[i] : 0.f); };
+        for (int i = threadIdx.x; i < n; i += 256) { const float v = y_at(i); ss = fmaf(v, v, ss); }
         const float sy = 1.0f / sqrtf(block_sum_256(ss, red) / (float)n + eps);
         ss = 0.f;
         for (int i = threadIdx.x; i < n; i += 256) {
-            const float v = xr[i] + (yr[i] + (y_bias ? y_bias[i] : 0.f)) * sy * w_post[i];
+            const float v = xr[i] + y_at(i) * sy * w_post[i];
             if (!row_index) xr[i] = v;
+            if (out && !w) out[(int64_t)row * n + i] = from_f32<TOut>(v);
             ss = fmaf(v, v, ss);
         }
-        if (!out) return;
+        if (!out || !w) return;
         const float sx = 1.0f / sqrtf(block_sum_256(ss, red) / (float)n + eps);
         for (int i = threadIdx.x; i < n; i += 256) {
             float v = xr[i];
-            if (row_index) v += (yr[i] + (y_bias ? y_bias[i] : 0.f)) * sy * w_post[i];     // x was not updated: form the sum again
+            if (row_index) v += y_at(i) * sy * w_post[i];                                   // x was not updated: form the sum again
             out[(int64_t)row * n + i] = from_f32<TOut>(v * sx * w[i]);
         }
     }
@@ -524,6 +529,15 @@ xielu_rows_kernel(const float* __restrict__ x, int64_t ld, const float* __restri
     } else {
         for (int i = 0; i < 4 && c + i < ff; ++i) dst[i] = from_f32<TOut>(xielu_f(src[i] + (bias ? bias[c + i] : 0.f), pos, neg));
     }
+}
+
+__global__ void cast_rows_kernel(const float* __restrict__ x, int64_t ldx, __nv_bfloat16* __restrict__ out, int64_t ld_out, int64_t total, int n) {
+    pdl_wait();
+    pdl_trigger();
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total) return;
+    const int64_t r = i / n;
+    out[r * ld_out + (i - r * n)] = __float2bfloat16_rn(x[r * ldx + (i - r * n)]);
 }
 
 __global__ void softcap_kernel(float* __restrict__ x, int64_t total, float cap) {
@@ -690,17 +704,22 @@ void glu_packed(const float* gate_up, void* out, int64_t rows, int32_t ff, int64
 
 void group_rms_norm_gate(const float* o, int64_t ldo, const float* weight, const float* gate, int64_t ld_gate, void* out, int32_t num_tokens, int32_t n,
                          int32_t groups, float eps, int32_t gate_act, int32_t out_dtype, int64_t stream) {
+    group_rms_norm_gate_into(o, ldo, weight, gate, ld_gate, out, n, num_tokens, n, groups, eps, gate_act, out_dtype, stream);
+}
+
+void group_rms_norm_gate_into(const float* o, int64_t ldo, const float* weight, const float* gate, int64_t ld_gate, void* out, int64_t ld_out, int32_t num_tokens, int32_t n,
+                              int32_t groups, float eps, int32_t gate_act, int32_t out_dtype, int64_t stream) {
     if (num_tokens == 0) return;
-    B200_REQUIRE(o && out && n > 0 && groups > 0 && n % groups == 0 && ldo >= n && (!gate || ld_gate >= n) && groups <= 65535 && (gate_act == 0 || gate_act == 1),
+    B200_REQUIRE(o && out && n > 0 && groups > 0 && n % groups == 0 && ldo >= n && ld_out >= n && (!gate || ld_gate >= n) && groups <= 65535 && (gate_act == 0 || gate_act == 1),
                  kErrBadArg, "group_rms_norm_gate: bad arguments");
     cudaStream_t st = as_stream(stream);
     const int glen = n / groups;
-    const bool vec = glen % 4 == 0 && glen <= 1024 && ldo % 4 == 0 && (!gate || ld_gate % 4 == 0) &&
-                     (((uintptr_t)o | (uintptr_t)weight | (uintptr_t)gate | (uintptr_t)out) & 15) == 0 && (out_dtype == B200_F32 || out_dtype == B200_BF16);
+    const bool vec = glen % 4 == 0 && glen <= 1024 && ldo % 4 == 0 && ld_out % 4 == 0 && (!gate || ld_gate % 4 == 0) &&
+                     (((uintptr_t)o | (uintptr_t)weight | (uintptr_t)gate) & 15) == 0 && ((uintptr_t)out & (out_dtype == B200_F32 ? 15 : 7)) == 0 && (out_dtype == B200_F32 || out_dtype == B200_BF16);
     if (vec) {
         const int64_t items = (int64_t)num_tokens * groups;
         const dim3 g8((unsigned)((items + 7) / 8));
-#define GRW(TO, KV) launch_pdl(group_rms_norm_gate_warp_kernel<TO, KV>, g8, dim3(256), 0, st, o, ldo, weight, gate, ld_gate, (TO*)out, items, (int)groups, (int)n, glen, eps, (int)gate_act)
+#define GRW(TO, KV) launch_pdl(group_rms_norm_gate_warp_kernel<TO, KV>, g8, dim3(256), 0, st, o, ldo, weight, gate, ld_gate, (TO*)out, items, (int)groups, ld_out, glen, eps, (int)gate_act)
 #define GRW_ALL(TO) do { if (glen <= 128) GRW(TO, 1); else if (glen <= 256) GRW(TO, 2); else if (glen <= 512) GRW(TO, 4); else GRW(TO, 8); } while (0)
         if (out_dtype == B200_F32) GRW_ALL(float);
         else GRW_ALL(__nv_bfloat16);
@@ -712,9 +731,9 @@ void group_rms_norm_gate(const float* o, int64_t ldo, const float* weight, const
     }
     const dim3 grid(groups, num_tokens);
     if (out_dtype == B200_F32)
-        launch_pdl(group_rms_norm_gate_kernel<float>, grid, dim3(128), 0, st, o, ldo, weight, gate, ld_gate, (float*)out, n, n / groups, eps, gate_act);
+        launch_pdl(group_rms_norm_gate_kernel<float>, grid, dim3(128), 0, st, o, ldo, weight, gate, ld_gate, (float*)out, ld_out, n / groups, eps, gate_act);
     else if (out_dtype == B200_BF16)
-        launch_pdl(group_rms_norm_gate_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, o, ldo, weight, gate, ld_gate, (__nv_bfloat16*)out, n, n / groups, eps, gate_act);
+        launch_pdl(group_rms_norm_gate_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, o, ldo, weight, gate, ld_gate, (__nv_bfloat16*)out, ld_out, n / groups, eps, gate_act);
     else { set_error(kErrUnsupported, "group_rms_norm_gate: out dtype %d (f32 / bf16)", out_dtype); return; }
     count_launch();
     check_launch("group_rms_norm_gate");
@@ -766,15 +785,20 @@ void add_rms_norm(float* x, const float* y1, int64_t ld1, const float* y2, int64
 
 void post_norm_add_rms_norm(float* x, const float* y, int64_t ldy, const float* y_bias, const float* post_weight, const float* weight, void* out, const int32_t* row_index,
                             int32_t rows, int32_t n, float eps, int32_t out_dtype, int64_t stream) {
+    B200_REQUIRE((weight == nullptr) == (out == nullptr), kErrBadArg, "post_norm_add_rms_norm: weight and out come together");
+    scaled_post_norm_add(x, y, ldy, 1.0f, y_bias, post_weight, weight, out, row_index, rows, n, eps, out_dtype, stream);
+}
+
+void scaled_post_norm_add(float* x, const float* y, int64_t ldy, float y_scale, const float* y_bias, const float* post_weight, const float* weight, void* out,
+                          const int32_t* row_index, int32_t rows, int32_t n, float eps, int32_t out_dtype, int64_t stream) {
     if (rows == 0) return;
-    B200_REQUIRE(x && y && post_weight && rows > 0 && n > 0 && ldy >= n && ((weight == nullptr) == (out == nullptr)) && (out || !row_index), kErrBadArg,
-                 "post_norm_add_rms_norm: bad arguments");
+    B200_REQUIRE(x && y && post_weight && rows > 0 && n > 0 && ldy >= n && (out || !weight) && (out || !row_index), kErrBadArg, "post_norm_add_rms_norm: bad arguments");
     B200_REQUIRE(!out || out_dtype == B200_F32 || out_dtype == B200_BF16, kErrUnsupported, "post_norm_add_rms_norm: out dtype %d (f32 / bf16)", out_dtype);
     const bool vec = n % 4 == 0 && ldy % 4 == 0 &&
                      (((uintptr_t)x | (uintptr_t)y | (uintptr_t)y_bias | (uintptr_t)post_weight | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
     const int kv = !vec ? 0 : n <= 1024 ? 1 : n <= 2048 ? 2 : n <= 4096 ? 4 : n <= 8192 ? 8 : 0;
     cudaStream_t st = as_stream(stream);
-#define PNA(TO, KV) launch_pdl(post_norm_add_rms_norm_kernel<TO, KV>, dim3(rows), dim3(256), 0, st, x, y, ldy, y_bias, post_weight, weight, (TO*)out, row_index, (int)n, eps)
+#define PNA(TO, KV) launch_pdl(post_norm_add_rms_norm_kernel<TO, KV>, dim3(rows), dim3(256), 0, st, x, y, ldy, y_bias, post_weight, weight, (TO*)out, row_index, (int)n, eps, y_scale)
 #define PNA_ALL(TO) do { if (kv == 1) PNA(TO, 1); else if (kv == 2) PNA(TO, 2); else if (kv == 4) PNA(TO, 4); else if (kv == 8) PNA(TO, 8); else PNA(TO, 0); } while (0)
     if (!out || out_dtype == B200_F32) PNA_ALL(float);
     else PNA_ALL(__nv_bfloat16);
@@ -795,6 +819,15 @@ void xielu_rows(const float* x, int64_t ld, const float* bias, void* out, int32_
     else { set_error(kErrUnsupported, "xielu_rows: out dtype %d (f32 / bf16)", out_dtype); return; }
     count_launch();
     check_launch("xielu_rows");
+}
+
+void cast_rows_bf16(const float* x, int64_t ldx, void* out, int64_t ld_out, int32_t rows, int32_t n, int64_t stream) {
+    if (rows == 0 || n == 0) return;
+    B200_REQUIRE(x && out && rows > 0 && n > 0 && ldx >= n && ld_out >= n, kErrBadArg, "cast_rows_bf16: bad arguments");
+    const int64_t total = (int64_t)rows * n;
+    launch_pdl(cast_rows_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, as_stream(stream), x, ldx, (__nv_bfloat16*)out, ld_out, total, (int)n);
+    count_launch();
+    check_launch("cast_rows_bf16");
 }
 
 void softcap_inplace(float* x, int64_t total, float cap, int64_t stream) {

@@ -19,7 +19,11 @@ kernels of ``seq_ops``.  Sizes and constants are constructor arguments so that a
   ChannelDecayLinearAttention  linear attention with a decay per token and key row from a low-rank map, per-head norm times a SiLU gate
   TalkingAttentionMixer  softmax attention whose heads mix their scores, values cached turned by their position, optionally over another layer's cache
                        (csrc/attention_talking.cu)
+  TokenShiftLinearAttention  linear attention whose projections each read their own mix of a token and the one before it, decays exp(-exp(.)) per token and
+                       key row, a bonus weight for the current token, per-head norm times a SiLU gate
+  ChannelDecayDeltaMixer  the gated delta rule with a decay per token and key row and a low-rank sigmoid gate on the normed heads (csrc/gated_delta.cu)
   ParallelMixer        two mixers side by side on one input (one fused projection), half the sum of their normed outputs
+  ParallelSumMixer     two mixers side by side, a scaled sum of their outputs as they are (one fused input and one fused output projection)
 
 Activations that feed a matrix product are of the model's compute dtype (bf16 or f32); products come back in f32 and everything
 between them (norms, convolution, recurrence, softmax) is 32-bit.
@@ -100,12 +104,17 @@ class PagedAttentionMixer:
 
     ``head_norm`` "before" / "after": q and k are normed head by head over dk, before or after the rotation (q.norm / k.norm are then [dk], shared by the
     heads, or absent for a norm without weight); ``interleaved``: the rotation pairs neighbours (2i, 2i + 1) instead of (i, i + dims/2); biases q.b / k.b /
-    v.b are added in the projection; sink [H]: exp(sink[h]) joins the softmax denominator of head h (a key without a value whose score is not scaled)."""
+    v.b are added in the projection; sink [H]: exp(sink[h]) joins the softmax denominator of head h (a key without a value whose score is not scaled).
+
+    ``keep_first``: keys at positions below it stay visible whatever the window; ``softcap``: scores become softcap tanh(s / softcap); ``gate`` "element": g is
+    [H dv, D], one sigmoid gate per output entry; a bias o.b [D] is left to the caller (``out_bias``), who adds it where the output is read next."""
     kind = "kv"
 
     def __init__(self, w: Dict[str, torch.Tensor], heads: int, kv_heads: int, dk: int, dv: int, scale: float, eps: float, dtype: torch.dtype,
                  rot: Optional[dict] = None, chunk: int = 0, window: int = 0, block_size: int = 64, max_pos: int = 4096, q_temp: Optional[dict] = None,
-                 value_norm: bool = False, head_norm: str = "none", interleaved: bool = False):
+                 value_norm: bool = False, head_norm: str = "none", interleaved: bool = False, keep_first: int = 0, softcap: float = 0.0, gate: str = "head"):
+        if gate not in ("head", "element") or keep_first < 0 or softcap < 0:
+            raise BackendError(f"PagedAttentionMixer: gate {gate!r} (head / element), keep_first {keep_first}, softcap {softcap}")
         if heads % kv_heads:
             raise BackendError("PagedAttentionMixer: heads must be a multiple of kv_heads")
         if head_norm not in ("none", "before", "after") or (head_norm != "none" and (q_temp or value_norm)):
@@ -123,6 +132,14 @@ class PagedAttentionMixer:
         if self.per_head and (q_temp or value_norm):
             raise BackendError("PagedAttentionMixer: biases / neighbour pairs do not combine with a query temperature or normed values")
         self.has_gate = "g" in w
+        self.keep_first, self.softcap, self.element_gate = int(keep_first), float(softcap), gate == "element" and self.has_gate
+        want = {"q": heads * dk, "k": kv_heads * dk, "v": kv_heads * dv, **({"g": heads * (dv if gate == "element" else 1)} if self.has_gate else {})}
+        for name, n in want.items():
+            if w[name].shape[0] != n:
+                raise BackendError(f"PagedAttentionMixer: {name} is {tuple(w[name].shape)}, expected {n} rows")
+        if tuple(w["o"].shape)[1] != heads * dv:
+            raise BackendError(f"PagedAttentionMixer: o {tuple(w['o'].shape)} for {heads} heads of {dv}")
+        self.out_bias = w["o.b"].float().contiguous() if "o.b" in w else None
         self.off_g = heads * dk + kv_heads * (dk + dv)
         self.w_in = torch.cat([w["q"], w["k"], w["v"]] + ([w["g"]] if self.has_gate else []), 0).to(dtype).contiguous()
         self.q_temp = (float(q_temp["coef"]), int(q_temp["every"])) if q_temp else None
@@ -155,17 +172,30 @@ class PagedAttentionMixer:
 
     def forward(self, h: torch.Tensor, batch: StepBatch, cache, proj: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``proj``: the product of ``w_in`` with the input when the caller has it already (columns of a wider fused projection)"""
+        return ops.linear(self.attend(h, batch, cache, proj), self.w_o)
+
+    def attend(self, h: torch.Tensor, batch: StepBatch, cache, proj: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """What the output projection reads, [T, H dv] in the compute dtype (into ``out``, row stride allowed, when given)"""
         k_cache, v_cache = cache
         if self.rot and batch.max_position >= self.cos.shape[0]:
             self.ensure_positions(max(2 * self.cos.shape[0], batch.max_position + 1))
         if proj is None:
             proj = ops.linear(h, self.w_in)
+        selected = out is not None or self.keep_first > 0 or self.softcap > 0 or self.element_gate
+        if selected and self.has_gate and not self.element_gate:
+            raise BackendError("PagedAttentionMixer: one gate per head does not combine with kept tokens, a score cap or a given output")
+        q_dtype = torch.float32 if selected else self.q_dtype
         if self.per_head:
             q = ops.qk_head_norm_rope_cache(proj, self.bias, self.q_norm, self.k_norm, self.cos, self.sin, batch, k_cache, v_cache, self.H, self.G, self.dk, self.dv,
-                                            self.rot_dims, self.eps, interleaved=self.interleaved, norm=self.head_norm, q_dtype=self.q_dtype)
+                                            self.rot_dims, self.eps, interleaved=self.interleaved, norm=self.head_norm, q_dtype=q_dtype)
         else:
             q = ops.qk_norm_rope_cache(proj, self.q_norm, self.k_norm, self.cos, self.sin, batch, k_cache, v_cache, self.H, self.G, self.dk, self.dv,
-                                       self.rot_dims, self.eps, self.q_dtype, q_temp=self.q_temp, v_unit_rms=self.value_norm)
+                                       self.rot_dims, self.eps, q_dtype, q_temp=self.q_temp, v_unit_rms=self.value_norm)
+        if selected:
+            if out is None:
+                out = torch.empty((q.shape[0], self.H * self.dv), dtype=self.dtype, device=q.device)
+            return ops.paged_attention_selected(q, k_cache, v_cache, batch, self.H, self.scale, self.chunk, self.window, self.keep_first, self.softcap, self.sink,
+                                                proj[:, self.off_g:self.off_g + self.H * self.dv] if self.element_gate else None, out)
         if self.decode_kernel and batch.pure_decode and batch.num_seqs <= 256:
             # without a chunk mask the whole table is one chunk
             a = ops.paged_attention_decode_chunked(q, k_cache, v_cache, batch, self.H, self.G, self.dk, self.block_size, self.scale,
@@ -177,7 +207,7 @@ class PagedAttentionMixer:
                                                 self.window, self.sink, torch.float32 if (self.has_gate and self.q_dtype == torch.float32) else self.dtype)
         if self.has_gate:
             a = ops.head_gate(a, proj[:, self.off_g:], self.H, self.dv, self.dtype)
-        return ops.linear(a, self.w_o)
+        return a
 
 
 class PooledWindowAttentionMixer:
@@ -229,12 +259,13 @@ class PooledWindowAttentionMixer:
 
 
 class GatedMlp:
-    """down(act(gate x) * (up x)), act the tanh GELU or SiLU; gate, up [ff, D], down [D, ff]."""
+    """down(act(gate x) * (up x)), act the tanh GELU or SiLU, or "clamped": down(g sigmoid(1.702 g) (u + 1)) with g = min(gate x, limit), u = clamp(up x, +-limit);
+    gate, up [ff, D], down [D, ff]."""
 
-    def __init__(self, w: Dict[str, torch.Tensor], dtype: torch.dtype, act: str = "gelu_tanh"):
-        if act not in ("gelu_tanh", "silu"):
+    def __init__(self, w: Dict[str, torch.Tensor], dtype: torch.dtype, act: str = "gelu_tanh", limit: float = 0.0):
+        if act not in ("gelu_tanh", "silu", "clamped"):
             raise BackendError(f"GatedMlp: unknown activation {act!r}")
-        self.dtype, self.act = dtype, act
+        self.dtype, self.act, self.limit = dtype, act, float(limit)
         self.w_in = torch.cat([w["gate"], w["up"]], 0).to(dtype).contiguous()
         self.w_down = w["down"].to(dtype).contiguous()
 
@@ -244,7 +275,7 @@ class GatedMlp:
             proj = ops.linear(h, self.w_in)
         if self.act == "gelu_tanh":
             return ops.linear(ops.gelu_tanh_mul(proj, self.dtype), self.w_down)
-        return ops.linear(ops.glu_packed(proj, self.act, self.dtype), self.w_down)
+        return ops.linear(ops.glu_packed(proj, self.act, self.dtype, self.limit), self.w_down)
 
 
 class UngatedMlp:
@@ -692,3 +723,162 @@ class ParallelMixer:
         b = self.right.forward(h, batch, state, proj=proj[:, self.split:])
         y = ops.rms_norm_ex(a, self.left_out, self.eps, 0.0, torch.float32)
         return ops.rms_norm_ex(b, self.right_out, self.eps, 0.0, torch.float32, residual=y, out=y)
+
+
+class TokenShiftLinearAttention:
+    """Linear attention over shifted tokens.  With x' the previous token's x (zeros before the first), each of r, k, v, g, w reads x + (x' - x) mu.*; r, k, v = W of their
+    mixes [H n], w = exp(-exp(w2 tanh(w1 mix_w) + w0)) per token and key row; per head o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t, then S_t = diag(w_t) S_(t-1) + k_t v_t^T;
+    each head's o over its root mean square, times norm [H n], times silu(W_g mix_g), then o [D, H n].  The mixes are formed from the f32 stream, the second map of the
+    decay runs in 32 bits whatever the compute dtype.  ``norm_scale`` multiplies the norm's weight."""
+    kind = "state"
+    w_in = None                                  # no projection of the plain input: every one reads a mix of its own
+
+    def __init__(self, w: Dict[str, torch.Tensor], heads: int, dim: int, eps: float, dtype: torch.dtype, norm_scale: float = 1.0):
+        self.H, self.n, self.eps, self.dtype = heads, dim, eps, dtype
+        N = self.N = heads * dim
+        self.D = w["r"].shape[1]
+        self.rank = w["w1"].shape[0]
+        for name in ("r", "k", "v", "g", "w2"):
+            if w[name].shape[0] != N:
+                raise BackendError(f"TokenShiftLinearAttention: {name} is {tuple(w[name].shape)}, expected {N} rows")
+        if w["w2"].shape[1] != self.rank or w["w0"].numel() != N or w["u"].numel() != N or w["norm"].numel() != N or tuple(w["o"].shape)[1] != N:
+            raise BackendError(f"TokenShiftLinearAttention: w2 {tuple(w['w2'].shape)} / w0 / u / norm / o {tuple(w['o'].shape)} for {heads} x {dim}")
+        self.mu = torch.stack([w["mu." + a].float().flatten() for a in "rkvgw"], 0).contiguous()
+        self.w_mix = torch.stack([w[a] for a in "rkvg"], 0).to(dtype).contiguous()             # [4, N, D]
+        self.w1 = w["w1"].to(dtype).contiguous()
+        self.w2, self.w0, self.u = w["w2"].float().contiguous(), w["w0"].float().flatten().contiguous(), w["u"].float().flatten().contiguous()
+        self.norm = (w["norm"].float().flatten() * norm_scale).contiguous()
+        self.w_o = w["o"].to(dtype).contiguous()
+        # bf16, TMA-sized operands: the four products of the mixes run as ONE grouped product, every mix padded to whole row tiles
+        self.grouped = dtype == torch.bfloat16 and self.D % 8 == 0 and N % 8 == 0 and self.D >= 64 and N >= 64
+        self._tile_mix = {}
+        self.kernel = None                       # None: chosen by the step's shape (tests force one)
+
+    def state_shapes(self):
+        return ((self.D,), (self.H, self.n, self.n))
+
+    def forward(self, x: torch.Tensor, batch: StepBatch, cache) -> torch.Tensor:
+        return ops.linear(self.attend(x, batch, cache), self.w_o)
+
+    def attend(self, x: torch.Tensor, batch: StepBatch, cache, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """x: the input rows in f32.  What the output projection reads, [T, H n] in the compute dtype (into ``out``, row stride allowed, when given)"""
+        prev, S = cache
+        T = x.shape[0]
+        tile = 1 if not self.grouped else 32 if T <= 32 else 64 if T <= 64 else 128
+        Tp = -(-T // tile) * tile
+        mix = ops.token_shift_mix(x, self.mu, prev, batch, torch.empty((5, Tp, self.D), dtype=self.dtype, device=x.device))
+        rkvg = torch.empty((4 * Tp, self.N), dtype=torch.float32, device=x.device)
+        if self.grouped:
+            if (Tp, tile) not in self._tile_mix:
+                self._tile_mix[Tp, tile] = (torch.arange(4 * Tp // tile, dtype=torch.int32, device=x.device) // (Tp // tile)).to(torch.int32)
+            ops.linear_grouped(mix[:4].view(4 * Tp, self.D), self.w_mix, self._tile_mix[Tp, tile], rkvg, tile)
+        else:
+            for i in range(4):
+                ops.linear(mix[i, :T], self.w_mix[i], out=rkvg[i * Tp:i * Tp + T])
+        w = ops.low_rank_map(ops.linear(mix[4, :T], self.w1), self.w2, self.w0, "double_exp", in_tanh=True)
+        o = ops.linear_attention_channel(rkvg, 0, Tp * self.N, 2 * Tp * self.N, w, S, batch, self.H, self.n, self.n, kernel=self.kernel, bonus=self.u, rows=T)
+        return ops.group_rms_norm_gate(o, self.norm, rkvg[3 * Tp:3 * Tp + T], self.H, self.eps, self.dtype, gate_act="silu", out=out)
+
+
+LOW_RANK_GATE_ROWS = 256          # steps with more rows take the second factor of the output gate on the tensor cores (bf16)
+
+
+class ChannelDecayDeltaMixer:
+    """The gated delta rule with a decay per token and key row.  q, k = W h [G dk], v = W h [H dv], each through a short causal convolution and SiLU; q and k unit vectors
+    per head (q also times dk^-1/2); beta = sigmoid(b h) per head; g = exp(-exp(A_log) softplus(a2 (a1 h) + dt_bias)) [H dk]; per head S <- diag(g) S; u = beta (v - S^T k);
+    S <- S + k u^T; o = S^T q; each head's o over its root mean square, times norm [dv] (shared by the heads), times sigmoid(g2 (g1 h)) [H dv], then o [D, H dv].
+    weights: q, k, v, b, a1 [rank, D], a2 [H dk, rank], g1 [rank', D], g2 [H dv, rank'], A_log [H], dt_bias [H dk], q.conv / k.conv / v.conv [channels, taps], norm, o.
+    The second map of the decay runs in 32 bits whatever the compute dtype.  ``norm_scale`` multiplies the norm's weight."""
+    kind = "state"
+
+    def __init__(self, w: Dict[str, torch.Tensor], heads: int, kv_heads: int, dk: int, dv: int, taps: int, eps: float, dtype: torch.dtype, norm_scale: float = 1.0):
+        if heads % kv_heads:
+            raise BackendError("ChannelDecayDeltaMixer: heads must be a multiple of kv_heads")
+        self.H, self.G, self.dk, self.dv, self.taps, self.eps, self.dtype = heads, kv_heads, dk, dv, taps, eps, dtype
+        self.N, self.C = heads * dv, 2 * kv_heads * dk + heads * dv
+        self.ra, self.rg = w["a1"].shape[0], w["g1"].shape[0]
+        want = {"q": kv_heads * dk, "k": kv_heads * dk, "v": heads * dv, "b": heads, "a2": heads * dk, "g2": heads * dv}
+        for name, n in want.items():
+            if w[name].shape[0] != n:
+                raise BackendError(f"ChannelDecayDeltaMixer: {name} is {tuple(w[name].shape)}, expected {n} rows")
+        if (w["a2"].shape[1] != self.ra or w["g2"].shape[1] != self.rg or w["A_log"].numel() != heads or w["dt_bias"].numel() != heads * dk or w["norm"].numel() != dv
+                or tuple(w["o"].shape)[1] != self.N):
+            raise BackendError(f"ChannelDecayDeltaMixer: a2 {tuple(w['a2'].shape)} / g2 {tuple(w['g2'].shape)} / A_log / dt_bias / norm / o {tuple(w['o'].shape)}")
+        self.w_in = torch.cat([w["q"], w["k"], w["v"], w["a1"], w["g1"], w["b"]], 0).to(dtype).contiguous()
+        self.off_a = self.C
+        self.off_g = self.off_a + self.ra
+        self.off_b = self.off_g + self.rg
+        self.conv = torch.cat([w["q.conv"], w["k.conv"], w["v.conv"]], 0).float().contiguous()
+        if self.conv.shape != (self.C, taps):
+            raise BackendError(f"ChannelDecayDeltaMixer: convolution taps {tuple(self.conv.shape)} != {(self.C, taps)}")
+        self.a2, self.dt_bias, self.A_log = w["a2"].float().contiguous(), w["dt_bias"].float().flatten().contiguous(), w["A_log"].float().flatten().contiguous()
+        self.g2_f32, self.g2 = w["g2"].float().contiguous(), w["g2"].to(dtype).contiguous()
+        self.norm = (w["norm"].float().flatten().repeat(heads) * norm_scale).contiguous()
+        self.w_o = w["o"].to(dtype).contiguous()
+        self.kernel = None                       # None: chosen by the step's shape (tests force one)
+
+    def state_shapes(self):
+        return ((max(self.taps - 1, 1), self.C), (self.H, self.dv, self.dk))
+
+    def forward(self, h: torch.Tensor, batch: StepBatch, cache, proj: Optional[torch.Tensor] = None) -> torch.Tensor:
+        return ops.linear(self.attend(h, batch, cache, proj), self.w_o)
+
+    def attend(self, h: torch.Tensor, batch: StepBatch, cache, proj: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """What the output projection reads, [T, H dv] in the compute dtype (into ``out``, row stride allowed, when given)"""
+        conv_state, S = cache
+        if proj is None:
+            proj = ops.linear(h, self.w_in)
+        T = proj.shape[0]
+        y = ops.causal_conv(proj[:, :self.C], self.conv, conv_state, batch, act="silu")
+        g = ops.low_rank_map(proj[:, self.off_a:self.off_a + self.ra], self.a2, self.dt_bias, "softplus_exp", log_rate=self.A_log)
+        o = ops.gated_delta_rule_channel(y, proj, self.off_b, g, S, batch, self.H, self.G, self.dk, self.dv, kernel=self.kernel)
+        zg = proj[:, self.off_g:self.off_g + self.rg]
+        if self.dtype == torch.bfloat16 and T > LOW_RANK_GATE_ROWS:
+            gate = ops.linear(ops.cast_rows(zg), self.g2)
+        else:
+            gate = ops.low_rank_map(zg, self.g2_f32, None, "plain")
+        return ops.group_rms_norm_gate(o, self.norm, gate, self.H, self.eps, self.dtype, gate_act="sigmoid", out=out)
+
+
+class ParallelSumMixer:
+    """Two mixers on the same input, left_scale * left + right_scale * right.  ``left`` (PagedAttentionMixer) keeps a paged cache, ``right`` a state; projections that read
+    the input itself are one product, and so are the two output projections: both sides write their rows into one buffer that meets [W_o left | W_o right].  The
+    scales touch no 16-bit weight: the right one enters through the right side's norm weight (``right`` is built with ``norm_scale`` = ``right_factor(...)``), and
+    ``forward`` returns y with the sum = out_scale * y + out_bias, which the closing norm's kernel forms in f32."""
+    kind = "both"
+
+    @staticmethod
+    def right_factor(left_scale: float, right_scale: float) -> float:
+        return float(right_scale) / float(left_scale) if left_scale else float(right_scale)
+
+    def __init__(self, left: PagedAttentionMixer, right, left_scale: float):
+        self.left, self.right = left, right
+        self.out_scale = float(left_scale) if left_scale else 1.0
+        self.w_in = left.w_in if right.w_in is None else torch.cat([left.w_in, right.w_in], 0).contiguous()
+        self.split = left.w_in.shape[0]
+        self.KL, self.KR = left.H * left.dv, right.N
+        w_left = left.w_o if left_scale else torch.zeros_like(left.w_o)
+        self.w_o = torch.cat([w_left, right.w_o], 1).contiguous()
+        self.out_bias = None if left.out_bias is None or not left_scale else (left.out_bias * self.out_scale).contiguous()
+        self.dtype = left.dtype
+        for side in (left, right):                          # the fused matrices hold the weights from here on
+            side.w_o = None
+        if right.w_in is not None:
+            left.w_in = right.w_in = None
+
+    def cache_shape(self):
+        return self.left.cache_shape()
+
+    def state_shapes(self):
+        return self.right.state_shapes()
+
+    def forward(self, x: torch.Tensor, h: torch.Tensor, batch: StepBatch, kv, state) -> torch.Tensor:
+        """x: the input rows in f32, h: the same in the compute dtype"""
+        proj = ops.linear(h, self.w_in)
+        z = torch.empty((h.shape[0], self.KL + self.KR), dtype=self.dtype, device=h.device)
+        self.left.attend(h, batch, kv, proj=proj[:, :self.split], out=z[:, :self.KL])
+        if self.w_in.shape[0] > self.split:
+            self.right.attend(h, batch, state, proj=proj[:, self.split:], out=z[:, self.KL:])
+        else:
+            self.right.attend(x, batch, state, out=z[:, self.KL:])
+        return ops.linear(z, self.w_o)

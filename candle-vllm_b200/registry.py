@@ -26,7 +26,7 @@ def architecture_of(config: dict) -> str:
 
 
 # the source group (build.GROUPS) whose library alone serves an architecture, for a first start from a source-only checkout
-_BUILD_GROUP = {"Gobesun": "ragged", "Guvusun": "latent", "Panarax": "hybrid", "Dofevik": "window", "Sigalorn": "talking"}
+_BUILD_GROUP = {"Gobesun": "ragged", "Guvusun": "latent", "Panarax": "hybrid", "Dofevik": "window", "Sigalorn": "talking", "Tavevik": "sliding"}
 
 
 def build_group_of(path: str) -> str:
@@ -71,6 +71,11 @@ def _sigalorn(path, **kw):
     return SigalornModel.from_pretrained(path, **kw)
 
 
+def _tavevik(path, **kw):
+    from .tavevik import TavevikModel
+    return TavevikModel.from_pretrained(path, **kw)
+
+
 def _llama(path, **kw):
     from .llama import load_dense_checkpoint
     return load_dense_checkpoint(path, **kw)
@@ -81,4 +86,5 @@ register_model("Guvusun", _guvusun)
 register_model("Panarax", _panarax)
 register_model("Dofevik", _dofevik)
 register_model("Sigalorn", _sigalorn)
+register_model("Tavevik", _tavevik)
 register_model("LlamaForCausalLM", _llama)

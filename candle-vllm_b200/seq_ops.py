@@ -571,13 +571,17 @@ def glu_packed(gate_up: torch.Tensor, act: str, out_dtype: torch.dtype, limit: f
 
 
 def group_rms_norm_gate(o: torch.Tensor, weight: Optional[torch.Tensor], gate: Optional[torch.Tensor], groups: int, eps: float, out_dtype: torch.dtype,
-                        gate_act: str = "sigmoid") -> torch.Tensor:
-    """o f32 [T, n] -> o / rms(o over each of ``groups`` equal runs) * weight * act(gate)"""
+                        gate_act: str = "sigmoid", out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """o f32 [T, n] -> o / rms(o over each of ``groups`` equal runs) * weight * act(gate), into ``out`` (row stride allowed) when given"""
     T, n = o.shape
-    out = torch.empty((T, n), dtype=out_dtype, device=o.device)
+    if out is None:
+        out = torch.empty((T, n), dtype=out_dtype, device=o.device)
+    elif out.dtype != out_dtype or out.shape != o.shape or out.stride(1) != 1:
+        raise BackendError(f"group_rms_norm_gate: out {tuple(out.shape)} {out.dtype}, expected {tuple(o.shape)} {out_dtype}")
     pitch = lambda t: t.stride(0) if T > 1 else max(n, t.stride(0))
-    lib().group_rms_norm_gate(_ptr(o), C.c_int64(pitch(o)), _ptr(weight), _ptr(gate), C.c_int64(0 if gate is None else pitch(gate)), _ptr(out), C.c_int32(T), C.c_int32(n),
-                              C.c_int32(groups), C.c_float(eps), C.c_int32({"sigmoid": 0, "silu": 1}[gate_act]), C.c_int32(_tag(out_dtype)), _stream(o.device))
+    lib().group_rms_norm_gate_into(_ptr(o), C.c_int64(pitch(o)), _ptr(weight), _ptr(gate), C.c_int64(0 if gate is None else pitch(gate)), _ptr(out), C.c_int64(pitch(out)),
+                                   C.c_int32(T), C.c_int32(n), C.c_int32(groups), C.c_float(eps), C.c_int32({"sigmoid": 0, "silu": 1}[gate_act]), C.c_int32(_tag(out_dtype)),
+                                   _stream(o.device))
     check("group_rms_norm_gate")
     return out
 
@@ -791,21 +795,25 @@ def paged_attention_sigmoid_pooled(q: torch.Tensor, k_cache: torch.Tensor, v_cac
 # ---- norm after and before a sublayer in one pass, xIELU, logit cap, decays per key row, heads that mix their scores --------------------------
 
 def post_norm_add_rms_norm(x: torch.Tensor, y: torch.Tensor, post_weight: torch.Tensor, weight: Optional[torch.Tensor], eps: float, out_dtype: Optional[torch.dtype] = None,
-                           y_bias: Optional[torch.Tensor] = None, row_index: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
-    """The step between two sublayers that are normed before and after, on the f32 stream x [T, n] (contiguous): x += rms_norm(y + y_bias) * post_weight in place,
-    then rms_norm(x) * weight -> [T, n] of ``out_dtype``.  ``weight`` None: the sum alone (returns None).  ``row_index`` (i32 [R]): only those rows are summed and
-    normed ([R, n] comes back) and x is left as it is."""
+                           y_bias: Optional[torch.Tensor] = None, row_index: Optional[torch.Tensor] = None, y_scale: float = 1.0,
+                           copy: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """The step between two sublayers that are normed before and after, on the f32 stream x [T, n] (contiguous): x += rms_norm(y_scale y + y_bias) * post_weight in
+    place, then rms_norm(x) * weight -> [T, n] of ``out_dtype``.  ``weight`` None: the sum alone (returns None); ``copy`` ([T, n], bf16 or f32) then also receives the
+    new x.  ``row_index`` (i32 [R]): only those rows are summed and normed ([R, n] comes back) and x is left as it is."""
     T, n = x.shape
     if x.dtype != torch.float32 or not x.is_contiguous() or y.dtype != torch.float32 or y.shape != x.shape or y.stride(1) != 1:
         raise BackendError("post_norm_add_rms_norm: an f32 contiguous stream and an f32 sublayer output of its shape")
+    if copy is not None and (weight is not None or row_index is not None or copy.shape != x.shape or not copy.is_contiguous()):
+        raise BackendError("post_norm_add_rms_norm: a copy of the stream is whole, contiguous and comes without an opening norm")
     if weight is None and row_index is not None:
         return None
     rows = T if row_index is None else row_index.shape[0]
-    out = None if weight is None else torch.empty((rows, n), dtype=out_dtype, device=x.device)
-    lib().post_norm_add_rms_norm(_ptr(x), _ptr(y), C.c_int64(y.stride(0) if T > 1 else max(n, y.stride(0))), _ptr(y_bias), _ptr(post_weight), _ptr(weight), _ptr(out),
-                                 _ptr(row_index), C.c_int32(rows), C.c_int32(n), C.c_float(eps), C.c_int32(_tag(out_dtype) if out is not None else DType.F32), _stream(x.device))
+    out = copy if weight is None else torch.empty((rows, n), dtype=out_dtype, device=x.device)
+    lib().scaled_post_norm_add(_ptr(x), _ptr(y), C.c_int64(y.stride(0) if T > 1 else max(n, y.stride(0))), C.c_float(y_scale), _ptr(y_bias), _ptr(post_weight), _ptr(weight),
+                               _ptr(out), _ptr(row_index), C.c_int32(rows), C.c_int32(n), C.c_float(eps), C.c_int32(_tag(out.dtype) if out is not None else DType.F32),
+                               _stream(x.device))
     check("post_norm_add_rms_norm")
-    return out
+    return None if weight is None else out
 
 
 def xielu(x: torch.Tensor, bias: Optional[torch.Tensor], pos: float, neg: float, out_dtype: torch.dtype) -> torch.Tensor:
@@ -831,22 +839,40 @@ def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
 
 def low_rank_decay(y: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], tau: float) -> torch.Tensor:
     """sigmoid(weight y + bias)^(1 / tau): y f32 [T, rank] (row stride allowed), weight f32 [channels, rank] -> f32 [T, channels]; 32-bit throughout"""
+    return low_rank_map(y, weight, bias, "root_sigmoid", tau=tau)
+
+
+LOW_RANK_FORMS = {"root_sigmoid": 0, "double_exp": 1, "softplus_exp": 2, "plain": 3}
+
+
+def low_rank_map(y: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], form: str, tau: float = 1.0, log_rate: Optional[torch.Tensor] = None,
+                 in_tanh: bool = False) -> torch.Tensor:
+    """The second factor of a low-rank map in 32 bits: z = weight y + bias (y f32 [T, rank], row stride allowed, through tanh first with ``in_tanh``; weight f32
+    [channels, rank]) -> f32 [T, channels]: "root_sigmoid" sigmoid(z)^(1 / tau), "double_exp" exp(-exp(z)), "softplus_exp" exp(-exp(log_rate) softplus(z)) with one
+    log_rate per equal run of channels, "plain" z"""
     T, R = y.shape
     N = weight.shape[0]
     if y.dtype != torch.float32 or weight.dtype != torch.float32 or y.stride(1) != 1 or weight.shape[1] != R or not weight.is_contiguous():
-        raise BackendError(f"low_rank_decay: y {tuple(y.shape)} {y.dtype}, weight {tuple(weight.shape)} {weight.dtype}")
-    alpha = torch.empty((T, N), dtype=torch.float32, device=y.device)
-    lib().low_rank_decay(_ptr(y), C.c_int64(y.stride(0) if T > 1 else max(R, y.stride(0))), _ptr(weight), _ptr(bias), _ptr(alpha), C.c_int32(T), C.c_int32(N), C.c_int32(R),
-                         C.c_float(tau), _stream(y.device))
-    check("low_rank_decay")
-    return alpha
+        raise BackendError(f"low_rank_map: y {tuple(y.shape)} {y.dtype}, weight {tuple(weight.shape)} {weight.dtype}")
+    if form not in LOW_RANK_FORMS or (form == "softplus_exp" and (log_rate is None or log_rate.dtype != torch.float32 or N % log_rate.numel())):
+        raise BackendError(f"low_rank_map: form {form!r} for {N} channels")
+    out = torch.empty((T, N), dtype=torch.float32, device=y.device)
+    lib().low_rank_map(_ptr(y), C.c_int64(y.stride(0) if T > 1 else max(R, y.stride(0))), _ptr(weight), _ptr(bias), _ptr(out), C.c_int32(T), C.c_int32(N), C.c_int32(R),
+                       C.c_int32(1 if in_tanh else 0), C.c_int32(LOW_RANK_FORMS[form]), C.c_float(tau), _ptr(log_rate),
+                       C.c_int32(N // log_rate.numel() if log_rate is not None else 1), _stream(y.device))
+    check("low_rank_map")
+    return out
 
 
 def linear_attention_channel(proj: torch.Tensor, off_q: int, off_k: int, off_v: int, alpha: torch.Tensor, state: torch.Tensor, batch: StepBatch, heads: int, dk: int, dv: int,
-                             q_scale: float = 1.0, kernel: Optional[str] = None) -> torch.Tensor:
+                             q_scale: float = 1.0, kernel: Optional[str] = None, bonus: Optional[torch.Tensor] = None, rows: Optional[int] = None) -> torch.Tensor:
     """``linear_attention`` with a decay per token and key row: S <- diag(alpha_t) S + k v^T, o = S^T q per head; alpha f32 [T, H dk], state f32 [slots, H, dv, dk]
-    advanced in place -> f32 [T, H dv].  The same three kernels ("step", "token", "chunked"), chosen by the step's shape the same way."""
-    T = proj.shape[0]
+    advanced in place -> f32 [T, H dv].  The same three kernels ("step", "token", "chunked"), chosen by the step's shape the same way.  ``bonus`` f32 [H, dk]: the
+    output is read before the token's own decay and write, o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t.  ``rows``: rows of the step when ``proj`` has more (its
+    operands are then slabs of rows of one matrix, the offsets counted in elements)."""
+    T = proj.shape[0] if rows is None else rows
+    if bonus is not None and (bonus.dtype != torch.float32 or bonus.numel() != heads * dk or not bonus.is_contiguous()):
+        raise BackendError(f"linear_attention_channel: bonus {tuple(bonus.shape)} {bonus.dtype} for {heads} x {dk}")
     if alpha.dtype != torch.float32 or alpha.shape != (T, heads * dk) or not alpha.is_contiguous():
         raise BackendError(f"linear_attention_channel: decays {tuple(alpha.shape)} {alpha.dtype} for {T} rows of {heads} x {dk}")
     out = torch.empty((T, heads * dv), dtype=torch.float32, device=proj.device)
@@ -860,10 +886,10 @@ def linear_attention_channel(proj: torch.Tensor, off_q: int, off_k: int, off_v: 
     except KeyError:
         raise BackendError(f"linear_attention_channel: unknown kernel {kernel!r}")
     scratch = torch.empty((need,), dtype=torch.float32, device=proj.device) if mode == 2 else None
-    lib().linear_attention_channel(_ptr(proj), C.c_int64(proj.stride(0) if T > 1 else proj.shape[1]), C.c_int32(off_q), C.c_int32(off_k), C.c_int32(off_v), _ptr(alpha),
-                                   C.c_int64(heads * dk), C.c_float(q_scale), _ptr(state), _ptr(out), _ptr(scratch), _ptr(batch.cu_seqlens), _ptr(batch.seq_slots),
-                                   _ptr(batch.seq_start), C.c_int32(T), C.c_int32(batch.num_seqs), C.c_int32(batch.max_rows), C.c_int32(mode), C.c_int32(heads),
-                                   C.c_int32(dk), C.c_int32(dv), _stream(proj.device))
+    lib().linear_attention_channel_bonus(_ptr(proj), C.c_int64(proj.stride(0) if T > 1 else proj.shape[1]), C.c_int64(off_q), C.c_int64(off_k), C.c_int64(off_v), _ptr(alpha),
+                                         C.c_int64(heads * dk), _ptr(bonus), C.c_float(q_scale), _ptr(state), _ptr(out), _ptr(scratch), _ptr(batch.cu_seqlens),
+                                         _ptr(batch.seq_slots), _ptr(batch.seq_start), C.c_int32(T), C.c_int32(batch.num_seqs), C.c_int32(batch.max_rows), C.c_int32(mode),
+                                         C.c_int32(heads), C.c_int32(dk), C.c_int32(dv), _stream(proj.device))
     check("linear_attention_channel")
     return out
 
@@ -935,4 +961,72 @@ def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                                  C.c_int32(bs), C.c_float(scale), C.c_int32(chunk), C.c_int32(window), C.c_int32(1 if one_sink else 0), C.c_int32(splits), _ptr(part), C.c_int32(1 if plain else 0),
                                  C.c_int32(_tag(k_cache.dtype)), C.c_int32(_tag(out_dtype)), _stream(q.device))
     check("talking_attention_rows")
+    return out
+
+
+# ---- kept first tokens, capped scores and element-wise gates on the paged attention; token shift; the delta rule with a decay per key row --------------
+
+def cast_rows(x: torch.Tensor) -> torch.Tensor:
+    """f32 rows (row stride allowed) -> contiguous bf16"""
+    T, n = x.shape
+    out = torch.empty((T, n), dtype=torch.bfloat16, device=x.device)
+    lib().cast_rows_bf16(_ptr(x), C.c_int64(x.stride(0) if T > 1 else max(n, x.stride(0))), _ptr(out), C.c_int64(n), C.c_int32(T), C.c_int32(n), _stream(x.device))
+    check("cast_rows_bf16")
+    return out
+
+
+def paged_attention_selected(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: StepBatch, heads: int, scale: float, chunk: int, window: int,
+                             keep_first: int, softcap: float, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], out: torch.Tensor) -> torch.Tensor:
+    """``paged_attention_varlen_sink`` with kept first tokens (a key at a position below ``keep_first`` stays visible whatever the window), scores softcap tanh(s /
+    softcap) (0 = as they are) and, with ``gate`` f32 [T, H dv] (row stride allowed), the outputs times sigmoid(gate) entry by entry; writes into ``out`` [T, H dv]
+    (row stride allowed)"""
+    T = q.shape[0]
+    nb, bs, G, dk = k_cache.shape
+    dv = v_cache.shape[3]
+    if out.shape != (T, heads * dv) or out.stride(1) != 1 or (gate is not None and (gate.dtype != torch.float32 or gate.shape != out.shape or gate.stride(1) != 1)):
+        raise BackendError(f"paged_attention_selected: out {tuple(out.shape)} / gate for {T} rows of {heads} x {dv}")
+    pitch = lambda t: 0 if t is None else (t.stride(0) if T > 1 else max(heads * dv, t.stride(0)))
+    lib().paged_attention_varlen_ex(_ptr(out), C.c_int64(pitch(out)), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), C.c_int32(batch.block_tables.shape[1]),
+                                    _ptr(batch.token_seq), _ptr(batch.positions), _ptr(batch.cu_seqlens), _ptr(batch.cu_seqlens_k), C.c_int32(batch.num_seqs), C.c_int32(T),
+                                    C.c_int32(heads), C.c_int32(G), C.c_int32(dk), C.c_int32(dv), C.c_int32(bs), C.c_float(scale), C.c_int32(chunk), C.c_int32(window),
+                                    C.c_int32(keep_first), C.c_float(softcap), _ptr(sink), _ptr(gate), C.c_int64(pitch(gate)), C.c_int32(_tag(q.dtype)),
+                                    C.c_int32(_tag(k_cache.dtype)), C.c_int32(_tag(out.dtype)), _stream(q.device))
+    check("paged_attention_varlen_ex")
+    return out
+
+
+def token_shift_mix(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, batch: StepBatch, out: torch.Tensor) -> torch.Tensor:
+    """out[m, t] = x[t] + (x[t - 1] - x[t]) * mu[m]: x f32 [T, D], mu f32 [M, D], out [M, >= T, D]; the row before an entry's first comes from state f32 [slots, D] (zeros
+    at a sequence's start), which takes the entry's last row"""
+    T, D = x.shape
+    M = mu.shape[0]
+    if (x.dtype != torch.float32 or x.stride(1) != 1 or mu.dtype != torch.float32 or not mu.is_contiguous() or mu.shape[1] != D or state.shape[1:] != (D,) or not out.is_contiguous()
+            or out.dim() != 3 or out.shape[0] != M or out.shape[1] < T or out.shape[2] != D):
+        raise BackendError(f"token_shift_mix: x {tuple(x.shape)} {x.dtype}, mu {tuple(mu.shape)}, state {tuple(state.shape)}, out {tuple(out.shape)}")
+    lib().token_shift_mix(_ptr(x), C.c_int64(x.stride(0) if T > 1 else max(D, x.stride(0))), _ptr(mu), _ptr(state), _ptr(out), C.c_int64(out.shape[1]), _ptr(batch.token_seq),
+                          _ptr(batch.cu_seqlens), _ptr(batch.seq_slots), _ptr(batch.seq_start), C.c_int32(T), C.c_int32(D), C.c_int32(M), C.c_int32(_tag(out.dtype)),
+                          _stream(x.device))
+    check("token_shift_mix")
+    return out
+
+
+def gated_delta_rule_channel(qkv: torch.Tensor, proj: torch.Tensor, off_b: int, decay: torch.Tensor, state: torch.Tensor, batch: StepBatch, heads: int, kv_heads: int, dk: int,
+                             dv: int, kernel: Optional[str] = None) -> torch.Tensor:
+    """``gated_delta_rule`` with a decay per token and key row: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; decay f32 [T, H dk]; the same three
+    kernels ("step", "token", "tiled"), chosen by the step's shape the same way"""
+    T = qkv.shape[0]
+    if decay.dtype != torch.float32 or decay.shape != (T, heads * dk) or not decay.is_contiguous() or not qkv.is_contiguous():
+        raise BackendError(f"gated_delta_rule_channel: decays {tuple(decay.shape)} {decay.dtype} for {T} rows of {heads} x {dk}")
+    out = torch.empty((T, heads * dv), dtype=torch.float32, device=qkv.device)
+    if kernel is None:
+        kernel = "step" if batch.pure_decode else "token"
+    try:
+        mode = {"token": 0, "step": 1, "tiled": 2}[kernel]
+    except KeyError:
+        raise BackendError(f"gated_delta_rule_channel: unknown kernel {kernel!r}")
+    scratch = None
+    lib().gated_delta_rule_channel(_ptr(qkv), _ptr(proj), C.c_int64(proj.stride(0) if T > 1 else proj.shape[1]), C.c_int32(off_b), _ptr(decay), _ptr(state), _ptr(out),
+                                   _ptr(scratch), _ptr(batch.cu_seqlens), _ptr(batch.seq_slots), _ptr(batch.seq_start), C.c_int32(T), C.c_int32(batch.num_seqs),
+                                   C.c_int32(batch.max_rows), C.c_int32(mode), C.c_int32(heads), C.c_int32(kv_heads), C.c_int32(dk), C.c_int32(dv), _stream(qkv.device))
+    check("gated_delta_rule_channel")
     return out

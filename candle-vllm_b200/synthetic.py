@@ -566,3 +566,88 @@ def sigalorn_weights(cfg: dict, seed: int = 0, rank: int = 16, device="cpu") -> 
             out[p + "mlp.up"], out[p + "mlp.up.b"], out[p + "mlp.down"], out[p + "mlp.down.b"] = lin(ff, D), rnd(ff, std=0.3), lin(D, ff), rnd(D, std=0.3)
             out[p + "mlp.act"] = rnd(2)
     return {k: v.to(torch.bfloat16).to(device) for k, v in out.items()}
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Tavevik: random checkpoints of any shape (tests and bench.py)
+# ---------------------------------------------------------------------------------------------------------------------
+def _tavevik_layer(kind: str, left: dict, right: dict, left_scale: float, right_scale: float, ff: int, limit: float) -> dict:
+    return dict(type=kind, mixer=dict(left=left, right=right, left_scale=left_scale, right_scale=right_scale), mlp=dict(ff=ff, kind="dense", limit=limit) if ff else None)
+
+
+def _tavevik_left(heads, kv_heads, dim, vdim, window, rot_dims, base, scale) -> dict:
+    left = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=dim ** -0.5 if scale is None else scale)
+    if rot_dims:
+        left["rot"] = dict(base=base, dims=rot_dims)
+    if window:
+        left["mask"] = dict(size=window)
+    return left
+
+
+def tavevik_shift_layer(heads: int, kv_heads: int, dim: int, vdim: int, m_heads: int, m_dim: int, window: int = 0, keep_first: int = 0, rot_dims: int = 0, base: float = 10000.0,
+                        scale: float = None, softcap: float = 20.0, left_scale: float = 0.9, right_scale: float = 1.3, ff: int = 0, limit: float = 2.0) -> dict:
+    """windowed attention with kept first tokens and capped scores beside linear attention over shifted tokens"""
+    left = _tavevik_left(heads, kv_heads, dim, vdim, window, rot_dims, base, scale)
+    if window and keep_first:
+        left["mask"]["keep_first"] = keep_first
+    if softcap:
+        left["softcap"] = softcap
+    return _tavevik_layer("parallel", left, dict(heads=m_heads, dim=m_dim), left_scale, right_scale, ff, limit)
+
+
+def tavevik_delta_layer(heads: int, kv_heads: int, dim: int, vdim: int, m_heads: int, m_kv_heads: int, m_dim: int, m_vdim: int, conv: int = 4, window: int = 0, rot_dims: int = 0,
+                        base: float = 10000.0, scale: float = None, left_scale: float = 1.1, right_scale: float = 0.7, ff: int = 0, limit: float = 2.0) -> dict:
+    """windowed attention with biases and a sink beside the delta rule with a decay per key row"""
+    left = _tavevik_left(heads, kv_heads, dim, vdim, window, rot_dims, base, scale)
+    return _tavevik_layer("parallel_2", left, dict(heads=m_heads, kv_heads=m_kv_heads, dim=m_dim, vdim=m_vdim, conv=conv), left_scale, right_scale, ff, limit)
+
+
+def tavevik_config(width: int, vocab: int, layers: list, eps: float = 1e-6) -> dict:
+    return dict(architecture="Tavevik", layers=layers, norm=dict(eps=eps), vocab=vocab, width=width)
+
+
+def tavevik_weights(cfg: dict, seed: int = 0, ranks=(16, 12, 20), device="cpu") -> dict:
+    """name -> bf16 tensor with magnitudes that keep every mechanism visible in the logits: scores of a few units, decays from nearly one to nearly zero within a layer, sinks
+    that carry weight, activations on both sides of the clamp.  ``ranks``: the token-shift decay's, the delta rule's decay's and gate's low ranks."""
+    g = torch.Generator().manual_seed(seed)
+    D, V = cfg["width"], cfg["vocab"]
+    out = {}
+    rnd = lambda *shape, std=1.0: (torch.randn(*shape, generator=g) * std)
+    uni = lambda n, lo, hi: torch.rand(n, generator=g) * (hi - lo) + lo
+    lin = lambda n, k, gain=1.0: rnd(n, k, std=gain * k ** -0.5)
+    norm = lambda n: 1.0 + rnd(n, std=0.25)
+    out["embed"], out["final.norm"] = rnd(V, D), norm(D) * 0.3
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        lm, rm = m["left"], m["right"]
+        H, G, dk, dv = lm["heads"], lm["kv_heads"], lm["dim"], lm["vdim"]
+        out[p + "norm1"] = norm(D)
+        a = p + "mix.left."
+        out[a + "q"], out[a + "k"], out[a + "v"], out[a + "o"] = lin(H * dk, D), lin(G * dk, D), lin(G * dv, D), lin(D, H * dv, 2.0)
+        out[a + "q.norm"], out[a + "k.norm"] = norm(dk) * 1.4, norm(dk) * 1.4
+        r = p + "mix.right."
+        if L["type"] == "parallel":
+            out[a + "g"] = lin(H * dv, D)
+            N, R = rm["heads"] * rm["dim"], ranks[0]
+            for x in "rkvgw":
+                out[r + "mu." + x] = uni(D, 0.0, 1.0)
+            for x in "rkvg":
+                out[r + x] = lin(N, D, 1.3)
+            out[r + "w1"], out[r + "w2"], out[r + "w0"] = lin(R, D), lin(N, R, 1.2), uni(N, -6.0, 0.5)
+            out[r + "u"], out[r + "norm"], out[r + "o"] = rnd(rm["heads"], rm["dim"]), norm(N), lin(D, N, 2.0)
+        else:
+            for x, n in (("q", H * dk), ("k", G * dk), ("v", G * dv), ("o", D)):
+                out[a + x + ".b"] = rnd(n, std=0.4)
+            out[a + "sink"] = rnd(H) + 1.5
+            mh, mg, mk, mv, taps = rm["heads"], rm["kv_heads"], rm["dim"], rm["vdim"], rm["conv"]
+            for x, n in (("q", mg * mk), ("k", mg * mk), ("v", mh * mv)):
+                out[r + x], out[r + x + ".conv"] = lin(n, D, 1.3), rnd(n, taps, std=0.6)
+            out[r + "b"], out[r + "A_log"] = lin(mh, D), uni(mh, -1.5, 1.0)
+            out[r + "a1"], out[r + "a2"], out[r + "dt_bias"] = lin(ranks[1], D), lin(mh * mk, ranks[1], 1.2), uni(mh * mk, -6.0, 1.0)
+            out[r + "g1"], out[r + "g2"] = lin(ranks[2], D), lin(mh * mv, ranks[2], 1.5)
+            out[r + "norm"], out[r + "o"] = norm(mv), lin(D, mh * mv, 2.0)
+        if L.get("mlp"):
+            ff = L["mlp"]["ff"]
+            out[p + "norm2"] = norm(D)
+            out[p + "mlp.gate"], out[p + "mlp.up"], out[p + "mlp.down"] = lin(ff, D, 1.5), lin(ff, D, 1.5), lin(D, ff)
+    return {k: v.to(torch.bfloat16).to(device) for k, v in out.items()}

@@ -730,6 +730,45 @@ void talking_attention_prefill(void* out, const void* q, const void* key_cache, 
                                int32_t num_tokens, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t block_size, float scale, int32_t chunk,
                                int32_t window, int32_t one_sink, int64_t stream);
 
+/* ---- kept first tokens and capped scores, token shift with a bonus recurrence, the delta rule with a decay per key row, scaled closing norm ----------
+ * paged_attention_varlen_ex: paged_attention_varlen_sink with kept first tokens (a key at a position below keep_first is seen by every later query, whatever the
+ *   window), scores softcap tanh(s / softcap) (softcap 0 = as they are), gate f32 [T, H dv] (row pitch ld_gate, or null): the output times sigmoid(gate) entry by
+ *   entry, and an output row pitch ld_out.
+ * token_shift_mix: out[m, t] = x[t] + (x[t - 1] - x[t]) * mu[m] for m < mixes (<= 8): x f32 [T, dim] (row pitch ldx), mu f32 [mixes, dim], out [mixes, slab_rows, dim]
+ *   of F32 / BF16 (rows from num_tokens on are left as they are); the row before an entry's first is state f32 [slots, dim] (zeros at a sequence's start), which
+ *   then takes the entry's last row.
+ * low_rank_map: out f32 [T, channels] = f(weight y' + bias), y' = y or tanh(y) (in_tanh); form 0: sigmoid(z)^(1 / tau), 1: exp(-exp(z)), 2: exp(-exp(log_rate[c /
+ *   channels_per_rate]) softplus(z)), 3: z.  32-bit throughout.
+ * linear_attention_channel_bonus: linear_attention_channel whose output is read before the token's decay and write: o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t,
+ *   bonus f32 [H, dk] (null: linear_attention_channel itself).  Offsets are 64-bit: q, k and v may be matrices of their own with one row pitch.
+ * gated_delta_rule_channel: gated_delta_rule with a decay per token and key row: S <- diag(g_t) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; decay f32 [T, H dk].
+ *   mode 0: token by token, any step; 1: every entry brings exactly one row; 2: over tiles of 16 tokens (dk <= 128, scratch =
+ *   gated_delta_channel_scratch(...) floats).  dk <= 512 in modes 0 and 1.
+ * scaled_post_norm_add: post_norm_add_rms_norm of y_scale * y + y_bias; with weight null and out given, out takes the new x as it is.
+ * group_rms_norm_gate_into: group_rms_norm_gate with an output row pitch ld_out.
+ * cast_rows_bf16: out BF16 [rows, n] (row pitch ld_out) = x f32 (row pitch ldx). */
+void paged_attention_varlen_ex(void* out, int64_t ld_out, const void* q, const void* key_cache, const void* value_cache, const int32_t* block_tables, int32_t table_width,
+                               const int32_t* token_seq, const int32_t* positions, const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, int32_t num_seqs,
+                               int32_t num_tokens, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int32_t block_size, float scale, int32_t chunk,
+                               int32_t window, int32_t keep_first, float softcap, const float* sink, const float* gate, int64_t ld_gate, int32_t q_dtype,
+                               int32_t cache_dtype, int32_t out_dtype, int64_t stream);
+void token_shift_mix(const float* x, int64_t ldx, const float* mu, float* state, void* out, int64_t slab_rows, const int32_t* token_seq, const int32_t* cu_seqlens,
+                     const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens, int32_t dim, int32_t mixes, int32_t out_dtype, int64_t stream);
+void low_rank_map(const float* y, int64_t ldy, const float* weight, const float* bias, float* out, int32_t num_tokens, int32_t channels, int32_t rank, int32_t in_tanh,
+                  int32_t form, float tau, const float* log_rate, int32_t channels_per_rate, int64_t stream);
+void linear_attention_channel_bonus(const float* proj, int64_t ld, int64_t off_q, int64_t off_k, int64_t off_v, const float* alpha, int64_t lda, const float* bonus,
+                                    float q_scale, float* state, float* out, float* scratch, const int32_t* cu_seqlens, const int32_t* seq_slots,
+                                    const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t max_rows, int32_t mode, int32_t num_heads, int32_t dk,
+                                    int32_t dv, int64_t stream);
+void gated_delta_rule_channel(const float* qkv, const float* proj, int64_t ld_proj, int32_t off_b, const float* decay, float* state, float* out, float* scratch,
+                              const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t max_rows,
+                              int32_t mode, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int64_t stream);
+void scaled_post_norm_add(float* x, const float* y, int64_t ldy, float y_scale, const float* y_bias, const float* post_weight, const float* weight, void* out,
+                          const int32_t* row_index, int32_t rows, int32_t n, float eps, int32_t out_dtype, int64_t stream);
+void group_rms_norm_gate_into(const float* o, int64_t ldo, const float* weight, const float* gate, int64_t ld_gate, void* out, int64_t ld_out, int32_t num_tokens, int32_t n,
+                              int32_t groups, float eps, int32_t gate_act, int32_t out_dtype, int64_t stream);
+void cast_rows_bf16(const float* x, int64_t ldx, void* out, int64_t ld_out, int32_t rows, int32_t n, int64_t stream);
+
 #ifdef __cplusplus
 }
 #endif
