@@ -43,7 +43,8 @@ SYMBOLS = [
     "mla_paged_attention_window",
     "post_norm_add_rms_norm", "xielu_rows", "softcap_inplace", "low_rank_decay", "linear_attention_channel", "qkv_norm_rope_cache", "talking_attention_rows",
     "talking_attention_prefill_supported", "talking_attention_prefill",
-    "paged_attention_varlen_ex", "token_shift_mix", "low_rank_map", "linear_attention_channel_bonus", "gated_delta_rule_channel", "scaled_post_norm_add",
+    "paged_attention_varlen_ex", "token_shift_mix", "low_rank_map", "linear_attention_channel_bonus", "gated_delta_rule_channel", "gated_delta_channel_chunked_scratch", "gated_delta_channel_chunked",
+    "paged_attention_rows_supported", "paged_attention_rows", "scaled_post_norm_add",
     "group_rms_norm_gate_into", "cast_rows_bf16",
 ]
 
@@ -69,14 +70,14 @@ GROUP_SYMBOLS = {
                          "moe_align", "moe_gather_rows", "moe_combine_rows"],
     "talking": _COMMON + ["low_rank_decay", "low_rank_map", "linear_attention_channel", "linear_attention_channel_bonus", "linear_attention_chunked_scratch", "qkv_norm_rope_cache", "talking_attention_rows",
                          "talking_attention_prefill_supported", "talking_attention_prefill"],
-    "sliding": _COMMON + ["causal_conv_ex", "gated_delta_rule_channel", "low_rank_map", "token_shift_mix", "linear_attention_channel_bonus", "linear_attention_chunked_scratch",
-                         "qk_head_norm_rope_cache", "paged_attention_varlen_ex", "linear_grouped"],
+    "sliding": _COMMON + ["causal_conv_ex", "gated_delta_rule_channel", "gated_delta_channel_chunked_scratch", "gated_delta_channel_chunked", "low_rank_map", "token_shift_mix", "linear_attention_channel_bonus", "linear_attention_chunked_scratch",
+                         "qk_head_norm_rope_cache", "paged_attention_varlen_ex", "paged_attention_rows_supported", "paged_attention_rows", "linear_grouped"],
 }
 _RESTYPES = {"b200_last_error_message": C.c_char_p, "paged_attention_decode_workspace_bytes": C.c_size_t, "qmatmul_workspace_bytes": C.c_size_t,
              "moe_gemm_workspace_bytes": C.c_size_t, "moe_gemm_fp8_workspace_bytes": C.c_size_t, "mla_paged_decode_workspace_bytes": C.c_size_t,
              "b200_llama_create": C.c_void_p, "b200_llama_peer_inbox_bytes": C.c_size_t, "b200_ipc_alloc": C.c_void_p, "b200_ipc_open": C.c_void_p,
              "b200_llama_logits": C.c_void_p, "b200_llama_next_tokens": C.c_void_p, "b200_llama_kernel_launches": C.c_int64,
-             "b200_total_kernel_launches": C.c_longlong, "moe_align_rows": C.c_int64, "linear_attention_chunked_scratch": C.c_int64}
+             "b200_total_kernel_launches": C.c_longlong, "moe_align_rows": C.c_int64, "linear_attention_chunked_scratch": C.c_int64, "gated_delta_channel_chunked_scratch": C.c_int64}
 
 
 def _open(path: str, symbols) -> C.CDLL:

@@ -54,8 +54,8 @@ GROUPS = {"ragged": ["lib", "linear_generic", "dense_gemm", "norm_act", "gated_d
           "talking": ["lib", "linear_generic", "dense_gemm", "norm_act", "linear_recurrence", "attention_varlen", "attention_prefill", "attention_talking", "elementwise"],
           # windowed attention with kept first tokens beside token-shift linear attention or a delta rule with a decay per key row: both linear kernels (the tcgen05 one
           # also grouped), norms, the recurrences, the per-head preparation, the attention over the paged cache, argmax
-          "sliding": ["lib", "linear_generic", "dense_gemm", "norm_act", "linear_recurrence", "gated_delta", "attention_window", "attention_varlen", "attention_prefill",
-                      "elementwise"]}
+          "sliding": ["lib", "linear_generic", "dense_gemm", "norm_act", "linear_recurrence", "gated_delta", "delta_chunk", "attention_window", "attention_varlen",
+                      "attention_prefill", "attention_rows", "elementwise"]}
 
 
 def so_path(group=None) -> str:

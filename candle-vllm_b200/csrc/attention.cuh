@@ -48,5 +48,10 @@ struct PrefillExtras {
 void paged_attention_prefill_tc(void* out, const void* q, const void* kc, const void* vc, const uint32_t* block_tables, const uint32_t* cu_q,
                                 const uint32_t* cu_k, int num_seqs, int total_q, int num_heads, int num_kv_heads, int max_blocks, int64_t num_blocks,
                                 float scale, int window, int dtype, cudaStream_t st, int chunk = 0, const PrefillExtras* extras = nullptr);
+// the same kernel with key and value sizes of their own (multiples of 8 up to 128), kept first tokens, capped scores, one gate per output entry, an output pitch; bf16
+bool paged_attention_prefill_sel_supported(int dk, int dv, int block_size, const void* q, const void* kc, const void* vc);
+void paged_attention_prefill_sel(void* out, int64_t ld_out, const void* q, const void* kc, const void* vc, const uint32_t* block_tables, const uint32_t* cu_q,
+                                 const uint32_t* cu_k, int num_seqs, int total_q, int num_heads, int num_kv_heads, int dk, int dv, int max_blocks, float scale, int chunk,
+                                 int window, int keep_first, float softcap, const float* sink, const float* gate, int64_t ld_gate, cudaStream_t st);
 
 }  // namespace b200

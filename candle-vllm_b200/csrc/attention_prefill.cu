@@ -13,6 +13,8 @@
 // bottom-right mask (+ optional sliding window) applied only on the pages that touch the diagonal.  FlashAttention-2 dataflow; the
 // arithmetic is ~4 * T_q * T_k * 128 flop per head against T_k * 512 B of page reads per 64 rows, i.e. tensor-bound.
 // Covers: flash layout, head_dim 128, block 64, 16-bit cache of the model dtype; everything else stays on the generic kernel.
+// A further form (kSel) serves key and value sizes of their own (multiples of 8 up to 128: the TMA boxes are 64 entries wide and fill what lies past a row with
+// zeros), kept first tokens beside a window, capped scores, one sigmoid gate per output entry and an output row pitch.
 #include <cuda.h>
 
 #include <type_traits>
@@ -23,11 +25,11 @@ namespace b200 {
 
 namespace {
 
-constexpr int kHd = 128, kPg = 64, kHalf = 32;
+constexpr int kHd = 128, kPg = 64, kHalf = 32;          // head size of the plain forms, tokens per page and per half page
 constexpr int kQTile = 64, kPfWarps = 4, kPfThreads = kPfWarps * 32;
 constexpr int kSub = kHalf * 64 * 2;                    // one swizzled sub-tile: 32 tokens x 64 dims x 2 B = 4 KB
-constexpr int kStage = 2 * 4 * kSub;                    // 64 tokens: 2 halves x (K lo, K hi, V lo, V hi) = 32 KB
-constexpr int kPfSmem = 2 * kStage + 64;
+constexpr int stage_bytes(int dk, int dv) { return 2 * (dk / 64 + dv / 64) * kSub; }       // 64 tokens: 2 halves x (K lo, K hi, V lo, V hi) = 32 KB at 128 + 128
+constexpr int prefill_smem(int dk, int dv) { return 2 * stage_bytes(dk, dv) + 64; }
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void mbar_init(uint32_t bar, uint32_t count) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count)); }
@@ -70,6 +72,7 @@ __device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4],
 template <typename T> __device__ __forceinline__ uint32_t pack2(float lo, float hi);
 template <> __device__ __forceinline__ uint32_t pack2<__nv_bfloat16>(float lo, float hi) { __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi); return *reinterpret_cast<uint32_t*>(&v); }
 template <> __device__ __forceinline__ uint32_t pack2<__half>(float lo, float hi) { __half2 v = __floats2half2_rn(lo, hi); return *reinterpret_cast<uint32_t*>(&v); }
+__device__ __forceinline__ float fast_rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ float fast_exp2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
 struct PrefillParams {
@@ -82,15 +85,24 @@ struct PrefillParams {
     const float* head_bias;         // [H] or null (sigmoid mode): added to every score of head h
     const float* kp; const float* vp;   // f32 pooled caches [nb, per_block, G, 128] or null: mean keys / values of blocks of `pool` positions
     int pool, per_block;
+    int dk, dv;                     // real key and value size (kSel)
+    int keep_first;                 // kSel: keys at positions below it are seen whatever the window
+    float cap_log2, cap_in;         // kSel: scores become cap tanh(s scale / cap): cap log2(e), and 2 scale log2(e) / cap; cap_log2 0 = as they are
+    const float* gate; int64_t ldg; // kSel: [T, H dv] or null: the output times sigmoid(gate) entry by entry
+    int64_t ldo;                    // kSel: output row pitch
 };
 
 // kSigmoid: the weight of a visible key is sigmoid(score * scale + head_bias[h]); no running maximum, no denominator.
 // With pooled caches, a row at position i also sees, like keys, the pooled entries of the blocks b with b pool + pool - 1 <= i - window; entry b lives
 // in the page of its last position at index b - floor(page 64 / pool).  Pooled tiles of 64 entries are gathered, converted to 16 bits and laid out
 // in shared memory like a page by all threads (the second stage buffer, before the page walk needs it), then take the same MMA path as a page.
-template <typename T, bool kSigmoid, bool kPooled>
+// kDK, kDV: key and value size rounded up to 64 or 128.
+template <typename T, bool kSigmoid, bool kPooled, bool kSel, int kDK, int kDV>
 __global__ void __launch_bounds__(kPfThreads, 2)
 paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap, const PrefillParams p) {
+    static_assert(kSel || (kDK == kHd && kDV == kHd), "the plain forms have 128-wide heads");
+    constexpr int kKSubs = kDK / 64, kVSubs = kDV / 64, kHalfBytes = (kKSubs + kVSubs) * kSub, kStage = stage_bytes(kDK, kDV);
+    const int hk = kSel ? p.dk : kDK, hv = kSel ? p.dv : kDV;
     extern __shared__ __align__(1024) uint8_t smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
@@ -118,6 +130,10 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
     if (p.chunk > 0) first_key = max(first_key, (pos0 / p.chunk) * p.chunk);       // row 0 has the earliest chunk start of the tile
     const int page_lo = first_key / kPg, page_hi = last_pos / kPg;  // pages [page_lo, page_hi] hold every visible key
     const uint32_t* table = p.block_tables + (int64_t)seq * p.max_blocks;
+    // kept first tokens: their pages come first, unless the walk reaches them anyway
+    const int kept_pages = kSel ? min((min(p.keep_first, klen) + kPg - 1) / kPg, page_lo) : 0;
+    const int num_pages = kept_pages + page_hi - page_lo + 1;
+    auto page_at = [&](int i) { return kSel && i < kept_pages ? i : page_lo + i - kept_pages; };
 
     if (threadIdx.x == 0) {
         mbar_init(bars, 1);
@@ -132,31 +148,32 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
         mbar_expect_tx(bar, kStage);
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-            tma_load_4d(dst + h * 4 * kSub, &kmap, bar, 0, kvh, h * kHalf, blk);
-            tma_load_4d(dst + h * 4 * kSub + kSub, &kmap, bar, 64, kvh, h * kHalf, blk);
-            tma_load_4d(dst + h * 4 * kSub + 2 * kSub, &vmap, bar, 0, kvh, h * kHalf, blk);
-            tma_load_4d(dst + h * 4 * kSub + 3 * kSub, &vmap, bar, 64, kvh, h * kHalf, blk);
+#pragma unroll
+            for (int c = 0; c < kKSubs; ++c) tma_load_4d(dst + h * kHalfBytes + c * kSub, &kmap, bar, c * 64, kvh, h * kHalf, blk);
+#pragma unroll
+            for (int c = 0; c < kVSubs; ++c) tma_load_4d(dst + h * kHalfBytes + (kKSubs + c) * kSub, &vmap, bar, c * 64, kvh, h * kHalf, blk);
         }
     };
-    if (threadIdx.x == 0) issue(page_lo, 0);
+    if (threadIdx.x == 0) issue(page_at(0), 0);
 
     // ---- Q fragments of this warp's 16 rows (rows r0 = 16 warp + g and r0 + 8), zero beyond the sequence ------------------------
     const T* qbase = static_cast<const T*>(p.q);
     const int r_lo = warp * 16 + g, r_hi = r_lo + 8;
-    uint32_t qa[8][4];
+    uint32_t qa[kDK / 16][4];
 #pragma unroll
-    for (int ks = 0; ks < 8; ++ks) {
+    for (int ks = 0; ks < kDK / 16; ++ks) {
         const int c = ks * 16 + 2 * t;
-        const T* ql = qbase + ((int64_t)(q_begin + q0 + r_lo) * p.num_heads + head) * kHd + c;
-        const T* qh = qbase + ((int64_t)(q_begin + q0 + r_hi) * p.num_heads + head) * kHd + c;
-        qa[ks][0] = r_lo < rows ? *reinterpret_cast<const uint32_t*>(ql) : 0u;
-        qa[ks][1] = r_hi < rows ? *reinterpret_cast<const uint32_t*>(qh) : 0u;
-        qa[ks][2] = r_lo < rows ? *reinterpret_cast<const uint32_t*>(ql + 8) : 0u;
-        qa[ks][3] = r_hi < rows ? *reinterpret_cast<const uint32_t*>(qh + 8) : 0u;
+        const T* ql = qbase + ((int64_t)(q_begin + q0 + r_lo) * p.num_heads + head) * hk + c;
+        const T* qh = qbase + ((int64_t)(q_begin + q0 + r_hi) * p.num_heads + head) * hk + c;
+        const bool in0 = !kSel || c < hk, in1 = !kSel || c + 8 < hk;       // sizes are multiples of 8: a pair lies inside a head or outside
+        qa[ks][0] = r_lo < rows && in0 ? *reinterpret_cast<const uint32_t*>(ql) : 0u;
+        qa[ks][1] = r_hi < rows && in0 ? *reinterpret_cast<const uint32_t*>(qh) : 0u;
+        qa[ks][2] = r_lo < rows && in1 ? *reinterpret_cast<const uint32_t*>(ql + 8) : 0u;
+        qa[ks][3] = r_hi < rows && in1 ? *reinterpret_cast<const uint32_t*>(qh + 8) : 0u;
     }
-    float o[16][4];
+    float o[kDV / 8][4];
 #pragma unroll
-    for (int i = 0; i < 16; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    for (int i = 0; i < kDV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     // with a sink the running maximum starts from it and the running sum from 1 (kept by one thread of the four that share a row)
     const float sink_log2 = (!kSigmoid && p.sink) ? p.sink[head] * 1.4426950408889634f : -INFINITY;
     float m_lo = sink_log2, m_hi = sink_log2, l_lo = (sink_log2 != -INFINITY && t == 0) ? 1.f : 0.f, l_hi = l_lo;
@@ -182,7 +199,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
         for (int nt = 0; nt < 4; ++nt) {
             const int row = nt * 8 + (lane & 7);
 #pragma unroll
-            for (int kp = 0; kp < 4; ++kp) {
+            for (int kp = 0; kp < kDK / 32; ++kp) {
                 const int chunk = kp * 4 + (lane >> 3);
                 uint32_t kb[4];
                 ldmatrix_x4(kb, kt + (chunk >> 3) * kSub + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
@@ -202,13 +219,22 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
                 if constexpr (pooled) {
                     ok_lo = tok < seen_lo; ok_hi = tok < seen_hi;
                 } else if (need_mask) {
-                    ok_lo = tok <= pos_lo && (p.window <= 0 || tok > pos_lo - p.window) && tok >= cs_lo;
-                    ok_hi = tok <= pos_hi && (p.window <= 0 || tok > pos_hi - p.window) && tok >= cs_hi;
+                    const bool kept = kSel && tok < p.keep_first;
+                    ok_lo = tok <= pos_lo && (p.window <= 0 || tok > pos_lo - p.window || kept) && tok >= cs_lo;
+                    ok_hi = tok <= pos_hi && (p.window <= 0 || tok > pos_hi - p.window || kept) && tok >= cs_hi;
                 }
                 if constexpr (kSigmoid) {
                     sacc[nt][e] = ok_lo ? __fdividef(1.0f, 1.0f + fast_exp2(-fmaf(sacc[nt][e], p.scale_log2, bias_log2))) : 0.f;
                     sacc[nt][2 + e] = ok_hi ? __fdividef(1.0f, 1.0f + fast_exp2(-fmaf(sacc[nt][2 + e], p.scale_log2, bias_log2))) : 0.f;
                 } else {
+                    if (kSel && p.cap_log2 > 0.f) {
+                        // cap tanh(x) = cap - 2 cap / (1 + e^(2x)), in units of log2: the error is absolute, a few ulp of the cap
+                        sacc[nt][e] = ok_lo ? fmaf(-2.f * p.cap_log2, fast_rcp(1.0f + fast_exp2(sacc[nt][e] * p.cap_in)), p.cap_log2) : -INFINITY;
+                        sacc[nt][2 + e] = ok_hi ? fmaf(-2.f * p.cap_log2, fast_rcp(1.0f + fast_exp2(sacc[nt][2 + e] * p.cap_in)), p.cap_log2) : -INFINITY;
+                        mx_lo = fmaxf(mx_lo, sacc[nt][e]);
+                        mx_hi = fmaxf(mx_hi, sacc[nt][2 + e]);
+                        continue;
+                    }
                     sacc[nt][e] = ok_lo ? sacc[nt][e] * p.scale_log2 : -INFINITY;
                     sacc[nt][2 + e] = ok_hi ? sacc[nt][2 + e] * p.scale_log2 : -INFINITY;
                     mx_lo = fmaxf(mx_lo, sacc[nt][e]);
@@ -237,15 +263,16 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
                 pa[nt][0] = pack2<T>(p0, p1); pa[nt][1] = pack2<T>(p2, p3);
             }
 #pragma unroll
-            for (int i = 0; i < 16; ++i) { o[i][0] *= c_lo; o[i][1] *= c_lo; o[i][2] *= c_hi; o[i][3] *= c_hi; }
+            for (int i = 0; i < kDV / 8; ++i) { o[i][0] *= c_lo; o[i][1] *= c_lo; o[i][2] *= c_hi; o[i][3] *= c_hi; }
         }
         // ---- O += P V : 2 k-steps (16 tokens) x 16 n-tiles (8 dims).  V rows past the context hold whatever the block contains:
         // their P is exactly 0 only if V is finite, so rows beyond klen are zeroed in shared memory first (as in the decode kernel);
         // a pooled tile is built with zeros past its last entry
         if (!pooled && tok0 + kHalf > klen) {   // (pooled is a compile-time constant here)
             __syncwarp();
-            for (int r = max(klen - tok0, 0) + (lane >> 4); r < kHalf; r += 2) {
-                const int ch = lane & 15;
+            constexpr int kCh = kDV / 8;                        // 16-byte groups of a value row
+            for (int r = max(klen - tok0, 0) + lane / kCh; r < kHalf; r += 32 / kCh) {
+                const int ch = lane % kCh;
                 *reinterpret_cast<int4*>(smem + (vt - smem_base) + (ch >> 3) * kSub + r * 128 + (((ch & 7) ^ (r & 7)) << 4)) = make_int4(0, 0, 0, 0);
             }
             __syncwarp();
@@ -255,7 +282,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
             const uint32_t a[4] = {pa[2 * ktk][0], pa[2 * ktk][1], pa[2 * ktk + 1][0], pa[2 * ktk + 1][1]};
             const int row = ktk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
 #pragma unroll
-            for (int np = 0; np < 8; ++np) {
+            for (int np = 0; np < kDV / 16; ++np) {
                 const int chunk = np * 2 + (lane >> 4);
                 uint32_t vb[4];
                 ldmatrix_x4_trans(vb, vt + (chunk >> 3) * kSub + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
@@ -274,7 +301,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
                 {
                     const int e = threadIdx.x >> 1, part = threadIdx.x & 1;          // entry of the tile, and which 64 of its 128 entries
                     const int b = b0 + e, r = e & 31;
-                    uint8_t* kdst = smem + kStage + (e >> 5) * 4 * kSub + part * kSub + r * 128;
+                    uint8_t* kdst = smem + kStage + (e >> 5) * kHalfBytes + part * kSub + r * 128;
                     const float* src[2] = {nullptr, nullptr};
                     if (b < seen_tile) {
                         const int page = (b * p.pool + p.pool - 1) / kPg;
@@ -298,8 +325,8 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
 #pragma unroll 1
                 for (int h = 0; h < 2; ++h) {
                     if (b0 + h * kHalf >= warp_seen) break;
-                    const uint32_t kt = smem_base + kStage + h * 4 * kSub;
-                    process(kt, kt + 2 * kSub, b0 + h * kHalf, std::true_type{});
+                    const uint32_t kt = smem_base + kStage + h * kHalfBytes;
+                    process(kt, kt + kKSubs * kSub, b0 + h * kHalf, std::true_type{});
                 }
                 __syncthreads();
             }
@@ -308,18 +335,18 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
         }
     }
 
-    for (int page = page_lo, it = 0; page <= page_hi; ++page, ++it) {
-        const int stage = it & 1;
-        if (threadIdx.x == 0 && page + 1 <= page_hi) issue(page + 1, stage ^ 1);      // that stage was drained before the last __syncthreads
+    for (int it = 0; it < num_pages; ++it) {
+        const int stage = it & 1, page = page_at(it);
+        if (threadIdx.x == 0 && it + 1 < num_pages) issue(page_at(it + 1), stage ^ 1);      // that stage was drained before the last __syncthreads
         mbar_wait(bars + stage * 8, (it >> 1) & 1);
 #pragma unroll 1
         for (int h = 0; h < 2; ++h) {
             const int tok0 = page * kPg + h * kHalf;                 // first token of this 32-token half
             if (tok0 > warp_max_pos) break;                          // entirely in the future of every row of this warp
-            if (p.window > 0 && tok0 + kHalf - 1 < warp_min_pos - p.window + 1) continue;      // entirely before every row's window
+            if (p.window > 0 && tok0 + kHalf - 1 < warp_min_pos - p.window + 1 && !(kSel && tok0 < p.keep_first)) continue;      // entirely before every row's window
             if (tok0 + kHalf - 1 < warp_min_cs) continue;                                      // entirely before every row's chunk
-            const uint32_t kt = smem_base + stage * kStage + h * 4 * kSub;
-            process(kt, kt + 2 * kSub, tok0, std::false_type{});
+            const uint32_t kt = smem_base + stage * kStage + h * kHalfBytes;
+            process(kt, kt + kKSubs * kSub, tok0, std::false_type{});
         }
         __syncthreads();                                             // every warp is done with this stage before it is refilled
     }
@@ -332,8 +359,33 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
         inv_lo = l_lo > 0.f ? 1.f / l_lo : 0.f; inv_hi = l_hi > 0.f ? 1.f / l_hi : 0.f;
     }
     T* obase = static_cast<T*>(p.out);
+    if constexpr (kSel) {
+        // a gate meets the f32 sums; a pair of entries is one store when the rows allow it
+        const bool pairs = (p.ldo & 1) == 0 && (reinterpret_cast<uintptr_t>(obase) & 3) == 0;
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+        for (int half = 0; half < 2; ++half) {
+            if ((half ? r_hi : r_lo) >= rows) continue;
+            const int64_t row = q_begin + q0 + (half ? r_hi : r_lo);
+            const float inv = half ? inv_hi : inv_lo;
+            T* orow = obase + row * p.ldo + head * hv;
+            const float* grow = p.gate ? p.gate + row * p.ldg + head * hv : nullptr;
+#pragma unroll
+            for (int i = 0; i < kDV / 8; ++i) {
+                const int c = i * 8 + 2 * t;
+                if (c >= hv) continue;
+                float a = o[i][2 * half] * inv, b = o[i][2 * half + 1] * inv;
+                if (grow) {
+                    a *= fast_rcp(1.0f + fast_exp2(-1.4426950408889634f * grow[c]));
+                    b *= fast_rcp(1.0f + fast_exp2(-1.4426950408889634f * grow[c + 1]));
+                }
+                if (pairs) *reinterpret_cast<uint32_t*>(orow + c) = pack2<T>(a, b);
+                else { orow[c] = from_f32<T>(a); orow[c + 1] = from_f32<T>(b); }
+            }
+        }
+        return;
+    }
+#pragma unroll
+    for (int i = 0; i < kDV / 8; ++i) {
         if (r_lo < rows)
             *reinterpret_cast<uint32_t*>(obase + ((int64_t)(q_begin + q0 + r_lo) * p.num_heads + head) * kHd + i * 8 + 2 * t) = pack2<T>(o[i][0] * inv_lo, o[i][1] * inv_lo);
         if (r_hi < rows)
@@ -354,11 +406,11 @@ EncodeTiledFn encode_fn() {
     }
     return fn;
 }
-bool make_kv_map(CUtensorMap* map, const void* cache, int64_t num_blocks, int kvh, int dtype) {
+bool make_kv_map(CUtensorMap* map, const void* cache, int64_t num_blocks, int kvh, int dtype, int hd = kHd) {
     EncodeTiledFn enc = encode_fn();
     if (!enc) return false;
-    const cuuint64_t dims[4] = {(cuuint64_t)kHd, (cuuint64_t)kvh, (cuuint64_t)kPg, (cuuint64_t)num_blocks};
-    const cuuint64_t strides[3] = {(cuuint64_t)kHd * 2, (cuuint64_t)kvh * kHd * 2, (cuuint64_t)kPg * kvh * kHd * 2};
+    const cuuint64_t dims[4] = {(cuuint64_t)hd, (cuuint64_t)kvh, (cuuint64_t)kPg, (cuuint64_t)num_blocks};
+    const cuuint64_t strides[3] = {(cuuint64_t)hd * 2, (cuuint64_t)kvh * hd * 2, (cuuint64_t)kPg * kvh * hd * 2};
     const cuuint32_t box[4] = {64, 1, (cuuint32_t)kHalf, 1};
     const cuuint32_t estr[4] = {1, 1, 1, 1};
     return enc(map, dtype == B200_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 4, const_cast<void*>(cache), dims, strides,
@@ -385,15 +437,15 @@ void paged_attention_prefill_tc(void* out, const void* q, const void* kc, const 
         return;
     }
     PrefillParams p{q, out, block_tables, cu_q, cu_k, num_seqs, num_heads, num_kv_heads, max_blocks, window, chunk, scale * 1.4426950408889634f,
-                    nullptr, nullptr, nullptr, nullptr, 0, 0};
+                    nullptr, nullptr, nullptr, nullptr, 0, 0, kHd, kHd, 0, 0.f, 0.f, nullptr, 0, (int64_t)num_heads * kHd};
     bool sigmoid = false;
     if (extras) {
         p.sink = extras->sink; p.head_bias = extras->head_bias; sigmoid = extras->sigmoid;
         if (extras->pooled_keys && extras->pool > 0) { p.kp = extras->pooled_keys; p.vp = extras->pooled_values; p.pool = extras->pool; p.per_block = extras->per_block; }
     }
     const int tiles = total_q / kQTile + num_seqs;                   // >= sum of ceil(q_len / 64)
-#define PF_LAUNCH(TT, SG, PL) do { ensure_dynamic_smem(reinterpret_cast<const void*>(paged_attn_prefill_kernel<TT, SG, PL>), kPfSmem); \
-        paged_attn_prefill_kernel<TT, SG, PL><<<dim3(tiles, num_heads), kPfThreads, kPfSmem, st>>>(km, vm, p); } while (0)
+#define PF_LAUNCH(TT, SG, PL) do { ensure_dynamic_smem(reinterpret_cast<const void*>(paged_attn_prefill_kernel<TT, SG, PL, false, kHd, kHd>), prefill_smem(kHd, kHd)); \
+        paged_attn_prefill_kernel<TT, SG, PL, false, kHd, kHd><<<dim3(tiles, num_heads), kPfThreads, prefill_smem(kHd, kHd), st>>>(km, vm, p); } while (0)
     const bool pooled = p.kp != nullptr && p.window > 0;                 // pooled entries come with the sigmoid form only
     if (pooled && !sigmoid) { set_error(kErrUnsupported, "paged_attention_prefill: pooled entries need the sigmoid form"); return; }
     if (dtype == B200_BF16) { if (pooled) PF_LAUNCH(__nv_bfloat16, true, true); else if (sigmoid) PF_LAUNCH(__nv_bfloat16, true, false); else PF_LAUNCH(__nv_bfloat16, false, false); }
@@ -401,6 +453,33 @@ void paged_attention_prefill_tc(void* out, const void* q, const void* kc, const 
 #undef PF_LAUNCH
     count_launch();
     check_launch("paged_attention_prefill");
+}
+
+bool paged_attention_prefill_sel_supported(int dk, int dv, int block_size, const void* q, const void* kc, const void* vc) {
+    return dk % 8 == 0 && dv % 8 == 0 && dk > 0 && dv > 0 && dk <= 128 && dv <= 128 && block_size == kPg && ((uintptr_t)q & 3) == 0 &&
+           (((uintptr_t)kc | (uintptr_t)vc) & 15) == 0 && encode_fn() != nullptr;
+}
+
+void paged_attention_prefill_sel(void* out, int64_t ld_out, const void* q, const void* kc, const void* vc, const uint32_t* block_tables, const uint32_t* cu_q,
+                                 const uint32_t* cu_k, int num_seqs, int total_q, int num_heads, int num_kv_heads, int dk, int dv, int max_blocks, float scale, int chunk,
+                                 int window, int keep_first, float softcap, const float* sink, const float* gate, int64_t ld_gate, cudaStream_t st) {
+    CUtensorMap km, vm;
+    const int64_t num_blocks = (int64_t)1 << 22;
+    if (!make_kv_map(&km, kc, num_blocks, num_kv_heads, B200_BF16, dk) || !make_kv_map(&vm, vc, num_blocks, num_kv_heads, B200_BF16, dv)) {
+        set_error(kErrCuda, "paged_attention_prefill: cuTensorMapEncodeTiled failed");
+        return;
+    }
+    constexpr float kLog2e = 1.4426950408889634f;
+    PrefillParams p{q, out, block_tables, cu_q, cu_k, num_seqs, num_heads, num_kv_heads, max_blocks, window, chunk, scale * kLog2e, sink, nullptr, nullptr, nullptr, 0, 0,
+                    dk, dv, keep_first, softcap * kLog2e, softcap > 0.f ? 2.f * scale * kLog2e / softcap : 0.f, gate, ld_gate, ld_out};
+    const int tiles = total_q / kQTile + num_seqs;                   // >= sum of ceil(q_len / 64)
+#define PS_LAUNCH(DK, DV) do { ensure_dynamic_smem(reinterpret_cast<const void*>(paged_attn_prefill_kernel<__nv_bfloat16, false, false, true, DK, DV>), prefill_smem(DK, DV)); \
+        paged_attn_prefill_kernel<__nv_bfloat16, false, false, true, DK, DV><<<dim3(tiles, num_heads), kPfThreads, prefill_smem(DK, DV), st>>>(km, vm, p); } while (0)
+    if (dk <= 64) { if (dv <= 64) PS_LAUNCH(64, 64); else PS_LAUNCH(64, 128); }
+    else { if (dv <= 64) PS_LAUNCH(128, 64); else PS_LAUNCH(128, 128); }
+#undef PS_LAUNCH
+    count_launch();
+    check_launch("paged_attention_prefill_sel");
 }
 
 }  // namespace b200

@@ -294,6 +294,13 @@ void paged_attention_varlen_ex(void* out, int64_t ld_out, const void* q, const v
                                    window, B200_BF16, st, chunk, &extras);
         return;
     }
+    // the same kernel in its general form: other sizes, kept tokens, capped scores, gates
+    if (!no_tc && q_dtype == B200_BF16 && out_dtype == B200_BF16 && cache_dtype == B200_BF16 && cu_seqlens_q && cu_seqlens_k && num_seqs > 0 &&
+        paged_attention_prefill_sel_supported(dk, dv, block_size, q, key_cache, value_cache)) {
+        paged_attention_prefill_sel(out, ld_out, q, key_cache, value_cache, (const uint32_t*)block_tables, (const uint32_t*)cu_seqlens_q, (const uint32_t*)cu_seqlens_k,
+                                    num_seqs, num_tokens, num_heads, num_kv_heads, dk, dv, table_width, scale, chunk, window, keep_first, softcap, sink, gate, ld_gate, st);
+        return;
+    }
     B200_REQUIRE(dv <= 32 * kMaxVPerLane && dk <= 2048, kErrUnsupported, "paged_attention_varlen: value size %d > %d or key size %d > 2048", dv,
                  32 * kMaxVPerLane, dk);
     const int64_t items = (int64_t)num_tokens * num_heads;

@@ -15,6 +15,7 @@
 //                           registers and walks the portion in tiles of 16 tokens staged through shared memory, the next
 //                           tile in flight while the current one is applied.  Decode (one token per entry) is one read and
 //                           one write of the state.
+//   gated_delta_rule_channel  the same with one decay per token and key row, S <- diag(g_t) S, handed in as f32 [T, H dk] (delta_chunk.cu: over chunks).
 //   gated_rms_norm          out = o / rms(o over dv) * w * silu(gate), per (token, head).
 #include "common.cuh"
 
@@ -789,19 +790,19 @@ void gated_delta_rule_tiled(const float* qkv, const float* proj, int64_t ld_proj
     check_launch("gated_delta_rule_tiled");
 }
 
-void gated_delta_rule_channel(const float* qkv, const float* proj, int64_t ld_proj, int32_t off_b, const float* decay, float* state, float* out, float* scratch,
-                              const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t max_rows,
-                              int32_t mode, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int64_t stream) {
+void gated_delta_rule_channel(const float* qkv, const float* proj, int64_t ld_proj, int32_t off_b, const float* decay, float* state, float* out,
+                              const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t single_rows,
+                              int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int64_t stream) {
     if (num_seqs == 0 || num_tokens == 0) return;
     B200_REQUIRE(qkv && proj && decay && state && out && cu_seqlens && seq_slots && seq_start, kErrBadArg, "gated_delta_rule_channel: null pointer");
-    B200_REQUIRE(num_heads > 0 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && dk > 0 && dv > 0 && num_seqs <= 65535 && max_rows > 0 && mode >= 0 && mode <= 2 &&
-                 (mode != 1 || num_tokens == num_seqs), kErrBadArg, "gated_delta_rule_channel: bad sizes");
+    B200_REQUIRE(num_heads > 0 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && dk > 0 && dv > 0 && num_seqs <= 65535 &&
+                 (!single_rows || num_tokens == num_seqs), kErrBadArg, "gated_delta_rule_channel: bad sizes");
     B200_REQUIRE(dk <= 512, kErrUnsupported, "gated_delta_rule_channel: key size %d > 512", dk);
     cudaStream_t st = as_stream(stream);
     const dim3 grid(ceil_div(dv, 16), num_heads, num_seqs);
     const float* none = nullptr;
 #define GDC(R) do { \
-        if (mode == 1) { \
+        if (single_rows) { \
             launch_pdl(gated_delta_step_kernel<R, true>, grid, dim3(128), 0, st, qkv, proj, ld_proj, off_b, 0, none, none, decay, state, out, seq_slots, seq_start, num_heads, \
                        num_kv_heads, dk, dv); \
         } else { \

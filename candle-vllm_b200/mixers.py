@@ -156,6 +156,7 @@ class PagedAttentionMixer:
         self.decode_kernel = (self.q_dtype == torch.bfloat16 and self.chunk % block_size == 0 and self.window == 0 and heads // kv_heads in (1, 2, 4, 8) and
                               self.sink is None)
         self._scratch = {}
+        self.selected_tc = ops.selected_tensor_cores(heads, kv_heads, dk, dv, block_size, dtype) and self.chunk == 0
         self.cos = self.sin = None
         self._device = self.w_in.device
         if rot:
@@ -184,7 +185,7 @@ class PagedAttentionMixer:
         selected = out is not None or self.keep_first > 0 or self.softcap > 0 or self.element_gate
         if selected and self.has_gate and not self.element_gate:
             raise BackendError("PagedAttentionMixer: one gate per head does not combine with kept tokens, a score cap or a given output")
-        q_dtype = torch.float32 if selected else self.q_dtype
+        q_dtype = (torch.bfloat16 if self.selected_tc else torch.float32) if selected else self.q_dtype
         if self.per_head:
             q = ops.qk_head_norm_rope_cache(proj, self.bias, self.q_norm, self.k_norm, self.cos, self.sin, batch, k_cache, v_cache, self.H, self.G, self.dk, self.dv,
                                             self.rot_dims, self.eps, interleaved=self.interleaved, norm=self.head_norm, q_dtype=q_dtype)

@@ -975,18 +975,41 @@ def cast_rows(x: torch.Tensor) -> torch.Tensor:
     return out
 
 
+SELECTED_PREFILL_MIN_ROWS = 8     # steps in which some entry brings at least this many rows take the tile kernel (bf16); shorter portions go row by row
+SELECTED_ROW_BLOCKS = 592         # four blocks of four warps per SM: steps with fewer rows cut the visible keys of every row into runs
+
+
+def selected_tensor_cores(heads: int, kv_heads: int, dk: int, dv: int, block_size: int, dtype: torch.dtype) -> bool:
+    """do both tensor-core kernels of ``paged_attention_selected`` take these sizes?  (q is then handed over in 16 bits)"""
+    return dtype == torch.bfloat16 and block_size == 64 and bool(lib().paged_attention_rows_supported(C.c_int32(heads), C.c_int32(kv_heads), C.c_int32(dk), C.c_int32(dv)))
+
+
 def paged_attention_selected(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch: StepBatch, heads: int, scale: float, chunk: int, window: int,
-                             keep_first: int, softcap: float, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], out: torch.Tensor) -> torch.Tensor:
+                             keep_first: int, softcap: float, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], out: torch.Tensor,
+                             splits: Optional[int] = None) -> torch.Tensor:
     """``paged_attention_varlen_sink`` with kept first tokens (a key at a position below ``keep_first`` stays visible whatever the window), scores softcap tanh(s /
     softcap) (0 = as they are) and, with ``gate`` f32 [T, H dv] (row stride allowed), the outputs times sigmoid(gate) entry by entry; writes into ``out`` [T, H dv]
-    (row stride allowed)"""
+    (row stride allowed).  A bf16 q (``selected_tensor_cores``) takes the tensor cores: tiles of 64 rows for portions of prompts, else row by row with the visible keys
+    in ``splits`` runs (None: enough blocks to fill the device, from the table width, so that a captured step keeps its choice)."""
     T = q.shape[0]
     nb, bs, G, dk = k_cache.shape
     dv = v_cache.shape[3]
     if out.shape != (T, heads * dv) or out.stride(1) != 1 or (gate is not None and (gate.dtype != torch.float32 or gate.shape != out.shape or gate.stride(1) != 1)):
         raise BackendError(f"paged_attention_selected: out {tuple(out.shape)} / gate for {T} rows of {heads} x {dv}")
     pitch = lambda t: 0 if t is None else (t.stride(0) if T > 1 else max(heads * dv, t.stride(0)))
-    lib().paged_attention_varlen_ex(_ptr(out), C.c_int64(pitch(out)), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), C.c_int32(batch.block_tables.shape[1]),
+    W = batch.block_tables.shape[1]
+    if q.dtype == torch.bfloat16 and chunk == 0 and (splits is not None or batch.max_rows < SELECTED_PREFILL_MIN_ROWS):
+        if splits is None:
+            longest = W * bs if window <= 0 else min(window + keep_first, W * bs)
+            splits = max(1, min(SELECTED_ROW_BLOCKS // (T * G * -(-heads // G // 16)), longest // 128, 64))
+        part = torch.empty((T * heads * splits * (dv + 2),), dtype=torch.float32, device=q.device) if splits > 1 else None
+        lib().paged_attention_rows(_ptr(out), C.c_int64(pitch(out)), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), C.c_int32(W), _ptr(batch.token_seq),
+                                   _ptr(batch.positions), C.c_int32(T), C.c_int32(heads), C.c_int32(G), C.c_int32(dk), C.c_int32(dv), C.c_int32(bs), C.c_float(scale),
+                                   C.c_int32(window), C.c_int32(keep_first), C.c_float(softcap), _ptr(sink), _ptr(gate), C.c_int64(pitch(gate)), C.c_int32(splits), _ptr(part),
+                                   _stream(q.device))
+        check("paged_attention_rows")
+        return out
+    lib().paged_attention_varlen_ex(_ptr(out), C.c_int64(pitch(out)), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), C.c_int32(W),
                                     _ptr(batch.token_seq), _ptr(batch.positions), _ptr(batch.cu_seqlens), _ptr(batch.cu_seqlens_k), C.c_int32(batch.num_seqs), C.c_int32(T),
                                     C.c_int32(heads), C.c_int32(G), C.c_int32(dk), C.c_int32(dv), C.c_int32(bs), C.c_float(scale), C.c_int32(chunk), C.c_int32(window),
                                     C.c_int32(keep_first), C.c_float(softcap), _ptr(sink), _ptr(gate), C.c_int64(pitch(gate)), C.c_int32(_tag(q.dtype)),
@@ -1010,23 +1033,36 @@ def token_shift_mix(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, batc
     return out
 
 
+CHUNKED_DELTA_MIN_ROWS = 32              # steps in which some entry brings at least this many rows take the chunked form of the rule
+CHUNKED_DELTA_SCRATCH = 1 << 32          # bytes of scratch above which a step stays on the token-by-token kernel
+
+
 def gated_delta_rule_channel(qkv: torch.Tensor, proj: torch.Tensor, off_b: int, decay: torch.Tensor, state: torch.Tensor, batch: StepBatch, heads: int, kv_heads: int, dk: int,
                              dv: int, kernel: Optional[str] = None) -> torch.Tensor:
-    """``gated_delta_rule`` with a decay per token and key row: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; decay f32 [T, H dk]; the same three
-    kernels ("step", "token", "tiled"), chosen by the step's shape the same way"""
+    """``gated_delta_rule`` with a decay per token and key row: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; decay f32 [T, H dk].  Three kernels:
+    "step" (every entry brings one token), "token" (token by token, any step) and "chunked" (over chunks of 64 tokens, for portions of prompts; key sizes up to 128);
+    ``kernel`` forces one, None chooses by the step's shape."""
     T = qkv.shape[0]
     if decay.dtype != torch.float32 or decay.shape != (T, heads * dk) or not decay.is_contiguous() or not qkv.is_contiguous():
         raise BackendError(f"gated_delta_rule_channel: decays {tuple(decay.shape)} {decay.dtype} for {T} rows of {heads} x {dk}")
     out = torch.empty((T, heads * dv), dtype=torch.float32, device=qkv.device)
+    ld_proj = C.c_int64(proj.stride(0) if T > 1 else proj.shape[1])
+    need = int(lib().gated_delta_channel_chunked_scratch(C.c_int32(T), C.c_int32(batch.num_seqs), C.c_int32(heads), C.c_int32(dk), C.c_int32(dv)))
     if kernel is None:
         kernel = "step" if batch.pure_decode else "token"
-    try:
-        mode = {"token": 0, "step": 1, "tiled": 2}[kernel]
-    except KeyError:
+        if dk <= 128 and batch.max_rows >= CHUNKED_DELTA_MIN_ROWS and need * 4 <= CHUNKED_DELTA_SCRATCH and -(-batch.max_rows // 64) * batch.num_seqs <= 65535:
+            kernel = "chunked"
+    if kernel == "chunked":
+        scratch = torch.empty((need,), dtype=torch.float32, device=qkv.device)
+        lib().gated_delta_channel_chunked(_ptr(qkv), _ptr(proj), ld_proj, C.c_int32(off_b), _ptr(decay), _ptr(state), _ptr(out), _ptr(scratch), _ptr(batch.cu_seqlens),
+                                          _ptr(batch.seq_slots), _ptr(batch.seq_start), C.c_int32(T), C.c_int32(batch.num_seqs), C.c_int32(batch.max_rows),
+                                          C.c_int32(heads), C.c_int32(kv_heads), C.c_int32(dk), C.c_int32(dv), _stream(qkv.device))
+        check("gated_delta_channel_chunked")
+        return out
+    if kernel not in ("step", "token"):
         raise BackendError(f"gated_delta_rule_channel: unknown kernel {kernel!r}")
-    scratch = None
-    lib().gated_delta_rule_channel(_ptr(qkv), _ptr(proj), C.c_int64(proj.stride(0) if T > 1 else proj.shape[1]), C.c_int32(off_b), _ptr(decay), _ptr(state), _ptr(out),
-                                   _ptr(scratch), _ptr(batch.cu_seqlens), _ptr(batch.seq_slots), _ptr(batch.seq_start), C.c_int32(T), C.c_int32(batch.num_seqs),
-                                   C.c_int32(batch.max_rows), C.c_int32(mode), C.c_int32(heads), C.c_int32(kv_heads), C.c_int32(dk), C.c_int32(dv), _stream(qkv.device))
+    lib().gated_delta_rule_channel(_ptr(qkv), _ptr(proj), ld_proj, C.c_int32(off_b), _ptr(decay), _ptr(state), _ptr(out), _ptr(batch.cu_seqlens), _ptr(batch.seq_slots),
+                                   _ptr(batch.seq_start), C.c_int32(T), C.c_int32(batch.num_seqs), C.c_int32(1 if kernel == "step" else 0), C.c_int32(heads),
+                                   C.c_int32(kv_heads), C.c_int32(dk), C.c_int32(dv), _stream(qkv.device))
     check("gated_delta_rule_channel")
     return out

@@ -742,8 +742,12 @@ void talking_attention_prefill(void* out, const void* q, const void* key_cache, 
  * linear_attention_channel_bonus: linear_attention_channel whose output is read before the token's decay and write: o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t,
  *   bonus f32 [H, dk] (null: linear_attention_channel itself).  Offsets are 64-bit: q, k and v may be matrices of their own with one row pitch.
  * gated_delta_rule_channel: gated_delta_rule with a decay per token and key row: S <- diag(g_t) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; decay f32 [T, H dk].
- *   mode 0: token by token, any step; 1: every entry brings exactly one row; 2: over tiles of 16 tokens (dk <= 128, scratch =
- *   gated_delta_channel_scratch(...) floats).  dk <= 512 in modes 0 and 1.
+ *   single_rows != 0: every entry brings exactly one row; else token by token, any step.  dk <= 512.
+ * gated_delta_channel_chunked: the same over chunks of 64 tokens (dk <= 128; scratch = gated_delta_channel_chunked_scratch(...) floats, 16-byte aligned; max_rows = the
+ *   most rows any entry brings).
+ * paged_attention_rows: paged_attention_varlen_ex without a chunk rule for rows taken one at a time (decoded tokens, short portions), q / caches / out BF16, on tensor
+ *   cores: dk and dv multiples of 8 up to 128 (paged_attention_rows_supported: 1 if the sizes fit).  splits > 1: every row's visible keys are cut into that many runs,
+ *   part = T * H * splits * (dv + 2) floats.
  * scaled_post_norm_add: post_norm_add_rms_norm of y_scale * y + y_bias; with weight null and out given, out takes the new x as it is.
  * group_rms_norm_gate_into: group_rms_norm_gate with an output row pitch ld_out.
  * cast_rows_bf16: out BF16 [rows, n] (row pitch ld_out) = x f32 (row pitch ldx). */
@@ -760,9 +764,18 @@ void linear_attention_channel_bonus(const float* proj, int64_t ld, int64_t off_q
                                     float q_scale, float* state, float* out, float* scratch, const int32_t* cu_seqlens, const int32_t* seq_slots,
                                     const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t max_rows, int32_t mode, int32_t num_heads, int32_t dk,
                                     int32_t dv, int64_t stream);
-void gated_delta_rule_channel(const float* qkv, const float* proj, int64_t ld_proj, int32_t off_b, const float* decay, float* state, float* out, float* scratch,
-                              const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t max_rows,
-                              int32_t mode, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int64_t stream);
+void gated_delta_rule_channel(const float* qkv, const float* proj, int64_t ld_proj, int32_t off_b, const float* decay, float* state, float* out,
+                              const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t single_rows,
+                              int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int64_t stream);
+int64_t gated_delta_channel_chunked_scratch(int32_t num_tokens, int32_t num_seqs, int32_t num_heads, int32_t dk, int32_t dv);
+void gated_delta_channel_chunked(const float* qkv, const float* proj, int64_t ld_proj, int32_t off_b, const float* decay, float* state, float* out, float* scratch,
+                                 const int32_t* cu_seqlens, const int32_t* seq_slots, const int32_t* seq_start, int32_t num_tokens, int32_t num_seqs, int32_t max_rows,
+                                 int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv, int64_t stream);
+int32_t paged_attention_rows_supported(int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv);
+void paged_attention_rows(void* out, int64_t ld_out, const void* q, const void* key_cache, const void* value_cache, const int32_t* block_tables, int32_t table_width,
+                          const int32_t* token_seq, const int32_t* positions, int32_t num_tokens, int32_t num_heads, int32_t num_kv_heads, int32_t dk, int32_t dv,
+                          int32_t block_size, float scale, int32_t window, int32_t keep_first, float softcap, const float* sink, const float* gate, int64_t ld_gate,
+                          int32_t splits, float* part, int64_t stream);
 void scaled_post_norm_add(float* x, const float* y, int64_t ldy, float y_scale, const float* y_bias, const float* post_weight, const float* weight, void* out,
                           const int32_t* row_index, int32_t rows, int32_t n, float eps, int32_t out_dtype, int64_t stream);
 void group_rms_norm_gate_into(const float* o, int64_t ldo, const float* weight, const float* gate, int64_t ld_gate, void* out, int64_t ld_out, int32_t num_tokens, int32_t n,
