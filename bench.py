@@ -49,11 +49,11 @@ def parse():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--cpu-seconds", type=float, default=20.0)
     ap.add_argument("--parity-steps", type=int, default=3, help="decode steps compared against a TP=1 engine before timing (0 = off)")
-    ap.add_argument("--arch", default="llama", choices=["llama", "gobesun", "guvusun", "panarax", "dofevik", "sigalorn"],
+    ap.add_argument("--arch", default="llama", choices=["llama", "gobesun", "guvusun", "panarax", "dofevik", "sigalorn", "tavevik"],
                     help="llama = the metric (default, unchanged).  gobesun = prefill / decode throughput of the Gobesun decoder at layer sizes of real "
                          "models (random weights), beside a dense bf16 Llama of equal width / heads / ff / depth, with a per-kernel roofline table; "
-                         "one JSON line, single GPU.  guvusun / panarax / dofevik / sigalorn = the same for those decoders (panarax and sigalorn beside a Gobesun, dofevik "
-                         "beside a Guvusun of equal size).")
+                         "one JSON line, single GPU.  guvusun / panarax / dofevik / sigalorn / tavevik = the same for those decoders (panarax, sigalorn and tavevik "
+                         "beside a Gobesun, dofevik beside a Guvusun of equal size).")
     ap.add_argument("--arch-sizes", default="w2048,w4096")
     return ap.parse_args()
 
@@ -1695,6 +1695,228 @@ def run_sigalorn(args):
                       "gpu_launches": int(pkg.lib().b200_total_kernel_launches() - l0), "sizes": results}))
 
 
+# ------------------------------------------------------------------------------------------------
+# --arch tavevik: windowed attention side by side with token-shift linear attention or a delta rule with a decay per key row, beside a Gobesun (delta rule and
+# chunk-masked attention layers) of equal size
+# ------------------------------------------------------------------------------------------------
+TAVEVIK_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv=4, dim=128, vdim=128, ff=5632, vocab=32000, layers=8, window=2048, keep=4, ranks=(64, 128, 128)),
+    "w4096": dict(width=4096, heads=32, kv=8, dim=128, vdim=128, ff=11008, vocab=32000, layers=4, window=2048, keep=4, ranks=(64, 128, 128)),
+    # attention heads of unequal key and value size, all over one kv head
+    "w2048mq": dict(width=2048, heads=16, kv=1, dim=64, vdim=128, ff=5632, vocab=32000, layers=8, window=1024, keep=16, ranks=(64, 128, 128)),
+}
+
+
+def run_tavevik(args):
+    import torch
+    import candle_vllm_b200 as pkg
+    from candle_vllm_b200 import seq_ops as ops, synthetic as S
+    from candle_vllm_b200.engine import ModelRunner
+    from candle_vllm_b200.gobesun import GobesunConfig, GobesunModel
+    from candle_vllm_b200.inputs import prepare_step
+    from candle_vllm_b200.tavevik import TavevikConfig, TavevikModel
+
+    torch.cuda.set_device(0)
+    dev = "cuda"
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else \
+        {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "fallback": True}
+    HBM, TC = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    props = torch.cuda.get_device_properties(0)
+    F32 = props.multi_processor_count * 128 * 2 * 1.965e9            # nominal f32 multiply-add rate: the recurrences are 32-bit by definition
+    K, W = max(args.steps, 1), max(args.warmup, 3)
+    P, B, CTX, hd = 4096, 32, 1024, 128
+    bf = torch.bfloat16
+    l0 = pkg.lib().b200_total_kernel_launches()
+
+    def timed(fn, reps, warm=3):
+        for _ in range(warm):
+            fn()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(reps):
+            fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / reps * 1e-3
+
+    def once(fn):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize(); e0.record()
+        r = fn()
+        e1.record(); torch.cuda.synchronize()
+        return r, e0.elapsed_time(e1) * 1e-3
+
+    names = ["linear", "linear_grouped", "rms_norm_ex", "post_norm_add_rms_norm", "gelu_tanh_mul", "glu_packed", "embedding_scaled", "cast_rows", "causal_conv_silu", "causal_conv",
+             "token_shift_mix", "gated_delta_rule", "gated_delta_rule_channel", "gated_rms_norm", "group_rms_norm_gate", "low_rank_map", "linear_attention_channel",
+             "qk_norm_rope_cache", "qk_head_norm_rope_cache", "paged_attention_varlen_sink", "paged_attention_decode_chunked", "paged_attention_selected"]
+
+    def key_of(n, a, k):
+        if n == "linear":
+            return f"linear[{a[1].shape[0]}x{a[1].shape[1]}]"
+        if n == "linear_grouped":
+            return "linear_grouped[" + "x".join(str(v) for v in a[1].shape) + "]"
+        if n == "low_rank_map":
+            return f"low_rank_map[{a[3]}, rank {a[1].shape[1]}]"
+        if n == "paged_attention_selected":
+            return "paged_attention_selected[" + ("cap, kept, gate]" if a[9] > 0 else "sink]")
+        return n
+
+    def measure(model, V):
+        """(prefill s, decode s per step incl. host, decode s per step device, {(tag, kernel): [s]})"""
+        blocks_per = -(-(CTX + K + W + 8) // 64)
+        runner = ModelRunner(model, B * blocks_per + P // 64 + 1, B + 1, 64, decode_graphs=True, max_blocks_per_seq=blocks_per)
+        toks = torch.randint(0, V, (P,), generator=torch.Generator().manual_seed(1)).tolist()
+
+        def prefill():
+            runner.admit(10 ** 6)
+            runner.execute([dict(seq_id=10 ** 6, tokens=toks, want=[P - 1])])
+            runner.release(10 ** 6)
+        pre = timed(prefill, 3, 2)
+        for i in range(B):
+            runner.admit(i)
+        for i in range(0, B, 4):
+            runner.execute([dict(seq_id=j, tokens=toks[:CTX], want=[]) for j in range(i, i + 4)])
+        step_entries = lambda: [dict(seq_id=j, tokens=[toks[j]], want=[0]) for j in range(B)]
+        dec = timed(lambda: runner.execute(step_entries()), K, W)
+        dec_dev = timed(runner._graphs[B].graph.replay, K, 3)
+        kern = {}
+        orig = {n: getattr(ops, n) for n in names}
+
+        def instrument(tag):
+            def wrap(n):
+                def f(*a, **k):
+                    r, s = once(lambda: orig[n](*a, **k))
+                    kern.setdefault((tag, key_of(n, a, k)), []).append(s)
+                    return r
+                return f
+            for n in names:
+                setattr(ops, n, wrap(n))
+        instrument("prefill")
+        prefill(); kern.clear(); prefill()
+        runner.decode_graphs = False
+        instrument("decode")
+        runner.execute(step_entries())
+        for k in [k for k in kern if k[0] == "decode"]:
+            kern.pop(k)
+        runner.execute(step_entries())
+        for n in names:
+            setattr(ops, n, orig[n])
+        del runner
+        torch.cuda.empty_cache()
+        return pre, dec, dec_dev, kern
+
+    sampler = ClockSampler(0); sampler.start()
+    results = {}
+    for name in [n for n in (args.arch_sizes.split(",") + (["w2048mq"] if "w2048" in args.arch_sizes.split(",") else [])) if n in TAVEVIK_SIZES]:
+        z = TAVEVIK_SIZES[name]
+        D, H, G, dk, dv, ff, V, NL, win, keep = (z[k] for k in ("width", "heads", "kv", "dim", "vdim", "ff", "vocab", "layers", "window", "keep"))
+        SH, SD, Gd = D // 64, 64, H // 2                                # token-shift heads of 64; delta rule: H heads of 128 over H / 2 key heads, like the Gobesun's
+        layers = []
+        for i in range(NL):
+            layers.append(S.tavevik_shift_layer(H, G, dk, dv, SH, SD, win, keep, dk, 1e6, softcap=30.0, ff=ff, limit=7.0) if i % 2 == 0 else
+                          S.tavevik_delta_layer(H, G, dk, dv, H, Gd, hd, hd, 4, win, dk // 2, 1e6, ff=ff, limit=7.0))
+        cfg = S.tavevik_config(D, V, layers)
+        model = TavevikModel(TavevikConfig.from_dict(cfg), S.tavevik_weights(cfg, 0, z["ranks"]), dtype=bf, block_size=64, max_pos=P + 64, device=dev)
+        t_pre, t_dec, t_dec_dev, t_kern = measure(model, V)
+        del model
+        torch.cuda.empty_cache()
+        # ---- Gobesun of equal width / heads / ff / depth
+        glayers = [S.gobesun_attention_layer(H, max(G, 2), hd, hd, 2048, hd, ff=ff, base=1e6) if i % 2 == 0 else S.gobesun_delta_layer(H, Gd, hd, hd, conv=4, ff=ff)
+                   for i in range(NL)]
+        gcfg = S.gobesun_config(D, V, glayers)
+        gmodel = GobesunModel(GobesunConfig.from_dict(gcfg), S.gobesun_weights(gcfg, 0), dtype=bf, block_size=64, max_pos=P + 64, device=dev)
+        g_pre, g_dec, g_dec_dev, g_kern = measure(gmodel, V)
+        del gmodel
+        torch.cuda.empty_cache()
+        # ---- like kernels of other models, same heads and sizes, timed alone the way the models' calls are: the linear attention whose output is read after the write
+        # (Sigalorn) and its low-rank decays
+        like = {}
+        for tag, entries, T in (("prefill", [dict(tokens=[0] * P, start=0, block_table=list(range(P // 64)), state_slot=0, want=[])], P),
+                                ("decode", [dict(tokens=[0], start=CTX, block_table=list(range(CTX // 64 + 1)), state_slot=j, want=[]) for j in range(B)], B)):
+            bt = ops.StepBatch.from_host(prepare_step(entries, 64), dev)
+            pr, al, st = torch.randn(T, 3 * D, device=dev) * 0.1, torch.full((T, D), 0.97, device=dev), torch.zeros(B, SH, SD, SD, device=dev)
+            y, w, b = torch.randn(T, 64, device=dev), torch.randn(D, 64, device=dev), torch.randn(D, device=dev)
+            calls = {"linear_attention_channel[after the write]": lambda: ops.linear_attention_channel(pr, 0, D, 2 * D, al, st, bt, SH, SD, SD),
+                     "low_rank_map[root_sigmoid, rank 64]": lambda: ops.low_rank_decay(y, w, b, 16.0)}
+            for key, call in calls.items():
+                for _ in range(3):
+                    call()
+                like[(tag, key)] = [once(call)[1] for _ in range(5)]
+            del pr, al, st
+        torch.cuda.empty_cache()
+        med = lambda v: (sorted(v)[(len(v) - 1) // 2] + sorted(v)[len(v) // 2]) / 2
+        esz = 2
+        Cd = 2 * Gd * hd + H * hd
+
+        def work(side, tag, key, T):
+            """algorithmic work of one call: ("bytes", n) against the measured copy bandwidth, ("flops", n) against the measured bf16 GEMM rate, ("f32", n) against
+            the nominal f32 multiply-add rate"""
+            pre = tag == "prefill"
+            if key.startswith("linear["):
+                n, k = (int(v) for v in key[7:-1].split("x"))
+                if n == V and pre:
+                    T = 1
+                return ("flops", 2.0 * T * n * k) if (pre and T > 1) else ("bytes", n * k * esz + T * (k * esz + n * 4))
+            if key.startswith("linear_grouped["):
+                e, n, k = (int(v) for v in key[15:-1].split("x"))
+                return ("flops", 2.0 * e * T * n * k) if pre else ("bytes", e * (n * k * esz + T * (k * esz + n * 4)))
+            if key.startswith("low_rank_map["):
+                r = int(key[:-1].split("rank ")[1])
+                return ("f32", 2.0 * T * D * r) if pre else ("bytes", T * (D + r) * 4 + D * r * 4)
+            state = lambda h, k, v: (1 if pre else T) * 2 * h * k * v * 4              # one read and one write of every entry's state
+            mine = side == "tavevik"
+            kdim, vdim, kvh = (dk, dv, G) if mine else (hd, hd, max(G, 2))
+            if mine:
+                seen = sum(min(i + 1, win + min(keep, max(0, i + 1 - win))) for i in range(T)) if pre else T * min(CTX + 1, win + keep)
+            else:
+                seen = sum(i % 2048 + 1 for i in range(T)) if pre else T * (CTX % 2048 + 1)
+            att = ("flops", 2.0 * H * (kdim + vdim) * seen) if pre else ("bytes", seen * kvh * (kdim + vdim) * esz)
+            qkv = T * ((H * kdim + kvh * (kdim + vdim)) * 4 + H * kdim * esz + kvh * (kdim + vdim) * esz)
+            if key.startswith("paged_attention_selected") or key in ("paged_attention_varlen_sink", "paged_attention_decode_chunked"):
+                return att
+            return {
+                "rms_norm_ex": ("bytes", T * D * (4 + esz)), "post_norm_add_rms_norm": ("bytes", T * D * (12 + esz)), "gelu_tanh_mul": ("bytes", T * ff * (8 + esz)),
+                "glu_packed": ("bytes", T * ff * (8 + esz)), "embedding_scaled": ("bytes", T * D * (esz + 4)), "cast_rows": ("bytes", T * D * (4 + esz)),
+                "causal_conv_silu": ("bytes", T * Cd * 8), "causal_conv": ("bytes", T * Cd * 8), "token_shift_mix": ("bytes", T * D * (4 + 5 * esz)),
+                "gated_rms_norm": ("bytes", T * H * hd * (8 + esz)), "group_rms_norm_gate": ("bytes", T * D * (8 + esz)),
+                "gated_delta_rule": ("f32", 6.0 * T * H * hd * hd) if pre else ("bytes", T * (Cd + H * hd) * 4 + state(H, hd, hd)),
+                "gated_delta_rule_channel": ("f32", 6.0 * T * H * hd * hd) if pre else ("bytes", T * (Cd + 2 * H * hd) * 4 + state(H, hd, hd)),
+                "linear_attention_channel": ("f32", 4.0 * T * D * SD) if pre else ("bytes", T * 5 * D * 4 + state(SH, SD, SD)),
+                "linear_attention_channel[after the write]": ("f32", 4.0 * T * D * SD) if pre else ("bytes", T * 5 * D * 4 + state(SH, SD, SD)),
+                "qk_norm_rope_cache": ("bytes", qkv), "qk_head_norm_rope_cache": ("bytes", qkv),
+            }.get(key)
+
+        def table(side, kern, tag, T):
+            out = {}
+            for (tg, key), v in kern.items():
+                if tg != tag:
+                    continue
+                t = med(v)
+                e = {"us": round(t * 1e6, 1), "calls_per_step": len(v)}
+                w = work(side, tag, key, T)
+                if w:
+                    roof = w[1] / {"bytes": HBM, "flops": TC, "f32": F32}[w[0]]
+                    e.update(bound=w[0], roofline_us=round(roof * 1e6, 2), frac_of_roofline=round(roof / t, 3))
+                out[key] = e
+            return out
+        side = lambda nm, pre, dec, dec_dev, kern: {
+            "prefill_tokens_per_s": round(P / pre), "prefill_ms": round(pre * 1e3, 2), "decode_tokens_per_s": round(B / dec), "decode_ms_per_step": round(dec * 1e3, 3),
+            "decode": "CUDA-graph replay incl. host metadata and H2D", "decode_ms_per_step_device": round(dec_dev * 1e3, 3),
+            "decode_tokens_per_s_device": round(B / dec_dev), "kernels_prefill": table(nm, kern, "prefill", P), "kernels_decode": table(nm, kern, "decode", B)}
+        results[name] = {"tavevik": side("tavevik", t_pre, t_dec, t_dec_dev, t_kern), "gobesun": side("gobesun", g_pre, g_dec, g_dec_dev, g_kern),
+                         "like_kernels": {"prefill": table("like", like, "prefill", P), "decode": table("like", like, "decode", B)},
+                         "shape": dict(z, prompt=P, decode_batch=B, decode_ctx=CTX, shift_heads=SH, shift_dim=SD, delta_heads=H, delta_dim=hd)}
+    clocks = sampler.stop()
+    first = results[next(iter(results))]
+    print(json.dumps({"metric": "Tavevik prefill / decode tokens/s beside a Gobesun of equal size", "value": first["tavevik"]["decode_tokens_per_s"],
+                      "unit": UNIT, "n_gpus": 1, "steps": K, "warmup": W, "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "arch": "tavevik",
+                      "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "f32_fma_tflops_nominal": round(F32 / 1e12, 1),
+                                "source": "fallback" if peaks.get("fallback") else "MEASURED_PEAKS.json"},
+                      "l2": "weights and activations of a step exceed L2 (126 MB)", "clocks": clocks,
+                      "gpu_launches": int(pkg.lib().b200_total_kernel_launches() - l0), "sizes": results}))
+
+
 def main():
     args = parse()
     if args.arch == "gobesun":
@@ -1702,6 +1924,9 @@ def main():
         return
     if args.arch == "sigalorn":
         run_sigalorn(args)
+        return
+    if args.arch == "tavevik":
+        run_tavevik(args)
         return
     if args.arch == "dofevik":
         run_dofevik(args)

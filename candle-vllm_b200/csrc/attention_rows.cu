@@ -3,19 +3,22 @@
 //
 // A row at position i sees the keys j <= i with i - j < window (window 0 = all) or j < keep_first; its visible positions are numbered 0 .. n - 1 (the kept ones
 // that lie before the window, then the window), so the window's start costs nothing and no key outside is read.  A block owns one row, one key / value head with
-// up to 16 of the query heads that share it (the 16 rows of the MMA tile) and one of `splits` runs of the visible keys; its four warps take 16 keys at a time in
+// up to 16 of the query heads that share it (the 16 rows of the MMA tile) and one of `splits` runs of the visible keys; its eight warps take 16 keys at a time in
 // turn, each with its own online softmax, and join at the end through shared memory.
 //
-// Nothing is staged: keys and values are read from global memory straight into the operand layout of mma.m16n8k16, 16 bytes per lane.  The contraction over the
-// head does not care about the order of its terms, so the four lanes of a key row read 16 neighbouring bytes each (entries 32 c + 8 t ..) and the query fragments
-// are put together in the same order.  A value fragment pairs two keys per register: a lane reads 16 bytes (columns 64 c + 8 g ..) of its four key rows and
-// pairs them by byte permutes; the columns come out permuted, which the store undoes.
+// Keys and values are fetched in the operand layout of mma.m16n8k16, 16 bytes per lane and copy.  The contraction over the head does not care about the order of
+// its terms, so the four lanes of a key row take 16 neighbouring bytes each (entries 32 c + 8 t ..) and the query fragments are put together in the same order.  A
+// value fragment pairs two keys per register: a lane takes 16 bytes (columns 64 c + 8 g ..) of its four key rows and pairs them by byte permutes; the columns come out
+// permuted, which the store undoes.  The copies are cp.async into a ring of three tiles whose places belong to one lane each: a lane reads back only what it
+// asked for itself, so the ring needs no barrier and two tiles are always on their way.
+#include <algorithm>
+
 #include "common.cuh"
 
 namespace b200 {
 namespace {
 
-constexpr int kRowWarps = 4, kRowThreads = kRowWarps * 32;
+constexpr int kRowWarps = 8, kRowThreads = kRowWarps * 32;
 constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
@@ -24,6 +27,11 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) { __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi); return *reinterpret_cast<uint32_t*>(&v); }
+
+constexpr int kRing = 3;
+__device__ __forceinline__ void copy16(uint4* dst, const void* src, bool ok) {        // zeros where the source does not exist
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
 
 struct RowsArgs {
     void* out; int64_t ldo;
@@ -50,7 +58,8 @@ attention_rows_kernel(const RowsArgs A) {
     pdl_wait();
     pdl_trigger();
     constexpr int kKC = kDK / 32, kVC = kDV / 64;       // 16-byte loads per key row and lane; per value row and lane
-    extern __shared__ float sm[];                       // [warps][16][kDV] sums, [warps][16] maxima, [warps][16] weight sums
+    constexpr int kPieces = 2 * kKC + 4 * kVC;          // copies of a lane per tile
+    extern __shared__ __align__(16) float sm[];         // the ring [warps][kRing][kPieces][32] of 16 bytes; then [warps][16][kDV] sums, maxima, weight sums
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
     const int rep = A.H / A.G, head_groups = (rep + 15) / 16;
     const int t = blockIdx.x, kvh = blockIdx.y / head_groups, hg = blockIdx.y % head_groups, split = blockIdx.z;
@@ -88,51 +97,52 @@ attention_rows_kernel(const RowsArgs A) {
         const int j = n < kept ? n : lo + n - kept;
         return table[j / A.block_size] * A.block_size + j % A.block_size;
     };
-    uint4 kb[2][kKC], vb[4][kVC];
-    auto load_keys = [&](int slot) {
+    uint4* ring = reinterpret_cast<uint4*>(sm) + (int64_t)warp * kRing * kPieces * 32 + lane;
+    auto fetch = [&](int tile, int stage) {
+        if (tile < tile1) {
+            const int slot = locate(tile);
+            uint4* dst = ring + stage * kPieces * 32;
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-            const int64_t s = __shfl_sync(0xffffffffu, slot, half * 8 + g);
-            const __nv_bfloat16* kr = A.kc + (s * A.G + kvh) * A.dk;
+            for (int half = 0; half < 2; ++half) {
+                const int64_t s = __shfl_sync(0xffffffffu, slot, half * 8 + g);
+                const __nv_bfloat16* kr = A.kc + (s * A.G + kvh) * A.dk;
 #pragma unroll
-            for (int c = 0; c < kKC; ++c) {
-                const int d = 32 * c + 8 * t4;
-                kb[half][c] = d < A.dk ? __ldg(reinterpret_cast<const uint4*>(kr + d)) : make_uint4(0, 0, 0, 0);
+                for (int c = 0; c < kKC; ++c) {
+                    const int d = 32 * c + 8 * t4;
+                    copy16(dst + (half * kKC + c) * 32, kr + (d < A.dk ? d : 0), d < A.dk);
+                }
+            }
+#pragma unroll
+            for (int r = 0; r < 4; ++r) {               // key rows 2 t4, 2 t4 + 1, 2 t4 + 8, 2 t4 + 9
+                const int64_t s = __shfl_sync(0xffffffffu, slot, 2 * t4 + (r & 1) + (r >> 1) * 8);
+                const __nv_bfloat16* vr = A.vc + (s * A.G + kvh) * A.dv;
+#pragma unroll
+                for (int c = 0; c < kVC; ++c) {
+                    const int d = 64 * c + 8 * g;
+                    copy16(dst + (2 * kKC + r * kVC + c) * 32, vr + (d < A.dv ? d : 0), d < A.dv);
+                }
             }
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");           // an empty group past the last tile: the count of groups stays that of the tiles
     };
-    auto load_values = [&](int slot) {
+    int stage = 0;
 #pragma unroll
-        for (int r = 0; r < 4; ++r) {                   // key rows 2 t4, 2 t4 + 1, 2 t4 + 8, 2 t4 + 9
-            const int64_t s = __shfl_sync(0xffffffffu, slot, 2 * t4 + (r & 1) + (r >> 1) * 8);
-            const __nv_bfloat16* vr = A.vc + (s * A.G + kvh) * A.dv;
-#pragma unroll
-            for (int c = 0; c < kVC; ++c) {
-                const int d = 64 * c + 8 * g;
-                vb[r][c] = d < A.dv ? __ldg(reinterpret_cast<const uint4*>(vr + d)) : make_uint4(0, 0, 0, 0);
-            }
-        }
-    };
-    int slot = 0;
-    if (tile0 + warp < tile1) {
-        slot = locate(tile0 + warp);
-        load_keys(slot);
-    }
+    for (int i = 0; i < kRing - 1; ++i) fetch(tile0 + warp + i * kRowWarps, i);
     for (int tile = tile0 + warp; tile < tile1; tile += kRowWarps) {
-        load_values(slot);                              // in flight under the scores
+        fetch(tile + (kRing - 1) * kRowWarps, stage == 0 ? kRing - 1 : stage - 1);         // the place read in the previous turn
+        asm volatile("cp.async.wait_group %0;" ::"n"(kRing - 1) : "memory");
+        const uint4* src = ring + stage * kPieces * 32;
+        stage = stage == kRing - 1 ? 0 : stage + 1;
         float s[2][4];
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             s[half][0] = s[half][1] = s[half][2] = s[half][3] = 0.f;
 #pragma unroll
             for (int c = 0; c < kKC; ++c) {
-                mma_bf16(s[half], qa[2 * c], kb[half][c].x, kb[half][c].y);
-                mma_bf16(s[half], qa[2 * c + 1], kb[half][c].z, kb[half][c].w);
+                const uint4 kb = src[(half * kKC + c) * 32];
+                mma_bf16(s[half], qa[2 * c], kb.x, kb.y);
+                mma_bf16(s[half], qa[2 * c + 1], kb.z, kb.w);
             }
-        }
-        if (tile + kRowWarps < tile1) {                 // the next tile's keys travel under the softmax and the value product
-            slot = locate(tile + kRowWarps);
-            load_keys(slot);
         }
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
@@ -165,8 +175,8 @@ attention_rows_kernel(const RowsArgs A) {
         for (int i = 0; i < kDV / 8; ++i) { o[i][0] *= c_lo; o[i][1] *= c_lo; o[i][2] *= c_hi; o[i][3] *= c_hi; }
 #pragma unroll
         for (int c = 0; c < kVC; ++c) {
-            const uint32_t r0[4] = {vb[0][c].x, vb[0][c].y, vb[0][c].z, vb[0][c].w}, r1[4] = {vb[1][c].x, vb[1][c].y, vb[1][c].z, vb[1][c].w};
-            const uint32_t r2[4] = {vb[2][c].x, vb[2][c].y, vb[2][c].z, vb[2][c].w}, r3[4] = {vb[3][c].x, vb[3][c].y, vb[3][c].z, vb[3][c].w};
+            const uint4 v0 = src[(2 * kKC + c) * 32], v1 = src[(2 * kKC + kVC + c) * 32], v2 = src[(2 * kKC + 2 * kVC + c) * 32], v3 = src[(2 * kKC + 3 * kVC + c) * 32];
+            const uint32_t r0[4] = {v0.x, v0.y, v0.z, v0.w}, r1[4] = {v1.x, v1.y, v1.z, v1.w}, r2[4] = {v2.x, v2.y, v2.z, v2.w}, r3[4] = {v3.x, v3.y, v3.z, v3.w};
 #pragma unroll
             for (int w = 0; w < 4; ++w) {               // columns 64 c + 8 g + 2 w and + 1
                 mma_bf16(o[8 * c + 2 * w], pa, __byte_perm(r0[w], r1[w], 0x5410), __byte_perm(r2[w], r3[w], 0x5410));
@@ -177,7 +187,8 @@ attention_rows_kernel(const RowsArgs A) {
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1); l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
 
-    // join the warps: accumulator i = 8 c + e, columns 2 t4 and 2 t4 + 1 of the fragment are entries 64 c + 16 t4 + e and 64 c + 16 t4 + 8 + e of the head
+    // join the warps, over the ring once every warp is done with its tiles: accumulator i = 8 c + e, columns 2 t4 and 2 t4 + 1 of the fragment are entries 64 c + 16 t4 + e and 64 c + 16 t4 + 8 + e of the head
+    __syncthreads();
     float* sums = sm;
     float* ms = sm + kRowWarps * 16 * kDV;
     float* ls = ms + kRowWarps * 16;
@@ -265,7 +276,7 @@ void paged_attention_rows(void* out, int64_t ld_out, const void* q, const void* 
     cudaStream_t st = as_stream(stream);
     const dim3 grid(num_tokens, num_kv_heads * ((num_heads / num_kv_heads + 15) / 16), splits);
 #define PAR(DK, DV) do { \
-        const int smem = kRowWarps * 16 * (DV + 2) * (int)sizeof(float); \
+        const int smem = std::max(kRowWarps * 16 * (DV + 2) * (int)sizeof(float), kRowWarps * kRing * (DK / 16 + DV / 16) * 512); \
         ensure_dynamic_smem(reinterpret_cast<const void*>(attention_rows_kernel<DK, DV>), smem); \
         launch_pdl(attention_rows_kernel<DK, DV>, grid, dim3(kRowThreads), (size_t)smem, st, A); } while (0)
     if (dk <= 64) { if (dv <= 64) PAR(64, 64); else PAR(64, 128); }

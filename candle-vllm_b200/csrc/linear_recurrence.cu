@@ -96,6 +96,80 @@ causal_conv_roll_kernel(const float* __restrict__ x, int64_t ldx, const float* _
     }
 }
 
+// Steps of many rows: a thread walks 16 rows of kV channels with the taps and the inputs of the last kK - 1 rows in registers, so that every input is read once.
+// kK is the number of taps rounded up; the taps that do not exist are zero and oldest, so the sum is the one above term by term.
+constexpr int kConvRows = 16;
+template <typename TOut, int kK, int kV>
+__global__ void __launch_bounds__(128)
+causal_conv_walk_kernel(const float* __restrict__ x, int64_t ldx, const float* __restrict__ in_bias, const float* __restrict__ taps,
+                        const float* __restrict__ out_bias, const float* __restrict__ conv_state, TOut* __restrict__ y, int64_t ldy,
+                        const int32_t* __restrict__ token_seq, const int32_t* __restrict__ cu_seqlens, const int32_t* __restrict__ seq_slots,
+                        const int32_t* __restrict__ seq_start, int T, int C, int K, int act, int add_input) {
+    pdl_wait();
+    pdl_trigger();
+    const int c = (blockIdx.x * 128 + threadIdx.x) * kV;
+    const int t_begin = blockIdx.y * kConvRows, t_end = min(T, t_begin + kConvRows);
+    if (c >= C) return;
+    auto load = [&](const float* p, float (&v)[kV]) {
+        if constexpr (kV == 4) { const float4 f = *reinterpret_cast<const float4*>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+        else v[0] = *p;
+    };
+    float w[kK][kV], h[kK][kV], ib[kV], ob[kV];      // taps and inputs, oldest first; h[kK - 1] is the current row
+#pragma unroll
+    for (int j = 0; j < kV; ++j) {
+        ib[j] = in_bias ? in_bias[c + j] : 0.f;
+        ob[j] = out_bias ? out_bias[c + j] : 0.f;
+#pragma unroll
+        for (int k = 0; k < kK; ++k) { const int d = kK - 1 - k; w[k][j] = d < K ? taps[(int64_t)(c + j) * K + (K - 1 - d)] : 0.f; h[k][j] = 0.f; }
+    }
+    int entry = -1;
+    for (int t = t_begin; t < t_end; ++t) {
+        const int b = token_seq[t];
+        if (b != entry) {                            // the rows before this one: earlier rows of the entry, the state, or nothing
+            entry = b;
+            const int i = t - cu_seqlens[b];
+            const bool fresh = seq_start[b] == 0;
+            const float* st = conv_state + (int64_t)seq_slots[b] * (K > 1 ? K - 1 : 1) * C + c;
+#pragma unroll
+            for (int k = 1; k < kK; ++k) {           // shifted down by one below: h[k] is the row kK - k rows back
+                const int src = i - (kK - k);
+                if (kK - k >= K || (src < 0 && fresh)) {
+#pragma unroll
+                    for (int j = 0; j < kV; ++j) h[k][j] = 0.f;
+                } else if (src >= 0) {
+                    load(x + (int64_t)(t - (kK - k)) * ldx + c, h[k]);
+#pragma unroll
+                    for (int j = 0; j < kV; ++j) h[k][j] += ib[j];
+                } else {
+                    load(st + (int64_t)(K - 1 + src) * C, h[k]);
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k + 1 < kK; ++k)
+#pragma unroll
+            for (int j = 0; j < kV; ++j) h[k][j] = h[k + 1][j];
+        load(x + (int64_t)t * ldx + c, h[kK - 1]);
+        float o[kV];
+        TOut q[kV];
+#pragma unroll
+        for (int j = 0; j < kV; ++j) {
+            h[kK - 1][j] += ib[j];
+            o[j] = 0.f;
+#pragma unroll
+            for (int k = 0; k < kK; ++k) o[j] = fmaf(w[k][j], h[k][j], o[j]);
+            o[j] += ob[j];
+            if (act == 1) o[j] = silu_f(o[j]);
+            if (add_input) o[j] += h[kK - 1][j];
+            q[j] = from_f32<TOut>(o[j]);
+        }
+        TOut* dst = y + (int64_t)t * ldy + c;
+        if constexpr (kV == 1) *dst = q[0];
+        else if constexpr (sizeof(TOut) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(q);
+        else *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(q);
+    }
+}
+
 // Steps in which every entry brings one row: the convolution and the roll of the state in one kernel (a thread owns its channel's state column)
 template <typename TOut>
 __global__ void __launch_bounds__(128)
@@ -1131,13 +1205,13 @@ __device__ __forceinline__ float low_rank_value(float z, int form, float inv_tau
     return z;
 }
 
+// few rows: 256 channels x kTok tokens per block, a thread keeps 16 weights of its channel at a time and meets the tokens' inner values with them
 template <int kTok>
 __global__ void __launch_bounds__(256)
-low_rank_decay_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ alpha, int T, int N,
-                      int R, float inv_tau, int in_tanh, int form, const float* __restrict__ log_rate, int channels_per_rate) {
+low_rank_rows_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ out, int T, int N,
+                     int R, float inv_tau, int in_tanh, int form, const float* __restrict__ log_rate, int channels_per_rate) {
     pdl_wait();
     pdl_trigger();
-    // 256 channels x kTok tokens per block: a thread keeps 16 weights of its channel at a time and meets the tokens' inner values with them
     __shared__ __align__(16) float ys[kTok][16];
     const int n = blockIdx.x * 256 + threadIdx.x, t0 = blockIdx.y * kTok;
     float z[kTok];
@@ -1177,7 +1251,75 @@ low_rank_decay_kernel(const float* __restrict__ y, int64_t ldy, const float* __r
     const float lr = form == 2 ? log_rate[n / channels_per_rate] : 0.f;
 #pragma unroll
     for (int i = 0; i < kTok; ++i)
-        if (t0 + i < T) alpha[(int64_t)(t0 + i) * N + n] = low_rank_value(z[i], form, inv_tau, lr);
+        if (t0 + i < T) out[(int64_t)(t0 + i) * N + n] = low_rank_value(z[i], form, inv_tau, lr);
+}
+
+// many rows: tiles of 64 tokens x 128 channels, 16 inner values at a time through shared memory (both operands stored inner value first), a thread makes 8 tokens x 4
+// neighbouring channels
+__global__ void __launch_bounds__(256)
+low_rank_tile_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ out, int T, int N,
+                     int R, float inv_tau, int in_tanh, int form, const float* __restrict__ log_rate, int channels_per_rate) {
+    pdl_wait();
+    pdl_trigger();
+    __shared__ __align__(16) float ys[16][64 + 4], ws[16][128 + 4];
+    const int n0 = blockIdx.x * 128, t0 = blockIdx.y * 64;
+    const int tx = threadIdx.x & 31, ty = threadIdx.x >> 5;
+    float acc[8][4], ry[4], rw[8];
+#pragma unroll
+    for (int l = 0; l < 4; ++l) {
+        const int n = n0 + tx * 4 + l;
+        const float b = (n < N && bias) ? bias[n] : 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) acc[i][l] = b;
+    }
+    auto fetch = [&](int r0) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int e = threadIdx.x + 256 * i, t = e >> 4, r = e & 15;
+            ry[i] = (t0 + t < T && r0 + r < R) ? y[(int64_t)(t0 + t) * ldy + r0 + r] : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int e = threadIdx.x + 256 * i, n = e >> 4, r = e & 15;
+            rw[i] = (n0 + n < N && r0 + r < R) ? w[(int64_t)(n0 + n) * R + r0 + r] : 0.f;
+        }
+    };
+    fetch(0);
+    for (int r0 = 0; r0 < R; r0 += 16) {
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { const int e = threadIdx.x + 256 * i; ys[e & 15][e >> 4] = in_tanh ? tanhf(ry[i]) : ry[i]; }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) { const int e = threadIdx.x + 256 * i; ws[e & 15][e >> 4] = rw[i]; }
+        __syncthreads();
+        if (r0 + 16 < R) fetch(r0 + 16);
+#pragma unroll
+        for (int r = 0; r < 16; ++r) {
+            const float4 a = *reinterpret_cast<const float4*>(&ys[r][ty * 8]), b = *reinterpret_cast<const float4*>(&ys[r][ty * 8 + 4]),
+                         v = *reinterpret_cast<const float4*>(&ws[r][tx * 4]);
+            const float yv[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w}, wv[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+#pragma unroll
+                for (int l = 0; l < 4; ++l) acc[i][l] = fmaf(wv[l], yv[i], acc[i][l]);
+        }
+    }
+    float lr[4];
+#pragma unroll
+    for (int l = 0; l < 4; ++l) lr[l] = form == 2 && n0 + tx * 4 + l < N ? log_rate[(n0 + tx * 4 + l) / channels_per_rate] : 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int t = t0 + ty * 8 + i, n = n0 + tx * 4;
+        if (t >= T || n >= N) continue;
+        float o[4];
+#pragma unroll
+        for (int l = 0; l < 4; ++l) o[l] = low_rank_value(acc[i][l], form, inv_tau, lr[l]);
+        float* dst = out + (int64_t)t * N + n;
+        if (N % 4 == 0) { *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]); continue; }
+#pragma unroll
+        for (int l = 0; l < 4; ++l)
+            if (n + l < N) dst[l] = o[l];
+    }
 }
 
 __global__ void __launch_bounds__(256)
@@ -1529,13 +1671,23 @@ void causal_conv_ex(const float* x, int64_t ldx, const float* in_bias, const flo
         check_launch("causal_conv_ex");
         return;
     }
-    if (out_dtype == B200_F32)
+    B200_REQUIRE(out_dtype == B200_F32 || out_dtype == B200_BF16, kErrUnsupported, "causal_conv_ex: out dtype %d (f32 / bf16)", out_dtype);
+    if (num_tokens > 256 && num_taps <= 8) {
+        const bool vec = channels % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && (((uintptr_t)x | (uintptr_t)conv_state | (uintptr_t)y) & 15) == 0;
+        const dim3 walk(ceil_div(channels, vec ? 512 : 128), ceil_div(num_tokens, kConvRows));
+#define CCW(TO, KK, V) launch_pdl(causal_conv_walk_kernel<TO, KK, V>, walk, dim3(128), 0, st, x, ldx, in_bias, taps, out_bias, (const float*)conv_state, (TO*)y, ldy, token_seq, \
+                                  cu_seqlens, seq_slots, seq_start, (int)num_tokens, channels, num_taps, act, add_input)
+#define CCW_V(TO, KK) do { if (vec) CCW(TO, KK, 4); else CCW(TO, KK, 1); } while (0)
+        if (out_dtype == B200_F32) { if (num_taps <= 4) CCW_V(float, 4); else CCW_V(float, 8); }
+        else { if (num_taps <= 4) CCW_V(__nv_bfloat16, 4); else CCW_V(__nv_bfloat16, 8); }
+#undef CCW_V
+#undef CCW
+    } else if (out_dtype == B200_F32)
         launch_pdl(causal_conv_ex_kernel<float>, grid, dim3(128), 0, st, x, ldx, in_bias, taps, out_bias, (const float*)conv_state, (float*)y, ldy, token_seq,
                    cu_seqlens, seq_slots, seq_start, channels, num_taps, act, add_input);
-    else if (out_dtype == B200_BF16)
+    else
         launch_pdl(causal_conv_ex_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, x, ldx, in_bias, taps, out_bias, (const float*)conv_state, (__nv_bfloat16*)y, ldy,
                    token_seq, cu_seqlens, seq_slots, seq_start, channels, num_taps, act, add_input);
-    else { set_error(kErrUnsupported, "causal_conv_ex: out dtype %d (f32 / bf16)", out_dtype); return; }
     count_launch();
     if (num_taps > 1) {
         launch_pdl(causal_conv_roll_kernel, dim3(ceil_div(channels, 128), num_seqs), dim3(128), 0, st, x, ldx, in_bias, conv_state, cu_seqlens, seq_slots, seq_start,
@@ -1690,15 +1842,12 @@ void low_rank_map(const float* y, int64_t ldy, const float* weight, const float*
                  (form != 2 || (log_rate && channels_per_rate > 0 && channels % channels_per_rate == 0)), kErrBadArg, "low_rank_map: bad arguments");
     cudaStream_t st = as_stream(stream);
     const float inv_tau = form == 0 ? 1.0f / tau : 0.f;
-    // few rows: short blocks, many of them
-    const int tok = num_tokens <= 256 ? 2 : 32;
-    const dim3 grid(ceil_div(channels, 256), ceil_div(num_tokens, tok));
-    if (tok == 2)
-        launch_pdl(low_rank_decay_kernel<2>, grid, dim3(256), 0, st, y, ldy, weight, bias, out, (int)num_tokens, (int)channels, (int)rank, inv_tau, (int)in_tanh, (int)form,
-                   log_rate, (int)channels_per_rate);
+    if (num_tokens <= 256)
+        launch_pdl(low_rank_rows_kernel<2>, dim3(ceil_div(channels, 256), ceil_div(num_tokens, 2)), dim3(256), 0, st, y, ldy, weight, bias, out, (int)num_tokens, (int)channels,
+                   (int)rank, inv_tau, (int)in_tanh, (int)form, log_rate, (int)channels_per_rate);
     else
-        launch_pdl(low_rank_decay_kernel<32>, grid, dim3(256), 0, st, y, ldy, weight, bias, out, (int)num_tokens, (int)channels, (int)rank, inv_tau, (int)in_tanh, (int)form,
-                   log_rate, (int)channels_per_rate);
+        launch_pdl(low_rank_tile_kernel, dim3(ceil_div(channels, 128), ceil_div(num_tokens, 64)), dim3(256), 0, st, y, ldy, weight, bias, out, (int)num_tokens, (int)channels,
+                   (int)rank, inv_tau, (int)in_tanh, (int)form, log_rate, (int)channels_per_rate);
     count_launch();
     check_launch("low_rank_map");
 }

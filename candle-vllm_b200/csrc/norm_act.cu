@@ -407,6 +407,23 @@ add_rms_norm_kernel(float* __restrict__ x, const float* __restrict__ y1, int64_t
 }
 
 
+// the gated forms of glu_packed without a row factor, rows of whole aligned groups of four
+template <typename TOut>
+__global__ void __launch_bounds__(256)
+glu_rows_kernel(const float* __restrict__ gu, TOut* __restrict__ out, int ff, int64_t ld, int act, float limit) {
+    pdl_wait();
+    pdl_trigger();
+    const int64_t r = blockIdx.x;
+    const int c = (blockIdx.y * 256 + threadIdx.x) * 4;
+    if (c >= ff) return;
+    const float4 g = *reinterpret_cast<const float4*>(gu + r * ld + c), u = *reinterpret_cast<const float4*>(gu + r * ld + ff + c);
+    alignas(16) const TOut o[4] = {from_f32<TOut>(glu_value(g.x, u.x, act, limit)), from_f32<TOut>(glu_value(g.y, u.y, act, limit)), from_f32<TOut>(glu_value(g.z, u.z, act, limit)),
+                       from_f32<TOut>(glu_value(g.w, u.w, act, limit))};
+    TOut* dst = out + r * ff + c;
+    if (sizeof(TOut) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(o);
+    else *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(o);
+}
+
 // act 3 of glu_packed without a row factor: out = relu(x)^2 over rows of ff entries (pitch ld), four entries per thread when rows allow 16-byte loads
 template <typename TOut>
 __global__ void __launch_bounds__(256)
@@ -690,6 +707,15 @@ void glu_packed(const float* gate_up, void* out, int64_t rows, int32_t ff, int64
         const dim3 g2((unsigned)rows, (unsigned)((ff + 1023) / 1024));
         if (out_dtype == B200_F32) launch_pdl(relu2_rows_kernel<float>, g2, dim3(256), 0, st, gate_up, (float*)out, ff, ld, vec);
         else launch_pdl(relu2_rows_kernel<__nv_bfloat16>, g2, dim3(256), 0, st, gate_up, (__nv_bfloat16*)out, ff, ld, vec);
+        count_launch();
+        check_launch("glu_packed");
+        return;
+    }
+    if (act != 3 && !row_scale && rows <= 0x7fffffff && ff % 4 == 0 && ld % 4 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 15) == 0 &&
+        (out_dtype == B200_F32 || out_dtype == B200_BF16)) {
+        const dim3 g2((unsigned)rows, (unsigned)((ff + 1023) / 1024));
+        if (out_dtype == B200_F32) launch_pdl(glu_rows_kernel<float>, g2, dim3(256), 0, st, gate_up, (float*)out, ff, ld, act, limit);
+        else launch_pdl(glu_rows_kernel<__nv_bfloat16>, g2, dim3(256), 0, st, gate_up, (__nv_bfloat16*)out, ff, ld, act, limit);
         count_launch();
         check_launch("glu_packed");
         return;

@@ -845,8 +845,12 @@ class ParallelSumMixer:
     """Two mixers on the same input, left_scale * left + right_scale * right.  ``left`` (PagedAttentionMixer) keeps a paged cache, ``right`` a state; projections that read
     the input itself are one product, and so are the two output projections: both sides write their rows into one buffer that meets [W_o left | W_o right].  The
     scales touch no 16-bit weight: the right one enters through the right side's norm weight (``right`` is built with ``norm_scale`` = ``right_factor(...)``), and
-    ``forward`` returns y with the sum = out_scale * y + out_bias, which the closing norm's kernel forms in f32."""
+    ``forward`` returns y with the sum = out_scale * y + out_bias, which the closing norm's kernel forms in f32.
+
+    The two sides share nothing between the projection of the input and the output projection: the right one runs on a stream of its own beside the left one (a
+    branch of its own in a captured step)."""
     kind = "both"
+    _side_streams: Dict[torch.device, "torch.cuda.Stream"] = {}
 
     @staticmethod
     def right_factor(left_scale: float, right_scale: float) -> float:
@@ -875,11 +879,22 @@ class ParallelSumMixer:
 
     def forward(self, x: torch.Tensor, h: torch.Tensor, batch: StepBatch, kv, state) -> torch.Tensor:
         """x: the input rows in f32, h: the same in the compute dtype"""
-        proj = ops.linear(h, self.w_in)
         z = torch.empty((h.shape[0], self.KL + self.KR), dtype=self.dtype, device=h.device)
+        main = torch.cuda.current_stream(h.device)
+        if h.device not in self._side_streams:
+            self._side_streams[h.device] = torch.cuda.Stream(device=h.device)
+        side = self._side_streams[h.device]
+        shared = self.w_in.shape[0] > self.split            # the right side's first product is part of the left side's
+        proj = ops.linear(h, self.w_in) if shared else None
+        # what this method hands to the side stream lives until the streams have met again; what the side stream allocates stays its own
+        side.wait_stream(main)
+        with torch.cuda.stream(side):
+            if shared:
+                self.right.attend(h, batch, state, proj=proj[:, self.split:], out=z[:, self.KL:])
+            else:
+                self.right.attend(x, batch, state, out=z[:, self.KL:])
+        if proj is None:
+            proj = ops.linear(h, self.w_in)
         self.left.attend(h, batch, kv, proj=proj[:, :self.split], out=z[:, :self.KL])
-        if self.w_in.shape[0] > self.split:
-            self.right.attend(h, batch, state, proj=proj[:, self.split:], out=z[:, self.KL:])
-        else:
-            self.right.attend(x, batch, state, out=z[:, self.KL:])
+        main.wait_stream(side)
         return ops.linear(z, self.w_o)

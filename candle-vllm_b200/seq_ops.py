@@ -976,7 +976,7 @@ def cast_rows(x: torch.Tensor) -> torch.Tensor:
 
 
 SELECTED_PREFILL_MIN_ROWS = 8     # steps in which some entry brings at least this many rows take the tile kernel (bf16); shorter portions go row by row
-SELECTED_ROW_BLOCKS = 592         # four blocks of four warps per SM: steps with fewer rows cut the visible keys of every row into runs
+SELECTED_ROW_BLOCKS = 148         # one block of eight warps per SM: steps with fewer rows cut the visible keys of every row into runs
 
 
 def selected_tensor_cores(heads: int, kv_heads: int, dk: int, dv: int, block_size: int, dtype: torch.dtype) -> bool:
@@ -1001,7 +1001,7 @@ def paged_attention_selected(q: torch.Tensor, k_cache: torch.Tensor, v_cache: to
     if q.dtype == torch.bfloat16 and chunk == 0 and (splits is not None or batch.max_rows < SELECTED_PREFILL_MIN_ROWS):
         if splits is None:
             longest = W * bs if window <= 0 else min(window + keep_first, W * bs)
-            splits = max(1, min(SELECTED_ROW_BLOCKS // (T * G * -(-heads // G // 16)), longest // 128, 64))
+            splits = max(1, min(SELECTED_ROW_BLOCKS // (T * G * -(-heads // G // 16)), longest // 256, 64))
         part = torch.empty((T * heads * splits * (dv + 2),), dtype=torch.float32, device=q.device) if splits > 1 else None
         lib().paged_attention_rows(_ptr(out), C.c_int64(pitch(out)), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), C.c_int32(W), _ptr(batch.token_seq),
                                    _ptr(batch.positions), C.c_int32(T), C.c_int32(heads), C.c_int32(G), C.c_int32(dk), C.c_int32(dv), C.c_int32(bs), C.c_float(scale),

@@ -143,6 +143,30 @@ def test_token_shift_in_unequal_batches(D, dtype):
         assert torch.equal(state[slots[i]].cpu(), xs[i][-1])
 
 
+@pytest.mark.parametrize("C,K", [(8, 1), (36, 2), (33, 3), (512, 4), (20, 6), (7, 8), (12, 11)])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_convolution_over_steps_of_many_rows(C, K, dtype):
+    g = torch.Generator().manual_seed(C)
+    lens, plans = [700, 3, 41, 290, 1], [[300, 1, 399], [2, 1], [5, 36], [1, 289], [1]]
+    xs, taps = [torch.randn(n, C, generator=g) for n in lens], torch.randn(C, K, generator=g)
+    want = [O.silu(O.short_conv(x.to(F64), taps.to(F64))) for x in xs]
+    ib, ob = torch.randn(C, generator=g), torch.randn(C, generator=g)
+    want2 = [O.short_conv(x.to(F64) + ib.to(F64), taps.to(F64)) + ob.to(F64) + x.to(F64) + ib.to(F64) for x in xs]
+    for plain in (True, False):
+        state, fed, pi, got = torch.full((6, max(K - 1, 1), C), 1e9, device=DEV), [0] * 5, [0] * 5, [[] for _ in lens]
+        while any(f < n for f, n in zip(fed, lens)):
+            live = [i for i in range(5) if fed[i] < lens[i]]
+            take = [min(plans[i][pi[i]], lens[i] - fed[i]) for i in live]
+            b = batch_of([dict(tokens=[0] * n, start=fed[i], block_table=list(range(11)), state_slot=5 - i, want=[]) for i, n in zip(live, take)])
+            x = dev(torch.cat([torch.cat([xs[i][fed[i]:fed[i] + n]] * 2, 1) for i, n in zip(live, take)]))[:, :C]
+            y = ops.causal_conv(x, dev(taps), state, b, out_dtype=dtype, act="silu") if plain else ops.causal_conv(x, dev(taps), state, b, dtype, dev(ib), dev(ob), add_input=True)
+            at = 0
+            for i, n in zip(live, take):
+                got[i].append(y[at:at + n]); at += n; fed[i] += n; pi[i] += 1
+        for i in range(5):
+            close(torch.cat(got[i]), (want if plain else want2)[i], 2e-6 if dtype == torch.float32 else 5e-3, f"sequence {i}")
+
+
 # ----------------------------------------------------------------------------------------------------------------------
 # the two recurrences
 # ----------------------------------------------------------------------------------------------------------------------
@@ -279,7 +303,7 @@ def test_a_memory_written_far_back(kernel):
             bb[1500] = -60.0                     # sigmoid -> 0: nothing is written
         want = O.delta_recurrence(O.unit(q.to(F64)) * dk ** -0.5, O.unit(k.to(F64)), v.to(F64), torch.sigmoid(bb.to(F64)), wd.to(F64))
         got = ops.gated_delta_rule_channel(p_cat(q, k, v), dev(bb), 0, dev(wd.view(T, -1)), torch.zeros(1, H, dv, dk, device=DEV), b, H, 1, dk, dv, kernel=kernel).cpu()
-        close(got.view(T, H, dv)[-1], want[-1], 2e-5, f"rewritten {rewrite}")
+        close(got.view(T, H, dv)[-1], want[-1], 6e-5, f"rewritten {rewrite}")
         assert float((want[-1] / want[-1].mean()).std()) < 0.2 if rewrite else float((want[-1] / want[-1].mean()).std()) > 0.2
 
 
