@@ -75,6 +75,15 @@ template <> __device__ __forceinline__ uint32_t pack2<__half>(float lo, float hi
 __device__ __forceinline__ float fast_rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 __device__ __forceinline__ float fast_exp2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
+// tanh(x) on [-1, 1] as x times a polynomial in x^2 (interpolation of tanh(x) / x at the Chebyshev points of [0, 1] in x^2): within 1.2e-7 in f32
+__device__ __forceinline__ float tanh_small(float x) {
+    const float t = x * x;
+    float r = 0.0010380251f;
+    r = fmaf(r, t, -0.0061943247f); r = fmaf(r, t, 0.020279707f); r = fmaf(r, t, -0.053451646f);
+    r = fmaf(r, t, 0.13325076f); r = fmaf(r, t, -0.33332828f); r = fmaf(r, t, 0.99999994f);
+    return x * r;
+}
+
 struct PrefillParams {
     const void* q; void* out;
     const uint32_t* block_tables; const uint32_t* cu_q; const uint32_t* cu_k;
@@ -87,7 +96,7 @@ struct PrefillParams {
     int pool, per_block;
     int dk, dv;                     // real key and value size (kSel)
     int keep_first;                 // kSel: keys at positions below it are seen whatever the window
-    float cap_log2, cap_in;         // kSel: scores become cap tanh(s scale / cap): cap log2(e), and 2 scale log2(e) / cap; cap_log2 0 = as they are
+    float cap_log2, cap_in, cap_x;  // kSel: scores become cap tanh(s scale / cap): cap log2(e), 2 scale log2(e) / cap, scale / cap; cap_log2 0 = as they are
     const float* gate; int64_t ldg; // kSel: [T, H dv] or null: the output times sigmoid(gate) entry by entry
     int64_t ldo;                    // kSel: output row pitch
 };
@@ -180,6 +189,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
     // sigmoid(x) = 1 / (1 + 2^(-x log2 e)): ex2.approx and an approximate reciprocal, both accurate to a few ulp, so that small weights keep their
     // RELATIVE accuracy (tanh.approx would be one operation, but its error is absolute: 2e-4 on a weight of 0.01 is 2 %)
     const float bias_log2 = (kSigmoid && p.head_bias) ? p.head_bias[head] * 1.4426950408889634f : 0.f;
+    const float score_unit = (kSel && p.cap_log2 > 0.f) ? 1.0f : p.scale_log2;                // capped scores are in units of log2 already
     const int pos_lo = pos0 + r_lo, pos_hi = pos0 + r_hi;          // last visible key of each of this thread's two rows
     const int warp_min_pos = pos0 + warp * 16, warp_max_pos = pos0 + warp * 16 + 15;
     const int cs_lo = p.chunk > 0 ? (pos_lo / p.chunk) * p.chunk : 0, cs_hi = p.chunk > 0 ? (pos_hi / p.chunk) * p.chunk : 0;
@@ -210,6 +220,25 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
         // ---- mask (only where the half touches the diagonal / window edge / context end; always for pooled entries) -------------
         const bool need_mask = pooled || tok0 + kHalf - 1 > warp_min_pos || (p.window > 0 && tok0 < warp_max_pos - p.window + 1) || tok0 < warp_max_cs;
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
+        if (kSel && p.cap_log2 > 0.f) {
+            // scores cap tanh(s scale / cap), in units of log2.  Scores within the cap (all of a warp's: the usual case) take the polynomial; else cap - 2 cap / (1 + e^(2x)),
+            // two special-function operations per score: the error of both is absolute, an ulp or two of the cap
+            float big = 0.f;
+#pragma unroll
+            for (int nt = 0; nt < 4; ++nt)
+                big = fmaxf(big, fmaxf(fmaxf(fabsf(sacc[nt][0]), fabsf(sacc[nt][1])), fmaxf(fabsf(sacc[nt][2]), fabsf(sacc[nt][3]))));
+            if (__all_sync(0xffffffffu, big * fabsf(p.cap_x) <= 1.0f)) {
+#pragma unroll
+                for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) sacc[nt][e] = p.cap_log2 * tanh_small(sacc[nt][e] * p.cap_x);
+            } else {
+#pragma unroll
+                for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) sacc[nt][e] = fmaf(-2.f * p.cap_log2, fast_rcp(1.0f + fast_exp2(sacc[nt][e] * p.cap_in)), p.cap_log2);
+            }
+        }
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) {
 #pragma unroll
@@ -227,16 +256,8 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap kmap, const __grid
                     sacc[nt][e] = ok_lo ? __fdividef(1.0f, 1.0f + fast_exp2(-fmaf(sacc[nt][e], p.scale_log2, bias_log2))) : 0.f;
                     sacc[nt][2 + e] = ok_hi ? __fdividef(1.0f, 1.0f + fast_exp2(-fmaf(sacc[nt][2 + e], p.scale_log2, bias_log2))) : 0.f;
                 } else {
-                    if (kSel && p.cap_log2 > 0.f) {
-                        // cap tanh(x) = cap - 2 cap / (1 + e^(2x)), in units of log2: the error is absolute, a few ulp of the cap
-                        sacc[nt][e] = ok_lo ? fmaf(-2.f * p.cap_log2, fast_rcp(1.0f + fast_exp2(sacc[nt][e] * p.cap_in)), p.cap_log2) : -INFINITY;
-                        sacc[nt][2 + e] = ok_hi ? fmaf(-2.f * p.cap_log2, fast_rcp(1.0f + fast_exp2(sacc[nt][2 + e] * p.cap_in)), p.cap_log2) : -INFINITY;
-                        mx_lo = fmaxf(mx_lo, sacc[nt][e]);
-                        mx_hi = fmaxf(mx_hi, sacc[nt][2 + e]);
-                        continue;
-                    }
-                    sacc[nt][e] = ok_lo ? sacc[nt][e] * p.scale_log2 : -INFINITY;
-                    sacc[nt][2 + e] = ok_hi ? sacc[nt][2 + e] * p.scale_log2 : -INFINITY;
+                    sacc[nt][e] = ok_lo ? sacc[nt][e] * score_unit : -INFINITY;
+                    sacc[nt][2 + e] = ok_hi ? sacc[nt][2 + e] * score_unit : -INFINITY;
                     mx_lo = fmaxf(mx_lo, sacc[nt][e]);
                     mx_hi = fmaxf(mx_hi, sacc[nt][2 + e]);
                 }
@@ -437,7 +458,7 @@ void paged_attention_prefill_tc(void* out, const void* q, const void* kc, const 
         return;
     }
     PrefillParams p{q, out, block_tables, cu_q, cu_k, num_seqs, num_heads, num_kv_heads, max_blocks, window, chunk, scale * 1.4426950408889634f,
-                    nullptr, nullptr, nullptr, nullptr, 0, 0, kHd, kHd, 0, 0.f, 0.f, nullptr, 0, (int64_t)num_heads * kHd};
+                    nullptr, nullptr, nullptr, nullptr, 0, 0, kHd, kHd, 0, 0.f, 0.f, 0.f, nullptr, 0, (int64_t)num_heads * kHd};
     bool sigmoid = false;
     if (extras) {
         p.sink = extras->sink; p.head_bias = extras->head_bias; sigmoid = extras->sigmoid;
@@ -471,7 +492,7 @@ void paged_attention_prefill_sel(void* out, int64_t ld_out, const void* q, const
     }
     constexpr float kLog2e = 1.4426950408889634f;
     PrefillParams p{q, out, block_tables, cu_q, cu_k, num_seqs, num_heads, num_kv_heads, max_blocks, window, chunk, scale * kLog2e, sink, nullptr, nullptr, nullptr, 0, 0,
-                    dk, dv, keep_first, softcap * kLog2e, softcap > 0.f ? 2.f * scale * kLog2e / softcap : 0.f, gate, ld_gate, ld_out};
+                    dk, dv, keep_first, softcap * kLog2e, softcap > 0.f ? 2.f * scale * kLog2e / softcap : 0.f, softcap > 0.f ? scale / softcap : 0.f, gate, ld_gate, ld_out};
     const int tiles = total_q / kQTile + num_seqs;                   // >= sum of ceil(q_len / 64)
 #define PS_LAUNCH(DK, DV) do { ensure_dynamic_smem(reinterpret_cast<const void*>(paged_attn_prefill_kernel<__nv_bfloat16, false, false, true, DK, DV>), prefill_smem(DK, DV)); \
         paged_attn_prefill_kernel<__nv_bfloat16, false, false, true, DK, DV><<<dim3(tiles, num_heads), kPfThreads, prefill_smem(DK, DV), st>>>(km, vm, p); } while (0)

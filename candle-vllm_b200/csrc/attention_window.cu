@@ -44,7 +44,7 @@ qk_head_norm_rope_cache_kernel(const float* __restrict__ proj, int64_t ld, const
     const int64_t slot = slot_mapping[t];
     const int half = rot_dims >> 1;
     const int units = H + G + (v_from_k ? 0 : G);
-    for (int u = warp; u < units; u += 8) {
+    for (int u = blockIdx.y * 8 + warp; u < units; u += 8 * gridDim.y) {
         if (u >= H + G) {                                  // a value head: bias, then the cache
             const int g = u - H - G;
             const int col0 = (H + G) * dk + g * dv;
@@ -275,7 +275,7 @@ void qk_head_norm_rope_cache(const float* proj, int64_t ld, const float* bias, c
     cudaStream_t st = as_stream(stream);
     const size_t smem = (size_t)8 * dk * sizeof(float);
 #define QHP(TC, TQ) do { ensure_dynamic_smem((const void*)qk_head_norm_rope_cache_kernel<TC, TQ>, (int)smem); \
-        launch_pdl(qk_head_norm_rope_cache_kernel<TC, TQ>, dim3(num_tokens), dim3(256), smem, st, proj, ld, bias, q_norm_w, k_norm_w, cos_t, sin_t, positions, \
+        launch_pdl(qk_head_norm_rope_cache_kernel<TC, TQ>, dim3(num_tokens, ceil_div(num_heads + 2 * num_kv_heads, 8)), dim3(256), smem, st, proj, ld, bias, q_norm_w, k_norm_w, cos_t, sin_t, positions, \
         slot_mapping, (TQ*)q_out, (TC*)key_cache, (TC*)value_cache, num_heads, num_kv_heads, dk, dv, rot_dims, interleaved, norm_mode, v_from_k, eps); } while (0)
     if (cache_dtype == B200_F32 && q_dtype == B200_F32) QHP(float, float);
     else if (cache_dtype == B200_BF16 && q_dtype == B200_F32) QHP(__nv_bfloat16, float);

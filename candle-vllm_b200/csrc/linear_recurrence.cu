@@ -1205,53 +1205,56 @@ __device__ __forceinline__ float low_rank_value(float z, int form, float inv_tau
     return z;
 }
 
-// few rows: 256 channels x kTok tokens per block, a thread keeps 16 weights of its channel at a time and meets the tokens' inner values with them
-template <int kTok>
+// few rows: 32 channels x 32 tokens per block (a lane per channel, a warp per four tokens), 64 inner values at a time through shared memory
 __global__ void __launch_bounds__(256)
 low_rank_rows_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ out, int T, int N,
                      int R, float inv_tau, int in_tanh, int form, const float* __restrict__ log_rate, int channels_per_rate) {
     pdl_wait();
     pdl_trigger();
-    __shared__ __align__(16) float ys[kTok][16];
-    const int n = blockIdx.x * 256 + threadIdx.x, t0 = blockIdx.y * kTok;
-    float z[kTok];
+    constexpr int kS = 64, kP = kS + 4;
+    __shared__ __align__(16) float ws[32][kP], ys[32][kP];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int n0 = blockIdx.x * 32, n = n0 + lane, t0 = blockIdx.y * 32;
+    float z[4];
     const float b = (n < N && bias) ? bias[n] : 0.f;
-    const bool fours = R % 4 == 0;               // weight rows are whole 16-byte words
 #pragma unroll
-    for (int i = 0; i < kTok; ++i) z[i] = b;
-    for (int r0 = 0; r0 < R; r0 += 16) {
-        float wr[16];
-        const float* wp = w + (int64_t)(n < N ? n : 0) * R + r0;
+    for (int i = 0; i < 4; ++i) z[i] = b;
+    float rw[8], ry[8];
+    auto fetch = [&](int r0) {
 #pragma unroll
-        for (int r = 0; r < 16; r += 4) {
-            if (fours) {
-                const float4 v = r0 + r < R ? *reinterpret_cast<const float4*>(wp + r) : make_float4(0.f, 0.f, 0.f, 0.f);
-                wr[r] = v.x; wr[r + 1] = v.y; wr[r + 2] = v.z; wr[r + 3] = v.w;
-            } else {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) wr[r + e] = r0 + r + e < R ? wp[r + e] : 0.f;
-            }
+        for (int i = 0; i < 8; ++i) {
+            const int e = threadIdx.x + 256 * i, j = e >> 6, r = r0 + (e & 63);
+            rw[i] = (n0 + j < N && r < R) ? w[(int64_t)(n0 + j) * R + r] : 0.f;
+            ry[i] = (t0 + j < T && r < R) ? y[(int64_t)(t0 + j) * ldy + r] : 0.f;
         }
-        __syncthreads();
-        for (int e = threadIdx.x; e < kTok * 16; e += 256) {
-            const int i = e >> 4, r = e & 15;
-            const float v = (t0 + i < T && r0 + r < R) ? y[(int64_t)(t0 + i) * ldy + r0 + r] : 0.f;
-            ys[i][r] = in_tanh ? tanhf(v) : v;
-        }
+    };
+    fetch(0);
+    for (int r0 = 0; r0 < R; r0 += kS) {
         __syncthreads();
 #pragma unroll
-        for (int i = 0; i < kTok; ++i)
+        for (int i = 0; i < 8; ++i) {
+            const int e = threadIdx.x + 256 * i;
+            ws[e >> 6][e & 63] = rw[i];
+            ys[e >> 6][e & 63] = in_tanh ? tanhf(ry[i]) : ry[i];
+        }
+        __syncthreads();
+        if (r0 + kS < R) fetch(r0 + kS);
+        if (t0 + warp * 4 >= T) continue;
+#pragma unroll 4
+        for (int r = 0; r < kS; r += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(&ws[lane][r]);
 #pragma unroll
-            for (int r = 0; r < 16; r += 4) {
-                const float4 v = *reinterpret_cast<const float4*>(&ys[i][r]);
-                z[i] = fmaf(wr[r], v.x, fmaf(wr[r + 1], v.y, fmaf(wr[r + 2], v.z, fmaf(wr[r + 3], v.w, z[i]))));
+            for (int i = 0; i < 4; ++i) {
+                const float4 q = *reinterpret_cast<const float4*>(&ys[warp * 4 + i][r]);
+                z[i] = fmaf(v.x, q.x, fmaf(v.y, q.y, fmaf(v.z, q.z, fmaf(v.w, q.w, z[i]))));
             }
+        }
     }
     if (n >= N) return;
     const float lr = form == 2 ? log_rate[n / channels_per_rate] : 0.f;
 #pragma unroll
-    for (int i = 0; i < kTok; ++i)
-        if (t0 + i < T) out[(int64_t)(t0 + i) * N + n] = low_rank_value(z[i], form, inv_tau, lr);
+    for (int i = 0; i < 4; ++i)
+        if (t0 + warp * 4 + i < T) out[(int64_t)(t0 + warp * 4 + i) * N + n] = low_rank_value(z[i], form, inv_tau, lr);
 }
 
 // many rows: tiles of 64 tokens x 128 channels, 16 inner values at a time through shared memory (both operands stored inner value first), a thread makes 8 tokens x 4
@@ -1843,7 +1846,7 @@ void low_rank_map(const float* y, int64_t ldy, const float* weight, const float*
     cudaStream_t st = as_stream(stream);
     const float inv_tau = form == 0 ? 1.0f / tau : 0.f;
     if (num_tokens <= 256)
-        launch_pdl(low_rank_rows_kernel<2>, dim3(ceil_div(channels, 256), ceil_div(num_tokens, 2)), dim3(256), 0, st, y, ldy, weight, bias, out, (int)num_tokens, (int)channels,
+        launch_pdl(low_rank_rows_kernel, dim3(ceil_div(channels, 32), ceil_div(num_tokens, 32)), dim3(256), 0, st, y, ldy, weight, bias, out, (int)num_tokens, (int)channels,
                    (int)rank, inv_tau, (int)in_tanh, (int)form, log_rate, (int)channels_per_rate);
     else
         launch_pdl(low_rank_tile_kernel, dim3(ceil_div(channels, 128), ceil_div(num_tokens, 64)), dim3(256), 0, st, y, ldy, weight, bias, out, (int)num_tokens, (int)channels,
