@@ -94,6 +94,101 @@ qk_head_norm_rope_cache_kernel(const float* __restrict__ proj, int64_t ld, const
     }
 }
 
+// The same for heads of up to 32 kN entries, a warp per head with everything in registers: a lane owns whole rotation pairs (the partner is never in another lane)
+// and strides over the entries that are not rotated; angles, weights and entries are all requested before the first of them is needed.
+template <typename TC, typename TQ, int kN>
+__global__ void __launch_bounds__(256)
+qk_head_norm_rope_cache_warp_kernel(const float* __restrict__ proj, int64_t ld, const float* __restrict__ bias, const float* __restrict__ q_w,
+                                    const float* __restrict__ k_w, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                                    const int32_t* __restrict__ positions, const int64_t* __restrict__ slot_mapping, TQ* __restrict__ q_out,
+                                    TC* __restrict__ k_cache, TC* __restrict__ v_cache, int H, int G, int dk, int dv, int rot_dims, int interleaved,
+                                    int norm_mode, int v_from_k, float eps) {
+    pdl_wait();
+    pdl_trigger();
+    constexpr int kPairs = kN / 2;
+    const int t = blockIdx.x, u = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (u >= H + G + (v_from_k ? 0 : G)) return;
+    const float* row = proj + (int64_t)t * ld;
+    const int pos = positions[t];
+    const int64_t slot = slot_mapping[t];
+    if (u >= H + G) {                                      // a value head: bias, then the cache
+        const int g = u - H - G, col0 = (H + G) * dk + g * dv;
+        if (slot < 0) return;
+        for (int i = lane; i < dv; i += 32) v_cache[(slot * G + g) * dv + i] = from_f32<TC>(row[col0 + i] + (bias ? bias[col0 + i] : 0.f));
+        return;
+    }
+    const bool is_q = u < H;
+    const float* x = row + u * dk;                         // q heads, then k heads, back to back
+    const float* xb = bias ? bias + u * dk : nullptr;
+    const float* w = is_q ? q_w : k_w;
+    const int rot = cos_t ? rot_dims : 0, half = rot >> 1;
+    float a[kPairs], b[kPairs], wa[kPairs], wb[kPairs], c[kPairs], s[kPairs], p[kN], wp[kN];
+#pragma unroll
+    for (int j = 0; j < kPairs; ++j) {
+        const int f = lane + 32 * j;
+        const bool in = f < half;
+        const int ia = in ? (interleaved ? 2 * f : f) : 0, ib = in ? (interleaved ? 2 * f + 1 : f + half) : 0;
+        a[j] = in ? x[ia] : 0.f; b[j] = in ? x[ib] : 0.f;
+        wa[j] = (in && w) ? w[ia] : 1.f; wb[j] = (in && w) ? w[ib] : 1.f;
+        c[j] = in ? cos_t[(int64_t)pos * half + f] : 1.f; s[j] = in ? sin_t[(int64_t)pos * half + f] : 0.f;
+        if (in && xb) { a[j] += xb[ia]; b[j] += xb[ib]; }
+    }
+#pragma unroll
+    for (int j = 0; j < kN; ++j) {
+        const int i = rot + lane + 32 * j;
+        const bool in = i < dk;
+        p[j] = in ? x[i] : 0.f;
+        wp[j] = (in && w) ? w[i] : 1.f;
+        if (in && xb) p[j] += xb[i];
+    }
+    auto square = [&]() {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < kPairs; ++j) ss = fmaf(a[j], a[j], fmaf(b[j], b[j], ss));
+#pragma unroll
+        for (int j = 0; j < kN; ++j) ss = fmaf(p[j], p[j], ss);
+        return 1.0f / sqrtf(warp_sum(ss) / (float)dk + eps);
+    };
+    auto scale = [&](float sc) {
+#pragma unroll
+        for (int j = 0; j < kPairs; ++j) { a[j] = a[j] * sc * wa[j]; b[j] = b[j] * sc * wb[j]; }
+#pragma unroll
+        for (int j = 0; j < kN; ++j) p[j] = p[j] * sc * wp[j];
+    };
+    if (!is_q && v_from_k && slot >= 0) {                  // the value of a token is its key head as projected
+        TC* v = v_cache + (slot * G + (u - H)) * dk;
+#pragma unroll
+        for (int j = 0; j < kPairs; ++j) {
+            const int f = lane + 32 * j;
+            if (f < half) { v[interleaved ? 2 * f : f] = from_f32<TC>(a[j]); v[interleaved ? 2 * f + 1 : f + half] = from_f32<TC>(b[j]); }
+        }
+#pragma unroll
+        for (int j = 0; j < kN; ++j)
+            if (rot + lane + 32 * j < dk) v[rot + lane + 32 * j] = from_f32<TC>(p[j]);
+    }
+    if (norm_mode == 1) scale(square());
+#pragma unroll
+    for (int j = 0; j < kPairs; ++j) {
+        const float e = a[j];
+        a[j] = e * c[j] - b[j] * s[j];
+        b[j] = b[j] * c[j] + e * s[j];
+    }
+    if (norm_mode == 2) scale(square());
+    if (!is_q && slot < 0) return;
+    auto put = [&](int i, float v) {
+        if (is_q) q_out[((int64_t)t * H + u) * dk + i] = from_f32<TQ>(v);
+        else k_cache[(slot * G + (u - H)) * dk + i] = from_f32<TC>(v);
+    };
+#pragma unroll
+    for (int j = 0; j < kPairs; ++j) {
+        const int f = lane + 32 * j;
+        if (f < half) { put(interleaved ? 2 * f : f, a[j]); put(interleaved ? 2 * f + 1 : f + half, b[j]); }
+    }
+#pragma unroll
+    for (int j = 0; j < kN; ++j)
+        if (rot + lane + 32 * j < dk) put(rot + lane + 32 * j, p[j]);
+}
+
 template <typename TC>
 __global__ void __launch_bounds__(256)
 pooled_cache_update_kernel(const TC* __restrict__ k_cache, const TC* __restrict__ v_cache, float* __restrict__ kp, float* __restrict__ vp,
@@ -274,14 +369,19 @@ void qk_head_norm_rope_cache(const float* proj, int64_t ld, const float* bias, c
                  kErrBadArg, "qk_head_norm_rope_cache: bad sizes");
     cudaStream_t st = as_stream(stream);
     const size_t smem = (size_t)8 * dk * sizeof(float);
-#define QHP(TC, TQ) do { ensure_dynamic_smem((const void*)qk_head_norm_rope_cache_kernel<TC, TQ>, (int)smem); \
-        launch_pdl(qk_head_norm_rope_cache_kernel<TC, TQ>, dim3(num_tokens, ceil_div(num_heads + 2 * num_kv_heads, 8)), dim3(256), smem, st, proj, ld, bias, q_norm_w, k_norm_w, cos_t, sin_t, positions, \
+    const dim3 grid(num_tokens, ceil_div(num_heads + (v_from_k ? 1 : 2) * num_kv_heads, 8));
+#define QHW(TC, TQ, N) launch_pdl(qk_head_norm_rope_cache_warp_kernel<TC, TQ, N>, grid, dim3(256), 0, st, proj, ld, bias, q_norm_w, k_norm_w, cos_t, sin_t, positions, \
+        slot_mapping, (TQ*)q_out, (TC*)key_cache, (TC*)value_cache, num_heads, num_kv_heads, dk, dv, rot_dims, interleaved, norm_mode, v_from_k, eps)
+#define QHP(TC, TQ) do { if (dk <= 64) { QHW(TC, TQ, 2); break; } if (dk <= 128) { QHW(TC, TQ, 4); break; } if (dk <= 256) { QHW(TC, TQ, 8); break; } \
+        ensure_dynamic_smem((const void*)qk_head_norm_rope_cache_kernel<TC, TQ>, (int)smem); \
+        launch_pdl(qk_head_norm_rope_cache_kernel<TC, TQ>, grid, dim3(256), smem, st, proj, ld, bias, q_norm_w, k_norm_w, cos_t, sin_t, positions, \
         slot_mapping, (TQ*)q_out, (TC*)key_cache, (TC*)value_cache, num_heads, num_kv_heads, dk, dv, rot_dims, interleaved, norm_mode, v_from_k, eps); } while (0)
     if (cache_dtype == B200_F32 && q_dtype == B200_F32) QHP(float, float);
     else if (cache_dtype == B200_BF16 && q_dtype == B200_F32) QHP(__nv_bfloat16, float);
     else if (cache_dtype == B200_BF16 && q_dtype == B200_BF16) QHP(__nv_bfloat16, __nv_bfloat16);
     else { set_error(kErrUnsupported, "qk_head_norm_rope_cache: cache dtype %d / q dtype %d", cache_dtype, q_dtype); return; }
 #undef QHP
+#undef QHW
     count_launch();
     check_launch("qk_head_norm_rope_cache");
 }

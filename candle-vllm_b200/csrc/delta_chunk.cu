@@ -9,7 +9,7 @@
 // responses of the recurrence itself, which contracts (beta <= 1, unit keys, decays <= 1), so they stay of order one.  Three kernels:
 //   delta_chunk_prepare  per (chunk, head), all at once: unit vectors, decay products, M, N, B, W = B K_P, U0 = B V, the rows P_t q_t and R_last,s k_s
 //   delta_chunk_walk     per (entry, head, 16 value columns) the walk over the chunks: U = U0 - W S0, then S_end; leaves U and the state entering every chunk
-//   delta_chunk_output   per (chunk, head, 64 value columns), all at once: o
+//   delta_chunk_output   per (chunk, head, 64 or 128 value columns), all at once: o
 // Decays enter as products only, each in [0, 1]: tokens in runs of four, prefix and suffix products inside a run, a table per key row of the products of whole runs
 // between two runs.  Nothing overflows, and a product that underflows is a contribution that has died.
 #include "common.cuh"
@@ -72,13 +72,17 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const float* qbase = A.qkv + (int64_t)tf * C + g * dk;
     const float* kbase = qbase + A.G * dk;
-    for (int t = warp; t < kC; t += 8) {
+#pragma unroll 4
+    for (int i = 0; i < kC / 8; ++i) {
+        const int t = warp + 8 * i;
         float qq = 0.f, kk = 0.f;
-        if (t < nt)
-            for (int r = lane; r < dk; r += 32) {
-                const float x = qbase[(int64_t)t * C + r], y = kbase[(int64_t)t * C + r];
-                qq = fmaf(x, x, qq); kk = fmaf(y, y, kk);
-            }
+#pragma unroll
+        for (int r4 = 0; r4 < kKD / 32; ++r4) {
+            const int r = lane + 32 * r4;
+            const bool ok = t < nt && r < dk;
+            const float x = ok ? qbase[(int64_t)t * C + r] : 0.f, y = ok ? kbase[(int64_t)t * C + r] : 0.f;
+            qq = fmaf(x, x, qq); kk = fmaf(y, y, kk);
+        }
         qq = warp_sum(qq); kk = warp_sum(kk);
         if (lane == 0) {
             qn[t] = (1.0f / sqrtf((float)dk)) / sqrtf(qq + 1e-6f);
@@ -101,7 +105,12 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
                 ra[i][t] = ok ? A.decay[(int64_t)(tf + j) * H * dk + h * dk + r0 + lane] : 1.f;
             }
     };
-    float am[4][4] = {}, an[4][4] = {};
+    // the 120 tiles (run of queries, earlier run of keys) below the diagonal go to threads 0 .. 239 in pairs: an even thread takes N's tile, an odd one M's
+    int tq = 1;
+    while (tq * (tq + 1) / 2 <= (int)(threadIdx.x >> 1) && tq < 15) ++tq;
+    const int tk = min((int)(threadIdx.x >> 1) - tq * (tq - 1) / 2, 15);
+    const bool has_tile = threadIdx.x < 240;
+    float as[4][4] = {};
     float dn[2][10] = {}, dm[2][6] = {};         // inside the thread's two runs, this lane's key rows: N for s <= t, M for s < t
     fetch(0);
     for (int r0 = 0; r0 < dk; r0 += 32) {
@@ -170,16 +179,19 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
             for (int i = 0; i < 8; ++i) KP[((warp + 8 * (i >> 2)) * 4 + (i & 3)) * kKp + r0 + lane] = 0.f;
         }
         if (r0 + 32 < dk) fetch(r0 + 32);
-        if (tx < ty) {                                         // a whole run of queries over a whole earlier run of keys
-#pragma unroll 4
+        if (has_tile) {
+            const float* left = (threadIdx.x & 1) ? &ka[0][tq * 4] : &qs[0][tq * 4];
+            const float* right = &kb[0][tk * 4];
+            const float* mid = mm + tq * 16 + tk;
+#pragma unroll 8
             for (int x = 0; x < 32; ++x) {
-                const float m = mm[x * kRunPitch + ty * 16 + tx];
-                const float4 q = *reinterpret_cast<const float4*>(&qs[x][ty * 4]), k = *reinterpret_cast<const float4*>(&ka[x][ty * 4]), e = *reinterpret_cast<const float4*>(&kb[x][tx * 4]);
-                const float qv[4] = {q.x, q.y, q.z, q.w}, kv[4] = {k.x, k.y, k.z, k.w}, ev[4] = {e.x * m, e.y * m, e.z * m, e.w * m};
+                const float m = mid[x * kRunPitch];
+                const float4 q = *reinterpret_cast<const float4*>(left + x * kLd), e = *reinterpret_cast<const float4*>(right + x * kLd);
+                const float qv[4] = {q.x, q.y, q.z, q.w}, ev[4] = {e.x * m, e.y * m, e.z * m, e.w * m};
 #pragma unroll
                 for (int i = 0; i < 4; ++i)
 #pragma unroll
-                    for (int l = 0; l < 4; ++l) { an[i][l] = fmaf(qv[i], ev[l], an[i][l]); am[i][l] = fmaf(kv[i], ev[l], am[i][l]); }
+                    for (int l = 0; l < 4; ++l) as[i][l] = fmaf(qv[i], ev[l], as[i][l]);
             }
         }
     }
@@ -192,15 +204,22 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
     }
     __syncthreads();                                           // the table has been read: its place takes M and B
     // N goes out through registers; tiles on the diagonal are filled by their runs' owners below, tiles above it are zero
-    if (tx != ty) {
-        const bool seen = tx < ty;
+    if (has_tile) {
+        if (threadIdx.x & 1) {
 #pragma unroll
-        for (int l = 0; l < 4; ++l)
-            *reinterpret_cast<float4*>(&Mt[tx * 4 + l][ty * 4]) = seen ? make_float4(am[0][l], am[1][l], am[2][l], am[3][l]) : make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int l = 0; l < 4; ++l) *reinterpret_cast<float4*>(&Mt[tk * 4 + l][tq * 4]) = make_float4(as[0][l], as[1][l], as[2][l], as[3][l]);
+        } else {
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
-            if (ty * 4 + i < nt)
-                *reinterpret_cast<float4*>(A.N + ((int64_t)(tf + ty * 4 + i) * H + h) * kC + tx * 4) = seen ? make_float4(an[i][0], an[i][1], an[i][2], an[i][3]) : make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int i = 0; i < 4; ++i)
+                if (tq * 4 + i < nt) *reinterpret_cast<float4*>(A.N + ((int64_t)(tf + tq * 4 + i) * H + h) * kC + tk * 4) = make_float4(as[i][0], as[i][1], as[i][2], as[i][3]);
+        }
+    }
+    if (tx > ty) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            *reinterpret_cast<float4*>(&Mt[tx * 4 + i][ty * 4]) = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (ty * 4 + i < nt) *reinterpret_cast<float4*>(A.N + ((int64_t)(tf + ty * 4 + i) * H + h) * kC + tx * 4) = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
     }
     if (lane == 0) {
 #pragma unroll
@@ -468,78 +487,90 @@ delta_chunk_walk_kernel(const DeltaChunkArgs A) {
 }
 
 // ---- the outputs ---------------------------------------------------------------------------------------------------------------------------------------
-constexpr int kOutFloats = 2 * 32 * kLd + 2 * kC * kLd;
+template <int kW> constexpr int out_floats() { return 32 * kLd + 32 * (kW + 4) + kC * kLd + kC * (kW + 4); }
 
-__global__ void __launch_bounds__(256, 3)
+// kW: value columns of a block (64 or 128); a thread makes four tokens x kW / 16 columns (groups of four, 64 columns apart)
+template <int kW>
+__global__ void __launch_bounds__(256, 2)
 delta_chunk_output_kernel(const DeltaChunkArgs A) {
     pdl_wait();
     pdl_trigger();
+    constexpr int kWp = kW + 4, kGr = kW / 64;
     extern __shared__ __align__(16) float sm[];
-    float (*qs)[kLd] = reinterpret_cast<float (*)[kLd]>(sm);                        // [32][68] P_t q_t: [key row][token]
-    float (*ss)[kLd] = reinterpret_cast<float (*)[kLd]>(sm + 32 * kLd);             // [32][68] the entering state: [key row][column]
-    float (*ns)[kLd] = reinterpret_cast<float (*)[kLd]>(sm + 2 * 32 * kLd);         // [64][68] N: [s][t]
-    float (*us)[kLd] = reinterpret_cast<float (*)[kLd]>(sm + 2 * 32 * kLd + kC * kLd);      // [64][68] u: [s][column]
+    float (*qs)[kLd] = reinterpret_cast<float (*)[kLd]>(sm);                                      // [32] P_t q_t: [key row][token]
+    float (*ss)[kWp] = reinterpret_cast<float (*)[kWp]>(sm + 32 * kLd);                           // [32] the entering state: [key row][column]
+    float (*ns)[kLd] = reinterpret_cast<float (*)[kLd]>(sm + 32 * kLd + 32 * kWp);                // [64] N: [s][t]
+    float (*us)[kWp] = reinterpret_cast<float (*)[kWp]>(sm + 32 * kLd + 32 * kWp + kC * kLd);     // [64] u: [s][column]
     const int h = blockIdx.y, b = blockIdx.z / A.max_chunks, c = blockIdx.z % A.max_chunks;
     const int t0 = A.cu[b], rows = A.cu[b + 1] - t0;
     if (c * kC >= rows) return;
     const int tf = t0 + c * kC, nt = min(kC, rows - c * kC);
-    const int dk = A.dk, dv = A.dv, H = A.H, c0 = blockIdx.x * 64;
+    const int dk = A.dk, dv = A.dv, H = A.H, c0 = blockIdx.x * kW;
     const float* Sc = A.Sc + ((int64_t)(chunk_base(A.cu, b) + c) * H + h) * dv * dk;
-    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-    float rq[8], rs[8];
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4, x = threadIdx.x & 31, j0 = threadIdx.x >> 5;
+    float rq[8], rs[8 * kGr];
     auto fetch = [&](int r0) {
+        const bool in = r0 + x < dk;
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-            const int e = threadIdx.x + 256 * i, j = e >> 5, x = e & 31;
-            rq[i] = (j < nt && r0 + x < dk) ? A.QP[((int64_t)(tf + j) * H + h) * dk + r0 + x] : 0.f;
-            rs[i] = (c0 + j < dv && r0 + x < dk) ? Sc[(int64_t)(c0 + j) * dk + r0 + x] : 0.f;
+            const int j = j0 + 8 * i;
+            rq[i] = (j < nt && in) ? A.QP[((int64_t)(tf + j) * H + h) * dk + r0 + x] : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < 8 * kGr; ++i) {
+            const int j = j0 + 8 * i;
+            rs[i] = (c0 + j < dv && in) ? Sc[(int64_t)(c0 + j) * dk + r0 + x] : 0.f;
         }
     };
     fetch(0);
     for (int e = threadIdx.x; e < kC * 64; e += 256) {
-        const int j = e >> 6, x = e & 63;
-        ns[x][j] = j < nt ? A.N[((int64_t)(tf + j) * H + h) * kC + x] : 0.f;
-        us[j][x] = (j < nt && c0 + x < dv) ? A.U[((int64_t)(tf + j) * H + h) * dv + c0 + x] : 0.f;
+        const int j = e >> 6, k = e & 63;
+        ns[k][j] = j < nt ? A.N[((int64_t)(tf + j) * H + h) * kC + k] : 0.f;
     }
-    float o[4][4] = {};
-    for (int r0 = 0; r0 < dk; r0 += 32) {
-        __syncthreads();
+    for (int e = threadIdx.x; e < kC * kW; e += 256) {
+        const int j = e / kW, k = e % kW;
+        us[j][k] = (j < nt && c0 + k < dv) ? A.U[((int64_t)(tf + j) * H + h) * dv + c0 + k] : 0.f;
+    }
+    float o[4][4 * kGr] = {};
+    auto multiply = [&](const float* left, const float* right) {       // one term: four tokens' factors times the columns' row
+        const float4 l4 = *reinterpret_cast<const float4*>(left);
+        const float l[4] = {l4.x, l4.y, l4.z, l4.w};
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int e = threadIdx.x + 256 * i;
-            qs[e & 31][e >> 5] = rq[i];
-            ss[e & 31][e >> 5] = rs[i];
-        }
-        __syncthreads();
-        if (r0 + 32 < dk) fetch(r0 + 32);
-#pragma unroll 8
-        for (int x = 0; x < 32; ++x) {
-            const float4 q4 = *reinterpret_cast<const float4*>(&qs[x][ty * 4]), s4 = *reinterpret_cast<const float4*>(&ss[x][tx * 4]);
-            const float q[4] = {q4.x, q4.y, q4.z, q4.w}, s[4] = {s4.x, s4.y, s4.z, s4.w};
+        for (int g = 0; g < kGr; ++g) {
+            const float4 r4 = *reinterpret_cast<const float4*>(right + 64 * g);
+            const float r[4] = {r4.x, r4.y, r4.z, r4.w};
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int l = 0; l < 4; ++l) o[i][l] = fmaf(q[i], s[l], o[i][l]);
+                for (int k = 0; k < 4; ++k) o[i][4 * g + k] = fmaf(l[i], r[k], o[i][4 * g + k]);
         }
+    };
+    for (int r0 = 0; r0 < dk; r0 += 32) {
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 8; ++i) qs[x][j0 + 8 * i] = rq[i];
+#pragma unroll
+        for (int i = 0; i < 8 * kGr; ++i) ss[x][j0 + 8 * i] = rs[i];
+        __syncthreads();
+        if (r0 + 32 < dk) fetch(r0 + 32);
+#pragma unroll 8
+        for (int k = 0; k < 32; ++k) multiply(&qs[k][ty * 4], &ss[k][tx * 4]);
     }
     const int last = min(nt, ty * 4 + 4);
 #pragma unroll 4
-    for (int s = 0; s < last; ++s) {
-        const float4 n4 = *reinterpret_cast<const float4*>(&ns[s][ty * 4]), u4 = *reinterpret_cast<const float4*>(&us[s][tx * 4]);
-        const float n[4] = {n4.x, n4.y, n4.z, n4.w}, u[4] = {u4.x, u4.y, u4.z, u4.w};
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-            for (int l = 0; l < 4; ++l) o[i][l] = fmaf(n[i], u[l], o[i][l]);
-    }
+    for (int k = 0; k < last; ++k) multiply(&ns[k][ty * 4], &us[k][tx * 4]);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int t = ty * 4 + i;
         if (t >= nt) continue;
 #pragma unroll
-        for (int l = 0; l < 4; ++l) {
-            const int cv = c0 + tx * 4 + l;
-            if (cv < dv) A.out[((int64_t)(tf + t) * H + h) * dv + cv] = o[i][l];
+        for (int g = 0; g < kGr; ++g) {
+            const int cv = c0 + 64 * g + tx * 4;
+            float* dst = A.out + ((int64_t)(tf + t) * H + h) * dv + cv;
+            if ((dv & 3) == 0) { if (cv < dv) *reinterpret_cast<float4*>(dst) = make_float4(o[i][4 * g], o[i][4 * g + 1], o[i][4 * g + 2], o[i][4 * g + 3]); continue; }
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+                if (cv + k < dv) dst[k] = o[i][4 * g + k];
         }
     }
 }
@@ -565,7 +596,7 @@ void gated_delta_channel_chunked(const float* qkv, const float* proj, int64_t ld
     B200_REQUIRE(qkv && proj && decay && state && out && scratch && cu_seqlens && seq_slots && seq_start, kErrBadArg, "gated_delta_channel_chunked: null pointer");
     B200_REQUIRE(num_heads > 0 && num_heads <= 65535 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && dk > 0 && dv > 0 && max_rows > 0 && num_seqs <= 65535, kErrBadArg,
                  "gated_delta_channel_chunked: bad sizes");
-    B200_REQUIRE(((uintptr_t)scratch & 15) == 0, kErrBadArg, "gated_delta_channel_chunked: scratch starts on a 16-byte border");
+    B200_REQUIRE((((uintptr_t)scratch | (uintptr_t)out) & 15) == 0, kErrBadArg, "gated_delta_channel_chunked: scratch and out start on 16-byte borders");
     B200_REQUIRE(dk <= 128, kErrUnsupported, "gated_delta_channel_chunked: key size %d > 128", dk);
     const int max_chunks = (max_rows + kC - 1) / kC;
     B200_REQUIRE((int64_t)max_chunks * num_seqs <= 65535, kErrUnsupported, "gated_delta_channel_chunked: %d chunks x %d entries exceed the grid", max_chunks, num_seqs);
@@ -591,9 +622,13 @@ void gated_delta_channel_chunked(const float* qkv, const float* proj, int64_t ld
     else if (dk <= 64) DCH(64);
     else DCH(128);
 #undef DCH
-    const int s3 = kOutFloats * (int)sizeof(float);
-    ensure_dynamic_smem(reinterpret_cast<const void*>(delta_chunk_output_kernel), s3);
-    launch_pdl(delta_chunk_output_kernel, dim3(ceil_div(dv, 64), num_heads, z), dim3(256), (size_t)s3, st, A);
+#define DCO(W) do { \
+        const int s3 = out_floats<W>() * (int)sizeof(float); \
+        ensure_dynamic_smem(reinterpret_cast<const void*>(delta_chunk_output_kernel<W>), s3); \
+        launch_pdl(delta_chunk_output_kernel<W>, dim3(ceil_div(dv, W), num_heads, z), dim3(256), (size_t)s3, st, A); } while (0)
+    if (dv <= 64) DCO(64);
+    else DCO(128);
+#undef DCO
     count_launch(3);
     check_launch("gated_delta_channel_chunked");
 }
