@@ -27,11 +27,12 @@ struct DeltaChunkArgs {
     float* state; float* out;                    // [slots, H, dv, dk], [T, H dv]
     const int32_t* cu; const int32_t* slots; const int32_t* start;
     int T, H, G, dk, dv, max_chunks;
-    float *W, *KE, *QP;                          // [T, H, dk]
-    float* N;                                    // [T, H, 64]
+    float *W, *KE;                               // [T, H, dk]
+    float* QP;                                   // [chunks, H, dk, 64]: tokens innermost, the layout the output kernel multiplies from
+    float* N;                                    // [chunks, H, 64 (s), 64 (t)]
     float* U;                                    // [T, H, dv]
     float* Pe;                                   // [chunks, H, dk] the product of a chunk's decays
-    float* Sc;                                   // [chunks, H, dv, dk] the state entering a chunk
+    float* Sc;                                   // [chunks, H, dk, dv] the state entering a chunk
 };
 
 __host__ __device__ __forceinline__ int64_t chunk_slots(int T, int B) { return (T + kC - 1) / kC + B; }
@@ -39,6 +40,12 @@ __device__ __forceinline__ int chunk_base(const int32_t* cu, int b) {      // ch
     int s = 0;
     for (int i = 0; i < b; ++i) s += (cu[i + 1] - cu[i] + kC - 1) / kC;
     return s;
+}
+
+__device__ __forceinline__ void cp_async(float* dst, const float* src, bool ok, bool wide) {       // 16 or 4 bytes; zeros where the source does not exist
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+    if (wide) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(ok ? 16 : 0) : "memory");
+    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(d), "l"(src), "r"(ok ? 4 : 0) : "memory");
 }
 
 constexpr int kPrepFloats(int kd) { return 3 * 32 * kLd + 32 * kRunPitch + 32 * 17 + kC * (kd + 4) + 3 * kC; }
@@ -68,6 +75,9 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
     if (c * kC >= rows) return;
     const int tf = t0 + c * kC, nt = min(kC, rows - c * kC);
     const int dk = A.dk, dv = A.dv, H = A.H, g = h / (H / A.G);
+    const int64_t ch = (int64_t)(chunk_base(A.cu, b) + c) * H + h;
+    float* QPt = A.QP + ch * dk * kC;
+    float* Nt = A.N + ch * kC * kC;
     const int C = 2 * A.G * dk + H * dv;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const float* qbase = A.qkv + (int64_t)tf * C + g * dk;
@@ -114,18 +124,18 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
     float dn[2][10] = {}, dm[2][6] = {};         // inside the thread's two runs, this lane's key rows: N for s <= t, M for s < t
     fetch(0);
     for (int r0 = 0; r0 < dk; r0 += 32) {
-        float q4[2][4], a4[2][4], b4[2][4];
+        float a4[2][4], b4[2][4];
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const int a = warp + 8 * i;
-            float p = 1.f, s = 1.f;
+            float p = 1.f, s = 1.f, q4[4];
 #pragma unroll
-            for (int t = 0; t < 4; ++t) { p *= ra[i][t]; q4[i][t] = rq[i][t] * p; a4[i][t] = rk[i][t] * p; }
+            for (int t = 0; t < 4; ++t) { p *= ra[i][t]; q4[t] = rq[i][t] * p; a4[i][t] = rk[i][t] * p; }
 #pragma unroll
             for (int t = 3; t >= 0; --t) { b4[i][t] = rk[i][t] * s; s *= ra[i][t]; }
             es[lane * 17 + a] = p;
-            *reinterpret_cast<float4*>(&qs[lane][a * 4]) = make_float4(q4[i][0], q4[i][1], q4[i][2], q4[i][3]);
+            *reinterpret_cast<float4*>(&qs[lane][a * 4]) = make_float4(q4[0], q4[1], q4[2], q4[3]);
             *reinterpret_cast<float4*>(&ka[lane][a * 4]) = make_float4(a4[i][0], a4[i][1], a4[i][2], a4[i][3]);
             *reinterpret_cast<float4*>(&kb[lane][a * 4]) = make_float4(b4[i][0], b4[i][1], b4[i][2], b4[i][3]);
             int n = 0, m = 0;
@@ -154,7 +164,7 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
             if (warp == 7) {
                 float m = 1.f;
                 for (int a = 0; a < 16; ++a) { mr[a * 17] = m; m *= er[a]; }
-                if (r0 + lane < dk) A.Pe[((int64_t)(chunk_base(A.cu, b) + c) * H + h) * dk + r0 + lane] = m;
+                if (r0 + lane < dk) A.Pe[ch * dk + r0 + lane] = m;
             }
         }
         __syncthreads();
@@ -169,9 +179,7 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
                     const int j = a * 4 + t;
                     KP[j * kKp + r0 + lane] = a4[i][t] * before;
                     if (j >= nt) continue;
-                    const int64_t at = ((int64_t)(tf + j) * H + h) * dk + r0 + lane;
-                    A.QP[at] = q4[i][t] * before;
-                    A.KE[at] = b4[i][t] * after;
+                    A.KE[((int64_t)(tf + j) * H + h) * dk + r0 + lane] = b4[i][t] * after;
                 }
             }
         } else if (r0 + lane < kKp) {
@@ -179,6 +187,14 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
             for (int i = 0; i < 8; ++i) KP[((warp + 8 * (i >> 2)) * 4 + (i & 3)) * kKp + r0 + lane] = 0.f;
         }
         if (r0 + 32 < dk) fetch(r0 + 32);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {                          // P_t q_t, a run of four tokens at a time
+            const int x = (threadIdx.x >> 4) + 16 * i;
+            if (r0 + x >= dk) continue;
+            const float before = mm[x * kRunPitch + tx * 17];
+            const float4 q = *reinterpret_cast<const float4*>(&qs[x][tx * 4]);
+            *reinterpret_cast<float4*>(QPt + (int64_t)(r0 + x) * kC + tx * 4) = make_float4(q.x * before, q.y * before, q.z * before, q.w * before);
+        }
         if (has_tile) {
             const float* left = (threadIdx.x & 1) ? &ka[0][tq * 4] : &qs[0][tq * 4];
             const float* right = &kb[0][tk * 4];
@@ -203,22 +219,20 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
         for (int n = 0; n < 6; ++n) dm[i][n] = warp_sum(dm[i][n]);
     }
     __syncthreads();                                           // the table has been read: its place takes M and B
-    // N goes out through registers; tiles on the diagonal are filled by their runs' owners below, tiles above it are zero
+    // tiles on the diagonal are filled by their runs' owners below, scores over later tokens are zero
     if (has_tile) {
-        if (threadIdx.x & 1) {
 #pragma unroll
-            for (int l = 0; l < 4; ++l) *reinterpret_cast<float4*>(&Mt[tk * 4 + l][tq * 4]) = make_float4(as[0][l], as[1][l], as[2][l], as[3][l]);
-        } else {
-#pragma unroll
-            for (int i = 0; i < 4; ++i)
-                if (tq * 4 + i < nt) *reinterpret_cast<float4*>(A.N + ((int64_t)(tf + tq * 4 + i) * H + h) * kC + tk * 4) = make_float4(as[i][0], as[i][1], as[i][2], as[i][3]);
+        for (int l = 0; l < 4; ++l) {
+            const float4 v = make_float4(as[0][l], as[1][l], as[2][l], as[3][l]);
+            if (threadIdx.x & 1) *reinterpret_cast<float4*>(&Mt[tk * 4 + l][tq * 4]) = v;
+            else *reinterpret_cast<float4*>(Nt + (tk * 4 + l) * kC + tq * 4) = v;
         }
     }
     if (tx > ty) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            *reinterpret_cast<float4*>(&Mt[tx * 4 + i][ty * 4]) = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (ty * 4 + i < nt) *reinterpret_cast<float4*>(A.N + ((int64_t)(tf + ty * 4 + i) * H + h) * kC + tx * 4) = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int l = 0; l < 4; ++l) {
+            *reinterpret_cast<float4*>(&Mt[tx * 4 + l][ty * 4]) = make_float4(0.f, 0.f, 0.f, 0.f);
+            *reinterpret_cast<float4*>(Nt + (tx * 4 + l) * kC + ty * 4) = make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
     if (lane == 0) {
@@ -229,12 +243,25 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
             *reinterpret_cast<float4*>(&Mt[a + 1][a]) = make_float4(0.f, 0.f, dm[i][3], dm[i][4]);
             *reinterpret_cast<float4*>(&Mt[a + 2][a]) = make_float4(0.f, 0.f, 0.f, dm[i][5]);
             *reinterpret_cast<float4*>(&Mt[a + 3][a]) = make_float4(0.f, 0.f, 0.f, 0.f);
-            const float n[4][4] = {{dn[i][0], 0.f, 0.f, 0.f}, {dn[i][1], dn[i][4], 0.f, 0.f}, {dn[i][2], dn[i][5], dn[i][7], 0.f}, {dn[i][3], dn[i][6], dn[i][8], dn[i][9]}};
-#pragma unroll
-            for (int t = 0; t < 4; ++t)
-                if (a + t < nt) *reinterpret_cast<float4*>(A.N + ((int64_t)(tf + a + t) * H + h) * kC + a) = make_float4(n[t][0], n[t][1], n[t][2], n[t][3]);
+            *reinterpret_cast<float4*>(Nt + a * kC + a) = make_float4(dn[i][0], dn[i][1], dn[i][2], dn[i][3]);
+            *reinterpret_cast<float4*>(Nt + (a + 1) * kC + a) = make_float4(0.f, dn[i][4], dn[i][5], dn[i][6]);
+            *reinterpret_cast<float4*>(Nt + (a + 2) * kC + a) = make_float4(0.f, 0.f, dn[i][7], dn[i][8]);
+            *reinterpret_cast<float4*>(Nt + (a + 3) * kC + a) = make_float4(0.f, 0.f, 0.f, dn[i][9]);
         }
     }
+    // the first 64 value columns travel while B is worked out
+    const float* vrow = A.qkv + (int64_t)tf * C + 2 * A.G * dk + h * dv;
+    const bool wide_v = (dv & 3) == 0 && (C & 3) == 0 && ((2 * A.G * dk) & 3) == 0 && ((uintptr_t)A.qkv & 15) == 0;
+    auto issue_values = [&](int c0) {
+        const int w = wide_v ? 4 : 1;
+        for (int e = threadIdx.x; e < kC * 64 / w; e += 256) {
+            const int j = e / (64 / w), x = (e % (64 / w)) * w;
+            const bool ok = j < nt && c0 + x < dv;
+            cp_async(&Vs[j][x], vrow + (ok ? (int64_t)j * C + c0 + x : 0), ok, wide_v);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    issue_values(0);
     __syncthreads();
     // ---- B in two halves of 32: the diagonal blocks column by column (a lane per column, everything in registers), then B21 = -B22 M21 B11 --------------
     if (warp < 2) {
@@ -314,11 +341,8 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
         if (kKD >= 64 || tx < 8) { product(KP + c0, kKp, acc); store(A.W, dk, c0, acc); }
     }
     for (int c0 = 0; c0 < dv; c0 += 64) {
-        __syncthreads();
-        for (int e = threadIdx.x; e < kC * 64; e += 256) {
-            const int j = e >> 6, x = e & 63;
-            Vs[j][x] = (j < nt && c0 + x < dv) ? A.qkv[(int64_t)(tf + j) * C + 2 * A.G * dk + h * dv + c0 + x] : 0.f;
-        }
+        if (c0 > 0) { __syncthreads(); issue_values(c0); }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         product(&Vs[0][0], kLd, acc);
         store(A.U, dv, c0, acc);
@@ -328,27 +352,27 @@ delta_chunk_prepare_kernel(const DeltaChunkArgs A) {
 // ---- the walk ------------------------------------------------------------------------------------------------------------------------------------------
 constexpr int kVB = 16, kVp = 20;                // value columns of a block and their pitch
 
+constexpr int kWalkThreads = 512;
 template <int kKD> constexpr int walk_stage_floats() { return 2 * kC * (kKD + 4) + kC * kVp + kKD; }
-template <int kKD> constexpr int walk_floats() { return 2 * walk_stage_floats<kKD>() + 4 * kC * kVp + kC * kVp + kKD * kVp + (256 / kKD) * kKD * kVp; }
-
-__device__ __forceinline__ void cp_async(float* dst, const float* src, bool ok, bool wide) {       // 16 or 4 bytes; zeros where the source does not exist
-    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
-    if (wide) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(ok ? 16 : 0) : "memory");
-    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(d), "l"(src), "r"(ok ? 4 : 0) : "memory");
+template <int kKD> constexpr int walk_red_floats() {          // partial sums: of the first product per share of the key rows, of the update per share of the tokens
+    constexpr int a = (kWalkThreads / 64) * kC * kVp, b = (kWalkThreads / kKD) * kKD * kVp;
+    return a > b ? a : b;
 }
+template <int kKD> constexpr int walk_floats() { return 2 * walk_stage_floats<kKD>() + walk_red_floats<kKD>() + kC * kVp + kKD * kVp; }
 
 template <int kKD>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(kWalkThreads)
 delta_chunk_walk_kernel(const DeltaChunkArgs A) {
     pdl_wait();
     pdl_trigger();
     constexpr int kKp = kKD + 4, kStage = walk_stage_floats<kKD>();
-    constexpr int kRG = kKD / 4, kSG = 64 / kRG;                       // update: groups of four key rows, shares of the tokens (4 column groups x kRG x kSG = 256)
+    constexpr int kKG = kWalkThreads / 64, kKs = kKD / kKG;            // first product: shares of the key rows and their size
+    constexpr int kRG = kKD / 4, kSG = kWalkThreads / (4 * kRG), kTs = kC / kSG;      // update: groups of four key rows, shares of the tokens and their size
+    static_assert(kKs % 4 == 0 && kTs * kSG == kC, "shares of whole fours");
     extern __shared__ __align__(16) float sm[];
-    float* red = sm + 2 * kStage;                                      // [4][64][20] partial products of the four quarters of the key rows
-    float* Us = red + 4 * kC * kVp;                                    // [64][20]
+    float* red = sm + 2 * kStage;                                      // [kKG][64][20] / [kSG][kKD][20]
+    float* Us = red + walk_red_floats<kKD>();                          // [64][20]
     float* S = Us + kC * kVp;                                          // [kKD][20]
-    float* part = S + kKD * kVp;                                       // [kSG][kKD][20]
     const int h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * kVB;
     const int t0 = A.cu[b], rows = A.cu[b + 1] - t0;
     if (rows <= 0) return;
@@ -361,20 +385,23 @@ delta_chunk_walk_kernel(const DeltaChunkArgs A) {
         float* U0 = Ks + kC * kKp;
         float* Pe = U0 + kC * kVp;
         const int tf = t0 + c * kC, nt = min(kC, rows - c * kC);
-        const int ek = wide_k ? 4 : 1, ev = wide_v ? 4 : 1;
-        for (int e = tid; e < kC * kKD / ek; e += 256) {
+        const float* Wg = A.W + ((int64_t)tf * H + h) * dk;
+        const float* Kg = A.KE + ((int64_t)tf * H + h) * dk;
+        const int ek = wide_k ? 4 : 1, ev = wide_v ? 4 : 1, ld = H * dk;
+        for (int e = tid; e < kC * kKD / ek; e += kWalkThreads) {
             const int j = e / (kKD / ek), r = (e % (kKD / ek)) * ek;
             const bool ok = j < nt && r < dk;
-            const int64_t at = ((int64_t)(tf + (ok ? j : 0)) * H + h) * dk + (ok ? r : 0);
-            cp_async(Ws + j * kKp + r, A.W + at, ok, wide_k);
-            cp_async(Ks + j * kKp + r, A.KE + at, ok, wide_k);
+            const int at = ok ? j * ld + r : 0;
+            cp_async(Ws + j * kKp + r, Wg + at, ok, wide_k);
+            cp_async(Ks + j * kKp + r, Kg + at, ok, wide_k);
         }
-        for (int e = tid; e < kC * kVB / ev; e += 256) {
+        const float* Ug = A.U + ((int64_t)tf * H + h) * dv;
+        for (int e = tid; e < kC * kVB / ev; e += kWalkThreads) {
             const int j = e / (kVB / ev), x = (e % (kVB / ev)) * ev;
             const bool ok = j < nt && c0 + x < dv;
-            cp_async(U0 + j * kVp + x, A.U + ((int64_t)(tf + (ok ? j : 0)) * H + h) * dv + (ok ? c0 + x : 0), ok, wide_v);
+            cp_async(U0 + j * kVp + x, Ug + (ok ? j * H * dv + c0 + x : 0), ok, wide_v);
         }
-        for (int e = tid; e < kKD / ek; e += 256) {
+        for (int e = tid; e < kKD / ek; e += kWalkThreads) {
             const int r = e * ek;
             const bool ok = r < dk;
             cp_async(Pe + r, A.Pe + ((int64_t)(base + c) * H + h) * dk + (ok ? r : 0), ok, wide_k);
@@ -384,11 +411,11 @@ delta_chunk_walk_kernel(const DeltaChunkArgs A) {
     issue(0, 0);
     const bool fresh = A.start[b] == 0;
     float* Sg = A.state + ((int64_t)A.slots[b] * H + h) * dv * dk;
-    for (int e = tid; e < kKD * kVB; e += 256) {
+    for (int e = tid; e < kKD * kVB; e += kWalkThreads) {
         const int x = e / kKD, r = e % kKD;
         S[r * kVp + x] = (!fresh && r < dk && c0 + x < dv) ? Sg[(int64_t)(c0 + x) * dk + r] : 0.f;
     }
-    // roles: first product -- column group cg, rows ig + 16 a, quarter kg of the key rows; update -- column group cg, key rows rg * 4 .., share sg of the tokens
+    // roles: first product -- column group cg, rows ig + 16 a, share kg of the key rows; update -- column group cg, key rows rg * 4 .., share sg of the tokens
     const int cg = tid & 3, ig = (tid >> 2) & 15, kg = tid >> 6, rg = (tid >> 2) % kRG, sg = (tid >> 2) / kRG;
     for (int c = 0; c < nc; ++c) {
         const int stage = c & 1, tf = t0 + c * kC, nt = min(kC, rows - c * kC);
@@ -404,14 +431,21 @@ delta_chunk_walk_kernel(const DeltaChunkArgs A) {
         }
         __syncthreads();
         // the state entering this chunk, for the outputs
-        float* Sc = A.Sc + ((int64_t)(base + c) * H + h) * dv * dk;
-        for (int e = tid; e < kKD * kVB; e += 256) {
-            const int x = e / kKD, r = e % kKD;
-            if (r < dk && c0 + x < dv) Sc[(int64_t)(c0 + x) * dk + r] = S[r * kVp + x];
+        float* Sc = A.Sc + ((int64_t)(base + c) * H + h) * dv * dk + c0;
+        for (int e = tid; e < kKD * 4; e += kWalkThreads) {
+            const int r = e >> 2, x = (e & 3) * 4;
+            if (r >= dk) continue;
+            const float4 v = *reinterpret_cast<const float4*>(S + r * kVp + x);
+            float* dst = Sc + (int64_t)r * dv + x;
+            if (wide_v) { if (c0 + x < dv) *reinterpret_cast<float4*>(dst) = v; continue; }
+            const float vv[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int l = 0; l < 4; ++l)
+                if (c0 + x + l < dv) dst[l] = vv[l];
         }
         float acc[4][4] = {};
-#pragma unroll 2
-        for (int k = kg * (kKD / 4); k < (kg + 1) * (kKD / 4); k += 4) {
+#pragma unroll
+        for (int k = kg * kKs; k < (kg + 1) * kKs; k += 4) {
             float4 s4[4], w4[4];
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
@@ -431,15 +465,14 @@ delta_chunk_walk_kernel(const DeltaChunkArgs A) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(red + (kg * kC + ig + 16 * i) * kVp + cg * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
         __syncthreads();
-        {
+        if (tid < kC * 4) {
             const int j = tid >> 2, x = (tid & 3) * 4;
-            const float4 u0 = *reinterpret_cast<const float4*>(U0 + j * kVp + x);
-            float4 r[4];
+            float4 u = *reinterpret_cast<const float4*>(U0 + j * kVp + x);
 #pragma unroll
-            for (int q = 0; q < 4; ++q) r[q] = *reinterpret_cast<const float4*>(red + (q * kC + j) * kVp + x);
-            float4 u;
-            u.x = u0.x - ((r[0].x + r[1].x) + (r[2].x + r[3].x)); u.y = u0.y - ((r[0].y + r[1].y) + (r[2].y + r[3].y));
-            u.z = u0.z - ((r[0].z + r[1].z) + (r[2].z + r[3].z)); u.w = u0.w - ((r[0].w + r[1].w) + (r[2].w + r[3].w));
+            for (int q = 0; q < kKG; ++q) {
+                const float4 r = *reinterpret_cast<const float4*>(red + (q * kC + j) * kVp + x);
+                u.x -= r.x; u.y -= r.y; u.z -= r.z; u.w -= r.w;
+            }
             *reinterpret_cast<float4*>(Us + j * kVp + x) = u;
             if (j < nt) {
                 float* dst = A.U + ((int64_t)(tf + j) * H + h) * dv + c0 + x;
@@ -454,8 +487,8 @@ delta_chunk_walk_kernel(const DeltaChunkArgs A) {
         }
         __syncthreads();
         float up[4][4] = {};
-#pragma unroll 4
-        for (int s = sg * (kC / kSG); s < (sg + 1) * (kC / kSG); ++s) {
+#pragma unroll 8
+        for (int s = sg * kTs; s < (sg + 1) * kTs; ++s) {
             const float4 k4 = *reinterpret_cast<const float4*>(Ks + s * kKp + rg * 4), u4 = *reinterpret_cast<const float4*>(Us + s * kVp + cg * 4);
             const float k[4] = {k4.x, k4.y, k4.z, k4.w}, u[4] = {u4.x, u4.y, u4.z, u4.w};
 #pragma unroll
@@ -464,73 +497,79 @@ delta_chunk_walk_kernel(const DeltaChunkArgs A) {
                 for (int l = 0; l < 4; ++l) up[i][l] = fmaf(k[i], u[l], up[i][l]);
         }
 #pragma unroll
-        for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(part + (sg * kKD + rg * 4 + i) * kVp + cg * 4) = make_float4(up[i][0], up[i][1], up[i][2], up[i][3]);
+        for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(red + (sg * kKD + rg * 4 + i) * kVp + cg * 4) = make_float4(up[i][0], up[i][1], up[i][2], up[i][3]);
         __syncthreads();
-        for (int e = tid; e < kKD * 4; e += 256) {
+        for (int e = tid; e < kKD * 4; e += kWalkThreads) {
             const int r = e >> 2, x = (e & 3) * 4;
             float4 s = *reinterpret_cast<const float4*>(S + r * kVp + x);
             const float pe = Pe[r];
             s.x *= pe; s.y *= pe; s.z *= pe; s.w *= pe;
 #pragma unroll
             for (int q = 0; q < kSG; ++q) {
-                const float4 v = *reinterpret_cast<const float4*>(part + (q * kKD + r) * kVp + x);
+                const float4 v = *reinterpret_cast<const float4*>(red + (q * kKD + r) * kVp + x);
                 s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
             }
             *reinterpret_cast<float4*>(S + r * kVp + x) = s;
         }
         __syncthreads();
     }
-    for (int e = tid; e < kKD * kVB; e += 256) {
+    for (int e = tid; e < kKD * kVB; e += kWalkThreads) {
         const int x = e / kKD, r = e % kKD;
         if (r < dk && c0 + x < dv) Sg[(int64_t)(c0 + x) * dk + r] = S[r * kVp + x];
     }
 }
 
 // ---- the outputs ---------------------------------------------------------------------------------------------------------------------------------------
-template <int kW> constexpr int out_floats() { return 32 * kLd + 32 * (kW + 4) + kC * kLd + kC * (kW + 4); }
+template <int kW> constexpr int out_floats() { return 2 * 32 * (kLd + kW + 4) + kC * kLd + kC * (kW + 4); }
 
-// kW: value columns of a block (64 or 128); a thread makes four tokens x kW / 16 columns (groups of four, 64 columns apart)
+// kW: value columns of a block (64 or 128); a thread makes four tokens x kW / 16 columns (groups of four, 64 columns apart).  All operands arrive by cp.async as they lie:
+// slabs of 32 key rows of P q and of the entering state (two buffers), N and u for the second term under the first one.
 template <int kW>
 __global__ void __launch_bounds__(256, 2)
 delta_chunk_output_kernel(const DeltaChunkArgs A) {
     pdl_wait();
     pdl_trigger();
-    constexpr int kWp = kW + 4, kGr = kW / 64;
-    extern __shared__ __align__(16) float sm[];
-    float (*qs)[kLd] = reinterpret_cast<float (*)[kLd]>(sm);                                      // [32] P_t q_t: [key row][token]
-    float (*ss)[kWp] = reinterpret_cast<float (*)[kWp]>(sm + 32 * kLd);                           // [32] the entering state: [key row][column]
-    float (*ns)[kLd] = reinterpret_cast<float (*)[kLd]>(sm + 32 * kLd + 32 * kWp);                // [64] N: [s][t]
-    float (*us)[kWp] = reinterpret_cast<float (*)[kWp]>(sm + 32 * kLd + 32 * kWp + kC * kLd);     // [64] u: [s][column]
+    constexpr int kWp = kW + 4, kGr = kW / 64, kSlab = 32 * (kLd + kWp);
+    extern __shared__ __align__(16) float sm[];             // two slabs: [32][68] P q, [32][kWp] state
+    float* ns = sm + 2 * kSlab;                             // [64][68] N: [s][t]
+    float* us = ns + kC * kLd;                              // [64][kWp] u: [s][column]
     const int h = blockIdx.y, b = blockIdx.z / A.max_chunks, c = blockIdx.z % A.max_chunks;
     const int t0 = A.cu[b], rows = A.cu[b + 1] - t0;
     if (c * kC >= rows) return;
     const int tf = t0 + c * kC, nt = min(kC, rows - c * kC);
     const int dk = A.dk, dv = A.dv, H = A.H, c0 = blockIdx.x * kW;
-    const float* Sc = A.Sc + ((int64_t)(chunk_base(A.cu, b) + c) * H + h) * dv * dk;
-    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4, x = threadIdx.x & 31, j0 = threadIdx.x >> 5;
-    float rq[8], rs[8 * kGr];
-    auto fetch = [&](int r0) {
-        const bool in = r0 + x < dk;
+    const int64_t ch = (int64_t)(chunk_base(A.cu, b) + c) * H + h;
+    const float* Sc = A.Sc + ch * dv * dk + c0;
+    const float* QPt = A.QP + ch * dk * kC;
+    const float* Nt = A.N + ch * kC * kC;
+    const float* Ug = A.U + ((int64_t)tf * H + h) * dv + c0;
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const bool wide_v = (dv & 3) == 0;
+    const int ev = wide_v ? 4 : 1;
+    auto issue = [&](int r0, int stage) {
+        float* qs = sm + stage * kSlab;
+        float* ss = qs + 32 * kLd;
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int j = j0 + 8 * i;
-            rq[i] = (j < nt && in) ? A.QP[((int64_t)(tf + j) * H + h) * dk + r0 + x] : 0.f;
+        for (int i = 0; i < 2; ++i) {
+            const int x = (threadIdx.x >> 4) + 16 * i, t = tx * 4;
+            const bool ok = r0 + x < dk;
+            cp_async(qs + x * kLd + t, QPt + (ok ? (r0 + x) * kC + t : 0), ok, true);
         }
-#pragma unroll
-        for (int i = 0; i < 8 * kGr; ++i) {
-            const int j = j0 + 8 * i;
-            rs[i] = (c0 + j < dv && in) ? Sc[(int64_t)(c0 + j) * dk + r0 + x] : 0.f;
+        for (int e = threadIdx.x; e < 32 * kW / ev; e += 256) {
+            const int x = e / (kW / ev), k = (e % (kW / ev)) * ev;
+            const bool ok = r0 + x < dk && c0 + k < dv;
+            cp_async(ss + x * kWp + k, Sc + (ok ? (int64_t)(r0 + x) * dv + k : 0), ok, wide_v);
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(0);
-    for (int e = threadIdx.x; e < kC * 64; e += 256) {
-        const int j = e >> 6, k = e & 63;
-        ns[k][j] = j < nt ? A.N[((int64_t)(tf + j) * H + h) * kC + k] : 0.f;
+    issue(0, 0);
+    for (int e = threadIdx.x; e < kC * 16; e += 256) cp_async(ns + (e >> 4) * kLd + (e & 15) * 4, Nt + e * 4, true, true);
+    for (int e = threadIdx.x; e < kC * kW / ev; e += 256) {
+        const int j = e / (kW / ev), k = (e % (kW / ev)) * ev;
+        const bool ok = j < nt && c0 + k < dv;
+        cp_async(us + j * kWp + k, Ug + (ok ? (int64_t)j * H * dv + k : 0), ok, wide_v);
     }
-    for (int e = threadIdx.x; e < kC * kW; e += 256) {
-        const int j = e / kW, k = e % kW;
-        us[j][k] = (j < nt && c0 + k < dv) ? A.U[((int64_t)(tf + j) * H + h) * dv + c0 + k] : 0.f;
-    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
     float o[4][4 * kGr] = {};
     auto multiply = [&](const float* left, const float* right) {       // one term: four tokens' factors times the columns' row
         const float4 l4 = *reinterpret_cast<const float4*>(left);
@@ -545,20 +584,24 @@ delta_chunk_output_kernel(const DeltaChunkArgs A) {
                 for (int k = 0; k < 4; ++k) o[i][4 * g + k] = fmaf(l[i], r[k], o[i][4 * g + k]);
         }
     };
-    for (int r0 = 0; r0 < dk; r0 += 32) {
+    for (int r0 = 0, stage = 0; r0 < dk; r0 += 32, stage ^= 1) {
+        const bool first = r0 == 0, more = r0 + 32 < dk;
+        if (more) issue(r0 + 32, stage ^ 1);
+        // the slab in use is the oldest group but one (N and u were asked for right after the first slab)
+        if (first) { if (more) asm volatile("cp.async.wait_group 2;" ::: "memory"); else asm volatile("cp.async.wait_group 1;" ::: "memory"); }
+        else { if (more) asm volatile("cp.async.wait_group 1;" ::: "memory"); else asm volatile("cp.async.wait_group 0;" ::: "memory"); }
         __syncthreads();
-#pragma unroll
-        for (int i = 0; i < 8; ++i) qs[x][j0 + 8 * i] = rq[i];
-#pragma unroll
-        for (int i = 0; i < 8 * kGr; ++i) ss[x][j0 + 8 * i] = rs[i];
-        __syncthreads();
-        if (r0 + 32 < dk) fetch(r0 + 32);
+        const float* qs = sm + stage * kSlab + ty * 4;
+        const float* ss = sm + stage * kSlab + 32 * kLd + tx * 4;
 #pragma unroll 8
-        for (int k = 0; k < 32; ++k) multiply(&qs[k][ty * 4], &ss[k][tx * 4]);
+        for (int k = 0; k < 32; ++k) multiply(qs + k * kLd, ss + k * kWp);
+        __syncthreads();
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
     const int last = min(nt, ty * 4 + 4);
 #pragma unroll 4
-    for (int k = 0; k < last; ++k) multiply(&ns[k][ty * 4], &us[k][tx * 4]);
+    for (int k = 0; k < last; ++k) multiply(ns + k * kLd + ty * 4, us + k * kWp + tx * 4);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int t = ty * 4 + i;
@@ -586,7 +629,7 @@ extern "C" {
 
 int64_t gated_delta_channel_chunked_scratch(int32_t num_tokens, int32_t num_seqs, int32_t num_heads, int32_t dk, int32_t dv) {
     const int64_t th = (int64_t)num_tokens * num_heads, sh = chunk_slots(num_tokens, num_seqs) * num_heads;
-    return 3 * round4(th * dk) + th * kC + round4(th * dv) + round4(sh * dk) + round4(sh * dv * dk);
+    return 2 * round4(th * dk) + sh * dk * kC + sh * kC * kC + round4(th * dv) + round4(sh * dk) + round4(sh * dv * dk);
 }
 
 void gated_delta_channel_chunked(const float* qkv, const float* proj, int64_t ld_proj, int32_t off_b, const float* decay, float* state, float* out, float* scratch,
@@ -606,8 +649,8 @@ void gated_delta_channel_chunked(const float* qkv, const float* proj, int64_t ld
     A.W = scratch;
     A.KE = A.W + round4(th * dk);
     A.QP = A.KE + round4(th * dk);
-    A.N = A.QP + round4(th * dk);
-    A.U = A.N + th * kC;
+    A.N = A.QP + sh * dk * kC;
+    A.U = A.N + sh * kC * kC;
     A.Pe = A.U + round4(th * dv);
     A.Sc = A.Pe + round4(sh * dk);
     cudaStream_t st = as_stream(stream);
@@ -617,7 +660,7 @@ void gated_delta_channel_chunked(const float* qkv, const float* proj, int64_t ld
         ensure_dynamic_smem(reinterpret_cast<const void*>(delta_chunk_prepare_kernel<KD>), s1); \
         ensure_dynamic_smem(reinterpret_cast<const void*>(delta_chunk_walk_kernel<KD>), s2); \
         launch_pdl(delta_chunk_prepare_kernel<KD>, dim3(1, num_heads, z), dim3(256), (size_t)s1, st, A); \
-        launch_pdl(delta_chunk_walk_kernel<KD>, dim3(ceil_div(dv, kVB), num_heads, num_seqs), dim3(256), (size_t)s2, st, A); } while (0)
+        launch_pdl(delta_chunk_walk_kernel<KD>, dim3(ceil_div(dv, kVB), num_heads, num_seqs), dim3(kWalkThreads), (size_t)s2, st, A); } while (0)
     if (dk <= 32) DCH(32);
     else if (dk <= 64) DCH(64);
     else DCH(128);
